@@ -35,7 +35,7 @@ typedef enum {
 
 /* Element types.  Values 0/1 match the reference's WeightPrecision (src/model.h:8-12) and GGMLType
  * F32/F16 (src/gguf.h:10-12). */
-typedef enum { LPP_F32 = 0, LPP_F16 = 1 } lpp_dtype;
+typedef enum { LPP_F32 = 0, LPP_F16 = 1, LPP_BF16 = 2 /* weights only */ } lpp_dtype;
 typedef enum { LPP_MEM_HOST = 0, LPP_MEM_DEVICE = 1 } lpp_memkind;
 
 /* Which reference tensor an upload carries: one value per transformerWeights member
@@ -53,7 +53,20 @@ typedef enum {
     LPP_T_W3 = 9,       /* w3 (up)               [F][D]   per layer                       */
     LPP_T_RMS_FINAL = 10, /* rms_final_weight    [D]                                      */
     LPP_T_W_CLS = 11,   /* w_cls                 [V][D]   (omit for tied embeddings)      */
-    LPP_T_COUNT = 12
+    /* Engines made by lpp_engine_create_layers only (no counterpart in the reference).  H heads with dim plain
+     * and rot rotated query/key dimensions and vdim value dimensions each, latent size rank; the shared ids above keep
+     * their meaning (RMS_ATT / RMS_FFN / RMS_FINAL are the norm weights before the mixer, before the feed-forward and
+     * before the classifier, WO is [D][H*vdim], W1 / W2 / W3 are gate / down / up). */
+    LPP_T_NORM1_B = 12,     /* LayerNorm bias before the mixer         [D]                    per layer */
+    LPP_T_NORM2_B = 13,     /* LayerNorm bias before the feed-forward  [D]                    per layer */
+    LPP_T_NORM_FINAL_B = 14,/* LayerNorm bias before the classifier    [D]                              */
+    LPP_T_LAT_Q = 15,       /* queries, per head dim plain then rot    [H*(dim+rot)][D]       per layer */
+    LPP_T_LAT_DKV = 16,     /* latent, then the shared key part        [rank+rot][D]          per layer */
+    LPP_T_LAT_NORM = 17,    /* RMS norm weight of the latent           [rank]                 per layer */
+    LPP_T_LAT_UK = 18,      /* latent -> plain keys, head by head      [H*dim][rank]          per layer */
+    LPP_T_LAT_UV = 19,      /* latent -> values, head by head          [H*vdim][rank]         per layer */
+    LPP_T_LAT_G = 20,       /* output gates, one per head              [H][D]                 per layer */
+    LPP_T_COUNT = 21
 } lpp_tensor;
 
 /* Engine flags (lpp_config.flags). */
@@ -66,6 +79,7 @@ typedef enum {
                                   * are mapped (lpp_tp_connect); default is the exchange fused into the GEMVs */
 #define LPP_FLAG_NO_PREFILL_GEMM 0x80u /* lpp_prefill feeds the prompt token by token (the reference's way) instead of
                                         * through the batched tensor-core path */
+#define LPP_FLAG_LATENT_CUDA_CORES 0x100u /* latent attention on the CUDA cores (the kernel of FP32 engines) whatever the sizes */
 #define LPP_FLAG_TP_LOCAL 0x40u  /* tensor parallelism without NCCL: the engine never loads or initialises NCCL and
                                   * nccl_id may be NULL; only the peer-memory exchange (lpp_tp_connect) can run */
 
@@ -87,6 +101,40 @@ typedef struct {
     int32_t tp_wait_ms;   /* the same for a wait on a tensor-parallel peer (0 = default, seconds)   */
 } lpp_config;
 
+/* A model as a list of layers, for designs whose layers differ from the reference's (or from one another).  A layer
+ * is  x += mixer(norm(x)),  then  x += W2 (act(W1 norm(x)) * (W3 norm(x)))  when it has a feed-forward. */
+typedef enum { LPP_MIXER_LATENT = 1 } lpp_mixer;
+typedef enum { LPP_NORM_RMS = 0, LPP_NORM_LAYER = 1 } lpp_norm;
+typedef enum { LPP_ACT_SILU = 0, LPP_ACT_GELU_TANH = 1 } lpp_act;
+
+typedef struct {
+    int32_t mixer;     /* lpp_mixer */
+    /* LPP_MIXER_LATENT: latent attention with a sigmoid gate per head.  score = (q_plain . k_plain + q_rot . k_rot) *
+     * scale over the positions of the window; the cache holds the normed latent and the rotated key part. */
+    int32_t heads, dim, rot_dim, vdim, kv_rank;
+    int32_t window;    /* positions a query sees, itself included; 0 = all before it */
+    float scale;
+    /* rotation of neighbouring pairs: the first rot_dims of the rot_dim rotated dimensions turn, pair i by pos * f_i with
+     * f_i = rot_base^(-2i/rot_dims); the rest pass unchanged */
+    int32_t rot_dims;
+    double rot_base;
+    /* YaRN stretching of the slow pairs; yarn_factor 0 = none */
+    double yarn_factor, yarn_original, yarn_fast, yarn_slow;
+    int32_t ff;        /* width of the feed-forward, 0 = the layer has none */
+    int32_t act;       /* lpp_act */
+} lpp_layer_desc;
+
+typedef struct {
+    int32_t dim, vocab_size, seq_len, n_layers;
+    int32_t norm;      /* lpp_norm of the norms before mixer, feed-forward and classifier */
+    float norm_eps;    /* of every norm */
+    int32_t weight_dtype; /* LPP_BF16 (with an LPP_F16 cache: batched prompts) or LPP_F32 (everything in FP32) */
+    int32_t kv_dtype;
+    int32_t device;
+    uint32_t flags;
+    int32_t ring_kb, wait_ms;
+} lpp_model_desc;
+
 /* Sampling parameters of one step: forward()'s temperature / penalty arguments
  * (src/model.h:164).  top-p is not part of the device sampler, as in src/sample.cu:210-214. */
 typedef struct {
@@ -100,6 +148,9 @@ typedef struct {
 /* nccl_id: 128-byte ncclUniqueId shared by all ranks when tp_size > 1 (from lpp_nccl_unique_id on
  * rank 0), NULL otherwise. */
 lpp_status lpp_engine_create(const lpp_config* cfg, const void* nccl_id, lpp_engine** out);
+/* The same engine for a model given layer by layer (one GPU; the classifier is the embedding unless w_cls is uploaded).
+ * Any sizes: the engine pads rows internally.  layers[n_layers] is copied. */
+lpp_status lpp_engine_create_layers(const lpp_model_desc* model, const lpp_layer_desc* layers, lpp_engine** out);
 lpp_status lpp_engine_destroy(lpp_engine* e);
 lpp_status lpp_nccl_unique_id(void* out128);
 
@@ -157,6 +208,13 @@ lpp_status lpp_decode(lpp_engine* e, int first_token, int start_pos, int n, cons
  * *device_ms (optional) receives the CUDA-event time. */
 lpp_status lpp_prefill(lpp_engine* e, const int* h_tokens, int n, int start_pos, float* device_ms);
 
+/* One portion of a sequence with logits: runs the n tokens at positions start_pos .. from the cache that earlier calls
+ * left (portions may be cut anywhere) and writes the logits of the n_want tokens want[0] < want[1] < ... (indices into
+ * h_tokens) to h_logits[n_want][vocab_size].  n_want may be 0.  Single tokens go through the step graph, longer portions
+ * through the batched path where the engine has one. */
+lpp_status lpp_extend(lpp_engine* e, const int* h_tokens, int n, int start_pos, const int* want, int n_want, float* h_logits,
+                      float* device_ms);
+
 /* cuda_sample (src/kernels.cuh:36, src/sample.cu:210-214) on caller-supplied logits: copies
  * h_logits[vocab_size] to the device and runs the engine's sampler on them. */
 lpp_status lpp_sample_logits(lpp_engine* e, const float* h_logits, const lpp_sample_params* sp,
@@ -169,6 +227,8 @@ lpp_status lpp_kv_prefill(lpp_engine* e, int layer, const void* k, const void* v
                           int memkind);
 /* Read one cache row (this rank's kv heads only) as FP32; h_k / h_v hold head_size floats. */
 lpp_status lpp_kv_read(lpp_engine* e, int layer, int kv_head, int pos, float* h_k, float* h_v);
+/* Latent attention: one cache row as FP32, kv_rank latent values then rot_dim rotated key values. */
+lpp_status lpp_latent_read(lpp_engine* e, int layer, int pos, float* h_row);
 /* Element offset, inside this engine's K (or V) cache allocation, of element `off` of kv head
  * `kv_head` (rank-local numbering) at `pos`: the reference's scatter index. */
 int64_t lpp_kv_index(const lpp_engine* e, int layer, int kv_head, int pos, int off);
@@ -186,7 +246,8 @@ int64_t lpp_step_bytes(const lpp_engine* e, int pos);
 /* Per-kernel-kind timing of one step at `pos`: the step is captured with a CUDA event-record node
  * before and after every kernel and replayed iters times (isolated kernel durations, no programmatic
  * overlap, no host launch latency).  kinds: 0 qkv gemv, 1 attention, 2 o_proj gemv, 3 gate|up gemv, 4 down gemv,
- * 5 lm-head gemv, 6 sampler, 7 all-reduce, 8-9 reserved.  ms[10] total device ms per step per
+ * 5 lm-head gemv, 6 sampler, 7 all-reduce, 8 latent query gemv, 9 latent value gemv
+ * (0 is the input gemv of a latent layer).  ms[10] total device ms per step per
  * kind, launches[10] launches per step, bytes[10] algorithmic bytes per step.  The sampler runs with the
  * temperature and penalty given in *sp (NULL = temperature 0, no penalty). */
 lpp_status lpp_profile_step(lpp_engine* e, int pos, int iters, const lpp_sample_params* sp, float* ms, int* launches,

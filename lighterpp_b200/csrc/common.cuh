@@ -3,9 +3,12 @@
 // the host, and the device-resident per-step state.
 #pragma once
 #include <cuda_runtime.h>
+#include <cuda_bf16.h>
 #include <cuda_fp16.h>
 #include <stdint.h>
 #include <math.h>
+
+#include <type_traits>
 
 namespace lpp {
 
@@ -55,6 +58,11 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// Barrier of the consumer threads of a GEMV CTA (its producer warp does not take part).
+__device__ __forceinline__ void consumer_barrier(int nthreads) {
+    asm volatile("bar.sync 1, %0;" ::"r"(nthreads) : "memory");
+}
+
 __device__ __forceinline__ uint32_t smem_u32(const void* p) {
     return static_cast<uint32_t>(__cvta_generic_to_shared(p));
 }
@@ -71,6 +79,43 @@ __device__ __forceinline__ uint4 ldg_stream_u4(const void* p) {
 __device__ __forceinline__ float2 half2_bits_to_float2(uint32_t u) {
     __half2 h = *reinterpret_cast<__half2*>(&u);
     return __half22float2(h);
+}
+
+// bfloat16 is the upper half of the FP32 word: widening is a shift or a mask.
+__device__ __forceinline__ float2 bf162_bits_to_float2(uint32_t u) {
+    return make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u));
+}
+// Two packed 16-bit elements of type T (FP16 or BF16) as FP32.
+template <typename T>
+__device__ __forceinline__ float2 unpack2(uint32_t u) {
+    if constexpr (std::is_same<T, __nv_bfloat16>::value)
+        return bf162_bits_to_float2(u);
+    else
+        return half2_bits_to_float2(u);
+}
+__device__ __forceinline__ float to_float(float v) { return v; }
+__device__ __forceinline__ float to_float(__half v) { return __half2float(v); }
+__device__ __forceinline__ float to_float(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <typename T>
+__device__ __forceinline__ T from_float(float v) {
+    if constexpr (std::is_same<T, __half>::value)
+        return __float2half_rn(v);
+    else if constexpr (std::is_same<T, __nv_bfloat16>::value)
+        return __float2bfloat16_rn(v);
+    else
+        return v;
+}
+
+// ------------------------------------------------------------------ activations of the gated feed-forward
+
+enum Act : int { kActSilu = 0, kActGeluTanh = 1 };
+
+// Argument of the sigmoid that either activation multiplies its input with: silu(z) = z sigmoid(z), and because
+// (1 + tanh(u)) / 2 = sigmoid(2u), gelu_tanh(z) = z sigmoid(2 sqrt(2/pi) (z + 0.044715 z^3)).
+__device__ __forceinline__ float act_gate_arg(int act, float z) {
+    if (act == kActSilu) return z;
+    const float kTwoSqrt2OverPi = 1.5957691216057308f;
+    return kTwoSqrt2OverPi * (z + 0.044715f * z * z * z);
 }
 
 // ------------------------------------------------------------------ programmatic dependent launch
@@ -196,7 +241,7 @@ __device__ __forceinline__ void bulk_prefetch_l2(const void* gsrc, uint32_t byte
 
 // ------------------------------------------------------------------ reproducible expf
 
-// exp(x) for float x, evaluated in double with only IEEE add/mul/fma, so the host twin (same
+// exp(x) for float x (Cody-Waite argument reduction, Taylor polynomial), evaluated in double with only IEEE add/mul/fma, so the host twin (same
 // source, compiled by the host compiler) returns the same bits as the device.  Relative error of
 // the double intermediate is < 1e-13, so the float result is the correctly rounded exp(x) except
 // when exp(x) lies within that distance of a rounding boundary.

@@ -15,6 +15,8 @@
 //   K, V cache [L][KVHl][S][hs]   FP16 (or FP32), the reference's index order
 //   rope [S][hs/2] (cos, sin)     built on the host with libm so rotations match the CPU path bit
 //                                 for bit
+// Engines made by lpp_engine_create_layers keep one allocation per matrix and layer (LatentLayer below): layers may
+// differ in every size, rows are padded with zeros to a multiple of 64 inputs.
 #include <cuda_runtime.h>
 #include <cuda_fp16.h>
 #include <dlfcn.h>
@@ -32,6 +34,7 @@
 #include "attention.cuh"
 #include "common.cuh"
 #include "gemv.cuh"
+#include "latent_attention.cuh"
 #include "ops.cuh"
 #include "prefill.cuh"
 #include "sampler.cuh"
@@ -123,7 +126,24 @@ static bool load() {
 
 // ------------------------------------------------------------------ engine
 
-enum Kind { kQkv = 0, kAttn = 1, kOproj = 2, kGateUp = 3, kDown = 4, kLmHead = 5, kSampler = 6, kAllReduce = 7, kKinds = 10 };
+enum Kind { kQkv = 0, kAttn = 1, kOproj = 2, kGateUp = 3, kDown = 4, kLmHead = 5, kSampler = 6, kAllReduce = 7, kLatQuery = 8, kLatValue = 9, kKinds = 10 };
+
+// One layer of latent attention with its feed-forward (latent.cuh).  Weight matrices: rows x pitch, pitch = inputs rounded
+// up to 64, zero padded; element type = weight_dtype.
+struct LatentLayer {
+    lpp_layer_desc d;
+    int rank_pitch, row_width;  // query / cache rows: latent part, whole
+    int dim_pitch, val_pitch;   // inputs per head of the query and of the value matrix
+    int vdim_rows;              // rows per head of the value matrix
+    int o_pitch, ff_pitch;      // inputs of the output projection and of the down projection
+    int q_plain_rows, q_rot_rows, latent_rows, in_rows;
+    void *w_in = nullptr, *w_uk = nullptr, *w_uv = nullptr, *wo = nullptr, *w13 = nullptr, *w2 = nullptr;
+    float *n1w = nullptr, *n1b = nullptr, *n2w = nullptr, *n2b = nullptr, *lat_w = nullptr;
+    const float2* rope = nullptr;
+    void* cache = nullptr;      // [seq_len][row_width]
+    CUtensorMap m_in, m_uk, m_uv, m_wo, m_w13, m_w2;    // weights (batched path)
+    CUtensorMap x_qn, x_olat, x_att, x_hb;              // activation blocks with this layer's widths
+};
 
 struct lpp_engine {
     lpp_config c;
@@ -137,7 +157,16 @@ struct lpp_engine {
     cudaStream_t stream = nullptr;
     // weights
     void *wqkv = nullptr, *wo = nullptr, *w13 = nullptr, *w2 = nullptr, *emb = nullptr, *wcls = nullptr;
-    float *rms_att = nullptr, *rms_ffn = nullptr, *rms_final = nullptr;
+    float *rms_att = nullptr, *rms_ffn = nullptr, *rms_final = nullptr, *final_b = nullptr;
+    // norms: RMS with the reference's epsilon unless the model says otherwise; Dp = width of a row in memory
+    int Dp = 0, Vp = 0;  // row pitch of width-sized vectors, classifier rows
+    bool layer_norm = false;
+    float norm_eps = 1e-5f;  // src/ops.cpp:20-32
+    // layers of lpp_engine_create_layers (empty for the reference's own architecture), buffers their steps share
+    std::vector<LatentLayer> lat;
+    std::vector<std::pair<lpp_layer_desc, float2*>> rope_tables;
+    float *lat_qplain = nullptr, *lat_raw = nullptr, *lat_gate = nullptr, *lat_part = nullptr;
+    void* lat_query = nullptr;
     bool wcls_owned = false;
     bool wcls_shard_only = false;  // an untied classifier of a tensor-parallel rank holds this rank's vocabulary rows only
     std::vector<unsigned char> got;  // upload bookkeeping: [tensor][layer]
@@ -177,8 +206,13 @@ struct lpp_engine {
 
     // batched prompt path (allocated by the first lpp_prefill)
     float *pf_x = nullptr, *pf_q = nullptr, *pf_part = nullptr;
-    __half *pf_xn = nullptr, *pf_att = nullptr, *pf_hb = nullptr;
-    int* pf_tokens = nullptr;
+    void *pf_xn = nullptr, *pf_att = nullptr, *pf_hb = nullptr;
+    int *pf_tokens = nullptr, *pf_rows = nullptr;
+    float* pf_logits = nullptr;
+    CUtensorMap pf_map_cls;
+    void *pf_qn = nullptr, *pf_olat = nullptr;      // latent attention: plain queries, attended latents (hi + lo operands)
+    __half* pf_lq = nullptr;                        // query rows
+    float *pf_lpart = nullptr, *pf_gate = nullptr;  // attention partials, gates
     CUtensorMap pf_map_wqkv, pf_map_wo, pf_map_w13, pf_map_w2, pf_map_xn, pf_map_att, pf_map_hb;
     bool pf_ready = false;
 
@@ -242,9 +276,15 @@ template <typename WT, int EPI>
 static cudaError_t launch_gemv_t(lpp_engine* e, GemvArgs& a, bool pdl, cudaStream_t s) {
     const int esz = sizeof(WT);
     const int groups = a.n_rows / kRowsPerGroup;
-    const size_t xbytes = align_up((size_t)a.K * 4, 128);
+    // Grouped rows: a CTA stages the inputs of every group its contiguous row pairs touch, plus the split weights.
+    auto staged_bytes = [&](int grid) -> size_t {
+        if (a.group_pairs <= 0) return align_up((size_t)a.K * 4, 128);
+        const int pairs = (groups + grid - 1) / grid;
+        const size_t n = (size_t)(pairs + a.group_pairs - 2) / a.group_pairs + 1;
+        return align_up(n * ((size_t)a.K + kLatentMaxSplits) * 4, 128);
+    };
     if (e->c.flags & LPP_FLAG_GEMV_LDG) {
-        const size_t smem = 128 + xbytes;
+        const size_t smem = 128 + staged_bytes(std::max(1, std::min(groups, e->num_sms * 4)));
         static bool attr_done[64] = {};
         if (!attr_done[e->c.device & 63]) {
             cudaError_t r = cudaFuncSetAttribute(gemv_ldg_kernel<WT, EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -259,12 +299,15 @@ static cudaError_t launch_gemv_t(lpp_engine* e, GemvArgs& a, bool pdl, cudaStrea
     int stage_target = kStageTarget;
     if (const char* sk = aid_env("LPP_STAGE_KB")) stage_target = std::max(1, atoi(sk)) * 1024;
     gemv_geometry(a, esz, stage_target);
+    const int grid = std::max(1, std::min(groups, e->num_sms));
+    const size_t xbytes = staged_bytes(grid);
+    a.xs_bytes = (int)xbytes;
     const size_t fixed = kGemvBarrierBytes + 128 + xbytes;
+    if (fixed >= e->smem_optin) return cudaErrorInvalidValue;
     size_t ring = (size_t)(e->c.ring_kb > 0 ? e->c.ring_kb : 128) * 1024;
     if (fixed + ring > e->smem_optin) ring = e->smem_optin - fixed;
     int ns = (int)(ring / ((size_t)kGemvConsumerWarps * a.stage_bytes));  // slots per consumer warp
     ns = std::max(2, std::min(ns, kGemvMaxStages));
-    const int grid = std::max(1, std::min(groups, e->num_sms));
     a.n_stages = ns;
     const size_t smem = fixed + (size_t)kGemvConsumerWarps * ns * a.stage_bytes;
     if (smem > e->smem_optin) return cudaErrorInvalidValue;
@@ -279,17 +322,25 @@ static cudaError_t launch_gemv_t(lpp_engine* e, GemvArgs& a, bool pdl, cudaStrea
 }
 
 static cudaError_t launch_gemv(lpp_engine* e, int epi, int w_dtype, GemvArgs& a, bool pdl, cudaStream_t s) {
-#define LPP_GEMV_CASE(E)                                                          \
-    case E:                                                                       \
-        return w_dtype == LPP_F16 ? launch_gemv_t<__half, E>(e, a, pdl, s)        \
-                                  : launch_gemv_t<float, E>(e, a, pdl, s);
+#define LPP_GEMV_CASE(E)                                                                \
+    case E:                                                                             \
+        if (w_dtype == LPP_BF16) return launch_gemv_t<__nv_bfloat16, E>(e, a, pdl, s);  \
+        return w_dtype == LPP_F16 ? launch_gemv_t<__half, E>(e, a, pdl, s) : launch_gemv_t<float, E>(e, a, pdl, s);
+#define LPP_GEMV_LATENT_CASE(E)                                                         \
+    case E:                                                                             \
+        return w_dtype == LPP_BF16 ? launch_gemv_t<__nv_bfloat16, E>(e, a, pdl, s) : launch_gemv_t<float, E>(e, a, pdl, s);
     switch (epi) {
         LPP_GEMV_CASE(kEpiStore)
         LPP_GEMV_CASE(kEpiResid)
         LPP_GEMV_CASE(kEpiSwiglu)
-        LPP_GEMV_CASE(kEpiQkv)
+        case kEpiQkv:
+            return w_dtype == LPP_F16 ? launch_gemv_t<__half, kEpiQkv>(e, a, pdl, s) : launch_gemv_t<float, kEpiQkv>(e, a, pdl, s);
+        LPP_GEMV_LATENT_CASE(kEpiLatentIn)
+        LPP_GEMV_LATENT_CASE(kEpiLatentQuery)
+        LPP_GEMV_LATENT_CASE(kEpiLatentValue)
     }
 #undef LPP_GEMV_CASE
+#undef LPP_GEMV_LATENT_CASE
     return cudaErrorInvalidValue;
 }
 
@@ -333,6 +384,94 @@ static cudaError_t launch_attn_mma(lpp_engine* e, const AttnArgs& a, bool pdl, c
 }
 static bool attn_mma_supported(const lpp_engine* e) {
     return e->c.kv_dtype == LPP_F16 && (e->hs == 64 || e->hs == 128) && (e->gqa == 1 || e->gqa == 2 || e->gqa == 4 || e->gqa == 8);
+}
+
+// ---- latent attention: the tensor-core kernel where query and key tiles fit shared memory, else the CUDA-core kernel
+
+constexpr int kLatMinChunk = 64;  // fewest keys worth a split of their own
+// Splits the step launches: as many as the window (or the cache) can fill.
+static int latent_decode_splits(const lpp_engine* e, const LatentLayer& y) {
+    const int keys = y.d.window > 0 ? std::min(y.d.window, e->c.seq_len) : e->c.seq_len;
+    return std::max(1, std::min(kLatentMaxSplits, (keys + kLatMinChunk - 1) / kLatMinChunk));
+}
+static bool latent_mma_supported(const lpp_engine* e, const LatentLayer& y) {
+    return e->c.kv_dtype == LPP_F16 && y.rank_pitch <= 512 && (size_t)latent_mma_smem<2>(y.row_width) <= e->smem_optin &&
+           !(e->c.flags & LPP_FLAG_LATENT_CUDA_CORES);
+}
+static int latent_tile_rows(int rows) { return rows <= 16 ? 16 : 32; }
+template <int MT, int NT>
+static cudaError_t launch_latent_mma(lpp_engine* e, const LatentAttnArgs& a, int splits, bool pdl, cudaStream_t s) {
+    static bool attr_done[64] = {};
+    if (!attr_done[e->c.device & 63]) {
+        const cudaError_t r = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)e->smem_optin);
+        if (r != cudaSuccess) return r;
+        attr_done[e->c.device & 63] = true;
+    }
+    const dim3 grid(splits, (a.n_tokens * a.heads + 16 * MT - 1) / (16 * MT));
+    return launch_kernel(latent_attn_mma_kernel<MT, NT>, grid, dim3(kLatentThreads), (size_t)latent_mma_smem<MT>(a.row_width), s, pdl, a);
+}
+static cudaError_t launch_latent_attn(lpp_engine* e, const LatentLayer& y, const LatentAttnArgs& a, bool pdl, cudaStream_t s) {
+    const int splits = a.max_splits, rp = a.rank_pitch;
+    if (latent_mma_supported(e, y)) {
+        if (latent_tile_rows(a.n_tokens * a.heads) == 16)
+            return rp <= 128   ? launch_latent_mma<1, 2>(e, a, splits, pdl, s)
+                   : rp <= 256 ? launch_latent_mma<1, 4>(e, a, splits, pdl, s)
+                               : launch_latent_mma<1, 8>(e, a, splits, pdl, s);
+        return rp <= 128   ? launch_latent_mma<2, 4>(e, a, splits, pdl, s)
+               : rp <= 256 ? launch_latent_mma<2, 8>(e, a, splits, pdl, s)
+                           : launch_latent_mma<2, 16>(e, a, splits, pdl, s);
+    }
+    const dim3 grid(splits, a.heads, a.n_tokens);
+    const size_t smem = (size_t)(a.row_width + kLatentTile) * 4;
+    if (e->c.kv_dtype == LPP_F32) return launch_kernel(latent_attn_kernel<float>, grid, dim3(kLatentThreads), smem, s, pdl, a);
+    return launch_kernel(latent_attn_kernel<__half>, grid, dim3(kLatentThreads), smem, s, pdl, a);
+}
+static LatentArgs latent_args(const lpp_engine* e, const LatentLayer& y) {
+    LatentArgs L = {};
+    L.heads = y.d.heads;
+    L.dim = y.d.dim;
+    L.rot = y.d.rot_dim;
+    L.vdim = y.d.vdim;
+    L.rank = y.d.kv_rank;
+    L.dim_pitch = y.dim_pitch;
+    L.rank_pitch = y.rank_pitch;
+    L.row_width = y.row_width;
+    L.vdim_rows = y.vdim_rows;
+    L.q_plain_rows = y.q_plain_rows;
+    L.q_rot_rows = y.q_rot_rows;
+    L.latent_rows = y.latent_rows;
+    L.cache_f32 = e->c.kv_dtype == LPP_F32;
+    L.rope = y.rope;
+    L.q_plain = e->lat_qplain;
+    L.latent = e->lat_raw;
+    L.gate = e->lat_gate;
+    L.query = e->lat_query;
+    L.cache = y.cache;
+    L.norm_w = y.lat_w;
+    L.norm_eps = e->norm_eps;
+    L.part = e->lat_part;
+    L.window = y.d.window;
+    L.max_splits = latent_decode_splits(e, y);
+    L.min_chunk = kLatMinChunk;
+    return L;
+}
+static LatentAttnArgs latent_attn_args(const lpp_engine* e, const LatentLayer& y) {
+    LatentAttnArgs a = {};
+    a.q = e->lat_query;
+    a.cache = y.cache;
+    a.part = e->lat_part;
+    a.st = e->st;
+    a.start_pos = -1;
+    a.n_tokens = 1;
+    a.heads = y.d.heads;
+    a.rank_pitch = y.rank_pitch;
+    a.row_width = y.row_width;
+    a.window = y.d.window;
+    a.max_splits = latent_decode_splits(e, y);
+    a.min_chunk = kLatMinChunk;
+    a.seq_len = e->c.seq_len;
+    a.scale = y.d.scale;
+    return a;
 }
 
 // ---- one decode step as a sequence of launches (captured into the graph, or run directly)
@@ -392,6 +531,8 @@ static void record_gemv(Recorder& R, int kind, int epi, GemvArgs a) {
     }
     a.vocab = e->c.vocab_size;
     a.seq_len = e->c.seq_len;
+    a.norm_eps = e->norm_eps;
+    a.norm_n = e->c.dim;
     R.mark(kind);
     R.check(launch_gemv(e, epi, e->c.weight_dtype, a, R.pdl(), R.s), "gemv launch");
     R.mark(-1);
@@ -582,80 +723,146 @@ static __global__ void tp_bump_kernel(unsigned int* epoch) {
     *epoch = *epoch + 1u;
 }
 
+// What the kernels after the mixer need to know about a layer, whichever way its weights are stored.
+struct LayerView {
+    const void *wo, *w13, *w2;
+    const float *norm2_w, *norm2_b;
+    int o_k, ff, ff_k;  // inputs of the output projection; feed-forward width (0 = none), inputs of the down projection
+    int act;
+};
+static LayerView layer_view(const lpp_engine* e, int l) {
+    if (!e->lat.empty()) {
+        const LatentLayer& y = e->lat[l];
+        return {y.wo, y.w13, y.w2, y.n2w, y.n2b, y.o_pitch, y.d.ff, y.ff_pitch, y.d.act == LPP_ACT_GELU_TANH ? kActGeluTanh : kActSilu};
+    }
+    const size_t D = e->c.dim, esz = e->esz;
+    return {(const char*)e->wo + (size_t)l * D * e->Dq * esz, (const char*)e->w13 + (size_t)l * 2 * e->Fl * D * esz,
+            (const char*)e->w2 + (size_t)l * D * e->Fl * esz, e->rms_ffn + (size_t)l * D, nullptr, e->Dq, e->Fl, e->Fl, kActSilu};
+}
+
+// Grouped-query attention of the reference: fused norm + QKV GEMV + RoPE + KV scatter, split-KV flash decode.
+static void record_gqa_mixer(Recorder& R, int l, float* cur) {
+    lpp_engine* e = R.e;
+    const lpp_config& c = e->c;
+    const int D = c.dim, qkv_rows = e->Dq + 2 * e->KVd;
+    GemvArgs a = {};
+    a.W = (const char*)e->wqkv + (size_t)l * qkv_rows * D * e->esz;
+    a.n_rows = qkv_rows;
+    a.K = D;
+    a.norm_w = e->rms_att + (size_t)l * D;
+    if (l == 0) {
+        a.emb = e->emb;
+        a.x_store = cur;
+    } else {
+        a.x = cur;
+        if (tp_peer_path(e)) tp_set_consumer(e, a, 2 * (l - 1) + 1, cur);  // the previous layer's down exchange
+    }
+    a.out = e->q;
+    a.q_rows = e->Dq;
+    a.kv_rows = e->KVd;
+    a.head_size = e->hs;
+    a.rope = e->rope;
+    const size_t lofs = (size_t)l * e->KVHl * c.seq_len * e->hs * e->kvesz;
+    a.k_cache = (char*)e->kcache + lofs;
+    a.v_cache = (char*)e->vcache + lofs;
+    a.kv_is_f32 = c.kv_dtype == LPP_F32;
+    // split-KV flash decode
+    AttnArgs at = {};
+    at.q = e->q;
+    at.k_cache = a.k_cache;
+    at.v_cache = a.v_cache;
+    at.out = e->att_out;
+    at.part = e->attn_part;
+    at.counters = e->attn_counters;
+    at.st = e->st;
+    at.seq_len = c.seq_len;
+    at.head_size = e->hs;
+    at.gqa = e->gqa;
+    at.n_splits = e->attn_splits;
+    at.n_kv_heads = e->KVHl;
+    if (const char* mc = aid_env("LPP_ATTN_CHUNK")) at.min_chunk = atoi(mc);  // timing experiments
+    set_prefetch(e, a, kQkv, l);
+    record_gemv(R, kQkv, kEpiQkv, a);
+    dim3 grid(e->attn_splits, e->KVHl, e->attn_z);
+    if (kind_skipped(e, kAttn)) return;
+    if (e->gtrace && R.kernels < 256) at.trace = e->gtrace + (size_t)R.kernels * e->num_sms * 8;
+    R.mark(kAttn);
+    if (attn_mma_supported(e) && !aid_env("LPP_ATTN_CUDA_CORES")) {
+        at.n_splits = e->attn_splits_long;
+        R.check(launch_attn_mma(e, at, R.pdl(), R.s), "attention (tensor-core) launch");
+    } else {
+        R.check(c.kv_dtype == LPP_F32 ? launch_attn_t<float>(e, at, grid, R.pdl(), R.s)
+                                      : launch_attn_t<__half>(e, at, grid, R.pdl(), R.s),
+                "attention launch");
+    }
+    R.mark(-1);
+    R.prev_kernel = true;
+    R.kernels++;
+}
+
+// Latent attention: input GEMV, query GEMV, attention over the window, value GEMV (latent.cuh).
+static void record_latent_mixer(Recorder& R, int l, float* cur) {
+    lpp_engine* e = R.e;
+    const LatentLayer& y = e->lat[l];
+    GemvArgs a = {};
+    a.lat = latent_args(e, y);
+    a.W = y.w_in;
+    a.n_rows = y.in_rows;
+    a.K = e->Dp;
+    a.norm_w = y.n1w;
+    a.norm_b = y.n1b;
+    if (l == 0) {
+        a.emb = e->emb;
+        a.x_store = cur;
+    } else {
+        a.x = cur;
+    }
+    record_gemv(R, kQkv, kEpiLatentIn, a);
+    GemvArgs q = {};
+    q.lat = a.lat;
+    q.W = y.w_uk;
+    q.n_rows = y.d.heads * y.rank_pitch;
+    q.K = y.dim_pitch;
+    q.x = e->lat_qplain;
+    q.group_pairs = y.rank_pitch / kRowsPerGroup;
+    record_gemv(R, kLatQuery, kEpiLatentQuery, q);
+    if (!kind_skipped(e, kAttn)) {
+        R.mark(kAttn);
+        R.check(launch_latent_attn(e, y, latent_attn_args(e, y), R.pdl(), R.s), "latent attention launch");
+        R.mark(-1);
+        R.prev_kernel = true;
+        R.kernels++;
+    }
+    GemvArgs v = {};
+    v.lat = a.lat;
+    v.W = y.w_uv;
+    v.n_rows = y.d.heads * y.vdim_rows;
+    v.K = y.val_pitch;
+    v.out = e->att_out;
+    v.group_pairs = y.vdim_rows / kRowsPerGroup;
+    record_gemv(R, kLatValue, kEpiLatentValue, v);
+}
+
 static void record_step(Recorder& R, bool with_sampler) {
     lpp_engine* e = R.e;
     const lpp_config& c = e->c;
-    const int D = c.dim, L = c.n_layers;
+    const int D = e->Dp, L = c.n_layers;
     const size_t esz = e->esz;
-    const int qkv_rows = e->Dq + 2 * e->KVd;
     const bool tp = c.tp_size > 1;
     const bool peers = tp_peer_path(e);  // fused exchange over peer memory instead of an NCCL all-reduce
     float* cur = e->xa;
     float* oth = e->xb;
     for (int l = 0; l < L; ++l) {
-        {  // fused RMSNorm + QKV GEMV + RoPE + KV scatter
-            GemvArgs a = {};
-            a.W = (const char*)e->wqkv + (size_t)l * qkv_rows * D * esz;
-            a.n_rows = qkv_rows;
-            a.K = D;
-            a.norm_w = e->rms_att + (size_t)l * D;
-            if (l == 0) {
-                a.emb = e->emb;
-                a.x_store = cur;
-            } else {
-                a.x = cur;
-                if (peers) tp_set_consumer(e, a, 2 * (l - 1) + 1, cur);  // the previous layer's down exchange
-            }
-            a.out = e->q;
-            a.q_rows = e->Dq;
-            a.kv_rows = e->KVd;
-            a.head_size = e->hs;
-            a.rope = e->rope;
-            const size_t lofs = (size_t)l * e->KVHl * c.seq_len * e->hs * e->kvesz;
-            a.k_cache = (char*)e->kcache + lofs;
-            a.v_cache = (char*)e->vcache + lofs;
-            a.kv_is_f32 = c.kv_dtype == LPP_F32;
-            // split-KV flash decode
-            AttnArgs at = {};
-            at.q = e->q;
-            at.k_cache = a.k_cache;
-            at.v_cache = a.v_cache;
-            at.out = e->att_out;
-            at.part = e->attn_part;
-            at.counters = e->attn_counters;
-            at.st = e->st;
-            at.seq_len = c.seq_len;
-            at.head_size = e->hs;
-            at.gqa = e->gqa;
-            at.n_splits = e->attn_splits;
-            at.n_kv_heads = e->KVHl;
-            if (const char* mc = aid_env("LPP_ATTN_CHUNK")) at.min_chunk = atoi(mc);  // timing experiments
-            {
-                set_prefetch(e, a, kQkv, l);
-                record_gemv(R, kQkv, kEpiQkv, a);
-                dim3 grid(e->attn_splits, e->KVHl, e->attn_z);
-                if (!kind_skipped(e, kAttn)) {
-                    if (e->gtrace && R.kernels < 256) at.trace = e->gtrace + (size_t)R.kernels * e->num_sms * 8;
-                    R.mark(kAttn);
-                    if (attn_mma_supported(e) && !aid_env("LPP_ATTN_CUDA_CORES")) {
-                        at.n_splits = e->attn_splits_long;
-                        R.check(launch_attn_mma(e, at, R.pdl(), R.s), "attention (tensor-core) launch");
-                    } else {
-                        R.check(c.kv_dtype == LPP_F32 ? launch_attn_t<float>(e, at, grid, R.pdl(), R.s)
-                                                      : launch_attn_t<__half>(e, at, grid, R.pdl(), R.s),
-                                "attention launch");
-                    }
-                    R.mark(-1);
-                    R.prev_kernel = true;
-                    R.kernels++;
-                }
-            }
-        }
+        if (!e->lat.empty())
+            record_latent_mixer(R, l, cur);
+        else
+            record_gqa_mixer(R, l, cur);
+        const LayerView v = layer_view(e, l);
         {  // o_proj + residual
             GemvArgs a = {};
-            a.W = (const char*)e->wo + (size_t)l * D * e->Dq * esz;
-            a.n_rows = D;
-            a.K = e->Dq;
+            a.W = v.wo;
+            a.n_rows = (c.dim + 1) & ~1;
+            a.K = v.o_k;
             a.x = e->att_out;
             a.resid = (!tp || c.tp_rank == 0) ? cur : nullptr;
             a.out = tp ? oth : cur;
@@ -667,23 +874,26 @@ static void record_step(Recorder& R, bool with_sampler) {
                 std::swap(cur, oth);
             }
         }
-        {  // fused RMSNorm + gate|up GEMV + SwiGLU
+        if (v.ff == 0) continue;  // a layer without a feed-forward
+        {  // fused norm + gate|up GEMV + gated activation
             GemvArgs a = {};
-            a.W = (const char*)e->w13 + (size_t)l * 2 * e->Fl * D * esz;
-            a.n_rows = 2 * e->Fl;
+            a.W = v.w13;
+            a.n_rows = 2 * v.ff;
             a.K = D;
             a.x = cur;
             if (peers) tp_set_consumer(e, a, 2 * l, cur);
-            a.norm_w = e->rms_ffn + (size_t)l * D;
+            a.norm_w = v.norm2_w;
+            a.norm_b = v.norm2_b;
+            a.act = v.act;
             a.out = e->hb;
             set_prefetch(e, a, kGateUp, l);
             record_gemv(R, kGateUp, kEpiSwiglu, a);
         }
         {  // down + residual
             GemvArgs a = {};
-            a.W = (const char*)e->w2 + (size_t)l * D * e->Fl * esz;
-            a.n_rows = D;
-            a.K = e->Fl;
+            a.W = v.w2;
+            a.n_rows = (c.dim + 1) & ~1;
+            a.K = v.ff_k;
             a.x = e->hb;
             a.resid = (!tp || c.tp_rank == 0) ? cur : nullptr;
             a.out = tp ? oth : cur;
@@ -696,14 +906,15 @@ static void record_step(Recorder& R, bool with_sampler) {
             }
         }
     }
-    {  // final RMSNorm + classifier
+    {  // final norm + classifier
         GemvArgs a = {};
         a.W = e->wcls;
-        a.n_rows = c.vocab_size;
+        a.n_rows = e->Vp;
         a.K = D;
         a.x = cur;
         if (peers) tp_set_consumer(e, a, 2 * (L - 1) + 1, cur);
         a.norm_w = e->rms_final;
+        a.norm_b = e->final_b;
         a.out = e->logits;
         const bool sharded = tp_cls_sharded(e);
         if (sharded) {
@@ -781,6 +992,69 @@ static bool dpl_supported(int hs) {
     return hs % 8 == 0 && (d == 2 || d == 4 || d == 6 || d == 8 || d == 12 || d == 16);
 }
 
+// Makes `device` current if it is a GPU this library runs on.
+static lpp_status open_device(int device, cudaDeviceProp* prop) {
+    int ndev = 0;
+    if (cudaGetDeviceCount(&ndev) != cudaSuccess || ndev == 0) {
+        (void)cudaGetLastError();
+        return fail(LPP_ERR_NO_DEVICE, "no CUDA device");
+    }
+    if (device < 0 || device >= ndev) return fail(LPP_ERR_INVALID_ARG, "device %d out of range", device);
+    CU(cudaSetDevice(device));
+    CU(cudaGetDeviceProperties(prop, device));
+    if (prop->major < 10) return fail(LPP_ERR_NO_DEVICE, "device is sm_%d%d; this library is built for sm_100a only", prop->major, prop->minor);
+    return LPP_OK;
+}
+
+// Buffers every kind of engine has: stream, one step's vectors, sampler scratch, step state.  att_n and hb_n are the
+// inputs of the output and of the down projection (the largest ones when layers differ).
+static lpp_status alloc_step_buffers(lpp_engine* e, size_t att_n, size_t hb_n) {
+    const lpp_config& c = e->c;
+    const size_t D = e->Dp;
+    CU(cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking));
+    CU(cudaEventCreate(&e->ev0));
+    CU(cudaEventCreate(&e->ev1));
+    CU(cudaMalloc(&e->xa, D * 4));
+    CU(cudaMalloc(&e->xb, D * 4));
+    CU(cudaMalloc(&e->att_out, att_n * 4));
+    CU(cudaMalloc(&e->hb, hb_n * 4));
+    CU(cudaMalloc(&e->logits, (size_t)e->Vp * 4));
+    // padded inputs stay what they are here: zero
+    CU(cudaMemsetAsync(e->xa, 0, D * 4, e->stream));
+    CU(cudaMemsetAsync(e->xb, 0, D * 4, e->stream));
+    CU(cudaMemsetAsync(e->att_out, 0, att_n * 4, e->stream));
+    CU(cudaMemsetAsync(e->hb, 0, hb_n * 4, e->stream));
+    CU(cudaMalloc(&e->samp_max, e->sample_blocks * 4));
+    CU(cudaMalloc(&e->samp_sum, e->sample_blocks * 4));
+    CU(cudaMalloc(&e->samp_idx, e->sample_blocks * 4));
+    CU(cudaMalloc(&e->samp_counter, 4));
+    CU(cudaMemsetAsync(e->samp_counter, 0, 4, e->stream));
+    e->exact_sampler = !(c.flags & LPP_FLAG_FAST_SAMPLER) && e->sample_blocks <= e->num_sms;
+    if (e->exact_sampler) {
+        CU(cudaMalloc(&e->ex_sync, 2 * sizeof(unsigned int)));
+        CU(cudaMemsetAsync(e->ex_sync, 0, 2 * sizeof(unsigned int), e->stream));
+        CU(cudaMalloc(&e->ex_block_sum, e->sample_blocks * sizeof(double)));
+        CU(cudaMalloc(&e->ex_entry_count, e->sample_blocks * sizeof(int)));
+        CU(cudaMalloc(&e->ex_entries, (size_t)e->sample_blocks * kExactMaxEntries * sizeof(ExactEntry)));
+        CU(cudaMalloc(&e->ex_scalars, 64 * sizeof(float)));
+    }
+    e->run_cap = std::max<int>(4096, c.seq_len);
+    CU(cudaMalloc(&e->r_values, (size_t)e->run_cap * 4));
+    CU(cudaMalloc(&e->out_tokens, (size_t)e->run_cap * 4));
+    CU(cudaMalloc(&e->st, sizeof(StepState)));
+    CU(cudaMemsetAsync(e->st, 0, sizeof(StepState), e->stream));
+    CU(cudaMallocHost(&e->h_st, sizeof(StepState)));
+    memset(e->h_st, 0, sizeof(StepState));
+    {
+        int khz = 0;  // SM clock in kHz = clocks per millisecond
+        CU(cudaDeviceGetAttribute(&khz, cudaDevAttrClockRate, c.device));
+        e->h_st->wait_cycles = c.wait_ms > 0 ? (long long)c.wait_ms * khz : 0;
+        e->h_st->tp_wait_cycles = c.tp_wait_ms > 0 ? (long long)c.tp_wait_ms * khz : 0;
+    }
+    CU(cudaMallocHost(&e->h_out, 16));
+    return LPP_OK;
+}
+
 extern "C" lpp_status lpp_engine_create(const lpp_config* cfg, const void* nccl_id, lpp_engine** out) {
     if (!cfg || !out) return fail(LPP_ERR_INVALID_ARG, "null argument");
     *out = nullptr;
@@ -808,17 +1082,8 @@ extern "C" lpp_status lpp_engine_create(const lpp_config* cfg, const void* nccl_
     if ((c.flags & LPP_FLAG_TP_LOCAL) && c.tp_size > kMaxTp)
         return fail(LPP_ERR_INVALID_ARG, "LPP_FLAG_TP_LOCAL supports at most %d ranks", kMaxTp);
 
-    int ndev = 0;
-    if (cudaGetDeviceCount(&ndev) != cudaSuccess || ndev == 0) {
-        (void)cudaGetLastError();
-        return fail(LPP_ERR_NO_DEVICE, "no CUDA device");
-    }
-    if (c.device < 0 || c.device >= ndev) return fail(LPP_ERR_INVALID_ARG, "device %d out of range", c.device);
-    CU(cudaSetDevice(c.device));
     cudaDeviceProp prop;
-    CU(cudaGetDeviceProperties(&prop, c.device));
-    if (prop.major < 10) return fail(LPP_ERR_NO_DEVICE, "device is sm_%d%d; this library is built for sm_100a only", prop.major, prop.minor);
-
+    TRY(open_device(c.device, &prop));
     TRACE("create: device %d ok (%s, %d SMs)", c.device, prop.name, prop.multiProcessorCount);
     lpp_engine* e = new lpp_engine();
     e->c = c;
@@ -844,6 +1109,8 @@ extern "C" lpp_status lpp_engine_create(const lpp_config* cfg, const void* nccl_
         return fail(LPP_ERR_TOO_LARGE, "vocab_size %d exceeds the sampler's %d", c.vocab_size, kSampleMaxBlocks * kSampleChunk);
     }
     e->got.assign((size_t)LPP_T_COUNT * c.n_layers, 0);
+    e->Dp = c.dim;
+    e->Vp = c.vocab_size;
 
     auto bail = [&](lpp_status s) {
         lpp_engine_destroy(e);
@@ -855,9 +1122,10 @@ extern "C" lpp_status lpp_engine_create(const lpp_config* cfg, const void* nccl_
         if (e_ != cudaSuccess)                                                                                 \
             return bail(fail(LPP_ERR_CUDA, "%s failed: %s (%s:%d)", #call, cudaGetErrorString(e_), __FILE__, __LINE__)); \
     } while (0)
-    CUB(cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking));
-    CUB(cudaEventCreate(&e->ev0));
-    CUB(cudaEventCreate(&e->ev1));
+    {
+        const lpp_status st = alloc_step_buffers(e, (size_t)e->Dq, (size_t)e->Fl);
+        if (st != LPP_OK) return bail(st);
+    }
     const size_t D = c.dim, L = c.n_layers, V = c.vocab_size, S = c.seq_len;
     const size_t esz = e->esz;
     CUB(cudaMalloc(&e->wqkv, L * (e->Dq + 2 * (size_t)e->KVd) * D * esz));
@@ -873,44 +1141,10 @@ extern "C" lpp_status lpp_engine_create(const lpp_config* cfg, const void* nccl_
     CUB(cudaMalloc(&e->vcache, kvbytes));
     CUB(cudaMemsetAsync(e->kcache, 0, kvbytes, e->stream));
     CUB(cudaMemsetAsync(e->vcache, 0, kvbytes, e->stream));
-    CUB(cudaMalloc(&e->xa, D * 4));
-    CUB(cudaMalloc(&e->xb, D * 4));
     CUB(cudaMalloc(&e->q, (size_t)e->Dq * 4));
-    CUB(cudaMalloc(&e->att_out, (size_t)e->Dq * 4));
-    CUB(cudaMalloc(&e->hb, (size_t)e->Fl * 4));
-    CUB(cudaMalloc(&e->logits, V * 4));
     CUB(cudaMalloc(&e->attn_part, (size_t)e->Hl * e->attn_splits * (hs + 2) * 4));
     CUB(cudaMalloc(&e->attn_counters, (size_t)e->KVHl * e->attn_z * 4));
     CUB(cudaMemsetAsync(e->attn_counters, 0, (size_t)e->KVHl * e->attn_z * 4, e->stream));
-    CUB(cudaMalloc(&e->samp_max, e->sample_blocks * 4));
-    CUB(cudaMalloc(&e->samp_sum, e->sample_blocks * 4));
-    CUB(cudaMalloc(&e->samp_idx, e->sample_blocks * 4));
-    CUB(cudaMalloc(&e->samp_counter, 4));
-    CUB(cudaMemsetAsync(e->samp_counter, 0, 4, e->stream));
-    e->exact_sampler = !(c.flags & LPP_FLAG_FAST_SAMPLER) && e->sample_blocks <= e->num_sms;
-    if (e->exact_sampler) {
-        CUB(cudaMalloc(&e->ex_sync, 2 * sizeof(unsigned int)));
-        CUB(cudaMemsetAsync(e->ex_sync, 0, 2 * sizeof(unsigned int), e->stream));
-        CUB(cudaMalloc(&e->ex_block_sum, e->sample_blocks * sizeof(double)));
-        CUB(cudaMalloc(&e->ex_entry_count, e->sample_blocks * sizeof(int)));
-        CUB(cudaMalloc(&e->ex_entries, (size_t)e->sample_blocks * kExactMaxEntries * sizeof(ExactEntry)));
-        CUB(cudaMalloc(&e->ex_scalars, 64 * sizeof(float)));
-    }
-    e->run_cap = std::max<int>(4096, c.seq_len);
-    CUB(cudaMalloc(&e->r_values, (size_t)e->run_cap * 4));
-    CUB(cudaMalloc(&e->out_tokens, (size_t)e->run_cap * 4));
-    CUB(cudaMalloc(&e->st, sizeof(StepState)));
-    CUB(cudaMemsetAsync(e->st, 0, sizeof(StepState), e->stream));
-    CUB(cudaMallocHost(&e->h_st, sizeof(StepState)));
-    memset(e->h_st, 0, sizeof(StepState));
-    {
-        int khz = 0;  // SM clock in kHz = clocks per millisecond
-        CUB(cudaDeviceGetAttribute(&khz, cudaDevAttrClockRate, c.device));
-        e->h_st->wait_cycles = c.wait_ms > 0 ? (long long)c.wait_ms * khz : 0;
-        e->h_st->tp_wait_cycles = c.tp_wait_ms > 0 ? (long long)c.tp_wait_ms * khz : 0;
-    }
-    CUB(cudaMallocHost(&e->h_out, 16));
-
     TRACE("create: buffers allocated");
     // rope table with libm, evaluated exactly like the reference loop (src/ops.cpp:36-40)
     {
@@ -953,6 +1187,178 @@ extern "C" lpp_status lpp_engine_create(const lpp_config* cfg, const void* nccl_
     return LPP_OK;
 }
 
+// ------------------------------------------------------------------ engines described layer by layer
+
+// cos / sin of every position and rotated pair.  Frequencies and angles in double, so a far position's angle is as exact as
+// a near one's; pairs beyond rot_dims do not turn.  Layers with the same rotation share a table.
+static lpp_status rope_table(lpp_engine* e, const lpp_layer_desc& d, const float2** out) {
+    *out = nullptr;
+    if (d.rot_dim == 0) return LPP_OK;
+    for (auto& t : e->rope_tables) {
+        const lpp_layer_desc& o = t.first;
+        if (o.rot_dim == d.rot_dim && o.rot_dims == d.rot_dims && o.rot_base == d.rot_base && o.yarn_factor == d.yarn_factor &&
+            o.yarn_original == d.yarn_original && o.yarn_fast == d.yarn_fast && o.yarn_slow == d.yarn_slow) {
+            *out = t.second;
+            return LPP_OK;
+        }
+    }
+    const int half = d.rot_dim / 2, S = e->c.seq_len;
+    std::vector<double> f(half, 0.0);
+    double mag = 1.0;
+    for (int i = 0; i < d.rot_dims / 2; ++i) f[i] = pow(d.rot_base, -2.0 * i / d.rot_dims);
+    if (d.yarn_factor != 0.0) {
+        // the pair whose wave makes `turns` turns over the original context, as a (fractional) dimension index
+        auto border = [&](double turns) {
+            return d.rot_dims * log(d.yarn_original / (2.0 * M_PI * turns)) / (2.0 * log(d.rot_base));
+        };
+        const double lo = std::max(floor(border(d.yarn_fast)), 0.0), hi = std::min(ceil(border(d.yarn_slow)), (double)d.rot_dims - 1.0);
+        for (int i = 0; i < d.rot_dims / 2; ++i) {
+            const double ramp = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0);
+            f[i] = f[i] / d.yarn_factor * ramp + f[i] * (1.0 - ramp);
+        }
+        mag = 0.1 * log(d.yarn_factor) + 1.0;
+    }
+    std::vector<float2> tab((size_t)S * half, make_float2(1.f, 0.f));
+    for (size_t p = 0; p < (size_t)S; ++p)
+        for (int i = 0; i < d.rot_dims / 2; ++i)
+            tab[p * half + i] = make_float2((float)(mag * cos((double)p * f[i])), (float)(mag * sin((double)p * f[i])));
+    float2* dev = nullptr;
+    CU(cudaMalloc(&dev, tab.size() * sizeof(float2)));
+    e->rope_tables.push_back({d, dev});
+    CU(cudaMemcpy(dev, tab.data(), tab.size() * sizeof(float2), cudaMemcpyHostToDevice));
+    *out = dev;
+    return LPP_OK;
+}
+
+static lpp_status zeroed(lpp_engine* e, void** p, size_t bytes) {
+    bytes = std::max<size_t>(bytes, 16);
+    CU(cudaMalloc(p, bytes));
+    CU(cudaMemsetAsync(*p, 0, bytes, e->stream));
+    return LPP_OK;
+}
+template <typename T>
+static lpp_status zeroed(lpp_engine* e, T** p, size_t bytes) {
+    return zeroed(e, reinterpret_cast<void**>(p), bytes);
+}
+
+static lpp_status setup_latent_layer(lpp_engine* e, LatentLayer& y) {
+    const lpp_layer_desc& d = y.d;
+    const size_t D2 = align_up(e->c.dim, 2), Dp = e->Dp, esz = e->esz;
+    TRY(zeroed(e, &y.w_in, (size_t)y.in_rows * Dp * esz));
+    TRY(zeroed(e, &y.w_uk, (size_t)d.heads * y.rank_pitch * y.dim_pitch * esz));
+    TRY(zeroed(e, &y.w_uv, (size_t)d.heads * y.vdim_rows * y.val_pitch * esz));
+    TRY(zeroed(e, &y.wo, D2 * y.o_pitch * esz));
+    TRY(zeroed(e, &y.n1w, Dp * 4));
+    TRY(zeroed(e, &y.lat_w, (size_t)y.rank_pitch * 4));
+    if (e->layer_norm) TRY(zeroed(e, &y.n1b, Dp * 4));
+    if (d.ff > 0) {
+        TRY(zeroed(e, &y.w13, (size_t)2 * d.ff * Dp * esz));
+        TRY(zeroed(e, &y.w2, D2 * y.ff_pitch * esz));
+        TRY(zeroed(e, &y.n2w, Dp * 4));
+        if (e->layer_norm) TRY(zeroed(e, &y.n2b, Dp * 4));
+    }
+    TRY(zeroed(e, &y.cache, (size_t)e->c.seq_len * y.row_width * e->kvesz));
+    return rope_table(e, d, &y.rope);
+}
+
+extern "C" lpp_status lpp_engine_create_layers(const lpp_model_desc* m, const lpp_layer_desc* layers, lpp_engine** out) {
+    if (!m || !layers || !out) return fail(LPP_ERR_INVALID_ARG, "null argument");
+    *out = nullptr;
+    if (m->dim <= 0 || m->vocab_size <= 0 || m->seq_len <= 0 || m->n_layers <= 0)
+        return fail(LPP_ERR_INVALID_ARG, "non-positive model dimension");
+    if (!((m->weight_dtype == LPP_BF16 && m->kv_dtype == LPP_F16) || (m->weight_dtype == LPP_F32 && m->kv_dtype == LPP_F32)))
+        return fail(LPP_ERR_INVALID_ARG, "weights / cache must be BF16 / F16 or F32 / F32");
+    if (m->norm != LPP_NORM_RMS && m->norm != LPP_NORM_LAYER) return fail(LPP_ERR_INVALID_ARG, "unknown norm %d", m->norm);
+    for (int l = 0; l < m->n_layers; ++l) {
+        const lpp_layer_desc& d = layers[l];
+        if (d.mixer != LPP_MIXER_LATENT) return fail(LPP_ERR_INVALID_ARG, "layer %d: unknown mixer %d", l, d.mixer);
+        if (d.heads <= 0 || d.dim <= 0 || d.rot_dim < 0 || d.vdim <= 0 || d.kv_rank <= 0 || d.window < 0 || d.ff < 0)
+            return fail(LPP_ERR_INVALID_ARG, "layer %d: bad size", l);
+        if (d.rot_dim % 2 || d.rot_dims % 2 || d.rot_dims < 0 || d.rot_dims > d.rot_dim)
+            return fail(LPP_ERR_INVALID_ARG, "layer %d: rotation of %d of %d dimensions", l, d.rot_dims, d.rot_dim);
+        if (d.rot_dims > 0 && !(d.rot_base > 0.0)) return fail(LPP_ERR_INVALID_ARG, "layer %d: bad rotation base", l);
+        if (d.yarn_factor != 0.0 && !(d.yarn_factor > 0.0 && d.yarn_original > 0.0 && d.yarn_fast > 0.0 && d.yarn_slow > 0.0))
+            return fail(LPP_ERR_INVALID_ARG, "layer %d: bad rotation scaling", l);
+        if (d.act != LPP_ACT_SILU && d.act != LPP_ACT_GELU_TANH) return fail(LPP_ERR_INVALID_ARG, "layer %d: unknown activation %d", l, d.act);
+        if (d.kv_rank > kLatentMaxPerThread * kLatentThreads) return fail(LPP_ERR_TOO_LARGE, "layer %d: kv_rank %d", l, d.kv_rank);
+    }
+    cudaDeviceProp prop;
+    TRY(open_device(m->device, &prop));
+    lpp_engine* e = new lpp_engine();
+    lpp_config& c = e->c;
+    c = {};
+    c.dim = m->dim;
+    c.n_layers = m->n_layers;
+    c.vocab_size = m->vocab_size;
+    c.seq_len = m->seq_len;
+    c.weight_dtype = m->weight_dtype;
+    c.kv_dtype = m->kv_dtype;
+    c.tp_size = 1;
+    c.device = m->device;
+    c.flags = m->flags;
+    c.ring_kb = m->ring_kb;
+    c.wait_ms = m->wait_ms;
+    e->esz = c.weight_dtype == LPP_BF16 ? 2 : 4;
+    e->kvesz = c.kv_dtype == LPP_F16 ? 2 : 4;
+    e->num_sms = prop.multiProcessorCount;
+    e->smem_optin = prop.sharedMemPerBlockOptin;
+    e->Dp = (int)align_up(c.dim, 64);
+    e->Vp = (int)align_up(c.vocab_size, 2);
+    e->layer_norm = m->norm == LPP_NORM_LAYER;
+    e->norm_eps = m->norm_eps;
+    e->sample_blocks = (c.vocab_size + kSampleChunk - 1) / kSampleChunk;
+    e->got.assign((size_t)LPP_T_COUNT * c.n_layers, 0);
+    auto bail = [&](lpp_status s) {
+        lpp_engine_destroy(e);
+        return s;
+    };
+    if (e->sample_blocks > kSampleMaxBlocks)
+        return bail(fail(LPP_ERR_TOO_LARGE, "vocab_size %d exceeds the sampler's %d", c.vocab_size, kSampleMaxBlocks * kSampleChunk));
+    e->lat.resize(c.n_layers);
+    size_t att_n = 64, hb_n = 64, qplain_n = 0, raw_n = 0, gate_n = 0, query_n = 0, part_n = 0;
+    for (int l = 0; l < c.n_layers; ++l) {
+        LatentLayer& y = e->lat[l];
+        const lpp_layer_desc& d = y.d = layers[l];
+        y.rank_pitch = (int)align_up(d.kv_rank, 16);
+        y.row_width = y.rank_pitch + (int)align_up(d.rot_dim, 16);
+        y.dim_pitch = (int)align_up(d.dim, 64);
+        y.val_pitch = (int)align_up(d.kv_rank, 64);
+        y.vdim_rows = (int)align_up(d.vdim, 2);
+        y.o_pitch = (int)align_up((size_t)d.heads * d.vdim, 64);
+        y.ff_pitch = (int)align_up(d.ff, 64);
+        y.q_plain_rows = (int)align_up((size_t)d.heads * d.dim, 2);
+        y.q_rot_rows = d.heads * d.rot_dim;
+        y.latent_rows = (int)align_up(d.kv_rank, 2);
+        y.in_rows = y.q_plain_rows + y.q_rot_rows + y.latent_rows + d.rot_dim + (int)align_up(d.heads, 2);
+        att_n = std::max(att_n, (size_t)y.o_pitch);
+        hb_n = std::max(hb_n, (size_t)y.ff_pitch);
+        qplain_n = std::max(qplain_n, (size_t)d.heads * y.dim_pitch);
+        raw_n = std::max(raw_n, (size_t)y.latent_rows);
+        gate_n = std::max(gate_n, align_up(d.heads, 2));
+        query_n = std::max(query_n, (size_t)d.heads * y.row_width);
+        part_n = std::max(part_n, (size_t)d.heads * kLatentMaxSplits * (y.rank_pitch + kLatentPartTail));
+    }
+    auto setup = [&]() -> lpp_status {
+        TRY(alloc_step_buffers(e, att_n, hb_n));
+        const size_t Dp = e->Dp;
+        TRY(zeroed(e, &e->emb, (size_t)e->Vp * Dp * e->esz));
+        TRY(zeroed(e, &e->rms_final, Dp * 4));
+        if (e->layer_norm) TRY(zeroed(e, &e->final_b, Dp * 4));
+        TRY(zeroed(e, &e->lat_qplain, qplain_n * 4));
+        TRY(zeroed(e, &e->lat_raw, raw_n * 4));
+        TRY(zeroed(e, &e->lat_gate, gate_n * 4));
+        TRY(zeroed(e, &e->lat_query, query_n * e->kvesz));
+        TRY(zeroed(e, &e->lat_part, part_n * 4));
+        for (LatentLayer& y : e->lat) TRY(setup_latent_layer(e, y));
+        CU(cudaStreamSynchronize(e->stream));
+        return LPP_OK;
+    };
+    const lpp_status st = setup();
+    if (st != LPP_OK) return bail(st);
+    *out = e;
+    return LPP_OK;
+}
+
 extern "C" lpp_status lpp_engine_destroy(lpp_engine* e) {
     if (!e) return LPP_OK;
     cudaSetDevice(e->c.device);
@@ -970,9 +1376,15 @@ extern "C" lpp_status lpp_engine_destroy(lpp_engine* e) {
                     e->rms_final, e->kcache, e->vcache, e->xa, e->xb, e->q, e->att_out, e->hb, e->logits,
                     e->attn_part, e->attn_counters, e->samp_max, e->samp_sum, e->samp_idx, e->samp_counter,
                     e->r_values, e->out_tokens, e->st, e->rope, e->stage, e->gtrace, e->pf_x, e->pf_q, e->pf_part, e->pf_xn, e->pf_att, e->pf_hb,
-                    e->pf_tokens, e->ex_sync, e->ex_block_sum, e->ex_entry_count, e->ex_entries, e->ex_scalars};
+                    e->pf_tokens, e->ex_sync, e->ex_block_sum, e->ex_entry_count, e->ex_entries, e->ex_scalars, e->final_b, e->lat_qplain,
+                    e->lat_raw, e->lat_gate, e->lat_query, e->lat_part, e->pf_rows, e->pf_logits, e->pf_qn, e->pf_olat, e->pf_lq,
+                    e->pf_lpart, e->pf_gate};
     for (void* p : bufs)
         if (p) cudaFree(p);
+    for (const LatentLayer& y : e->lat)
+        for (void* p : {y.w_in, y.w_uk, y.w_uv, y.wo, y.w13, y.w2, (void*)y.n1w, (void*)y.n1b, (void*)y.n2w, (void*)y.n2b, (void*)y.lat_w, y.cache})
+            if (p) cudaFree(p);
+    for (auto& t : e->rope_tables) cudaFree(t.second);
     if (e->h_st) cudaFreeHost(e->h_st);
     if (e->h_out) cudaFreeHost(e->h_out);
     if (e->ev0) cudaEventDestroy(e->ev0);
@@ -1004,47 +1416,169 @@ static lpp_status ensure_stage(lpp_engine* e, size_t bytes) {
     return LPP_OK;
 }
 
-// dst[r*dst_pitch + c] (dst_dtype) = src[(r0 + r)*src_pitch + c0 + c] (src_dtype), r < rows, c < cols
-static lpp_status put_block(lpp_engine* e, void* dst, size_t dst_pitch, int dst_dtype, const void* src,
-                            size_t src_pitch, size_t r0, size_t c0, int rows, int cols, int src_dtype, int memkind) {
-    const size_t sesz = src_dtype == LPP_F16 ? 2 : 4;
-    const char* s = (const char*)src + (r0 * src_pitch + c0) * sesz;
-    size_t spitch = src_pitch;
-    if (memkind == LPP_MEM_HOST) {
-        TRY(ensure_stage(e, (size_t)rows * cols * sesz));
-        CU(cudaMemcpy2DAsync(e->stage, (size_t)cols * sesz, s, src_pitch * sesz, (size_t)cols * sesz, rows,
-                             cudaMemcpyHostToDevice, e->stream));
-        s = (const char*)e->stage;
-        spitch = cols;
-    }
-    const long long total = (long long)rows * cols;
+// Element (r, c) of a block of rows x cols: source row r sits at src + ((r / group) * group_stride + r % group) * src_pitch
+// (group 0 = consecutive rows), destination dst + r * dst_row + c * dst_col; strides in elements.
+struct BlockShape {
+    int rows, cols;
+    size_t src_pitch;
+    int group = 0;
+    size_t group_stride = 0;
+    size_t dst_row = 0, dst_col = 1;
+};
+template <typename DT>
+static void launch_repack(DT* dst, const void* src, int src_dtype, const BlockShape& b, cudaStream_t s) {
+    const long long total = (long long)b.rows * b.cols;
     const int grid = (int)std::min<long long>((total + 255) / 256, 148 * 16);
-    if (dst_dtype == LPP_F16 && src_dtype == LPP_F16)
-        repack_kernel<__half, __half><<<grid, 256, 0, e->stream>>>((__half*)dst, dst_pitch, (const __half*)s, spitch, rows, cols);
-    else if (dst_dtype == LPP_F16 && src_dtype == LPP_F32)
-        repack_kernel<__half, float><<<grid, 256, 0, e->stream>>>((__half*)dst, dst_pitch, (const float*)s, spitch, rows, cols);
-    else if (dst_dtype == LPP_F32 && src_dtype == LPP_F16)
-        repack_kernel<float, __half><<<grid, 256, 0, e->stream>>>((float*)dst, dst_pitch, (const __half*)s, spitch, rows, cols);
+    const int group = b.group > 0 ? b.group : std::max(1, b.rows);
+    const long long gs = b.group > 0 ? (long long)b.group_stride : b.rows;
+    if (src_dtype == LPP_F16)
+        repack_kernel<DT, __half><<<grid, 256, 0, s>>>(dst, b.dst_row, b.dst_col, (const __half*)src, b.src_pitch, group, gs, b.rows, b.cols);
+    else if (src_dtype == LPP_BF16)
+        repack_kernel<DT, __nv_bfloat16><<<grid, 256, 0, s>>>(dst, b.dst_row, b.dst_col, (const __nv_bfloat16*)src, b.src_pitch, group, gs, b.rows, b.cols);
     else
-        repack_kernel<float, float><<<grid, 256, 0, e->stream>>>((float*)dst, dst_pitch, (const float*)s, spitch, rows, cols);
+        repack_kernel<DT, float><<<grid, 256, 0, s>>>(dst, b.dst_row, b.dst_col, (const float*)src, b.src_pitch, group, gs, b.rows, b.cols);
+}
+static size_t dtype_size(int t) { return t == LPP_F32 ? 4 : 2; }
+static lpp_status put_shape(lpp_engine* e, void* dst, int dst_dtype, const void* src, int src_dtype, int memkind, BlockShape b) {
+    const char* p = (const char*)src;
+    const size_t sesz = dtype_size(src_dtype);
+    if (memkind == LPP_MEM_HOST) {
+        // the rows from the first to the last one, compacted to `cols` columns
+        const size_t span = b.group > 0 ? (size_t)((b.rows - 1) / b.group) * b.group_stride + (b.rows - 1) % b.group + 1 : b.rows;
+        TRY(ensure_stage(e, span * b.cols * sesz));
+        CU(cudaMemcpy2DAsync(e->stage, (size_t)b.cols * sesz, p, b.src_pitch * sesz, (size_t)b.cols * sesz, span, cudaMemcpyHostToDevice, e->stream));
+        p = (const char*)e->stage;
+        b.src_pitch = b.cols;
+    }
+    if (dst_dtype == LPP_F16)
+        launch_repack((__half*)dst, p, src_dtype, b, e->stream);
+    else if (dst_dtype == LPP_BF16)
+        launch_repack((__nv_bfloat16*)dst, p, src_dtype, b, e->stream);
+    else
+        launch_repack((float*)dst, p, src_dtype, b, e->stream);
     CU(cudaGetLastError());
     // the staging buffer is reused by the next call and host memory may be freed by the caller
     CU(cudaStreamSynchronize(e->stream));
     return LPP_OK;
 }
 
+// dst[r*dst_pitch + c] (dst_dtype) = src[(r0 + r)*src_pitch + c0 + c] (src_dtype), r < rows, c < cols
+static lpp_status put_block(lpp_engine* e, void* dst, size_t dst_pitch, int dst_dtype, const void* src,
+                            size_t src_pitch, size_t r0, size_t c0, int rows, int cols, int src_dtype, int memkind) {
+    BlockShape b;
+    b.rows = rows;
+    b.cols = cols;
+    b.src_pitch = src_pitch;
+    b.dst_row = dst_pitch;
+    return put_shape(e, dst, dst_dtype, (const char*)src + (r0 * src_pitch + c0) * dtype_size(src_dtype), src_dtype, memkind, b);
+}
+
+// A tensor of an engine described layer by layer, into the padded layouts of LatentLayer.
+static lpp_status upload_latent(lpp_engine* e, int which, int l, const void* src, int dt, int memkind) {
+    const lpp_config& c = e->c;
+    LatentLayer& y = e->lat[l];
+    const lpp_layer_desc& d = y.d;
+    const int D = c.dim, wd = c.weight_dtype;
+    const size_t Dp = e->Dp, esz = e->esz;
+    auto vec = [&](float* dst, int n) { return put_block(e, dst, n, LPP_F32, src, n, 0, 0, 1, n, dt, memkind); };
+    auto mat = [&](void* dst, size_t pitch, int rows, int cols) { return put_block(e, dst, pitch, wd, src, cols, 0, 0, rows, cols, dt, memkind); };
+    auto in_row = [&](size_t r) { return (char*)y.w_in + r * Dp * esz; };
+    const bool norm_bias = which == LPP_T_NORM1_B || which == LPP_T_NORM2_B || which == LPP_T_NORM_FINAL_B;
+    if (norm_bias && !e->layer_norm) return fail(LPP_ERR_INVALID_ARG, "this model's norms have no bias");
+    const bool ff = which == LPP_T_RMS_FFN || which == LPP_T_NORM2_B || which == LPP_T_W1 || which == LPP_T_W2 || which == LPP_T_W3;
+    if (ff && d.ff == 0) return fail(LPP_ERR_INVALID_ARG, "layer %d has no feed-forward", l);
+    switch (which) {
+        case LPP_T_TOK_EMB: return mat(e->emb, Dp, c.vocab_size, D);
+        case LPP_T_W_CLS:
+            if (!e->wcls_owned) {
+                TRY(zeroed(e, &e->wcls, (size_t)e->Vp * Dp * esz));
+                e->wcls_owned = true;
+            }
+            return mat(e->wcls, Dp, c.vocab_size, D);
+        case LPP_T_RMS_FINAL: return vec(e->rms_final, D);
+        case LPP_T_NORM_FINAL_B: return vec(e->final_b, D);
+        case LPP_T_RMS_ATT: return vec(y.n1w, D);
+        case LPP_T_NORM1_B: return vec(y.n1b, D);
+        case LPP_T_RMS_FFN: return vec(y.n2w, D);
+        case LPP_T_NORM2_B: return vec(y.n2b, D);
+        case LPP_T_LAT_NORM: return vec(y.lat_w, d.kv_rank);
+        case LPP_T_LAT_Q: {  // per head dim plain rows, then rot rows: two sections of the input matrix
+            BlockShape b;
+            b.cols = D;
+            b.src_pitch = D;
+            b.group_stride = d.dim + d.rot_dim;
+            b.dst_row = Dp;
+            b.rows = d.heads * d.dim;
+            b.group = d.dim;
+            TRY(put_shape(e, in_row(0), wd, src, dt, memkind, b));
+            if (d.rot_dim == 0) return LPP_OK;
+            b.rows = d.heads * d.rot_dim;
+            b.group = d.rot_dim;
+            return put_shape(e, in_row(y.q_plain_rows), wd, (const char*)src + (size_t)d.dim * D * dtype_size(dt), dt, memkind, b);
+        }
+        case LPP_T_LAT_DKV: {  // the latent's section may end in a padding row
+            const size_t r0 = (size_t)y.q_plain_rows + y.q_rot_rows;
+            TRY(put_block(e, in_row(r0), Dp, wd, src, D, 0, 0, d.kv_rank, D, dt, memkind));
+            if (d.rot_dim == 0) return LPP_OK;
+            return put_block(e, in_row(r0 + y.latent_rows), Dp, wd, src, D, d.kv_rank, 0, d.rot_dim, D, dt, memkind);
+        }
+        case LPP_T_LAT_G: return mat(in_row((size_t)y.q_plain_rows + y.q_rot_rows + y.latent_rows + d.rot_dim), Dp, d.heads, D);
+        case LPP_T_LAT_UK:  // [heads][dim][rank] -> [heads][rank_pitch][dim_pitch]: the step multiplies by the transpose
+            for (int h = 0; h < d.heads; ++h) {
+                BlockShape b;
+                b.rows = d.dim;
+                b.cols = d.kv_rank;
+                b.src_pitch = d.kv_rank;
+                b.dst_row = 1;
+                b.dst_col = y.dim_pitch;
+                TRY(put_shape(e, (char*)y.w_uk + (size_t)h * y.rank_pitch * y.dim_pitch * esz, wd,
+                              (const char*)src + (size_t)h * d.dim * d.kv_rank * dtype_size(dt), dt, memkind, b));
+            }
+            return LPP_OK;
+        case LPP_T_LAT_UV:
+            for (int h = 0; h < d.heads; ++h)
+                TRY(put_block(e, (char*)y.w_uv + (size_t)h * y.vdim_rows * y.val_pitch * esz, y.val_pitch, wd, src, d.kv_rank,
+                              (size_t)h * d.vdim, 0, d.vdim, d.kv_rank, dt, memkind));
+            return LPP_OK;
+        case LPP_T_WO: return mat(y.wo, y.o_pitch, D, d.heads * d.vdim);
+        case LPP_T_W1: return put_block(e, y.w13, 2 * Dp, wd, src, D, 0, 0, d.ff, D, dt, memkind);                      // gate -> even rows
+        case LPP_T_W3: return put_block(e, (char*)y.w13 + Dp * esz, 2 * Dp, wd, src, D, 0, 0, d.ff, D, dt, memkind);  // up -> odd rows
+        case LPP_T_W2: return mat(y.w2, y.ff_pitch, D, d.ff);
+    }
+    return fail(LPP_ERR_INVALID_ARG, "tensor id %d does not belong to this model", which);
+}
+// Whether layer l of the model has tensor t.
+static bool tensor_expected(const lpp_engine* e, int t, int l) {
+    if (t == LPP_T_W_CLS) return false;  // optional
+    if (e->lat.empty()) return t < LPP_T_NORM1_B;
+    switch (t) {
+        case LPP_T_WQ: case LPP_T_WK: case LPP_T_WV: return false;
+        case LPP_T_NORM1_B: case LPP_T_NORM_FINAL_B: return e->layer_norm;
+        case LPP_T_NORM2_B: return e->layer_norm && e->lat[l].d.ff > 0;
+        case LPP_T_RMS_FFN: case LPP_T_W1: case LPP_T_W2: case LPP_T_W3: return e->lat[l].d.ff > 0;
+    }
+    return true;
+}
+static bool tensor_stacked(int t) { return !(t == LPP_T_TOK_EMB || t == LPP_T_RMS_FINAL || t == LPP_T_W_CLS || t == LPP_T_NORM_FINAL_B); }
+
 extern "C" lpp_status lpp_upload_tensor(lpp_engine* e, int which, int layer, const void* src, int src_dtype,
                                         int memkind) {
     if (!e || !src) return fail(LPP_ERR_INVALID_ARG, "null argument");
     if (which < 0 || which >= LPP_T_COUNT) return fail(LPP_ERR_INVALID_ARG, "unknown tensor id %d", which);
-    if (src_dtype != LPP_F16 && src_dtype != LPP_F32) return fail(LPP_ERR_INVALID_ARG, "bad src_dtype");
+    if (src_dtype != LPP_F16 && src_dtype != LPP_F32 && src_dtype != LPP_BF16) return fail(LPP_ERR_INVALID_ARG, "bad src_dtype");
     if (memkind != LPP_MEM_HOST && memkind != LPP_MEM_DEVICE) return fail(LPP_ERR_INVALID_ARG, "bad memkind");
     const lpp_config& c = e->c;
-    const bool stacked = !(which == LPP_T_TOK_EMB || which == LPP_T_RMS_FINAL || which == LPP_T_W_CLS);
+    const bool stacked = tensor_stacked(which);
     if (stacked && (layer < 0 || layer >= c.n_layers)) return fail(LPP_ERR_INVALID_ARG, "layer %d out of range", layer);
     if (!stacked) layer = 0;
     CU(cudaSetDevice(c.device));
     TRACE("upload tensor %d layer %d", which, layer);
+    if (!e->lat.empty()) {
+        TRY(upload_latent(e, which, layer, src, src_dtype, memkind));
+        e->got[(size_t)which * c.n_layers + layer] = 1;
+        e->finalized = false;
+        return LPP_OK;
+    }
     const size_t D = c.dim, F = c.hidden_dim, V = c.vocab_size, esz = e->esz;
     const size_t l = layer, r = c.tp_rank;
     const size_t qkv_rows = e->Dq + 2 * (size_t)e->KVd;
@@ -1053,6 +1587,7 @@ extern "C" lpp_status lpp_upload_tensor(lpp_engine* e, int which, int layer, con
     char* w13_l = (char*)e->w13 + l * 2 * e->Fl * D * esz;
     lpp_status s = LPP_OK;
     switch (which) {
+        default: return fail(LPP_ERR_INVALID_ARG, "tensor id %d does not belong to this model", which);
         case LPP_T_TOK_EMB:
             s = put_block(e, e->emb, D, wd, src, D, 0, 0, (int)V, (int)D, src_dtype, memkind);
             break;
@@ -1110,13 +1645,12 @@ extern "C" lpp_status lpp_finalize(lpp_engine* e) {
     if (!e) return fail(LPP_ERR_INVALID_ARG, "null argument");
     const lpp_config& c = e->c;
     CU(cudaSetDevice(c.device));
-    static const char* names[LPP_T_COUNT] = {"tok_emb", "rms_att", "wq", "wk", "wv", "wo", "rms_ffn", "w1", "w2", "w3", "rms_final", "w_cls"};
+    static const char* names[LPP_T_COUNT] = {"tok_emb", "rms_att", "wq", "wk", "wv", "wo", "rms_ffn", "w1", "w2", "w3", "rms_final", "w_cls",
+                                              "norm1_b", "norm2_b", "norm_final_b", "lat_q", "lat_dkv", "lat_norm", "lat_uk", "lat_uv", "lat_g"};
     for (int t = 0; t < LPP_T_COUNT; ++t) {
-        if (t == LPP_T_W_CLS) continue;
-        const bool stacked = !(t == LPP_T_TOK_EMB || t == LPP_T_RMS_FINAL);
-        const int n = stacked ? c.n_layers : 1;
+        const int n = tensor_stacked(t) ? c.n_layers : 1;
         for (int l = 0; l < n; ++l)
-            if (!e->got[(size_t)t * c.n_layers + l])
+            if (tensor_expected(e, t, l) && !e->got[(size_t)t * c.n_layers + l])
                 return fail(LPP_ERR_NOT_READY, "tensor %s (layer %d) was never uploaded", names[t], l);
     }
     if (c.tp_size > 1 && !e->comm && !tp_peer_path(e))
@@ -1145,7 +1679,8 @@ extern "C" lpp_status lpp_finalize(lpp_engine* e) {
         }
         TRACE("finalize: graphs captured (%d kernels per long-context step)", e->kernels_full);
     } else {
-        e->kernels_full = 5 * c.n_layers + 2 + (tp_cls_sharded(e) ? 1 : 0);
+        e->kernels_full = 2 + (tp_cls_sharded(e) ? 1 : 0);
+        for (int l = 0; l < c.n_layers; ++l) e->kernels_full += (e->lat.empty() ? 2 : 4) + 1 + (layer_view(e, l).ff > 0 ? 2 : 0);
     }
     e->finalized = true;
     return LPP_OK;
@@ -1298,170 +1833,338 @@ static lpp_status make_activation_map(CUtensorMap* m, const void* base, size_t t
     return LPP_OK;
 }
 
-// The tensor-core path takes FP16 weights, an FP16 cache and a single GPU; everything else is fed token by token.
+// The tensor-core path takes 16-bit weights, an FP16 cache and a single GPU; everything else is fed token by token.
 static bool prefill_batched(const lpp_engine* e) {
+    if (e->c.flags & LPP_FLAG_NO_PREFILL_GEMM) return false;
+    if (!e->lat.empty()) return e->c.weight_dtype == LPP_BF16 && e->c.kv_dtype == LPP_F16;
     return e->c.tp_size == 1 && e->c.weight_dtype == LPP_F16 && e->c.kv_dtype == LPP_F16 && e->hs <= 128 && e->gqa <= 8 &&
-           e->c.dim % 64 == 0 && e->Dq % 64 == 0 && e->Fl % 64 == 0 && !(e->c.flags & LPP_FLAG_NO_PREFILL_GEMM);
+           e->c.dim % 64 == 0 && e->Dq % 64 == 0 && e->Fl % 64 == 0;
+}
+
+template <typename T>
+static lpp_status allow_gemm_smem() {
+    CU(cudaFuncSetAttribute(prefill_gemm_umma_kernel<T, kPfResid>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes));
+    CU(cudaFuncSetAttribute(prefill_gemm_umma_kernel<T, kPfSwiglu>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes));
+    CU(cudaFuncSetAttribute(prefill_gemm_umma_kernel<T, kPfStore>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes));
+    return LPP_OK;
+}
+
+// Key splits of a prompt block's attention: enough CTAs for about one wave.
+static int latent_prefill_splits(const lpp_engine* e, const LatentLayer& y, int tokens) {
+    const int rows = tokens * y.d.heads;
+    const int tiles = latent_mma_supported(e, y) ? (rows + latent_tile_rows(rows) - 1) / latent_tile_rows(rows) : rows;
+    const int keys = std::min(e->c.seq_len, y.d.window > 0 ? y.d.window + latent_tile_rows(rows) / y.d.heads + 1 : e->c.seq_len);
+    return std::max(1, std::min({kLatentMaxSplits, (keys + kLatMinChunk - 1) / kLatMinChunk, e->num_sms / tiles}));
 }
 
 static lpp_status prefill_setup(lpp_engine* e) {
     if (e->pf_ready) return LPP_OK;
     const lpp_config& c = e->c;
-    const size_t D = c.dim, L = c.n_layers, T = kPrefillTokens;
-    const size_t qkv_rows = e->Dq + 2 * (size_t)e->KVd;
-    CU(cudaMalloc(&e->pf_x, T * D * 4));
-    CU(cudaMalloc(&e->pf_q, T * e->Dq * 4));
-    CU(cudaMalloc(&e->pf_xn, 2 * T * D * 2));  // hi plane, lo plane
-    CU(cudaMalloc(&e->pf_att, 2 * T * e->Dq * 2));  // hi plane, lo plane
-    CU(cudaMalloc(&e->pf_hb, 2 * T * e->Fl * 2));  // hi plane, lo plane
-    CU(cudaMalloc(&e->pf_part, (size_t)kPfMaxSplits * T * std::max<size_t>(D, qkv_rows) * 4));
-    CU(cudaMalloc(&e->pf_tokens, T * sizeof(int)));
-    CU(cudaMemsetAsync(e->pf_x, 0, T * D * 4, e->stream));
-    CU(cudaMemsetAsync(e->pf_xn, 0, 2 * T * D * 2, e->stream));
-    CU(cudaMemsetAsync(e->pf_att, 0, 2 * T * e->Dq * 2, e->stream));
-    CU(cudaMemsetAsync(e->pf_hb, 0, 2 * T * e->Fl * 2, e->stream));
-    CU(cudaMemsetAsync(e->pf_tokens, 0, T * sizeof(int), e->stream));
-    TRY(make_weight_map(&e->pf_map_wqkv, e->wqkv, L * qkv_rows, D, kUmmaM));
-    TRY(make_weight_map(&e->pf_map_wo, e->wo, L * D, e->Dq, kUmmaM));
-    TRY(make_weight_map(&e->pf_map_w13, e->w13, L * 2 * e->Fl, D, kUmmaM));
-    TRY(make_weight_map(&e->pf_map_w2, e->w2, L * D, e->Fl, kUmmaM));
+    const size_t D = e->Dp, L = c.n_layers, T = kPrefillTokens;
+    const bool latent = !e->lat.empty();
+    size_t part_rows = D, att_n = e->Dq, hb_n = e->Fl, qn_n = 0, olat_n = 0, lq_n = 0, lpart_n = 0, gate_n = 0;
+    const size_t qkv_rows = latent ? 0 : e->Dq + 2 * (size_t)e->KVd;
+    part_rows = std::max(part_rows, qkv_rows);
+    for (const LatentLayer& y : e->lat) {
+        const size_t H = y.d.heads;
+        part_rows = std::max(part_rows, (size_t)y.in_rows);
+        att_n = std::max(att_n, (size_t)y.o_pitch);
+        hb_n = std::max(hb_n, (size_t)y.ff_pitch);
+        qn_n = std::max(qn_n, H * y.dim_pitch);
+        olat_n = std::max(olat_n, H * y.val_pitch);
+        lq_n = std::max(lq_n, H * y.row_width);
+        for (size_t t = 1; t <= T; ++t)
+            lpart_n = std::max(lpart_n, t * H * latent_prefill_splits(e, y, (int)t) * (y.rank_pitch + kLatentPartTail));
+        gate_n = std::max(gate_n, H);
+    }
+    TRY(zeroed(e, &e->pf_x, T * D * 4));
+    TRY(zeroed(e, &e->pf_xn, 2 * T * D * 2));      // hi plane, lo plane
+    TRY(zeroed(e, &e->pf_att, 2 * T * att_n * 2));  // hi plane, lo plane
+    TRY(zeroed(e, &e->pf_hb, 2 * T * hb_n * 2));    // hi plane, lo plane
+    TRY(zeroed(e, &e->pf_part, (size_t)kPfMaxSplits * T * part_rows * 4));
+    TRY(zeroed(e, &e->pf_tokens, T * sizeof(int)));
+    TRY(zeroed(e, &e->pf_rows, T * sizeof(int)));
+    if (latent) {
+        TRY(zeroed(e, &e->pf_qn, 2 * T * qn_n * 2));
+        TRY(zeroed(e, &e->pf_olat, 2 * T * olat_n * 2));
+        TRY(zeroed(e, &e->pf_lq, T * lq_n * 2));
+        TRY(zeroed(e, &e->pf_lpart, lpart_n * 4));
+        TRY(zeroed(e, &e->pf_gate, T * gate_n * 4));
+        for (LatentLayer& y : e->lat) {
+            const size_t H = y.d.heads, D2 = align_up(c.dim, 2);
+            TRY(make_weight_map(&y.m_in, y.w_in, y.in_rows, D, kUmmaM));
+            TRY(make_weight_map(&y.m_uk, y.w_uk, H * y.rank_pitch, y.dim_pitch, kUmmaM));
+            TRY(make_weight_map(&y.m_uv, y.w_uv, H * y.vdim_rows, y.val_pitch, kUmmaM));
+            TRY(make_weight_map(&y.m_wo, y.wo, D2, y.o_pitch, kUmmaM));
+            TRY(make_activation_map(&y.x_qn, e->pf_qn, T, H * y.dim_pitch, kPrefillTokens));
+            TRY(make_activation_map(&y.x_olat, e->pf_olat, T, H * y.val_pitch, kPrefillTokens));
+            TRY(make_activation_map(&y.x_att, e->pf_att, T, y.o_pitch, kPrefillTokens));
+            if (y.d.ff > 0) {
+                TRY(make_weight_map(&y.m_w13, y.w13, 2 * (size_t)y.d.ff, D, kUmmaM));
+                TRY(make_weight_map(&y.m_w2, y.w2, D2, y.ff_pitch, kUmmaM));
+                TRY(make_activation_map(&y.x_hb, e->pf_hb, T, y.ff_pitch, kPrefillTokens));
+            }
+        }
+        TRY(allow_gemm_smem<__nv_bfloat16>());
+        CU(cudaFuncSetAttribute(prefill_gemm_umma_kernel<__nv_bfloat16, kPfLatentQuery>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes));
+        CU(cudaFuncSetAttribute(prefill_gemm_umma_kernel<__nv_bfloat16, kPfLatentValue>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes));
+    } else {
+        TRY(zeroed(e, &e->pf_q, T * e->Dq * 4));
+        TRY(make_weight_map(&e->pf_map_wqkv, e->wqkv, L * qkv_rows, D, kUmmaM));
+        TRY(make_weight_map(&e->pf_map_wo, e->wo, L * D, e->Dq, kUmmaM));
+        TRY(make_weight_map(&e->pf_map_w13, e->w13, L * 2 * e->Fl, D, kUmmaM));
+        TRY(make_weight_map(&e->pf_map_w2, e->w2, L * D, e->Fl, kUmmaM));
+        TRY(make_activation_map(&e->pf_map_att, e->pf_att, T, e->Dq, kPrefillTokens));
+        TRY(make_activation_map(&e->pf_map_hb, e->pf_hb, T, e->Fl, kPrefillTokens));
+        TRY(allow_gemm_smem<__half>());
+        CU(cudaFuncSetAttribute(prefill_gemm_umma_kernel<__half, kPfQkv>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes));
+        CU(cudaFuncSetAttribute(prefill_attention_mma_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, pf_attn_smem<64>()));
+        CU(cudaFuncSetAttribute(prefill_attention_mma_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, pf_attn_smem<128>()));
+    }
     TRY(make_activation_map(&e->pf_map_xn, e->pf_xn, T, D, kPrefillTokens));
-    TRY(make_activation_map(&e->pf_map_att, e->pf_att, T, e->Dq, kPrefillTokens));
-    TRY(make_activation_map(&e->pf_map_hb, e->pf_hb, T, e->Fl, kPrefillTokens));
-    CU(cudaFuncSetAttribute(prefill_gemm_umma_kernel<kPfQkv>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes));
-    CU(cudaFuncSetAttribute(prefill_gemm_umma_kernel<kPfResid>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes));
-    CU(cudaFuncSetAttribute(prefill_gemm_umma_kernel<kPfSwiglu>, cudaFuncAttributeMaxDynamicSharedMemorySize, kPfSmemBytes));
-    CU(cudaFuncSetAttribute(prefill_attention_mma_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, pf_attn_smem<64>()));
-    CU(cudaFuncSetAttribute(prefill_attention_mma_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, pf_attn_smem<128>()));
+    TRY(make_weight_map(&e->pf_map_cls, e->wcls, e->Vp, D, kUmmaM));
     e->pf_ready = true;
     return LPP_OK;
 }
 
-// Work items are tiles of 128 weight rows (the weight maps' box).  A GEMM whose row tiles do not fill the GPU is also
-// cut along K; its partial sums go to pf_part and are added up by the next prefill_norm_kernel (residual projections)
-// or by prefill_qkv_finish_kernel (QKV).
-static cudaError_t launch_prefill_gemm(lpp_engine* e, const CUtensorMap& wm, const CUtensorMap& xm, PrefillGemmArgs a) {
-    const int tiles = (a.n_rows + kUmmaM - 1) / kUmmaM;
-    const int n_kc = (a.K + kPfKc - 1) / kPfKc;
-    a.st = e->st;
-    a.splits = 1;
-    // QKV is cut too: its partial sums are finished by prefill_qkv_finish_kernel
-    if ((a.epi == kPfResid || a.epi == kPfQkv) && tiles < e->num_sms)
-        a.splits = std::max(1, std::min({kPfMaxSplits, n_kc, (e->num_sms + tiles - 1) / tiles}));
-    a.part = e->pf_part;
-    const dim3 g(std::min(tiles * a.splits, e->num_sms)), b(kUmmaThreads);
-    const size_t sm = (size_t)kPfSmemBytes;
-    if (a.epi == kPfResid) return launch_kernel(prefill_gemm_umma_kernel<kPfResid>, g, b, sm, e->stream, true, wm, xm, a);
-    if (a.epi == kPfSwiglu) return launch_kernel(prefill_gemm_umma_kernel<kPfSwiglu>, g, b, sm, e->stream, true, wm, xm, a);
-    const cudaError_t err = launch_kernel(prefill_gemm_umma_kernel<kPfQkv>, g, b, sm, e->stream, true, wm, xm, a);
-    if (err != cudaSuccess || a.splits == 1) return err;
-    return launch_kernel(prefill_qkv_finish_kernel, dim3(a.n_tokens, (a.n_rows / 2 + 255) / 256), dim3(256), 0, e->stream, true, a);
-}
-static int prefill_splits(const lpp_engine* e, int n_rows, int K) {  // what launch_prefill_gemm chooses for a residual GEMM
+// Ranges of K a GEMM is cut into so that its row tiles (128 weight rows: the weight maps' box) fill the GPU.
+static int prefill_splits(const lpp_engine* e, int n_rows, int K) {
     const int tiles = (n_rows + kUmmaM - 1) / kUmmaM, n_kc = (K + kPfKc - 1) / kPfKc;
     return tiles < e->num_sms ? std::max(1, std::min({kPfMaxSplits, n_kc, (e->num_sms + tiles - 1) / tiles})) : 1;
 }
 
-// One block of n <= kPrefillTokens prompt tokens at positions start_pos ..: seven kernels per layer; the last layer
-// stops after its K/V rows are written (nothing downstream of them is needed: the call produces no logits).
-static lpp_status prefill_block(lpp_engine* e, const int* h_tokens, int n, int start_pos) {
-    const lpp_config& c = e->c;
-    const int D = c.dim, L = c.n_layers;
-    const int qkv_rows = e->Dq + 2 * e->KVd;
-    const int s_o = prefill_splits(e, D, e->Dq), s_d = prefill_splits(e, D, e->Fl);
-    CU(cudaMemcpyAsync(e->pf_tokens, h_tokens, (size_t)n * sizeof(int), cudaMemcpyHostToDevice, e->stream));
-    for (int l = 0; l < L; ++l) {
-        // layer 0 takes the embedding rows; later layers first add the previous down projection's partial sums
-        CU(launch_kernel(prefill_norm_kernel, dim3(n), dim3(kPfNormThreads), 0, e->stream, l > 0, e->pf_x, (const int*)e->pf_tokens,
-                         (const __half*)(l == 0 ? e->emb : nullptr), c.vocab_size, (const float*)(e->rms_att + (size_t)l * D),
-                         e->pf_xn, D, n, (const float*)e->pf_part, l == 0 ? 1 : s_d, e->st));
-        const size_t lofs = (size_t)l * e->KVHl * c.seq_len * e->hs;
-        PrefillGemmArgs g = {};
-        g.n_tokens = n;
-        g.start_pos = start_pos;
-        g.n_rows = qkv_rows;
-        g.K = D;
-        g.row0 = l * qkv_rows;
-        g.epi = kPfQkv;
-        g.q = e->pf_q;
-        g.q_rows = e->Dq;
-        g.kv_rows = e->KVd;
-        g.head_size = e->hs;
-        g.seq_len = c.seq_len;
-        g.rope = e->rope;
-        g.k_cache = (__half*)e->kcache + lofs;
-        g.v_cache = (__half*)e->vcache + lofs;
-        CU(launch_prefill_gemm(e, e->pf_map_wqkv, e->pf_map_xn, g));
-        if (l == L - 1) break;
-        const dim3 agrid((n + kPfAttnRows - 1) / kPfAttnRows, e->KVHl);
-        const bool pf_mma = !aid_env("LPP_ATTN_CUDA_CORES");
-        if (pf_mma && e->hs == 64 && e->gqa <= 8)
-            CU(launch_kernel(prefill_attention_mma_kernel<64>, agrid, dim3(32 * e->gqa), pf_attn_smem<64>(), e->stream, true,
-                             (const float*)e->pf_q, (const __half*)g.k_cache, (const __half*)g.v_cache, e->pf_att, n, start_pos,
-                             c.seq_len, e->gqa, e->Dq));
-        else if (pf_mma && e->hs == 128 && e->gqa <= 8)
-            CU(launch_kernel(prefill_attention_mma_kernel<128>, agrid, dim3(32 * e->gqa), pf_attn_smem<128>(), e->stream, true,
-                             (const float*)e->pf_q, (const __half*)g.k_cache, (const __half*)g.v_cache, e->pf_att, n, start_pos,
-                             c.seq_len, e->gqa, e->Dq));
-        else
-            CU(launch_kernel(prefill_attention_kernel, dim3(n, e->KVHl), dim3(32 * e->gqa),
-                             (size_t)e->gqa * e->hs * sizeof(float), e->stream, true, (const float*)e->pf_q,
-                             (const __half*)g.k_cache, (const __half*)g.v_cache, e->pf_att, n, start_pos, c.seq_len, e->hs,
-                             e->gqa, e->Dq));
-        PrefillGemmArgs o = {};
-        o.n_tokens = n;
-        o.start_pos = start_pos;
-        o.n_rows = D;
-        o.K = e->Dq;
-        o.row0 = l * D;
-        o.epi = kPfResid;
-        o.x = e->pf_x;
-        CU(launch_prefill_gemm(e, e->pf_map_wo, e->pf_map_att, o));
-        CU(launch_kernel(prefill_norm_kernel, dim3(n), dim3(kPfNormThreads), 0, e->stream, true, e->pf_x, (const int*)e->pf_tokens,
-                         (const __half*)nullptr, c.vocab_size, (const float*)(e->rms_ffn + (size_t)l * D), e->pf_xn, D, n,
-                         (const float*)e->pf_part, s_o, e->st));
-        PrefillGemmArgs u = {};
-        u.n_tokens = n;
-        u.start_pos = start_pos;
-        u.n_rows = 2 * e->Fl;
-        u.K = D;
-        u.row0 = l * 2 * e->Fl;
-        u.epi = kPfSwiglu;
-        u.hb = e->pf_hb;
-        CU(launch_prefill_gemm(e, e->pf_map_w13, e->pf_map_xn, u));
-        PrefillGemmArgs d = {};
-        d.n_tokens = n;
-        d.start_pos = start_pos;
-        d.n_rows = D;
-        d.K = e->Fl;
-        d.row0 = l * D;
-        d.epi = kPfResid;
-        d.x = e->pf_x;
-        CU(launch_prefill_gemm(e, e->pf_map_w2, e->pf_map_hb, d));
-    }
+// A GEMM whose row tiles do not fill the GPU is also cut along K (a.splits); its partial sums go to pf_part and are added
+// up by the next prefill_norm_kernel (residual projections) or by a finishing kernel (input projections).
+template <typename T, int EPI>
+static cudaError_t launch_prefill_gemm_t(lpp_engine* e, const CUtensorMap& wm, const CUtensorMap& xm, const PrefillGemmArgs& a) {
+    const int tiles = (a.n_rows + kUmmaM - 1) / kUmmaM * std::max(1, a.groups);
+    return launch_kernel(prefill_gemm_umma_kernel<T, EPI>, dim3(std::min(tiles * a.splits, e->num_sms)), dim3(kUmmaThreads),
+                         (size_t)kPfSmemBytes, e->stream, true, wm, xm, a);
+}
+template <int EPI>
+static cudaError_t launch_prefill_gemm(lpp_engine* e, const CUtensorMap& wm, const CUtensorMap& xm, const PrefillGemmArgs& a) {
+    return e->c.weight_dtype == LPP_BF16 ? launch_prefill_gemm_t<__nv_bfloat16, EPI>(e, wm, xm, a)
+                                         : launch_prefill_gemm_t<__half, EPI>(e, wm, xm, a);
+}
+static PrefillGemmArgs prefill_gemm_args(const lpp_engine* e, int n_rows, int K, int n_tokens, int start_pos) {
+    PrefillGemmArgs a = {};
+    a.n_rows = n_rows;
+    a.K = K;
+    a.n_tokens = n_tokens;
+    a.start_pos = start_pos;
+    a.splits = 1;
+    a.part = e->pf_part;
+    a.st = e->st;
+    return a;
+}
+
+// x_rows -> normalised operands; `parts` > 1: the previous residual GEMM's partial sums are added to x first.
+static lpp_status prefill_norm(lpp_engine* e, int n, const float* w, const float* b, bool embed, int parts, const int* rows, bool pdl) {
+    PrefillNormArgs a = {};
+    a.x = e->pf_x;
+    a.tokens = e->pf_tokens;
+    a.emb = embed ? e->emb : nullptr;
+    a.vocab = e->c.vocab_size;
+    a.rows = rows;
+    a.norm_w = w;
+    a.norm_b = b;
+    a.norm_eps = e->norm_eps;
+    a.norm_n = e->c.dim;
+    a.out = e->pf_xn;
+    a.D = e->Dp;
+    a.part = e->pf_part;
+    a.splits = embed ? 1 : parts;
+    a.st = e->st;
+    if (e->c.weight_dtype == LPP_BF16)
+        CU(launch_kernel(prefill_norm_kernel<__nv_bfloat16>, dim3(n), dim3(kPfNormThreads), 0, e->stream, pdl, a));
+    else
+        CU(launch_kernel(prefill_norm_kernel<__half>, dim3(n), dim3(kPfNormThreads), 0, e->stream, pdl, a));
     return LPP_OK;
 }
 
-extern "C" lpp_status lpp_prefill(lpp_engine* e, const int* h_tokens, int n, int start_pos, float* device_ms) {
+// x += W . in  for the block: output and down projection.  Returns the number of partial sums the next norm adds.
+static lpp_status prefill_resid(lpp_engine* e, const CUtensorMap& wm, int row0, const CUtensorMap& xm, int K, int n, int start_pos, int* parts) {
+    PrefillGemmArgs g = prefill_gemm_args(e, (e->c.dim + 1) & ~1, K, n, start_pos);
+    g.row0 = row0;
+    g.x = e->pf_x;
+    g.x_pitch = e->Dp;
+    g.splits = *parts = prefill_splits(e, g.n_rows, K);
+    CU(launch_prefill_gemm<kPfResid>(e, wm, xm, g));
+    return LPP_OK;
+}
+
+// Grouped-query attention of a prompt block: K/V rows to the cache and, unless only those are wanted, the attended values
+// to pf_att.
+static lpp_status prefill_gqa_mixer(lpp_engine* e, int l, int n, int start_pos, bool cache_only) {
+    const lpp_config& c = e->c;
+    const int D = c.dim, qkv_rows = e->Dq + 2 * e->KVd;
+    const size_t lofs = (size_t)l * e->KVHl * c.seq_len * e->hs;
+    PrefillGemmArgs g = prefill_gemm_args(e, qkv_rows, D, n, start_pos);
+    g.row0 = l * qkv_rows;
+    g.epi = kPfQkv;
+    g.q = e->pf_q;
+    g.q_rows = e->Dq;
+    g.kv_rows = e->KVd;
+    g.head_size = e->hs;
+    g.seq_len = c.seq_len;
+    g.rope = e->rope;
+    g.k_cache = (__half*)e->kcache + lofs;
+    g.v_cache = (__half*)e->vcache + lofs;
+    g.splits = prefill_splits(e, qkv_rows, D);
+    const cudaError_t ge = launch_prefill_gemm_t<__half, kPfQkv>(e, e->pf_map_wqkv, e->pf_map_xn, g);
+    CU(ge);
+    if (g.splits > 1)
+        CU(launch_kernel(prefill_qkv_finish_kernel, dim3(n, (qkv_rows / 2 + 255) / 256), dim3(256), 0, e->stream, true, g));
+    if (cache_only) return LPP_OK;
+    const dim3 agrid((n + kPfAttnRows - 1) / kPfAttnRows, e->KVHl);
+    __half* att = (__half*)e->pf_att;
+    const bool pf_mma = !aid_env("LPP_ATTN_CUDA_CORES");
+    if (pf_mma && e->hs == 64 && e->gqa <= 8)
+        CU(launch_kernel(prefill_attention_mma_kernel<64>, agrid, dim3(32 * e->gqa), pf_attn_smem<64>(), e->stream, true,
+                         (const float*)e->pf_q, (const __half*)g.k_cache, (const __half*)g.v_cache, att, n, start_pos,
+                         c.seq_len, e->gqa, e->Dq));
+    else if (pf_mma && e->hs == 128 && e->gqa <= 8)
+        CU(launch_kernel(prefill_attention_mma_kernel<128>, agrid, dim3(32 * e->gqa), pf_attn_smem<128>(), e->stream, true,
+                         (const float*)e->pf_q, (const __half*)g.k_cache, (const __half*)g.v_cache, att, n, start_pos,
+                         c.seq_len, e->gqa, e->Dq));
+    else
+        CU(launch_kernel(prefill_attention_kernel, dim3(n, e->KVHl), dim3(32 * e->gqa),
+                         (size_t)e->gqa * e->hs * sizeof(float), e->stream, true, (const float*)e->pf_q,
+                         (const __half*)g.k_cache, (const __half*)g.v_cache, att, n, start_pos, c.seq_len, e->hs,
+                         e->gqa, e->Dq));
+    return LPP_OK;
+}
+
+// Latent attention of a prompt block: input GEMM (cut along K) and its finishing kernel, per-head query GEMM, attention in
+// key splits, their combination, per-head value GEMM with the gates.
+static lpp_status prefill_latent_mixer(lpp_engine* e, int l, int n, int start_pos, bool cache_only) {
+    typedef __nv_bfloat16 T;
+    const LatentLayer& y = e->lat[l];
+    const int H = y.d.heads;
+    PrefillGemmArgs g = prefill_gemm_args(e, y.in_rows, e->Dp, n, start_pos);
+    g.out = e->pf_part;
+    g.out_pitch = y.in_rows;
+    g.splits = prefill_splits(e, y.in_rows, e->Dp);
+    CU((launch_prefill_gemm_t<T, kPfStore>(e, y.m_in, e->pf_map_xn, g)));
+    PrefillLatentFinishArgs f = {};
+    f.part = e->pf_part;
+    f.n_rows = y.in_rows;
+    f.splits = g.splits;
+    f.start_pos = start_pos;
+    f.seq_len = e->c.seq_len;
+    f.qn = e->pf_qn;
+    f.gate = e->pf_gate;
+    f.st = e->st;
+    f.lat = latent_args(e, y);
+    f.lat.query = e->pf_lq;
+    const int q_sections = cache_only ? 0 : (y.q_plain_rows + y.q_rot_rows + 2 * kLatFinishThreads - 1) / (2 * kLatFinishThreads);
+    CU(launch_kernel(prefill_latent_finish_kernel<T>, dim3(n, 1 + q_sections), dim3(kLatFinishThreads), (size_t)y.latent_rows * 4, e->stream,
+                     true, f));
+    if (cache_only) return LPP_OK;
+    PrefillGemmArgs q = prefill_gemm_args(e, y.rank_pitch, y.dim_pitch, n, start_pos);
+    q.groups = H;
+    q.group_stride = y.rank_pitch;
+    q.group_pieces = y.dim_pitch / 64;
+    q.lat_query = e->pf_lq;
+    q.lat_pitch = y.row_width;
+    CU((launch_prefill_gemm_t<T, kPfLatentQuery>(e, y.m_uk, y.x_qn, q)));
+    LatentAttnArgs a = latent_attn_args(e, y);
+    a.q = e->pf_lq;
+    a.part = e->pf_lpart;
+    a.start_pos = start_pos;
+    a.n_tokens = n;
+    a.max_splits = latent_prefill_splits(e, y, n);
+    CU(launch_latent_attn(e, y, a, true, e->stream));
+    const int tile_rows = latent_mma_supported(e, y) ? latent_tile_rows(n * H) : 0;
+    CU(launch_kernel(prefill_latent_combine_kernel<T>, dim3(n * H), dim3(128), 0, e->stream, true, a, tile_rows, (T*)e->pf_olat, y.val_pitch));
+    PrefillGemmArgs v = prefill_gemm_args(e, y.vdim_rows, y.val_pitch, n, start_pos);
+    v.groups = H;
+    v.group_stride = y.vdim_rows;
+    v.group_pieces = y.val_pitch / 64;
+    v.hb = e->pf_att;
+    v.hb_pitch = y.o_pitch;
+    v.gate = e->pf_gate;
+    v.n_valid = y.d.vdim;
+    CU((launch_prefill_gemm_t<T, kPfLatentValue>(e, y.m_uv, y.x_olat, v)));
+    return LPP_OK;
+}
+
+// One block of n <= kPrefillTokens prompt tokens at positions start_pos ...  Without wanted logits the last layer stops
+// after its cache rows are written (nothing downstream of them is needed); otherwise the n_want rows `want` of the block go
+// through the final norm and the classifier and their logits are copied to h_logits.
+static lpp_status prefill_block(lpp_engine* e, const int* h_tokens, int n, int start_pos, const int* want, int n_want, float* h_logits) {
+    const lpp_config& c = e->c;
+    const int L = c.n_layers;
+    const bool latent = !e->lat.empty();
+    CU(cudaMemcpyAsync(e->pf_tokens, h_tokens, (size_t)n * sizeof(int), cudaMemcpyHostToDevice, e->stream));
+    if (n_want > 0) CU(cudaMemcpyAsync(e->pf_rows, want, (size_t)n_want * sizeof(int), cudaMemcpyHostToDevice, e->stream));
+    int parts = 1;
+    for (int l = 0; l < L; ++l) {
+        const bool cache_only = l == L - 1 && n_want == 0;
+        const LayerView v = layer_view(e, l);
+        // layer 0 takes the embedding rows; later layers first add the previous residual GEMM's partial sums
+        TRY(prefill_norm(e, n, latent ? e->lat[l].n1w : e->rms_att + (size_t)l * c.dim, latent ? e->lat[l].n1b : nullptr, l == 0, parts,
+                         nullptr, l > 0));
+        TRY(latent ? prefill_latent_mixer(e, l, n, start_pos, cache_only) : prefill_gqa_mixer(e, l, n, start_pos, cache_only));
+        if (cache_only) return LPP_OK;
+        TRY(prefill_resid(e, latent ? e->lat[l].m_wo : e->pf_map_wo, latent ? 0 : l * c.dim, latent ? e->lat[l].x_att : e->pf_map_att, v.o_k, n,
+                          start_pos, &parts));
+        if (v.ff == 0) continue;  // a layer without a feed-forward
+        TRY(prefill_norm(e, n, v.norm2_w, v.norm2_b, false, parts, nullptr, true));
+        PrefillGemmArgs u = prefill_gemm_args(e, 2 * v.ff, e->Dp, n, start_pos);
+        u.row0 = latent ? 0 : l * 2 * v.ff;
+        u.hb = e->pf_hb;
+        u.hb_pitch = v.ff_k;
+        u.act = v.act;
+        CU(launch_prefill_gemm<kPfSwiglu>(e, latent ? e->lat[l].m_w13 : e->pf_map_w13, e->pf_map_xn, u));
+        TRY(prefill_resid(e, latent ? e->lat[l].m_w2 : e->pf_map_w2, latent ? 0 : l * c.dim, latent ? e->lat[l].x_hb : e->pf_map_hb, v.ff_k, n,
+                          start_pos, &parts));
+    }
+    if (!e->pf_logits) CU(cudaMalloc(&e->pf_logits, (size_t)kPrefillTokens * e->Vp * 4));
+    TRY(prefill_norm(e, n_want, e->rms_final, e->final_b, false, parts, e->pf_rows, true));
+    PrefillGemmArgs g = prefill_gemm_args(e, e->Vp, e->Dp, n_want, start_pos);
+    g.out = e->pf_logits;
+    g.out_pitch = e->Vp;
+    CU(launch_prefill_gemm<kPfStore>(e, e->pf_map_cls, e->pf_map_xn, g));
+    CU(cudaMemcpy2DAsync(h_logits, (size_t)c.vocab_size * 4, e->pf_logits, (size_t)e->Vp * 4, (size_t)c.vocab_size * 4, n_want,
+                         cudaMemcpyDeviceToHost, e->stream));
+    return LPP_OK;
+}
+
+extern "C" lpp_status lpp_extend(lpp_engine* e, const int* h_tokens, int n, int start_pos, const int* want, int n_want, float* h_logits,
+                                 float* device_ms) {
     NEED_READY(e);
-    if (!h_tokens || n <= 0) return fail(LPP_ERR_INVALID_ARG, "bad argument");
-    if (start_pos < 0 || start_pos + n > e->c.seq_len) return fail(LPP_ERR_INVALID_ARG, "positions %d..%d outside [0, %d)", start_pos, start_pos + n - 1, e->c.seq_len);
+    if (!h_tokens || n <= 0 || n_want < 0 || (n_want > 0 && (!want || !h_logits))) return fail(LPP_ERR_INVALID_ARG, "bad argument");
+    if (start_pos < 0 || start_pos > e->c.seq_len - n) return fail(LPP_ERR_INVALID_ARG, "positions %d..%d outside [0, %d)", start_pos, start_pos + n - 1, e->c.seq_len);
     for (int i = 0; i < n; ++i)
         if (h_tokens[i] < 0 || h_tokens[i] >= e->c.vocab_size) return fail(LPP_ERR_INVALID_ARG, "token %d outside [0, %d)", h_tokens[i], e->c.vocab_size);
+    for (int i = 0; i < n_want; ++i)
+        if (want[i] < (i ? want[i - 1] + 1 : 0) || want[i] >= n) return fail(LPP_ERR_INVALID_ARG, "wanted tokens must ascend within the portion");
+    const size_t V = e->c.vocab_size;
+    int w = 0;  // wanted tokens served so far
     TRY(push_state(e, h_tokens[0], start_pos, nullptr, nullptr, 0, 0.f, 0, 0));  // clears the device status
-    if (prefill_batched(e)) {
+    if (prefill_batched(e) && !(n == 1 && n_want == 1)) {
         TRY(prefill_setup(e));
         CU(cudaEventRecord(e->ev0, e->stream));
-        for (int i = 0; i < n; i += kPrefillTokens) TRY(prefill_block(e, h_tokens + i, std::min(kPrefillTokens, n - i), start_pos + i));
+        for (int i = 0; i < n; i += kPrefillTokens) {
+            const int m = std::min(kPrefillTokens, n - i);
+            int rows[kPrefillTokens], k = 0;
+            while (w + k < n_want && want[w + k] < i + m) rows[k] = want[w + k] - i, ++k;
+            TRY(prefill_block(e, h_tokens + i, m, start_pos + i, rows, k, h_logits + (size_t)w * V));
+            w += k;
+        }
         CU(cudaEventRecord(e->ev1, e->stream));
     } else {
         // token by token through the step graph without its sampler, like the reference's prompt loop
         CU(cudaEventRecord(e->ev0, e->stream));
         for (int i = 0; i < n; ++i) {
-            TRY(push_state(e, h_tokens[i], start_pos + i, nullptr, nullptr, 0, 0.f, 0, 0));
+            if (i > 0) TRY(push_state(e, h_tokens[i], start_pos + i, nullptr, nullptr, 0, 0.f, 0, 0));
             TRY(run_step(e, false, start_pos + i));
-            // the pinned staging block of push_state is rewritten by the next token: the copy must have run
-            if (i + 1 < n) CU(cudaStreamSynchronize(e->stream));
+            if (w < n_want && want[w] == i)
+                CU(cudaMemcpyAsync(h_logits + (size_t)w++ * V, e->logits, V * 4, cudaMemcpyDeviceToHost, e->stream));
+            // the pinned staging block of push_state is rewritten by the next token (the copy must have run), and the
+            // next token's push would clear a status this one has set
+            if (i + 1 < n) TRY(pull_result(e, nullptr));
         }
         CU(cudaEventRecord(e->ev1, e->stream));
     }
@@ -1470,10 +2173,14 @@ extern "C" lpp_status lpp_prefill(lpp_engine* e, const int* h_tokens, int n, int
     return LPP_OK;
 }
 
+extern "C" lpp_status lpp_prefill(lpp_engine* e, const int* h_tokens, int n, int start_pos, float* device_ms) {
+    return lpp_extend(e, h_tokens, n, start_pos, nullptr, 0, nullptr, device_ms);
+}
+
 // ------------------------------------------------------------------ KV cache access
 
 extern "C" int64_t lpp_kv_index(const lpp_engine* e, int layer, int kv_head, int pos, int off) {
-    if (!e) return -1;
+    if (!e || !e->lat.empty()) return -1;
     const int64_t kvd = (int64_t)e->KVHl * e->hs, S = e->c.seq_len;
     return (int64_t)layer * (kvd * S) + (int64_t)kv_head * (S * e->hs) + (int64_t)pos * e->hs + off;
 }
@@ -1482,6 +2189,7 @@ extern "C" lpp_status lpp_kv_prefill(lpp_engine* e, int layer, const void* k, co
                                      int memkind) {
     if (!e || !k || !v) return fail(LPP_ERR_INVALID_ARG, "null argument");
     const lpp_config& c = e->c;
+    if (!e->lat.empty()) return fail(LPP_ERR_INVALID_ARG, "this model keeps latents, not keys and values");
     if (layer < 0 || layer >= c.n_layers || n_pos < 0 || n_pos > c.seq_len) return fail(LPP_ERR_INVALID_ARG, "layer/n_pos out of range");
     if (src_dtype != LPP_F16 && src_dtype != LPP_F32) return fail(LPP_ERR_INVALID_ARG, "bad src_dtype");
     CU(cudaSetDevice(c.device));
@@ -1504,6 +2212,7 @@ extern "C" lpp_status lpp_kv_prefill(lpp_engine* e, int layer, const void* k, co
 extern "C" lpp_status lpp_kv_read(lpp_engine* e, int layer, int kv_head, int pos, float* h_k, float* h_v) {
     if (!e || !h_k || !h_v) return fail(LPP_ERR_INVALID_ARG, "null argument");
     const lpp_config& c = e->c;
+    if (!e->lat.empty()) return fail(LPP_ERR_INVALID_ARG, "this model keeps latents, not keys and values");
     if (layer < 0 || layer >= c.n_layers || kv_head < 0 || kv_head >= e->KVHl || pos < 0 || pos >= c.seq_len)
         return fail(LPP_ERR_INVALID_ARG, "index out of range");
     CU(cudaSetDevice(c.device));
@@ -1522,6 +2231,20 @@ extern "C" lpp_status lpp_kv_read(lpp_engine* e, int layer, int kv_head, int pos
             h_v[i] = __half2float(tv[i]);
         }
     }
+    return LPP_OK;
+}
+
+extern "C" lpp_status lpp_latent_read(lpp_engine* e, int layer, int pos, float* h_row) {
+    if (!e || !h_row) return fail(LPP_ERR_INVALID_ARG, "null argument");
+    if (layer < 0 || layer >= (int)e->lat.size() || pos < 0 || pos >= e->c.seq_len) return fail(LPP_ERR_INVALID_ARG, "index out of range");
+    CU(cudaSetDevice(e->c.device));
+    CU(cudaStreamSynchronize(e->stream));
+    const LatentLayer& y = e->lat[layer];
+    std::vector<unsigned char> raw((size_t)y.row_width * e->kvesz);
+    CU(cudaMemcpy(raw.data(), (const char*)y.cache + (size_t)pos * raw.size(), raw.size(), cudaMemcpyDeviceToHost));
+    auto at = [&](int i) { return e->kvesz == 4 ? ((const float*)raw.data())[i] : __half2float(((const __half*)raw.data())[i]); };
+    for (int i = 0; i < y.d.kv_rank; ++i) h_row[i] = at(i);
+    for (int i = 0; i < y.d.rot_dim; ++i) h_row[y.d.kv_rank + i] = at(y.rank_pitch + i);
     return LPP_OK;
 }
 
@@ -1653,6 +2376,24 @@ static void kind_bytes(const lpp_engine* e, int pos, int64_t* b) {
     const lpp_config& c = e->c;
     const int64_t D = c.dim, L = c.n_layers, V = c.vocab_size, esz = e->esz;
     for (int k = 0; k < kKinds; ++k) b[k] = 0;
+    if (!e->lat.empty()) {
+        for (const LatentLayer& y : e->lat) {
+            const lpp_layer_desc& d = y.d;
+            const int64_t keys = d.window > 0 ? std::min<int64_t>(d.window, pos + 1) : pos + 1;
+            const int64_t row = d.kv_rank + d.rot_dim, H = d.heads;
+            b[kQkv] += (H * (d.dim + d.rot_dim) + row + H) * D * esz + 8 * D;
+            b[kLatQuery] += H * d.dim * d.kv_rank * esz;
+            b[kAttn] += (keys + 1) * row * e->kvesz;
+            b[kLatValue] += H * d.vdim * d.kv_rank * esz;
+            b[kOproj] += D * H * d.vdim * esz;
+            if (d.ff > 0) {
+                b[kGateUp] += (int64_t)2 * d.ff * D * esz + 8 * D;
+                b[kDown] += D * d.ff * esz;
+            }
+        }
+        b[kLmHead] = V * D * esz + 8 * D;
+        return;
+    }
     b[kQkv] = L * ((int64_t)(e->Dq + 2 * e->KVd) * D * esz + 4 * D) + 4 * D;  // + att norms + embedding row
     b[kAttn] = L * (int64_t)e->kvesz * 2 * e->KVd * ((int64_t)pos + 1) + L * (int64_t)e->kvesz * 2 * e->KVd;
     b[kOproj] = L * D * e->Dq * esz;

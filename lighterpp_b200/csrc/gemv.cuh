@@ -1,7 +1,8 @@
-// Batch-1 streaming GEMV family: out[n] = W[n,K] . x[K] with FP16 or FP32 weights, FP32 activations
+// Batch-1 streaming GEMV family: out[n] = W[n,K] . x[K] with FP16, BF16 or FP32 weights, FP32 activations
 // and FP32 accumulation.  One kernel template serves every matrix of the decode step; what differs
-// is the prologue (plain vector, RMSNorm'd vector, embedding row) and the epilogue (store,
-// residual add, SwiGLU, RoPE + KV-cache scatter).
+// is the prologue (plain vector, RMSNorm'd or LayerNorm'd vector, embedding row, per-head inputs, combination of
+// attention splits) and the epilogue (store, residual add, gated activation, RoPE + KV-cache scatter, and the
+// three projections of latent attention, latent.cuh).
 //
 // Replaces, from the reference tree: gemv_kernel / gemv_f16_kernel / convert_f32_to_f16_kernel
 // (src/matmul.cu:9-161), rmsnorm (src/RMSNorm.cu:11-71, fused as prologue), swiglu_kernel
@@ -23,10 +24,19 @@
 // when the activations arrive.  HBM traffic = the matrix once; x is re-read from L2 per CTA.
 #pragma once
 #include "common.cuh"
+#include "latent.cuh"
 
 namespace lpp {
 
-enum GemvEpi : int { kEpiStore = 0, kEpiResid = 1, kEpiSwiglu = 2, kEpiQkv = 3 };
+enum GemvEpi : int {
+    kEpiStore = 0,
+    kEpiResid = 1,
+    kEpiSwiglu = 2,
+    kEpiQkv = 3,
+    kEpiLatentIn = 4,     // query | latent | rotated key part | gate rows of latent attention
+    kEpiLatentQuery = 5,  // per head: query in the latent space
+    kEpiLatentValue = 6   // per head: value of the attended latent, times the head's gate
+};
 
 constexpr int kGemvConsumerWarps = 8;
 constexpr int kGemvRingThreads = (kGemvConsumerWarps + 1) * 32;  // + producer warp
@@ -48,8 +58,16 @@ struct GemvArgs {
     float* x_store;       // CTA 0 stores the un-normalised input vector here (nullptr = don't)
     StepState* st;        // token / pos / status
     int vocab, seq_len;
+    const float* norm_b;  // LayerNorm bias [K]: selects LayerNorm (mean taken off); nullptr = RMSNorm
+    float norm_eps;       // inside the root
+    int norm_n;           // inputs the statistics cover (0 = K); inputs norm_n .. K-1 are zero padding
+    // Grouped rows (heads): row pair g takes the K inputs of group g / group_pairs, x + group * K.  0 = one input
+    // vector for all rows.  No normalisation, no embedding.
+    int group_pairs;
+    LatentArgs lat;       // latent attention prologues and epilogues
     // ---- epilogue
     float* out;          // Store/Resid: [n_rows]; Swiglu: [n_rows/2]; Qkv: q vector [q_rows]
+    int act;             // Swiglu: activation of the gate (Act)
     const float* resid;  // Resid: added to the result when non-null
     int q_rows, kv_rows, head_size;  // Qkv: rows are q | k | v
     const float2* rope;              // Qkv: [seq_len][head_size/2] (cos, sin)
@@ -96,18 +114,15 @@ struct GemvArgs {
 
 // ------------------------------------------------------------------ x staging layouts
 //
-// FP16 weights: a lane multiplies 8 consecutive weights (one 16-byte vector) with 8 consecutive x.
+// 16-bit weights: a lane multiplies 8 consecutive weights (one 16-byte vector) with 8 consecutive x.
 // To keep both 16-byte x reads bank-conflict free the low and high halves of every 8-group live in
 // two separate planes.  FP32 weights: one 16-byte vector = 4 weights, x is stored naturally.
 template <typename WT>
-__device__ __forceinline__ int xs_index(int k, int K);
-template <>
-__device__ __forceinline__ int xs_index<__half>(int k, int K) {
-    return ((k >> 3) << 2) + (k & 3) + ((k & 4) ? (K >> 1) : 0);
-}
-template <>
-__device__ __forceinline__ int xs_index<float>(int k, int /*K*/) {
-    return k;
+__device__ __forceinline__ int xs_index(int k, int K) {
+    if constexpr (sizeof(WT) == 2)
+        return ((k >> 3) << 2) + (k & 3) + ((k & 4) ? (K >> 1) : 0);
+    else
+        return k;
 }
 
 __device__ __forceinline__ void gemv_stamp(const GemvArgs& a, int k) {
@@ -116,10 +131,6 @@ __device__ __forceinline__ void gemv_stamp(const GemvArgs& a, int k) {
         asm volatile("mov.u64 %0, %%globaltimer;" : "=l"(t));
         a.trace[(size_t)blockIdx.x * 8 + k] = t;
     }
-}
-
-__device__ __forceinline__ void consumer_barrier(int nthreads) {
-    asm volatile("bar.sync 1, %0;" ::"r"(nthreads) : "memory");
 }
 
 // Stores four consecutive inputs x[k..k+3] (k % 4 == 0) into the staging layout.
@@ -138,6 +149,45 @@ __device__ __forceinline__ float4* xs_ptr4(float* xs, int k, int K) {
         return reinterpret_cast<float4*>(xs + ((k >> 3) << 2) + ((k & 4) ? (K >> 1) : 0));
     else
         return reinterpret_cast<float4*>(xs + k);
+}
+
+__device__ __forceinline__ int norm_count(const GemvArgs& a) { return a.norm_n > 0 ? a.norm_n : a.K; }
+
+// Sum over NT threads of one value each; `slot` separates reductions that follow each other without a barrier.
+template <int NT>
+__device__ __forceinline__ float consumer_sum(float v, float* red, int tid, int slot) {
+    v = warp_sum(v);
+    if ((tid & 31) == 0) red[slot * (NT / 32) + (tid >> 5)] = v;
+    consumer_barrier(NT);
+    float tot = 0.f;
+#pragma unroll
+    for (int w = 0; w < NT / 32; ++w) tot += red[slot * (NT / 32) + w];
+    return tot;
+}
+
+// LayerNorm, in place, of the inputs that this thread staged itself (inputs tid * step .. + step - 1, then NT * step
+// further on, with step 1 or 4): the mean first, then the mean of the squared deviations from it.  Zero padding
+// beyond norm_n stays out of both and comes out as zero (its weight and bias are zero).
+template <typename WT, int NT>
+__device__ __forceinline__ void layer_norm_staged(const GemvArgs& a, float* xs, float* red, int tid, int step) {
+    const int K = a.K, n = norm_count(a);
+    float s = 0.f;
+    for (int k0 = tid * step; k0 < n; k0 += NT * step)
+        for (int k = k0; k < min(k0 + step, n); ++k) s += xs[xs_index<WT>(k, K)];
+    const float mean = __fdiv_rn(consumer_sum<NT>(s, red, tid, 0), (float)n);
+    float q = 0.f;
+    for (int k0 = tid * step; k0 < n; k0 += NT * step)
+        for (int k = k0; k < min(k0 + step, n); ++k) {
+            const float d = xs[xs_index<WT>(k, K)] - mean;
+            q = fmaf(d, d, q);
+        }
+    const float var = __fdiv_rn(consumer_sum<NT>(q, red, tid, 1), (float)n);
+    const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(var, a.norm_eps)));
+    for (int k0 = tid * step; k0 < K; k0 += NT * step)
+        for (int k = k0; k < min(k0 + step, K); ++k) {
+            float* p = xs + xs_index<WT>(k, K);
+            *p = k < n ? fmaf(__fmul_rn(*p - mean, scale), __ldg(a.norm_w + k), __ldg(a.norm_b + k)) : 0.f;
+        }
 }
 
 // Input staging when the input vector arrives through the tensor-parallel exchange: the sum, in rank
@@ -246,7 +296,7 @@ __device__ __forceinline__ void stage_input_peers(const GemvArgs& a, float* xs, 
         float tot = 0.f;
 #pragma unroll
         for (int w = 0; w < NT / 32; ++w) tot += red[w];
-        const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, (float)K), 1e-5f)));
+        const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, (float)K), a.norm_eps)));
         for (int i = tid; i < nv4; i += NT) {  // the elements this thread staged itself
             float4* p = xs_ptr4<WT>(xs, i << 2, K);
             const float4 v = *p, g = __ldg(reinterpret_cast<const float4*>(a.norm_w) + i);
@@ -267,12 +317,13 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
     const int nv4 = K >> 2;
     constexpr int kPer = 4;  // float4 per thread and pass: one pass covers 4*4*NT inputs
     const bool one_pass = nv4 <= kPer * NT;
-    float4 wr[kPer];
+    float4 wr[kPer], br[kPer];
     if (a.norm_w && one_pass) {
 #pragma unroll
         for (int j = 0; j < kPer; ++j) {
             const int i = tid + j * NT;
             if (i < nv4) wr[j] = __ldg(reinterpret_cast<const float4*>(a.norm_w) + i);
+            if (i < nv4 && a.norm_b) br[j] = __ldg(reinterpret_cast<const float4*>(a.norm_b) + i);
         }
     }
     // An input that arrives through the tensor-parallel exchange validates itself word by word (this
@@ -297,23 +348,21 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
         const bool store = a.x_store && blockIdx.x == 0;
         float ss = 0.f;
         for (int k = tid; k < K; k += NT) {
-            float v;
-            if constexpr (sizeof(WT) == 2)
-                v = __half2float(erow[k]);
-            else
-                v = erow[k];
+            const float v = to_float(erow[k]);
             ss = fmaf(v, v, ss);
             if (store) a.x_store[k] = v;
             xs[xs_index<WT>(k, K)] = v;
         }
-        if (a.norm_w) {
+        if (a.norm_b) {
+            layer_norm_staged<WT, NT>(a, xs, red, tid, 1);
+        } else if (a.norm_w) {
             ss = warp_sum(ss);
             if ((tid & 31) == 0) red[tid >> 5] = ss;
             consumer_barrier(NT);
             float tot = 0.f;
 #pragma unroll
             for (int w = 0; w < NT / 32; ++w) tot += red[w];
-            const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, (float)K), 1e-5f)));
+            const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, (float)norm_count(a)), a.norm_eps)));
             for (int k = tid; k < K; k += NT) {
                 const int i = xs_index<WT>(k, K);
                 xs[i] = __fmul_rn(__fmul_rn(xs[i], scale), a.norm_w[k]);
@@ -325,6 +374,48 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
 
     const float4* x4 = reinterpret_cast<const float4*>(a.x);
     auto load_x4 = [&](int i) -> float4 { return __ldcg(x4 + i); };
+    if (a.norm_b && one_pass) {
+        // LayerNorm from registers: the mean, then the mean of the squared deviations (zero padding beyond norm_n adds
+        // nothing to the first sum, is left out of the second one and has zero weight and bias)
+        const int n = norm_count(a);
+        float4 x[kPer];
+        float s = 0.f, q = 0.f;
+#pragma unroll
+        for (int j = 0; j < kPer; ++j) {
+            const int i = tid + j * NT;
+            x[j] = i < nv4 ? load_x4(i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int j = 0; j < kPer; ++j) s += (x[j].x + x[j].y) + (x[j].z + x[j].w);
+        const float mean = __fdiv_rn(consumer_sum<NT>(s, red, tid, 0), (float)n);
+#pragma unroll
+        for (int j = 0; j < kPer; ++j) {
+            const int k = (tid + j * NT) << 2;
+            x[j].x -= mean; x[j].y -= mean; x[j].z -= mean; x[j].w -= mean;
+            if (k + 0 < n) q = fmaf(x[j].x, x[j].x, q);
+            if (k + 1 < n) q = fmaf(x[j].y, x[j].y, q);
+            if (k + 2 < n) q = fmaf(x[j].z, x[j].z, q);
+            if (k + 3 < n) q = fmaf(x[j].w, x[j].w, q);
+        }
+        const float var = __fdiv_rn(consumer_sum<NT>(q, red, tid, 1), (float)n);
+        const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(var, a.norm_eps)));
+#pragma unroll
+        for (int j = 0; j < kPer; ++j) {
+            const int i = tid + j * NT;
+            if (i < nv4)
+                xs_store4<WT>(xs, i << 2, K,
+                              make_float4(fmaf(__fmul_rn(x[j].x, scale), wr[j].x, br[j].x), fmaf(__fmul_rn(x[j].y, scale), wr[j].y, br[j].y),
+                                          fmaf(__fmul_rn(x[j].z, scale), wr[j].z, br[j].z), fmaf(__fmul_rn(x[j].w, scale), wr[j].w, br[j].w)));
+        }
+        consumer_barrier(NT);
+        return;
+    }
+    if (a.norm_b) {  // wider rows: from the staged copy
+        for (int i = tid; i < nv4; i += NT) xs_store4<WT>(xs, i << 2, K, load_x4(i));
+        layer_norm_staged<WT, NT>(a, xs, red, tid, 4);
+        consumer_barrier(NT);
+        return;
+    }
     if (!a.norm_w) {
         for (int i = tid; i < nv4; i += NT) xs_store4<WT>(xs, i << 2, K, load_x4(i));
         consumer_barrier(NT);
@@ -355,7 +446,7 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
     float tot = 0.f;
 #pragma unroll
     for (int w = 0; w < NT / 32; ++w) tot += red[w];
-    const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, (float)K), 1e-5f)));
+    const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, (float)norm_count(a)), a.norm_eps)));
     auto normed = [&](float4 v, float4 w) {
         return make_float4(__fmul_rn(__fmul_rn(v.x, scale), w.x), __fmul_rn(__fmul_rn(v.y, scale), w.y),
                            __fmul_rn(__fmul_rn(v.z, scale), w.z), __fmul_rn(__fmul_rn(v.w, scale), w.w));
@@ -369,6 +460,31 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
     } else {
         for (int i = tid; i < nv4; i += NT)
             xs_store4<WT>(xs, i << 2, K, normed(load_x4(i), __ldg(reinterpret_cast<const float4*>(a.norm_w) + i)));
+    }
+    consumer_barrier(NT);
+}
+
+// Staging for grouped rows: inputs of groups first .. first + n - 1 (one per head), K each.  The query projection
+// reads the plain query parts; its last CTA also turns the raw latent of this token into a cache row.  The value
+// projection reads the attended latents, which it puts together from the partial results of the attention splits.
+template <typename WT, int EPI, int NT>
+__device__ __forceinline__ void stage_input_groups(const GemvArgs& a, float* xs, int tid, int first, int n) {
+    const int K = a.K, Kx = n * K;
+    pdl_wait();
+    if (tid == 0) gemv_stamp(a, 1);
+    if constexpr (EPI == kEpiLatentQuery) {
+        if (blockIdx.x == gridDim.x - 1) latent_norm_to_cache<NT>(a.lat, a.st, a.seq_len, xs, tid);
+        const float4* x4 = reinterpret_cast<const float4*>(a.x + (size_t)first * K);
+        for (int i = tid; i < Kx >> 2; i += NT) xs_store4<WT>(xs, i << 2, Kx, __ldcg(x4 + i));
+    } else {
+        // split weights behind the staged inputs: [n][kLatentMaxSplits]
+        float* wt = xs + Kx;
+        const int n_eff = latent_split_weights<NT>(a.lat, a.st, a.seq_len, wt, tid, first, n);
+        consumer_barrier(NT);
+        for (int i = tid; i < Kx >> 2; i += NT) {
+            const int g = (i << 2) / K, k = (i << 2) - g * K;
+            xs_store4<WT>(xs, i << 2, Kx, latent_combine4(a.lat, wt + g * kLatentMaxSplits, first + g, n_eff, k));
+        }
     }
     consumer_barrier(NT);
 }
@@ -410,15 +526,15 @@ __device__ __forceinline__ void dot_rows(const unsigned char* row0, const unsign
             }
             const float4 xl = lds_f4(xlo + (uint32_t)v * 16u), xh = lds_f4(xhi + (uint32_t)v * 16u);
             float2 p;
-            p = half2_bits_to_float2(w0.x); a0 = fmaf(p.x, xl.x, a0); b0 = fmaf(p.y, xl.y, b0);
-            p = half2_bits_to_float2(w0.y); a0 = fmaf(p.x, xl.z, a0); b0 = fmaf(p.y, xl.w, b0);
-            p = half2_bits_to_float2(w0.z); a0 = fmaf(p.x, xh.x, a0); b0 = fmaf(p.y, xh.y, b0);
-            p = half2_bits_to_float2(w0.w); a0 = fmaf(p.x, xh.z, a0); b0 = fmaf(p.y, xh.w, b0);
+            p = unpack2<WT>(w0.x); a0 = fmaf(p.x, xl.x, a0); b0 = fmaf(p.y, xl.y, b0);
+            p = unpack2<WT>(w0.y); a0 = fmaf(p.x, xl.z, a0); b0 = fmaf(p.y, xl.w, b0);
+            p = unpack2<WT>(w0.z); a0 = fmaf(p.x, xh.x, a0); b0 = fmaf(p.y, xh.y, b0);
+            p = unpack2<WT>(w0.w); a0 = fmaf(p.x, xh.z, a0); b0 = fmaf(p.y, xh.w, b0);
             if constexpr (NR == 2) {
-                p = half2_bits_to_float2(w1.x); a1 = fmaf(p.x, xl.x, a1); b1 = fmaf(p.y, xl.y, b1);
-                p = half2_bits_to_float2(w1.y); a1 = fmaf(p.x, xl.z, a1); b1 = fmaf(p.y, xl.w, b1);
-                p = half2_bits_to_float2(w1.z); a1 = fmaf(p.x, xh.x, a1); b1 = fmaf(p.y, xh.y, b1);
-                p = half2_bits_to_float2(w1.w); a1 = fmaf(p.x, xh.z, a1); b1 = fmaf(p.y, xh.w, b1);
+                p = unpack2<WT>(w1.x); a1 = fmaf(p.x, xl.x, a1); b1 = fmaf(p.y, xl.y, b1);
+                p = unpack2<WT>(w1.y); a1 = fmaf(p.x, xl.z, a1); b1 = fmaf(p.y, xl.w, b1);
+                p = unpack2<WT>(w1.z); a1 = fmaf(p.x, xh.x, a1); b1 = fmaf(p.y, xh.y, b1);
+                p = unpack2<WT>(w1.w); a1 = fmaf(p.x, xh.z, a1); b1 = fmaf(p.y, xh.w, b1);
             }
         }
     } else {
@@ -463,7 +579,7 @@ __device__ __forceinline__ void store_rows(const GemvArgs& a, int row, float v0,
 }
 
 // Writes the results of row pair `g` (rows 2g, 2g+1); called by one lane with the warp-reduced sums.
-template <int EPI>
+template <typename WT, int EPI>
 __device__ __forceinline__ void gemv_epilogue(const GemvArgs& a, int g, float v0, float v1) {
     const int row = g * kRowsPerGroup;
     if constexpr (EPI == kEpiStore) {
@@ -477,9 +593,16 @@ __device__ __forceinline__ void gemv_epilogue(const GemvArgs& a, int g, float v0
         }
         store_rows(a, row, v0, v1);
     } else if constexpr (EPI == kEpiSwiglu) {
-        // rows are interleaved (gate_i, up_i); hb = (h1*sigmoid(h1))*h3 (src/ops.cpp:78-87)
-        const float sig = __fdiv_rn(1.0f, 1.0f + expf(-v0));
+        // rows are interleaved (gate_i, up_i); hb = (h1*sigmoid(h1))*h3 (src/ops.cpp:78-87), or the tanh form of
+        // GELU in place of h1*sigmoid(h1)
+        const float sig = __fdiv_rn(1.0f, 1.0f + expf(-act_gate_arg(a.act, v0)));
         a.out[g] = __fmul_rn(__fmul_rn(v0, sig), v1);
+    } else if constexpr (EPI == kEpiLatentIn) {
+        latent_in_rows(a.lat, a.st, a.seq_len, row, v0, v1);
+    } else if constexpr (EPI == kEpiLatentQuery) {
+        latent_query_rows(a.lat, row, v0, v1);
+    } else if constexpr (EPI == kEpiLatentValue) {
+        latent_value_rows(a.lat, a.out, row, v0, v1);
     } else {  // kEpiQkv
         const int pos = a.st->pos;
         if (pos < 0 || pos >= a.seq_len) {
@@ -633,7 +756,21 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgs& a, unsigned char*
             asm volatile("" ::"f"(cs.x), "f"(cs.y));
         }
     }
-    stage_input<WT, kGemvConsumerWarps * 32>(a, xs, red, tid);
+    // grouped rows: the inputs of the groups this CTA's row pairs belong to are staged back to back
+    int first_group = 0, Kx = a.K;
+    if constexpr (EPI == kEpiLatentQuery || EPI == kEpiLatentValue) {
+        first_group = g0 / a.group_pairs;
+        const int n_groups = (g1 - 1) / a.group_pairs - first_group + 1;
+        Kx = n_groups * a.K;
+        stage_input_groups<WT, EPI, kGemvConsumerWarps * 32>(a, xs, tid, first_group, n_groups);
+    } else {
+        stage_input<WT, kGemvConsumerWarps * 32>(a, xs, red, tid);
+    }
+    // where the inputs of row pair p start among the staged ones
+    auto input_offset = [&](int p) -> int {
+        if constexpr (EPI == kEpiLatentQuery || EPI == kEpiLatentValue) return (p / a.group_pairs - first_group) * a.K;
+        return 0;
+    };
     if (tid == 0) gemv_stamp(a, 2);
 
     uint64_t* myfull = full + w * kGemvMaxStages;
@@ -672,14 +809,14 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgs& a, unsigned char*
             for (int i = 0; i < cnt; ++i) {
                 float acc0 = 0.f, acc1 = 0.f;
                 const unsigned char* r0 = st + (size_t)i * kRowsPerGroup * row_bytes;
-                if (!(a.debug & 1)) dot_rows<WT, 2, false>(r0, r0 + row_bytes, xs, a.K, 0, a.K, lane, acc0, acc1);
+                if (!(a.debug & 1)) dot_rows<WT, 2, false>(r0, r0 + row_bytes, xs, Kx, input_offset(p + i), a.K, lane, acc0, acc1);
                 acc0 = warp_sum(acc0);
                 acc1 = warp_sum(acc1);
                 if (lane == 0) {
                     if (EPI == kEpiResid && p + i == p0)
                         store_rows(a, p0 * kRowsPerGroup, acc0 + r_first.x, acc1 + r_first.y);
                     else
-                        gemv_epilogue<EPI>(a, p + i, acc0, acc1);
+                        gemv_epilogue<WT, EPI>(a, p + i, acc0, acc1);
                 }
             }
             release();
@@ -698,7 +835,7 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgs& a, unsigned char*
                     const int klen = min(a.kc, a.K - k0);
                     const unsigned char* st = myring + (size_t)slot * a.stage_bytes;
                     float dummy = 0.f;
-                    if (!(a.debug & 1)) dot_rows<WT, 1, false>(st, st, xs, a.K, k0, klen, lane, acc[r], dummy);
+                    if (!(a.debug & 1)) dot_rows<WT, 1, false>(st, st, xs, Kx, input_offset(p) + k0, klen, lane, acc[r], dummy);
                     release();
                 }
             if (!ok) break;
@@ -707,7 +844,7 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgs& a, unsigned char*
                 if (EPI == kEpiResid && p == p0)
                     store_rows(a, p0 * kRowsPerGroup, v0 + r_first.x, v1 + r_first.y);
                 else
-                    gemv_epilogue<EPI>(a, p, v0, v1);
+                    gemv_epilogue<WT, EPI>(a, p, v0, v1);
             }
         }
     }
@@ -745,16 +882,26 @@ __global__ void __launch_bounds__(kGemvLdgThreads) gemv_ldg_kernel(const GemvArg
     const int g1 = (int)(((long long)(blockIdx.x + 1) * groups) / gridDim.x);
     constexpr int NW = kGemvLdgThreads / 32;
 
-    stage_input<WT, kGemvLdgThreads>(a, xs, red, tid);
+    int first_group = 0, Kx = a.K;
+    if constexpr (EPI == kEpiLatentQuery || EPI == kEpiLatentValue) {
+        first_group = g0 / a.group_pairs;
+        const int n_groups = (g1 - 1) / a.group_pairs - first_group + 1;
+        Kx = n_groups * a.K;
+        stage_input_groups<WT, EPI, kGemvLdgThreads>(a, xs, tid, first_group, n_groups);
+    } else {
+        stage_input<WT, kGemvLdgThreads>(a, xs, red, tid);
+    }
     const unsigned char* W = reinterpret_cast<const unsigned char*>(a.W);
     const size_t row_bytes = (size_t)a.K * sizeof(WT);
     for (int g = g0 + warp; g < g1; g += NW) {
         float acc0 = 0.f, acc1 = 0.f;
         const unsigned char* r0 = W + (size_t)g * kRowsPerGroup * row_bytes;
-        dot_rows<WT, 2, true>(r0, r0 + row_bytes, xs, a.K, 0, a.K, lane, acc0, acc1);
+        int k0 = 0;
+        if constexpr (EPI == kEpiLatentQuery || EPI == kEpiLatentValue) k0 = (g / a.group_pairs - first_group) * a.K;
+        dot_rows<WT, 2, true>(r0, r0 + row_bytes, xs, Kx, k0, a.K, lane, acc0, acc1);
         acc0 = warp_sum(acc0);
         acc1 = warp_sum(acc1);
-        if (lane == 0) gemv_epilogue<EPI>(a, g, acc0, acc1);
+        if (lane == 0) gemv_epilogue<WT, EPI>(a, g, acc0, acc1);
     }
     pdl_launch_dependents();
 }

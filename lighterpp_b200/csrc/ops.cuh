@@ -20,25 +20,24 @@ static __global__ void convert_f16_to_f32_kernel(float* dst, const __half* src, 
     for (long long k = i; k < n; k += stride) dst[k] = __half2float(src[k]);
 }
 
-// Strided 2-D repack with optional dtype conversion: dst[r*dst_pitch + c] = src[r*src_pitch + c]
-// (pitches in elements).  Used to build the engine's fused weight layout from reference-layout
-// tensors (row slices, column slices, gate/up interleave).
+// Strided 2-D repack with optional type conversion: dst[r*dst_row + c*dst_col] = source element (r, c), where source
+// row r starts at src + ((r / group) * group_stride + r % group) * src_pitch (strides in elements).  Used to build the
+// engine's fused weight layouts from full tensors (row and column slices, gate/up interleave, per-head sections,
+// transposes).
 template <typename DT, typename ST>
-static __global__ void repack_kernel(DT* dst, long long dst_pitch, const ST* src, long long src_pitch, int rows,
-                              int cols) {
+static __global__ void repack_kernel(DT* dst, long long dst_row, long long dst_col, const ST* src, long long src_pitch, int group,
+                                     long long group_stride, int rows, int cols) {
     const long long total = (long long)rows * cols;
     const long long stride = (long long)gridDim.x * blockDim.x;
     for (long long k = (long long)blockIdx.x * blockDim.x + threadIdx.x; k < total; k += stride) {
         const long long r = k / cols, c = k % cols;
-        const ST v = src[r * src_pitch + c];
+        const ST v = src[((r / group) * group_stride + r % group) * src_pitch + c];
         DT o;
-        if constexpr (sizeof(DT) == 2 && sizeof(ST) == 4)
-            o = __float2half_rn(v);
-        else if constexpr (sizeof(DT) == 4 && sizeof(ST) == 2)
-            o = __half2float(v);
-        else
+        if constexpr (std::is_same<DT, ST>::value)
             o = v;
-        dst[r * dst_pitch + c] = o;
+        else
+            o = from_float<DT>(to_float(v));
+        dst[r * dst_row + c * dst_col] = o;
     }
 }
 

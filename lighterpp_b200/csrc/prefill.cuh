@@ -36,16 +36,26 @@ constexpr int kPfMaxSplits = 8;
 constexpr int kPfRingBytes = 192 * 1024;
 constexpr int kPfSmemBytes = 1024 /*barriers*/ + 1024 /*alignment slack*/ + kPfRingBytes;
 
-enum PfEpi : int { kPfQkv = 0, kPfResid = 1, kPfSwiglu = 2 };
+enum PfEpi : int {
+    kPfQkv = 0,
+    kPfResid = 1,
+    kPfSwiglu = 2,
+    kPfStore = 3,         // logits, or partial sums for a finishing kernel
+    kPfLatentQuery = 4,   // latent attention: a head's query in the latent space -> FP16 query rows
+    kPfLatentValue = 5    // latent attention: a head's value times its gate -> hi + lo operand
+};
 
-// An activation x is handed to the tensor cores as two FP16 numbers, hi = fp16(x) and lo = fp16(x - hi): the MMA
-// accumulates W.hi + W.lo in FP32, which keeps about 22 bits of x, so the batched pass carries FP32 activations
-// through FP16-operand MMAs like the token loop carries them through its FP32 arithmetic.  Every activation buffer
-// holds the hi plane [kPrefillTokens][cols] followed by the lo plane; one 4-D tensor map covers both.
-__device__ __forceinline__ void split_half(float x, __half& hi, __half& lo) {
-    hi = __float2half_rn(x);
-    lo = __float2half_rn(x - __half2float(hi));
+// An activation x is handed to the tensor cores as two numbers of the weights' 16-bit type, hi = round(x) and
+// lo = round(x - hi): the MMA accumulates W.hi + W.lo in FP32, which keeps about 22 bits of x with FP16 (17 with BF16),
+// so the batched pass carries FP32 activations through 16-bit-operand MMAs like the token loop carries them through its
+// FP32 arithmetic.  Every activation buffer holds the hi plane [kPrefillTokens][cols] followed by the lo plane; one
+// 4-D tensor map covers both.
+template <typename T>
+__device__ __forceinline__ void split_pair(float x, T& hi, T& lo) {
+    hi = from_float<T>(x);
+    lo = from_float<T>(x - to_float(hi));
 }
+__device__ __forceinline__ void split_half(float x, __half& hi, __half& lo) { split_pair(x, hi, lo); }
 
 struct PrefillGemmArgs {
     int n_rows, K;        // rows of the weight matrix, inputs per row
@@ -59,8 +69,23 @@ struct PrefillGemmArgs {
     // part[split][t][row] and the next kernel (prefill_norm_kernel) adds them to x in split order
     float* x;
     float* part;
-    // kPfSwiglu: hb[t][row/2] = silu(gate) * up   (rows interleaved gate, up; hb: FP16 [kPrefillTokens][n_rows/2])
-    __half* hb;
+    int x_pitch;          // row pitch of x and part (kPfResid)
+    // kPfSwiglu: hb[t][row/2] = act(gate) * up   (rows interleaved gate, up; hb: hi and lo plane [kPrefillTokens][hb_pitch])
+    void* hb;
+    int hb_pitch;
+    int act;
+    // kPfStore: out[split][t][row], rows of out_pitch floats
+    float* out;
+    int out_pitch;
+    // Grouped weights (heads): `groups` matrices of n_rows rows each, group_stride rows apart in the tensor map; group g
+    // multiplies the K inputs that start at 64-input piece g * group_pieces of the activations.  0 = one matrix.
+    int groups, group_stride, group_pieces;
+    // kPfLatentQuery: query rows (token * groups + group) of lat_pitch FP16 elements
+    __half* lat_query;
+    int lat_pitch;
+    // kPfLatentValue: column group * n_valid + row of hb (rows below n_valid), times gate[t][group]
+    const float* gate;
+    int n_valid;
     // kPfQkv: rows are q | k | v; RoPE on q and k, q -> FP32 [kPrefillTokens][q_rows], k/v -> cache at start_pos + t
     float* q;
     int q_rows, kv_rows, head_size, seq_len;
@@ -86,6 +111,9 @@ __device__ __forceinline__ void mma_f16_16816(float (&d)[4], uint32_t a0, uint32
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void ldmatrix_x2(uint32_t addr, uint32_t& r0, uint32_t& r1) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
 }
 __device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
@@ -146,9 +174,13 @@ constexpr int kUmmaThreads = (2 + kUmmaEpiWarps) * 32;
 constexpr int kUmmaN = 2 * kPrefillTokens;                         // MMA N: the 64 hi rows and the 64 lo rows of the activation tile
 constexpr int kUmmaAccCols = kUmmaN;                               // FP32 columns of one accumulator: W.hi | W.lo
 constexpr int kUmmaTmemCols = 2 * kUmmaAccCols;                    // power of two >= 32
-// Instruction descriptor: D = F32 (bits 4-5 = 1), A = B = F16 (0), both K-major (bits 15, 16 = 0),
-// N / 8 in bits 17-22, M / 16 in bits 24-28.
-constexpr uint32_t kUmmaIdesc = (1u << 4) | ((uint32_t)(kUmmaN >> 3) << 17) | ((uint32_t)(kUmmaM >> 4) << 24);
+// Instruction descriptor: D = F32 (bits 4-5 = 1), A and B of the same 16-bit type (bits 7-9 and 10-12: 0 = FP16,
+// 1 = BF16), both K-major (bits 15, 16 = 0), N / 8 in bits 17-22, M / 16 in bits 24-28.
+template <typename T>
+__host__ __device__ constexpr uint32_t umma_idesc() {
+    return (1u << 4) | (std::is_same<T, __nv_bfloat16>::value ? (1u << 7) | (1u << 10) : 0u) | ((uint32_t)(kUmmaN >> 3) << 17) |
+           ((uint32_t)(kUmmaM >> 4) << 24);
+}
 
 // Shared-memory matrix descriptor of a K-major operand tile with the 128-byte swizzle: start address / 16 in bits
 // 0-13, leading byte offset (unused for swizzled K-major, set to 1) in bits 16-29, stride between 8-row groups
@@ -198,44 +230,66 @@ __device__ __forceinline__ void tc_ld32(uint32_t taddr, float (&v)[32]) {
 // Epilogue of one thread: weight row `row`, tokens t0 .. t0+31 with the sums v[0..31].  Lanes are consecutive rows,
 // so for a fixed token a warp's stores are contiguous; the partner row (row ^ 1) of the rotation and SwiGLU pairs
 // is the neighbouring lane.  The rotation rounds like pf_qkv_store.
-template <int EPI>
-__device__ __forceinline__ void umma_epilogue(const PrefillGemmArgs& a, int split, int row, int t0, const float (&v)[32],
+template <typename T, int EPI>
+__device__ __forceinline__ void umma_epilogue(const PrefillGemmArgs& a, int split, int group, int row, int t0, const float (&v)[32],
                                               int lane) {
     const bool row_ok = row < a.n_rows;
     const int nt = min(32, a.n_tokens - t0);  // valid tokens of this half (may be <= 0)
     if constexpr (EPI == kPfResid) {
         if (a.splits > 1) {
-            float* p = a.part + ((size_t)split * kPrefillTokens + t0) * a.n_rows + row;
+            float* p = a.part + ((size_t)split * kPrefillTokens + t0) * a.x_pitch + row;
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-                if (row_ok && i < nt) p[(size_t)i * a.n_rows] = v[i];
+                if (row_ok && i < nt) p[(size_t)i * a.x_pitch] = v[i];
         } else {
-            float* p = a.x + (size_t)t0 * a.n_rows + row;
+            float* p = a.x + (size_t)t0 * a.x_pitch + row;
             float old[32];
 #pragma unroll
-            for (int i = 0; i < 32; ++i) old[i] = (row_ok && i < nt) ? p[(size_t)i * a.n_rows] : 0.f;
+            for (int i = 0; i < 32; ++i) old[i] = (row_ok && i < nt) ? p[(size_t)i * a.x_pitch] : 0.f;
 #pragma unroll
             for (int i = 0; i < 32; ++i)
-                if (row_ok && i < nt) p[(size_t)i * a.n_rows] = old[i] + v[i];  // x += W.xb (src/model.cpp:232, 239)
+                if (row_ok && i < nt) p[(size_t)i * a.x_pitch] = old[i] + v[i];  // x += W.xb (src/model.cpp:232, 239)
         }
+    } else if constexpr (EPI == kPfStore) {
+        float* p = a.out + ((size_t)split * kPrefillTokens + t0) * a.out_pitch + row;
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+            if (row_ok && i < nt) p[(size_t)i * a.out_pitch] = v[i];
+    } else if constexpr (EPI == kPfLatentQuery) {
+        __half* p = a.lat_query + ((size_t)t0 * a.groups + group) * a.lat_pitch + row;
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+            if (row_ok && i < nt) p[(size_t)i * a.groups * a.lat_pitch] = __float2half_rn(v[i]);
+    } else if constexpr (EPI == kPfLatentValue) {
+        T* p = reinterpret_cast<T*>(a.hb) + (size_t)t0 * a.hb_pitch + (size_t)group * a.n_valid + row;
+        const float* gate = a.gate + (size_t)t0 * a.groups + group;
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+            if (row < a.n_valid && i < nt) {
+                T hi, lo;
+                split_pair(v[i] * gate[(size_t)i * a.groups], hi, lo);
+                p[(size_t)i * a.hb_pitch] = hi;
+                p[(size_t)(kPrefillTokens + i) * a.hb_pitch] = lo;
+            }
     } else if constexpr (EPI == kPfSwiglu) {
         // rows interleaved (gate_i, up_i): the even lane finishes tokens 0..15 of the pair, the odd lane tokens 16..31;
         // each sends the partner the half it does not finish itself.  hb = (h1*sigmoid(h1))*h3 (src/ops.cpp:78-87)
-        // with the fast exponential and division (relative error ~1e-6, far below the FP16 weights' own rounding).
+        // with the fast exponential and division (relative error ~1e-6, far below the 16-bit weights' own rounding), or
+        // the tanh form of GELU in place of h1*sigmoid(h1).
         const bool even = (lane & 1) == 0;
-        __half* hb = a.hb + (size_t)(t0 + (even ? 0 : 16)) * (a.n_rows >> 1) + (row >> 1);
+        T* hb = reinterpret_cast<T*>(a.hb) + (size_t)(t0 + (even ? 0 : 16)) * a.hb_pitch + (row >> 1);
         const int nt_mine = nt - (even ? 0 : 16);
 #pragma unroll
         for (int k = 0; k < 16; ++k) {
             const float keep = even ? v[k] : v[k + 16], send = even ? v[k + 16] : v[k];
             const float recv = __shfl_xor_sync(0xffffffffu, send, 1);
             const float g = even ? keep : recv, u = even ? recv : keep;
-            const float r = __fdividef(g, 1.0f + __expf(-g)) * u;
-            __half hi, lo;
-            split_half(r, hi, lo);
+            const float r = __fdividef(g, 1.0f + __expf(-act_gate_arg(a.act, g))) * u;
+            T hi, lo;
+            split_pair(r, hi, lo);
             if (row_ok && k < nt_mine) {
-                hb[(size_t)k * (a.n_rows >> 1)] = hi;
-                hb[(size_t)(kPrefillTokens + k) * (a.n_rows >> 1)] = lo;
+                hb[(size_t)k * a.hb_pitch] = hi;
+                hb[(size_t)(kPrefillTokens + k) * a.hb_pitch] = lo;
             }
         }
     } else if (a.splits > 1) {  // kPfQkv cut along K: partial sums, finished by prefill_qkv_finish_kernel
@@ -293,7 +347,7 @@ __device__ unsigned long long g_pf_trace[160][48];
     } while (0)
 #endif
 
-template <int EPI>
+template <typename T, int EPI>
 static __global__ void __launch_bounds__(kUmmaThreads, 1) prefill_gemm_umma_kernel(const __grid_constant__ CUtensorMap w_map,
                                                                                    const __grid_constant__ CUtensorMap x_map,
                                                                                    const PrefillGemmArgs a) {
@@ -308,7 +362,8 @@ static __global__ void __launch_bounds__(kUmmaThreads, 1) prefill_gemm_umma_kern
     const uint32_t ring = (smem_u32(smem) + 1024u + 1023u) & ~1023u;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int unit = blockIdx.x, n_units = gridDim.x;
-    const int n_tiles = (a.n_rows + kUmmaM - 1) / kUmmaM;  // items along the rows
+    const int group_tiles = (a.n_rows + kUmmaM - 1) / kUmmaM;  // row tiles of one matrix
+    const int n_tiles = group_tiles * max(1, a.groups);        // items along the rows
     const int n_kc = (a.K + kPfKc - 1) / kPfKc;
     const int S = a.splits;
     const int n_items = n_tiles * S;
@@ -345,12 +400,13 @@ static __global__ void __launch_bounds__(kUmmaThreads, 1) prefill_gemm_umma_kern
             int early = 0;  // stages whose weights are already in flight
             // one copy per operand and stage: both 64-input weight sub-tiles / the four activation sub-tiles (hi, lo)
             auto load_w = [&](uint32_t dst, int kc, int wrow, int sl) { tma_load_3d(dst, &w_map, 0, wrow, 2 * kc, smem_u32(&full[sl])); };
-            auto load_x = [&](uint32_t dst, int kc, int sl) { tma_load_4d(dst, &x_map, 0, 0, 0, 2 * kc, smem_u32(&full[sl])); };
+            auto load_x = [&](uint32_t dst, int piece, int sl) { tma_load_4d(dst, &x_map, 0, 0, 0, piece, smem_u32(&full[sl])); };
             auto expect = [&](int sl) { mbar_arrive_expect_tx(&full[sl], kStage); };
             for (int item = unit; item < n_items && ok; item += n_units) {
                 const int tile = item / S, split = item - tile * S;
                 const int kc0 = (split * n_kc) / S, kc1 = ((split + 1) * n_kc) / S;
-                const int wrow = a.row0 + tile * kUmmaM;
+                const int group = tile / group_tiles, piece0 = group * a.group_pieces;
+                const int wrow = a.row0 + group * a.group_stride + (tile - group * group_tiles) * kUmmaM;
                 if (!waited) {
                     early = min(kc1 - kc0, kStages);
                     for (int i = 0; i < early; ++i) {
@@ -376,7 +432,7 @@ static __global__ void __launch_bounds__(kUmmaThreads, 1) prefill_gemm_umma_kern
                         load_w(dst, kc, wrow, slot);
                     }
                     PF_STAMP(2 + kc - kc0);
-                    load_x(dst + 2 * kUmmaSubW, kc, slot);
+                    load_x(dst + 2 * kUmmaSubW, piece0 + 2 * kc, slot);
                     if (++slot == kStages) {
                         slot = 0;
                         ++pass;
@@ -419,7 +475,7 @@ static __global__ void __launch_bounds__(kUmmaThreads, 1) prefill_gemm_umma_kern
 #pragma unroll
                         for (int ks = 0; ks < 4; ++ks) {  // 16 inputs = 32 bytes along the swizzled row per step
                             const uint32_t acc = (kc > kc0 || sub > 0 || ks > 0) ? 1u : 0u;
-                            tc_mma_f16(d_tmem, umma_desc(wt + ks * 32), umma_desc(xt + ks * 32), kUmmaIdesc, acc);
+                            tc_mma_f16(d_tmem, umma_desc(wt + ks * 32), umma_desc(xt + ks * 32), umma_idesc<T>(), acc);
                         }
                     }
                     tc_commit(&empty[slot]);  // arrives once the MMAs issued so far have read this stage
@@ -455,7 +511,8 @@ static __global__ void __launch_bounds__(kUmmaThreads, 1) prefill_gemm_umma_kern
             __syncwarp();
             if (lane == 0) mbar_arrive(&acc_empty[b]);
             if (tid == 64) PF_STAMP(35);
-            umma_epilogue<EPI>(a, split, tile * kUmmaM + quarter * 32 + lane, half * 32, v, lane);
+            const int group = tile / group_tiles;
+            umma_epilogue<T, EPI>(a, split, group, (tile - group * group_tiles) * kUmmaM + quarter * 32 + lane, half * 32, v, lane);
             if (tid == 64) PF_STAMP(36);
         }
     }
@@ -498,96 +555,138 @@ static __global__ void __launch_bounds__(256) prefill_qkv_finish_kernel(const Pr
     pf_qkv_store(a, row + 1, t, v.y, v.x);
 }
 
-// Rows of the residual stream -> RMS-normalised FP16 rows (MMA operands).  Layer 0 takes the embedding rows of
-// the prompt tokens and also writes them out as the FP32 residual stream.  grid: tokens.
+// Rows of the residual stream -> normalised rows (hi + lo MMA operands): RMSNorm, or LayerNorm when a bias is given.
+// Layer 0 takes the embedding rows of the prompt tokens and also writes them out as the FP32 residual stream.  With a
+// row list, block i takes row rows[i] (the positions whose logits are wanted).  D is the row pitch; the statistics cover
+// the first norm_n inputs, the rest is zero padding with zero weights.  grid: rows.
 constexpr int kPfNormThreads = 512;
-// Only the weights (emb, norm_w) are marked read-only: a pointer to data the preceding kernel produced must not be
-// `const __restrict__`, or its loads become invariant loads that the compiler may move above the dependency wait.
-static __global__ void __launch_bounds__(kPfNormThreads) prefill_norm_kernel(float* x, const int* tokens,
-                                                                            const __half* __restrict__ emb, int vocab,
-                                                                            const float* __restrict__ norm_w, __half* out,
-                                                                            int D, int n_tokens, const float* part,
-                                                                            int splits, StepState* st) {
-    __shared__ float red[kPfNormThreads / 32];
-    pdl_launch_dependents();
-    pdl_wait();
-    const int t = blockIdx.x, tid = threadIdx.x;
-    float4* xr = reinterpret_cast<float4*>(x + (size_t)t * D);
-    const int nv4 = D >> 2;  // D is a multiple of 8
-    constexpr int kMaxPer = 4;  // float4 per thread kept in registers for the second pass: rows up to 8192 wide
-    float4 v[kMaxPer];
-    int tok = 0;
-    if (emb) {
-        tok = tokens[t];
-        if (tok < 0 || tok >= vocab) {
-            if (tid == 0) atomicOr(&st->status, kStatusBadToken);
-            tok = 0;
-        }
-    }
-    const bool add_parts = !emb && splits > 1;
-    float ss = 0.f;
-#pragma unroll
-    for (int k = 0; k < kMaxPer; ++k) {
-        const int i = tid + k * kPfNormThreads;
-        if (i < nv4) {
-            // every load of this piece (the row and all partial sums) is issued before the first is used
-            float4 p[kPfMaxSplits];
-            if (emb) {
-                const uint2 h = *reinterpret_cast<const uint2*>(emb + (size_t)tok * D + 4 * (size_t)i);
-                const float2 lo = half2_bits_to_float2(h.x), hi = half2_bits_to_float2(h.y);
-                v[k] = make_float4(lo.x, lo.y, hi.x, hi.y);
-            } else {
-                v[k] = xr[i];
-            }
-            if (add_parts) {
-#pragma unroll
-                for (int s0 = 0; s0 < kPfMaxSplits; ++s0)
-                    if (s0 < splits) p[s0] = reinterpret_cast<const float4*>(part + ((size_t)s0 * kPrefillTokens + t) * D)[i];
-                // x += p_0 + p_1 + ... in range order
-#pragma unroll
-                for (int s0 = 0; s0 < kPfMaxSplits; ++s0)
-                    if (s0 < splits) {
-                        v[k].x += p[s0].x; v[k].y += p[s0].y; v[k].z += p[s0].z; v[k].w += p[s0].w;
-                    }
-            }
-            if (emb || add_parts) xr[i] = v[k];  // the residual stream as the next residual GEMM reads it
-            ss = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, ss))));
-        }
-    }
-    // rows wider than kMaxPer * kPfNormThreads * 4: the rest without register caching
-    for (int i = tid + kMaxPer * kPfNormThreads; i < nv4; i += kPfNormThreads) {
-        float4 w;
-        if (emb) {
-            const uint2 h = *reinterpret_cast<const uint2*>(emb + (size_t)tok * D + 4 * (size_t)i);
-            const float2 lo = half2_bits_to_float2(h.x), hi = half2_bits_to_float2(h.y);
-            w = make_float4(lo.x, lo.y, hi.x, hi.y);
-        } else {
-            w = xr[i];
-        }
-        if (add_parts)
-            for (int s0 = 0; s0 < splits; ++s0) {
-                const float4 q = reinterpret_cast<const float4*>(part + ((size_t)s0 * kPrefillTokens + t) * D)[i];
-                w.x += q.x; w.y += q.y; w.z += q.z; w.w += q.w;
-            }
-        if (emb || add_parts) xr[i] = w;
-        ss = fmaf(w.x, w.x, fmaf(w.y, w.y, fmaf(w.z, w.z, fmaf(w.w, w.w, ss))));
-    }
-    ss = warp_sum(ss);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
+struct PrefillNormArgs {
+    float* x;            // [kPrefillTokens][D]
+    const int* tokens;   // with emb
+    const void* emb;     // [vocab][D], nullptr = the rows of x
+    int vocab;
+    const int* rows;     // nullptr = block i takes row i
+    const float* norm_w;
+    const float* norm_b; // nullptr = RMSNorm
+    float norm_eps;
+    int norm_n;
+    void* out;           // [2 planes][kPrefillTokens][D]
+    int D;
+    const float* part;   // [splits][kPrefillTokens][D], added to x in order when splits > 1
+    int splits;
+    StepState* st;
+};
+__device__ __forceinline__ float norm_block_sum(float v, float* red, int tid) {
+    v = warp_sum(v);
+    if ((tid & 31) == 0) red[tid >> 5] = v;
     __syncthreads();
     float tot = 0.f;
 #pragma unroll
     for (int k = 0; k < kPfNormThreads / 32; ++k) tot += red[k];
-    const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, (float)D), 1e-5f)));
-    auto emit = [&](int i, const float4& xv) {
-        const float4 w = __ldg(reinterpret_cast<const float4*>(norm_w) + i);
-        const float y[4] = {__fmul_rn(__fmul_rn(xv.x, scale), w.x), __fmul_rn(__fmul_rn(xv.y, scale), w.y),
-                            __fmul_rn(__fmul_rn(xv.z, scale), w.z), __fmul_rn(__fmul_rn(xv.w, scale), w.w)};
-        __align__(8) __half hi[4], lo[4];
+    return tot;
+}
+// Only the weights (emb, norm_w, norm_b) are loaded as read-only data: a load of what the preceding kernel produced must
+// not become an invariant one, which the compiler may move above the dependency wait.
+template <typename T>
+static __global__ void __launch_bounds__(kPfNormThreads) prefill_norm_kernel(const PrefillNormArgs a) {
+    __shared__ float red[2][kPfNormThreads / 32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int tid = threadIdx.x, D = a.D, splits = a.splits;
+    const int t = a.rows ? *reinterpret_cast<const volatile int*>(a.rows + blockIdx.x) : (int)blockIdx.x;
+    float4* xr = reinterpret_cast<float4*>(a.x + (size_t)t * D);
+    const int nv4 = D >> 2;  // D is a multiple of 8
+    constexpr int kMaxPer = 4;  // float4 per thread kept in registers for the second pass: rows up to 8192 wide
+    float4 v[kMaxPer];
+    int tok = 0;
+    if (a.emb) {
+        tok = *reinterpret_cast<const volatile int*>(a.tokens + t);
+        if (tok < 0 || tok >= a.vocab) {
+            if (tid == 0) atomicOr(&a.st->status, kStatusBadToken);
+            tok = 0;
+        }
+    }
+    const bool add_parts = !a.emb && splits > 1;
+    // one piece of the row: the embedding, or the residual plus all partial sums in range order (every load issued
+    // before the first is used)
+    auto fetch = [&](int i) -> float4 {
+        float4 w, p[kPfMaxSplits];
+        if (a.emb) {
+            const uint2 h = __ldg(reinterpret_cast<const uint2*>(reinterpret_cast<const T*>(a.emb) + (size_t)tok * D + 4 * (size_t)i));
+            const float2 lo = unpack2<T>(h.x), hi = unpack2<T>(h.y);
+            w = make_float4(lo.x, lo.y, hi.x, hi.y);
+        } else {
+            w = xr[i];
+        }
+        if (add_parts) {
 #pragma unroll
-        for (int c = 0; c < 4; ++c) split_half(y[c], hi[c], lo[c]);
-        *reinterpret_cast<uint2*>(out + (size_t)t * D + 4 * (size_t)i) = *reinterpret_cast<const uint2*>(hi);
-        *reinterpret_cast<uint2*>(out + (size_t)(kPrefillTokens + t) * D + 4 * (size_t)i) = *reinterpret_cast<const uint2*>(lo);
+            for (int s0 = 0; s0 < kPfMaxSplits; ++s0)
+                if (s0 < splits) p[s0] = reinterpret_cast<const float4*>(a.part + ((size_t)s0 * kPrefillTokens + t) * D)[i];
+#pragma unroll
+            for (int s0 = 0; s0 < kPfMaxSplits; ++s0)
+                if (s0 < splits) {
+                    w.x += p[s0].x; w.y += p[s0].y; w.z += p[s0].z; w.w += p[s0].w;
+                }
+        }
+        if (a.emb || add_parts) xr[i] = w;  // the residual stream as the next residual GEMM reads it
+        return w;
+    };
+    const bool ln = a.norm_b != nullptr;
+    const float n = (float)a.norm_n;
+    float ss = 0.f;  // RMSNorm: sum of squares; LayerNorm: sum
+    auto first = [&](const float4& w) {
+        ss = ln ? ss + ((w.x + w.y) + (w.z + w.w)) : fmaf(w.x, w.x, fmaf(w.y, w.y, fmaf(w.z, w.z, fmaf(w.w, w.w, ss))));
+    };
+#pragma unroll
+    for (int k = 0; k < kMaxPer; ++k) {
+        const int i = tid + k * kPfNormThreads;
+        if (i < nv4) {
+            v[k] = fetch(i);
+            first(v[k]);
+        }
+    }
+    // rows wider than kMaxPer * kPfNormThreads * 4: the rest without register caching
+    for (int i = tid + kMaxPer * kPfNormThreads; i < nv4; i += kPfNormThreads) first(fetch(i));
+    float tot = norm_block_sum(ss, red[0], tid), mean = 0.f;
+    if (ln) {
+        mean = __fdiv_rn(tot, n);
+        float q = 0.f;
+        auto second = [&](int i, const float4& w) {
+            const float d[4] = {w.x - mean, w.y - mean, w.z - mean, w.w - mean};
+#pragma unroll
+            for (int c = 0; c < 4; ++c)
+                if (4 * i + c < a.norm_n) q = fmaf(d[c], d[c], q);
+        };
+#pragma unroll
+        for (int k = 0; k < kMaxPer; ++k) {
+            const int i = tid + k * kPfNormThreads;
+            if (i < nv4) second(i, v[k]);
+        }
+        for (int i = tid + kMaxPer * kPfNormThreads; i < nv4; i += kPfNormThreads) second(i, xr[i]);
+        tot = norm_block_sum(q, red[1], tid);
+    }
+    const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, n), a.norm_eps)));
+    T* out = reinterpret_cast<T*>(a.out) + (size_t)blockIdx.x * D;
+    auto emit = [&](int i, const float4& xv) {
+        const float4 w = __ldg(reinterpret_cast<const float4*>(a.norm_w) + i);
+        float y[4];
+        if (ln) {
+            const float4 b = __ldg(reinterpret_cast<const float4*>(a.norm_b) + i);
+            y[0] = fmaf(__fmul_rn(xv.x - mean, scale), w.x, b.x);
+            y[1] = fmaf(__fmul_rn(xv.y - mean, scale), w.y, b.y);
+            y[2] = fmaf(__fmul_rn(xv.z - mean, scale), w.z, b.z);
+            y[3] = fmaf(__fmul_rn(xv.w - mean, scale), w.w, b.w);
+        } else {
+            y[0] = __fmul_rn(__fmul_rn(xv.x, scale), w.x);
+            y[1] = __fmul_rn(__fmul_rn(xv.y, scale), w.y);
+            y[2] = __fmul_rn(__fmul_rn(xv.z, scale), w.z);
+            y[3] = __fmul_rn(__fmul_rn(xv.w, scale), w.w);
+        }
+        __align__(8) T hi[4], lo[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) split_pair(y[c], hi[c], lo[c]);
+        *reinterpret_cast<uint2*>(out + 4 * (size_t)i) = *reinterpret_cast<const uint2*>(hi);
+        *reinterpret_cast<uint2*>(out + (size_t)kPrefillTokens * D + 4 * (size_t)i) = *reinterpret_cast<const uint2*>(lo);
     };
 #pragma unroll
     for (int k = 0; k < kMaxPer; ++k) {

@@ -13,27 +13,31 @@ from typing import Dict, Iterable, Optional, Sequence, Tuple
 
 import numpy as np
 
-from .formats import ModelConfig
+from .formats import LayeredConfig, ModelConfig
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "liblpp_b200.so")
 
-LPP_F32, LPP_F16 = 0, 1
+LPP_F32, LPP_F16, LPP_BF16 = 0, 1, 2
 MEM_HOST, MEM_DEVICE = 0, 1
 FLAG_GEMV_LDG, FLAG_NO_PDL, FLAG_NO_GRAPH, FLAG_FAST_SAMPLER = 1, 2, 4, 16
 TENSOR_IDS = {"tok_emb": 0, "rms_att": 1, "wq": 2, "wk": 3, "wv": 4, "wo": 5, "rms_ffn": 6, "w1": 7, "w2": 8,
-              "w3": 9, "rms_final": 10, "w_cls": 11}
-_UNSTACKED = ("tok_emb", "rms_final", "w_cls")
+              "w3": 9, "rms_final": 10, "w_cls": 11,
+              # models described layer by layer
+              "norm1_b": 12, "norm2_b": 13, "norm_final_b": 14, "lat_q": 15, "lat_dkv": 16, "lat_norm": 17, "lat_uk": 18,
+              "lat_uv": 19, "lat_g": 20}
+_UNSTACKED = ("tok_emb", "rms_final", "w_cls", "norm_final_b")
 TP_HANDLE_BYTES = 64
-FLAG_TP_NCCL, FLAG_TP_LOCAL, FLAG_NO_PREFILL_GEMM = 32, 64, 128
+FLAG_TP_NCCL, FLAG_TP_LOCAL, FLAG_NO_PREFILL_GEMM, FLAG_LATENT_CUDA_CORES = 32, 64, 128, 256
+MIXERS, NORMS, ACTIVATIONS = {"latent": 1}, {"rms": 0, "layer": 1}, {"silu": 0, "gelu_tanh": 1}
 KINDS = ["qkv_gemv", "attention", "oproj_gemv", "gateup_gemv", "down_gemv", "lmhead_gemv", "sampler", "allreduce",
-         "reserved8", "reserved9"]
+         "latent_query_gemv", "latent_value_gemv"]
 
 # every symbol include/lpp_b200.h declares; tests check the built library exports all of them
 EXPORTS = [
-    "lpp_engine_create", "lpp_engine_destroy", "lpp_nccl_unique_id", "lpp_upload_tensor", "lpp_finalize",
-    "lpp_step", "lpp_step_logits", "lpp_decode", "lpp_prefill", "lpp_sample_logits", "lpp_kv_prefill", "lpp_kv_read",
-    "lpp_kv_index", "lpp_strerror", "lpp_last_error", "lpp_engine_stream", "lpp_kernels_per_step",
+    "lpp_engine_create", "lpp_engine_create_layers", "lpp_engine_destroy", "lpp_nccl_unique_id", "lpp_upload_tensor", "lpp_finalize",
+    "lpp_step", "lpp_step_logits", "lpp_decode", "lpp_prefill", "lpp_extend", "lpp_sample_logits", "lpp_kv_prefill", "lpp_kv_read",
+    "lpp_latent_read", "lpp_kv_index", "lpp_strerror", "lpp_last_error", "lpp_engine_stream", "lpp_kernels_per_step",
     "lpp_step_bytes", "lpp_profile_step", "lpp_profile_kind", "lpp_tp_export", "lpp_tp_connect", "lpp_op_convert_f32_to_f16", "lpp_op_gemv", "lpp_op_rmsnorm",
     "lpp_op_rope", "lpp_op_swiglu", "lpp_op_softmax_multihead", "lpp_op_scale_multihead",
     "lpp_op_aggregation_multihead", "lpp_op_residual_add", "lpp_op_scatter_kv", "lpp_op_multihead_gemv",
@@ -55,6 +59,19 @@ class Config(C.Structure):
                 ("ring_kb", C.c_int32), ("attn_splits", C.c_int32), ("wait_ms", C.c_int32), ("tp_wait_ms", C.c_int32)]
 
 
+class LayerDesc(C.Structure):
+    _fields_ = [("mixer", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32), ("rot_dim", C.c_int32), ("vdim", C.c_int32),
+                ("kv_rank", C.c_int32), ("window", C.c_int32), ("scale", C.c_float), ("rot_dims", C.c_int32),
+                ("rot_base", C.c_double), ("yarn_factor", C.c_double), ("yarn_original", C.c_double),
+                ("yarn_fast", C.c_double), ("yarn_slow", C.c_double), ("ff", C.c_int32), ("act", C.c_int32)]
+
+
+class ModelDesc(C.Structure):
+    _fields_ = [("dim", C.c_int32), ("vocab_size", C.c_int32), ("seq_len", C.c_int32), ("n_layers", C.c_int32),
+                ("norm", C.c_int32), ("norm_eps", C.c_float), ("weight_dtype", C.c_int32), ("kv_dtype", C.c_int32),
+                ("device", C.c_int32), ("flags", C.c_uint32), ("ring_kb", C.c_int32), ("wait_ms", C.c_int32)]
+
+
 class SampleParams(C.Structure):
     _fields_ = [("temperature", C.c_float), ("penalty", C.c_float)]
 
@@ -74,6 +91,7 @@ def load_library() -> C.CDLL:
     lib = C.CDLL(LIB_PATH)
     vp, ip, fp = C.c_void_p, C.POINTER(C.c_int), C.POINTER(C.c_float)
     lib.lpp_engine_create.argtypes = [C.POINTER(Config), vp, C.POINTER(vp)]
+    lib.lpp_engine_create_layers.argtypes = [C.POINTER(ModelDesc), C.POINTER(LayerDesc), C.POINTER(vp)]
     lib.lpp_engine_destroy.argtypes = [vp]
     lib.lpp_nccl_unique_id.argtypes = [vp]
     lib.lpp_upload_tensor.argtypes = [vp, C.c_int, C.c_int, vp, C.c_int, C.c_int]
@@ -84,6 +102,8 @@ def load_library() -> C.CDLL:
                                fp]
     lib.lpp_sample_logits.argtypes = [vp, fp, C.POINTER(SampleParams), ip, C.c_int, C.c_float, ip]
     lib.lpp_prefill.argtypes = [vp, ip, C.c_int, C.c_int, fp]
+    lib.lpp_extend.argtypes = [vp, ip, C.c_int, C.c_int, ip, C.c_int, fp, fp]
+    lib.lpp_latent_read.argtypes = [vp, C.c_int, C.c_int, fp]
     lib.lpp_kv_prefill.argtypes = [vp, C.c_int, vp, vp, C.c_int, C.c_int, C.c_int]
     lib.lpp_kv_read.argtypes = [vp, C.c_int, C.c_int, C.c_int, fp, fp]
     lib.lpp_kv_index.argtypes = [vp, C.c_int, C.c_int, C.c_int, C.c_int]
@@ -121,18 +141,28 @@ def _np_dtype_code(a: np.ndarray) -> int:
         return LPP_F32
     if a.dtype == np.float16:
         return LPP_F16
+    if a.dtype == np.uint16:  # numpy has no bfloat16: its bit patterns travel as uint16
+        return LPP_BF16
     raise TypeError(f"unsupported dtype {a.dtype}")
 
 
 class Engine:
     """One tensor-parallel rank of the decode engine on one GPU."""
 
-    def __init__(self, cfg: ModelConfig, weight_dtype: str = "f16", kv_dtype: str = "f16", *, device: int = 0,
+    def __init__(self, cfg, weight_dtype: str = "f16", kv_dtype: str = "f16", *, device: int = 0,
                  tp_rank: int = 0, tp_size: int = 1, nccl_id: Optional[bytes] = None, flags: int = 0,
                  ring_kb: int = 0, attn_splits: int = 0, wait_ms: int = 0, tp_wait_ms: int = 0):
+        """``cfg``: a ``ModelConfig`` (the reference's architecture) or a ``LayeredConfig`` (a list of layers)."""
         self.lib = load_library()
         self.cfg = cfg
-        self.weight_dtype = {"f32": LPP_F32, "f16": LPP_F16}[weight_dtype]
+        self.weight_dtype = {"f32": LPP_F32, "f16": LPP_F16, "bf16": LPP_BF16}[weight_dtype]
+        self.kv_dtype = {"f32": LPP_F32, "f16": LPP_F16}[kv_dtype]
+        if isinstance(cfg, LayeredConfig):
+            if tp_size != 1:
+                raise ValueError("models described layer by layer run on one GPU")
+            self.tp_rank, self.tp_size = 0, 1
+            self._create_layers(cfg, device, flags, ring_kb, wait_ms)
+            return
         c = Config(cfg.dim, cfg.hidden_dim, cfg.n_layers, cfg.n_heads, cfg.n_kv_heads, cfg.vocab_size, cfg.seq_len,
                    cfg.rope_base, self.weight_dtype, {"f32": LPP_F32, "f16": LPP_F16}[kv_dtype], tp_rank, tp_size,
                    device, flags, ring_kb, attn_splits, wait_ms, tp_wait_ms)
@@ -140,6 +170,23 @@ class Engine:
         h = C.c_void_p()
         idbuf = C.create_string_buffer(nccl_id, 128) if nccl_id is not None else None
         _check(self.lib.lpp_engine_create(C.byref(c), idbuf, C.byref(h)), "lpp_engine_create")
+        self.h = h
+
+    def _create_layers(self, cfg: LayeredConfig, device: int, flags: int, ring_kb: int, wait_ms: int) -> None:
+        layers = (LayerDesc * len(cfg.layers))()
+        for d, y in zip(layers, cfg.layers):
+            m, r = y.mixer, y.mixer.rotation
+            d.mixer = MIXERS["latent"]
+            d.heads, d.dim, d.rot_dim, d.vdim, d.kv_rank = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank
+            d.window, d.scale = m.window, m.scale
+            d.rot_dims, d.rot_base = r.dims, r.base
+            if r.yarn is not None:
+                d.yarn_factor, d.yarn_original, d.yarn_fast, d.yarn_slow = r.yarn.factor, r.yarn.original, r.yarn.fast, r.yarn.slow
+            d.ff, d.act = y.ff, ACTIVATIONS[y.act]
+        m = ModelDesc(cfg.dim, cfg.vocab_size, cfg.seq_len, len(cfg.layers), NORMS[cfg.norm], cfg.norm_eps,
+                      self.weight_dtype, self.kv_dtype, device, flags, ring_kb, wait_ms)
+        h = C.c_void_p()
+        _check(self.lib.lpp_engine_create_layers(C.byref(m), layers, C.byref(h)), "lpp_engine_create_layers")
         self.h = h
 
     # ---- weights -------------------------------------------------------------------------------
@@ -153,7 +200,7 @@ class Engine:
         else:  # torch tensor on the engine's device
             import torch
             a = array.contiguous()
-            code = {torch.float32: LPP_F32, torch.float16: LPP_F16}[a.dtype]
+            code = {torch.float32: LPP_F32, torch.float16: LPP_F16, torch.bfloat16: LPP_BF16}[a.dtype]
             ptr, kind = a.data_ptr(), (MEM_DEVICE if a.is_cuda else MEM_HOST)
             if a.is_cuda:
                 torch.cuda.current_stream(a.device).synchronize()
@@ -217,6 +264,18 @@ class Engine:
                                     C.byref(ms)), "lpp_prefill")
         return ms.value
 
+    def extend(self, tokens: Sequence[int], start_pos: int, want: Sequence[int] = ()) -> np.ndarray:
+        """Runs one portion of a sequence at positions ``start_pos ..`` on the cache of earlier calls; returns the logits
+        of the tokens ``want`` (ascending indices into ``tokens``) as [len(want), vocab]."""
+        toks = np.ascontiguousarray(tokens, dtype=np.int32)
+        w = np.ascontiguousarray(want, dtype=np.int32)
+        out = np.empty((w.size, self.cfg.vocab_size), dtype=np.float32)
+        ip, fp = C.POINTER(C.c_int), C.POINTER(C.c_float)
+        _check(self.lib.lpp_extend(self.h, toks.ctypes.data_as(ip), int(toks.size), int(start_pos),
+                                   w.ctypes.data_as(ip) if w.size else None, int(w.size),
+                                   out.ctypes.data_as(fp) if w.size else None, None), "lpp_extend")
+        return out
+
     def sample(self, logits: np.ndarray, temperature: float, penalty: float = 1.0, history: Sequence[int] = (),
                r: float = 0.0) -> int:
         """``cuda_sample`` (src/sample.cu:210-214) on given logits."""
@@ -253,6 +312,13 @@ class Engine:
         _check(self.lib.lpp_kv_read(self.h, layer, kv_head, pos, k.ctypes.data_as(fp), v.ctypes.data_as(fp)),
                "lpp_kv_read")
         return k, v
+
+    def latent_read(self, layer: int, pos: int) -> np.ndarray:
+        """One cache row of a latent-attention layer: normed latent, then the rotated key part."""
+        m = self.cfg.layers[layer].mixer
+        row = np.empty(m.kv_rank + m.rot_dim, dtype=np.float32)
+        _check(self.lib.lpp_latent_read(self.h, layer, pos, row.ctypes.data_as(C.POINTER(C.c_float))), "lpp_latent_read")
+        return row
 
     def kv_index(self, layer: int, kv_head: int, pos: int, off: int) -> int:
         return int(self.lib.lpp_kv_index(self.h, layer, kv_head, pos, off))
@@ -313,11 +379,7 @@ class Engine:
 
 
 def engine_from_file(path: str, **kw) -> Engine:
-    """Load a llama2.c ``.bin`` or GGUF model file into a new engine (src/main.cpp:44-113 dispatch)."""
-    from .formats import load_model
-    cfg, tensors = load_model(path)
-    wd = "f16" if tensors["wq"].dtype == np.float16 else "f32"
-    kw.setdefault("kv_dtype", "f16" if wd == "f16" else "f32")
-    e = Engine(cfg, wd, **kw)
-    e.load_weights(tensors)
-    return e
+    """Load a model file (llama2.c ``.bin``, GGUF: src/main.cpp:44-113 dispatch) or a model folder into a new engine;
+    see ``models.load_engine``."""
+    from .models import load_engine
+    return load_engine(path, **kw)

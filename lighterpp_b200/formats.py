@@ -9,12 +9,15 @@ Tensor naming used throughout this package (one name per reference ``transformer
 
     tok_emb [V,D]  rms_att [L,D]  wq [L,D,D]  wk [L,KV,D]  wv [L,KV,D]  wo [L,D,D]
     rms_ffn [L,D]  w1 [L,F,D]     w2 [L,D,F]  w3 [L,F,D]   rms_final [D]  w_cls [V,D] (optional)
+
+Besides them: model folders (``config.json`` + ``model.safetensors``), whose architectures ``models.py`` lists.
 """
 from __future__ import annotations
 
+import json
 import struct
-from dataclasses import dataclass, asdict
-from typing import Dict, Iterable, Optional, Tuple
+from dataclasses import dataclass, asdict, field
+from typing import Dict, Iterable, List, Optional, Tuple
 
 import numpy as np
 
@@ -44,6 +47,61 @@ class ModelConfig:
     @property
     def kv_dim(self) -> int:
         return self.dim * self.n_kv_heads // self.n_heads
+
+    def asdict(self):
+        return asdict(self)
+
+
+@dataclass
+class Yarn:
+    """Stretching of slowly turning pairs beyond the context a model was made for."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass
+class Rotation:
+    """Rotary positions on the first ``dims`` dimensions, neighbours paired, pair i turning base^(-2i/dims) per position."""
+    dims: int
+    base: float
+    yarn: Optional[Yarn] = None
+
+
+@dataclass
+class LatentMixer:
+    """Latent attention with a sigmoid gate per head; ``window`` 0 = all earlier positions."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    scale: float
+    rotation: Rotation
+    window: int = 0
+
+
+@dataclass
+class Layer:
+    mixer: LatentMixer
+    ff: int = 0  # 0 = no feed-forward
+    act: str = "silu"
+
+
+@dataclass
+class LayeredConfig:
+    """A model as a list of layers that may differ from one another; ``norm`` is "rms" or "layer"."""
+    dim: int
+    vocab_size: int
+    seq_len: int
+    layers: List[Layer] = field(default_factory=list)
+    norm: str = "rms"
+    norm_eps: float = 1e-5
+
+    @property
+    def n_layers(self) -> int:
+        return len(self.layers)
 
     def asdict(self):
         return asdict(self)
@@ -311,6 +369,37 @@ def read_gguf(path: str) -> Tuple[ModelConfig, Dict[str, np.ndarray], Dict[str, 
                 out[ours] = np.empty(shapes[ours], dtype=a.dtype)
             out[ours][layer] = a
     return c, out, meta
+
+
+# --------------------------------------------------------------------------- safetensors
+
+_SAFE_DTYPES = {"F32": np.dtype("<f4"), "F16": np.dtype("<f2"), "BF16": np.dtype("<u2"), "I32": np.dtype("<i4")}
+
+
+def read_safetensors(path: str) -> Dict[str, np.ndarray]:
+    """Every tensor of the file as a memory-mapped array.  bfloat16 tensors come as their bit patterns (uint16), which
+    is also how the engine's upload takes them."""
+    raw = np.memmap(path, dtype=np.uint8, mode="r")
+    if raw.size < 8:
+        raise ValueError(f"{path}: too short for a safetensors header")
+    n = struct.unpack("<Q", bytes(raw[:8]))[0]
+    if n > raw.size - 8:
+        raise ValueError(f"{path}: header of {n} bytes in a file of {raw.size}")
+    head = json.loads(bytes(raw[8:8 + n]))
+    out: Dict[str, np.ndarray] = {}
+    for name, t in head.items():
+        if name == "__metadata__":
+            continue
+        if t["dtype"] not in _SAFE_DTYPES:
+            raise ValueError(f"{path}: tensor {name} has unsupported type {t['dtype']}")
+        dt = _SAFE_DTYPES[t["dtype"]]
+        a, b = t["data_offsets"]
+        count = int(np.prod(t["shape"], dtype=np.int64))
+        if a < 0 or b - a != count * dt.itemsize or 8 + n + b > raw.size:
+            raise ValueError(f"{path}: tensor {name} does not fit the file")
+        out[name] = np.frombuffer(raw, dtype=np.uint8, count=b - a, offset=8 + n + a).view(dt).reshape(t["shape"]) \
+            if (8 + n + a) % dt.itemsize == 0 else np.frombuffer(bytes(raw[8 + n + a:8 + n + b]), dtype=dt).reshape(t["shape"])
+    return out
 
 
 def is_gguf(path: str) -> bool:
