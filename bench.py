@@ -1,6 +1,7 @@
 #!/usr/bin/env python
 """Benchmark of the batch-1 decode step (tokens/s and fraction of the HBM roofline).
 
+    python bench.py --layered rutenex-1b    (a layered design beside the existing model of equal size)
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference] [--workload NAME]
 
 A "step" is one decoded token: forward(token, pos) + fused sampler.  At N=1 the workload is the
@@ -34,6 +35,17 @@ WORKLOADS = {
     "stories15m": ("stories15m", 16, 1.0, 1.0),
     # long context: K/V cache pre-filled with 32768 positions of seeded N(0,1) values, then prompt + decode
     "llama-3-8b-32k": ("llama-3-8b-32k", 64, 0.8, 1.1, 32768),
+}
+
+
+# Layered designs beside the closest existing model of equal size (--layered NAME): same width, layers, feed-forward and
+# vocabulary; the existing model's heads are those of the Llama shape of that width.
+#   name: (width, layers, ff, vocab, mixer sizes, window, (llama heads, kv heads), prompt tokens)
+_MLA = dict(dim=128, rot_dim=64, vdim=128, kv_rank=512)
+LAYERED = {
+    "rutenex-1b": (2048, 16, 8192, 32768, dict(heads=16, **_MLA), 1024, (32, 8), 1024),
+    "rutenex-8b": (4096, 32, 14336, 32768, dict(heads=32, **_MLA), 4096, (32, 8), 1024),
+    "rutenex-300m": (1024, 24, 2816, 32768, dict(heads=16, dim=64, rot_dim=32, vdim=64, kv_rank=256), 512, (16, 4), 1024),
 }
 
 
@@ -460,6 +472,82 @@ def run_reference(args, rank, world):
             "e2e": {"value": cb["value"], "unit": "tok/s", "h2d_bytes_per_step": 0, "d2h_bytes_per_step": 0}}
 
 
+def layered_engines(name):
+    """(label, engine) of the layered design and of the existing model, random weights, one after the other."""
+    import torch
+    from lighterpp_b200 import engine as E
+    from lighterpp_b200.formats import LatentMixer, Layer, LayeredConfig, ModelConfig, Rotation, Yarn
+    from lighterpp_b200.models import ARCHITECTURES
+    width, layers, ff, vocab, mix, window, (heads, kv), n_prompt = LAYERED[name]
+    seq = n_prompt + 1024
+    g = torch.Generator(device="cuda")
+    g.manual_seed(7)
+    m = LatentMixer(scale=(mix["dim"] + mix["rot_dim"]) ** -0.5, window=window,
+                    rotation=Rotation(mix["rot_dim"], 1e6, Yarn(4.0, 4096, 32.0, 1.0)), **mix)
+    cfg = LayeredConfig(width, vocab, seq, [Layer(m, ff, "gelu_tanh") for _ in range(layers)], "layer", 1e-6)
+    eng = E.Engine(cfg, "bf16", "f16")
+    for ours, layer, tensor, shape in ARCHITECTURES["Rutenex"].tensors(cfg):
+        if len(shape) == 1:
+            t = torch.zeros(shape, device="cuda") if tensor.endswith(".b") else torch.ones(shape, device="cuda")
+        else:
+            t = torch.randn(shape, device="cuda", generator=g) * shape[1] ** -0.5
+        eng.upload(ours, t.to(torch.bfloat16), layer)
+    eng.finalize()
+    torch.cuda.empty_cache()
+    yield "rutenex", eng
+    eng.close()
+    cfg = ModelConfig(width, ff, layers, heads, kv, vocab, seq, 500000.0)
+    eng = E.Engine(cfg, "f16", "f16")
+    for tensor, l, t in gen_device_weights(cfg, "f16", True, 7):
+        eng.upload(tensor, t, max(l, 0))
+    eng.finalize()
+    torch.cuda.empty_cache()
+    yield "llama", eng
+    eng.close()
+
+
+def run_layered(args):
+    """Prompt and decode throughput of a layered design and of the existing model of equal size, with the fraction of the
+    measured copy bandwidth every decode kernel kind reaches in both."""
+    import torch
+    torch.cuda.set_device(0)
+    n_prompt = LAYERED[args.layered][-1]
+    peak, peak_kind = measured_peak()
+    line = {"metric": "batch-1 prompt and decode tok/s beside the existing model of equal size", "unit": "tok/s", "n_gpus": 1,
+            "steps": args.steps, "warmup": args.warmup, "data": "synthetic", "config": {"design": args.layered, "sizes": LAYERED[args.layered]},
+            "peak_gbs": peak, "peak_source": f"{peak_kind} copy bandwidth"}
+    with ClockSampler(0) as clk:
+        for label, eng in layered_engines(args.layered):
+            prompt = np.random.default_rng(1).integers(0, eng.cfg.vocab_size, n_prompt).astype(np.int32)
+            rs = np.random.default_rng(2).random(args.warmup + args.steps).astype(np.float32)
+            for _ in range(3):
+                eng.prefill(prompt[:-1], 0)
+            pf = sorted(eng.prefill(prompt[:-1], 0) for _ in range(5))[2]
+            out, _ = eng.decode(int(prompt[-1]), n_prompt - 1, args.warmup, 0.8, 1.1, prompt[-64:], 64, rs[:args.warmup])
+            pos = n_prompt - 1 + args.warmup
+            torch.cuda.synchronize()
+            _, ms = eng.decode(int(out[-1]), pos, args.steps, 0.8, 1.1, prompt[-64:], 64, rs[args.warmup:])
+            torch.cuda.synchronize()
+            us = ms * 1e3 / args.steps
+            gbs = eng.step_bytes(pos + args.steps // 2) / us / 1e3
+            kinds = {}
+            prof = eng.profile_step(pos, 10, 0.8, 1.1)
+            for k, v in prof.items():
+                if not v["launches"] or not v["bytes"]:
+                    continue
+                run = eng.profile_kind(pos, k, 10)
+                t = run["ms_per_launch"] * 1e3
+                per = v["bytes"] / v["launches"]
+                kinds[k] = {"us": round(t, 2), "isolated_us": round(v["ms"] * 1e3 / v["launches"], 2), "kib": round(per / 1024, 1),
+                            "frac_of_measured": round(per / t / 1e3 / peak, 3)}
+            line[label] = {"prompt_tok_s": round((n_prompt - 1) / pf * 1e3, 1), "prompt_ms": round(pf, 3),
+                           "decode_tok_s": round(1e6 / us, 1), "us_per_token": round(us, 1), "step_gbs": round(gbs, 1),
+                           "step_frac_of_measured": round(gbs / peak, 3), "kernels_per_step": eng.kernels_per_step, "kernels": kinds}
+    line["clocks"] = clk.summary()
+    line["value"] = line["rutenex"]["decode_tok_s"]
+    return line
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -467,6 +555,8 @@ def main():
     ap.add_argument("--warmup", type=int, default=16)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default=None, choices=sorted(WORKLOADS))
+    ap.add_argument("--layered", default=None, choices=sorted(LAYERED),
+                    help="instead of the workload: a layered design beside the existing model of equal size")
     ap.add_argument("--flags", type=int, default=0)
     ap.add_argument("--ring-kb", type=int, default=0)
     ap.add_argument("--cpu-seconds", type=float, default=15.0)
@@ -477,6 +567,10 @@ def main():
     if world != args.gpus and world == 1 and args.gpus > 1:
         print(json.dumps({"error": f"--gpus {args.gpus} needs torchrun with {args.gpus} ranks"}))
         sys.exit(2)
+    if args.layered:
+        args.warmup = max(args.warmup, 3)
+        print(json.dumps(run_layered(args)), flush=True)
+        return
     if args.workload is None:
         args.workload = "llama-3.2-1b" if world == 1 else "llama-3-8b"
     args.warmup = max(args.warmup, 3) if args.impl == "ours" else args.warmup

@@ -272,14 +272,14 @@ static void gemv_geometry(GemvArgs& a, int esz, int stage_target) {
     }
 }
 
-template <typename WT, int EPI>
-static cudaError_t launch_gemv_t(lpp_engine* e, GemvArgs& a, bool pdl, cudaStream_t s) {
+template <typename WT, int EPI, bool LN = false>
+static cudaError_t launch_gemv_t(lpp_engine* e, GemvArgsOf<EPI>& a, bool pdl, cudaStream_t s) {
     const int esz = sizeof(WT);
     const int groups = a.n_rows / kRowsPerGroup;
     // Grouped rows: a CTA stages the inputs of every group its contiguous row pairs touch, plus the split weights.
     auto staged_bytes = [&](int grid) -> size_t {
         if (a.group_pairs <= 0) return align_up((size_t)a.K * 4, 128);
-        const int pairs = (groups + grid - 1) / grid;
+        const int pairs = (groups + grid - 1) / grid;  // grid: CTAs with rows
         const size_t n = (size_t)(pairs + a.group_pairs - 2) / a.group_pairs + 1;
         return align_up(n * ((size_t)a.K + kLatentMaxSplits) * 4, 128);
     };
@@ -287,19 +287,21 @@ static cudaError_t launch_gemv_t(lpp_engine* e, GemvArgs& a, bool pdl, cudaStrea
         const size_t smem = 128 + staged_bytes(std::max(1, std::min(groups, e->num_sms * 4)));
         static bool attr_done[64] = {};
         if (!attr_done[e->c.device & 63]) {
-            cudaError_t r = cudaFuncSetAttribute(gemv_ldg_kernel<WT, EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+            cudaError_t r = cudaFuncSetAttribute(gemv_ldg_kernel<WT, EPI, LN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                  (int)e->smem_optin);
             if (r != cudaSuccess) return r;
             attr_done[e->c.device & 63] = true;
         }
-        const int grid = std::max(1, std::min(groups, e->num_sms * 4));
-        return launch_kernel(gemv_ldg_kernel<WT, EPI>, dim3(grid), dim3(kGemvLdgThreads), smem, s, pdl, a);
+        const int grid = std::max(1, std::min(groups, e->num_sms * 4)) + (EPI == kEpiLatentQuery ? 1 : 0);
+        return launch_kernel(gemv_ldg_kernel<WT, EPI, LN>, dim3(grid), dim3(kGemvLdgThreads), smem, s, pdl, a);
     }
     // LPP_STAGE_KB (timing experiments) overrides the 8 KiB stage size.
     int stage_target = kStageTarget;
     if (const char* sk = aid_env("LPP_STAGE_KB")) stage_target = std::max(1, atoi(sk)) * 1024;
     gemv_geometry(a, esz, stage_target);
-    const int grid = std::max(1, std::min(groups, e->num_sms));
+    // the query GEMV of latent attention: one CTA without rows (row_ctas in gemv.cuh)
+    const int extra = EPI == kEpiLatentQuery ? 1 : 0;
+    const int grid = std::max(1, std::min(groups, e->num_sms - extra));
     const size_t xbytes = staged_bytes(grid);
     a.xs_bytes = (int)xbytes;
     const size_t fixed = kGemvBarrierBytes + 128 + xbytes;
@@ -313,34 +315,51 @@ static cudaError_t launch_gemv_t(lpp_engine* e, GemvArgs& a, bool pdl, cudaStrea
     if (smem > e->smem_optin) return cudaErrorInvalidValue;
     static bool attr_done[64] = {};
     if (!attr_done[e->c.device & 63]) {
-        cudaError_t r = cudaFuncSetAttribute(gemv_ring_kernel<WT, EPI>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        cudaError_t r = cudaFuncSetAttribute(gemv_ring_kernel<WT, EPI, LN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              (int)e->smem_optin);
         if (r != cudaSuccess) return r;
         attr_done[e->c.device & 63] = true;
     }
-    return launch_kernel(gemv_ring_kernel<WT, EPI>, dim3(grid), dim3(kGemvRingThreads), smem, s, pdl, a);
+    return launch_kernel(gemv_ring_kernel<WT, EPI, LN>, dim3(grid + extra), dim3(kGemvRingThreads), smem, s, pdl, a);
 }
 
 static cudaError_t launch_gemv(lpp_engine* e, int epi, int w_dtype, GemvArgs& a, bool pdl, cudaStream_t s) {
-#define LPP_GEMV_CASE(E)                                                                \
-    case E:                                                                             \
-        if (w_dtype == LPP_BF16) return launch_gemv_t<__nv_bfloat16, E>(e, a, pdl, s);  \
+#define LPP_GEMV_CASE(E)                                                                                                \
+    case E:                                                                                                             \
+        if (w_dtype == LPP_BF16) return launch_gemv_t<__nv_bfloat16, E>(e, a, pdl, s);                                  \
         return w_dtype == LPP_F16 ? launch_gemv_t<__half, E>(e, a, pdl, s) : launch_gemv_t<float, E>(e, a, pdl, s);
-#define LPP_GEMV_LATENT_CASE(E)                                                         \
-    case E:                                                                             \
-        return w_dtype == LPP_BF16 ? launch_gemv_t<__nv_bfloat16, E>(e, a, pdl, s) : launch_gemv_t<float, E>(e, a, pdl, s);
+#define LPP_GEMV_LN_CASE(E)                                                                                             \
+    case E:                                                                                                             \
+        return w_dtype == LPP_BF16 ? launch_gemv_t<__nv_bfloat16, E, true>(e, a, pdl, s) : launch_gemv_t<float, E, true>(e, a, pdl, s);
+    if (a.norm_b) {
+        switch (epi) {
+            LPP_GEMV_LN_CASE(kEpiStore)
+            LPP_GEMV_LN_CASE(kEpiSwiglu)
+        }
+        return cudaErrorInvalidValue;
+    }
     switch (epi) {
         LPP_GEMV_CASE(kEpiStore)
         LPP_GEMV_CASE(kEpiResid)
         LPP_GEMV_CASE(kEpiSwiglu)
         case kEpiQkv:
             return w_dtype == LPP_F16 ? launch_gemv_t<__half, kEpiQkv>(e, a, pdl, s) : launch_gemv_t<float, kEpiQkv>(e, a, pdl, s);
-        LPP_GEMV_LATENT_CASE(kEpiLatentIn)
-        LPP_GEMV_LATENT_CASE(kEpiLatentQuery)
-        LPP_GEMV_LATENT_CASE(kEpiLatentValue)
     }
 #undef LPP_GEMV_CASE
-#undef LPP_GEMV_LATENT_CASE
+#undef LPP_GEMV_LN_CASE
+    return cudaErrorInvalidValue;
+}
+template <int EPI, bool LN>
+static cudaError_t launch_latent_gemv(lpp_engine* e, int w_dtype, GemvLatentArgs& a, bool pdl, cudaStream_t s) {
+    return w_dtype == LPP_BF16 ? launch_gemv_t<__nv_bfloat16, EPI, LN>(e, a, pdl, s) : launch_gemv_t<float, EPI, LN>(e, a, pdl, s);
+}
+static cudaError_t launch_gemv(lpp_engine* e, int epi, int w_dtype, GemvLatentArgs& a, bool pdl, cudaStream_t s) {
+    switch (epi) {
+        case kEpiLatentIn:
+            return a.norm_b ? launch_latent_gemv<kEpiLatentIn, true>(e, w_dtype, a, pdl, s) : launch_latent_gemv<kEpiLatentIn, false>(e, w_dtype, a, pdl, s);
+        case kEpiLatentQuery: return launch_latent_gemv<kEpiLatentQuery, false>(e, w_dtype, a, pdl, s);
+        case kEpiLatentValue: return launch_latent_gemv<kEpiLatentValue, false>(e, w_dtype, a, pdl, s);
+    }
     return cudaErrorInvalidValue;
 }
 
@@ -521,7 +540,8 @@ static bool kind_skipped(const lpp_engine* e, int kind) {
     return (skip_mask() & (1u << kind)) || (e->only_kind >= 0 && kind != e->only_kind);
 }
 
-static void record_gemv(Recorder& R, int kind, int epi, GemvArgs a) {
+template <typename Args>
+static void record_gemv(Recorder& R, int kind, int epi, Args a) {
     lpp_engine* e = R.e;
     if (kind_skipped(e, kind)) return;
     a.st = e->st;
@@ -804,7 +824,7 @@ static void record_gqa_mixer(Recorder& R, int l, float* cur) {
 static void record_latent_mixer(Recorder& R, int l, float* cur) {
     lpp_engine* e = R.e;
     const LatentLayer& y = e->lat[l];
-    GemvArgs a = {};
+    GemvLatentArgs a = {};
     a.lat = latent_args(e, y);
     a.W = y.w_in;
     a.n_rows = y.in_rows;
@@ -818,7 +838,7 @@ static void record_latent_mixer(Recorder& R, int l, float* cur) {
         a.x = cur;
     }
     record_gemv(R, kQkv, kEpiLatentIn, a);
-    GemvArgs q = {};
+    GemvLatentArgs q = {};
     q.lat = a.lat;
     q.W = y.w_uk;
     q.n_rows = y.d.heads * y.rank_pitch;
@@ -833,7 +853,7 @@ static void record_latent_mixer(Recorder& R, int l, float* cur) {
         R.prev_kernel = true;
         R.kernels++;
     }
-    GemvArgs v = {};
+    GemvLatentArgs v = {};
     v.lat = a.lat;
     v.W = y.w_uv;
     v.n_rows = y.d.heads * y.vdim_rows;
@@ -2143,7 +2163,7 @@ extern "C" lpp_status lpp_extend(lpp_engine* e, const int* h_tokens, int n, int 
     const size_t V = e->c.vocab_size;
     int w = 0;  // wanted tokens served so far
     TRY(push_state(e, h_tokens[0], start_pos, nullptr, nullptr, 0, 0.f, 0, 0));  // clears the device status
-    if (prefill_batched(e) && !(n == 1 && n_want == 1)) {
+    if (prefill_batched(e) && n > 1) {
         TRY(prefill_setup(e));
         CU(cudaEventRecord(e->ev0, e->stream));
         for (int i = 0; i < n; i += kPrefillTokens) {

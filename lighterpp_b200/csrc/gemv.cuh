@@ -58,13 +58,12 @@ struct GemvArgs {
     float* x_store;       // CTA 0 stores the un-normalised input vector here (nullptr = don't)
     StepState* st;        // token / pos / status
     int vocab, seq_len;
-    const float* norm_b;  // LayerNorm bias [K]: selects LayerNorm (mean taken off); nullptr = RMSNorm
+    const float* norm_b;  // LayerNorm bias [K] (kernels with LN set: mean taken off); unused by RMSNorm
     float norm_eps;       // inside the root
     int norm_n;           // inputs the statistics cover (0 = K); inputs norm_n .. K-1 are zero padding
     // Grouped rows (heads): row pair g takes the K inputs of group g / group_pairs, x + group * K.  0 = one input
     // vector for all rows.  No normalisation, no embedding.
     int group_pairs;
-    LatentArgs lat;       // latent attention prologues and epilogues
     // ---- epilogue
     float* out;          // Store/Resid: [n_rows]; Swiglu: [n_rows/2]; Qkv: q vector [q_rows]
     int act;             // Swiglu: activation of the gate (Act)
@@ -111,6 +110,15 @@ struct GemvArgs {
     long long tp_wait_cycles;            // limit of a wait on a peer in SM clocks (a kernel argument: the poll loop must
                                          // not pay a global load for it)
 };
+
+// The launches of latent attention carry its arguments too; the kernels of every other epilogue keep the short list.
+struct GemvLatentArgs : GemvArgs {
+    LatentArgs lat;
+};
+template <int EPI>
+constexpr bool is_latent_epi = EPI == kEpiLatentIn || EPI == kEpiLatentQuery || EPI == kEpiLatentValue;
+template <int EPI>
+using GemvArgsOf = std::conditional_t<is_latent_epi<EPI>, GemvLatentArgs, GemvArgs>;
 
 // ------------------------------------------------------------------ x staging layouts
 //
@@ -311,7 +319,7 @@ __device__ __forceinline__ void stage_input_peers(const GemvArgs& a, float* xs, 
 // RMS-normalises it (ss = 1/sqrt(mean(x^2) + 1e-5); out = x*ss*w, src/ops.cpp:20-32) and leaves it
 // in shared memory in the layout xs_index<WT> describes.  Executed by `NT` threads (tid 0..NT-1).
 // The norm weights are constants, so their loads are issued before the dependency wait.
-template <typename WT, int NT>
+template <typename WT, int NT, bool LN>
 __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float* red, int tid) {
     const int K = a.K;
     const int nv4 = K >> 2;
@@ -323,16 +331,19 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
         for (int j = 0; j < kPer; ++j) {
             const int i = tid + j * NT;
             if (i < nv4) wr[j] = __ldg(reinterpret_cast<const float4*>(a.norm_w) + i);
-            if (i < nv4 && a.norm_b) br[j] = __ldg(reinterpret_cast<const float4*>(a.norm_b) + i);
+            if constexpr (LN)
+                if (i < nv4) br[j] = __ldg(reinterpret_cast<const float4*>(a.norm_b) + i);
         }
     }
     // An input that arrives through the tensor-parallel exchange validates itself word by word (this
     // rank's own slot included): its flags can only be complete once every rank's producing GEMV has
     // stored all its rows, which in turn follows everything earlier in the step, so that case does not
     // wait for the local kernel to drain its peer stores and exit.
-    if (a.tp_in != nullptr) {
-        stage_input_peers<WT, NT>(a, xs, red, tid);
-        return;
+    if constexpr (!LN) {
+        if (a.tp_in != nullptr) {
+            stage_input_peers<WT, NT>(a, xs, red, tid);
+            return;
+        }
     }
     pdl_wait();  // activations / KV / step state come from the previous kernel
     if (tid == 0) gemv_stamp(a, 1);
@@ -353,7 +364,7 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
             if (store) a.x_store[k] = v;
             xs[xs_index<WT>(k, K)] = v;
         }
-        if (a.norm_b) {
+        if constexpr (LN) {
             layer_norm_staged<WT, NT>(a, xs, red, tid, 1);
         } else if (a.norm_w) {
             ss = warp_sum(ss);
@@ -374,106 +385,107 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
 
     const float4* x4 = reinterpret_cast<const float4*>(a.x);
     auto load_x4 = [&](int i) -> float4 { return __ldcg(x4 + i); };
-    if (a.norm_b && one_pass) {
-        // LayerNorm from registers: the mean, then the mean of the squared deviations (zero padding beyond norm_n adds
-        // nothing to the first sum, is left out of the second one and has zero weight and bias)
-        const int n = norm_count(a);
-        float4 x[kPer];
-        float s = 0.f, q = 0.f;
+    if constexpr (LN) {
+        if (one_pass) {
+            // LayerNorm from registers: the mean, then the mean of the squared deviations (zero padding beyond norm_n adds
+            // nothing to the first sum, is left out of the second one and has zero weight and bias)
+            const int n = norm_count(a);
+            float4 x[kPer];
+            float s = 0.f, q = 0.f;
 #pragma unroll
-        for (int j = 0; j < kPer; ++j) {
-            const int i = tid + j * NT;
-            x[j] = i < nv4 ? load_x4(i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int j = 0; j < kPer; ++j) {
+                const int i = tid + j * NT;
+                x[j] = i < nv4 ? load_x4(i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+#pragma unroll
+            for (int j = 0; j < kPer; ++j) s += (x[j].x + x[j].y) + (x[j].z + x[j].w);
+            const float mean = __fdiv_rn(consumer_sum<NT>(s, red, tid, 0), (float)n);
+#pragma unroll
+            for (int j = 0; j < kPer; ++j) {
+                const int k = (tid + j * NT) << 2;
+                x[j].x -= mean; x[j].y -= mean; x[j].z -= mean; x[j].w -= mean;
+                if (k + 0 < n) q = fmaf(x[j].x, x[j].x, q);
+                if (k + 1 < n) q = fmaf(x[j].y, x[j].y, q);
+                if (k + 2 < n) q = fmaf(x[j].z, x[j].z, q);
+                if (k + 3 < n) q = fmaf(x[j].w, x[j].w, q);
+            }
+            const float var = __fdiv_rn(consumer_sum<NT>(q, red, tid, 1), (float)n);
+            const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(var, a.norm_eps)));
+#pragma unroll
+            for (int j = 0; j < kPer; ++j) {
+                const int i = tid + j * NT;
+                if (i < nv4)
+                    xs_store4<WT>(xs, i << 2, K,
+                                  make_float4(fmaf(__fmul_rn(x[j].x, scale), wr[j].x, br[j].x), fmaf(__fmul_rn(x[j].y, scale), wr[j].y, br[j].y),
+                                              fmaf(__fmul_rn(x[j].z, scale), wr[j].z, br[j].z), fmaf(__fmul_rn(x[j].w, scale), wr[j].w, br[j].w)));
+            }
+            consumer_barrier(NT);
+            return;
         }
-#pragma unroll
-        for (int j = 0; j < kPer; ++j) s += (x[j].x + x[j].y) + (x[j].z + x[j].w);
-        const float mean = __fdiv_rn(consumer_sum<NT>(s, red, tid, 0), (float)n);
-#pragma unroll
-        for (int j = 0; j < kPer; ++j) {
-            const int k = (tid + j * NT) << 2;
-            x[j].x -= mean; x[j].y -= mean; x[j].z -= mean; x[j].w -= mean;
-            if (k + 0 < n) q = fmaf(x[j].x, x[j].x, q);
-            if (k + 1 < n) q = fmaf(x[j].y, x[j].y, q);
-            if (k + 2 < n) q = fmaf(x[j].z, x[j].z, q);
-            if (k + 3 < n) q = fmaf(x[j].w, x[j].w, q);
-        }
-        const float var = __fdiv_rn(consumer_sum<NT>(q, red, tid, 1), (float)n);
-        const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(var, a.norm_eps)));
-#pragma unroll
-        for (int j = 0; j < kPer; ++j) {
-            const int i = tid + j * NT;
-            if (i < nv4)
-                xs_store4<WT>(xs, i << 2, K,
-                              make_float4(fmaf(__fmul_rn(x[j].x, scale), wr[j].x, br[j].x), fmaf(__fmul_rn(x[j].y, scale), wr[j].y, br[j].y),
-                                          fmaf(__fmul_rn(x[j].z, scale), wr[j].z, br[j].z), fmaf(__fmul_rn(x[j].w, scale), wr[j].w, br[j].w)));
-        }
-        consumer_barrier(NT);
-        return;
-    }
-    if (a.norm_b) {  // wider rows: from the staged copy
+        // wider rows: from the staged copy
         for (int i = tid; i < nv4; i += NT) xs_store4<WT>(xs, i << 2, K, load_x4(i));
         layer_norm_staged<WT, NT>(a, xs, red, tid, 4);
         consumer_barrier(NT);
         return;
-    }
-    if (!a.norm_w) {
-        for (int i = tid; i < nv4; i += NT) xs_store4<WT>(xs, i << 2, K, load_x4(i));
+    } else {
+        if (!a.norm_w) {
+            for (int i = tid; i < nv4; i += NT) xs_store4<WT>(xs, i << 2, K, load_x4(i));
+            consumer_barrier(NT);
+            return;
+        }
+        float ss = 0.f;
+        float4 xr[kPer];
+        if (one_pass) {
+#pragma unroll
+            for (int j = 0; j < kPer; ++j) {
+                const int i = tid + j * NT;
+                if (i < nv4) xr[j] = load_x4(i);
+            }
+#pragma unroll
+            for (int j = 0; j < kPer; ++j) {
+                const int i = tid + j * NT;
+                if (i < nv4) ss = fmaf(xr[j].x, xr[j].x, fmaf(xr[j].y, xr[j].y, fmaf(xr[j].z, xr[j].z, fmaf(xr[j].w, xr[j].w, ss))));
+            }
+        } else {
+            for (int i = tid; i < nv4; i += NT) {
+                const float4 v = load_x4(i);
+                ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+            }
+        }
+        ss = warp_sum(ss);
+        if ((tid & 31) == 0) red[tid >> 5] = ss;
         consumer_barrier(NT);
-        return;
+        float tot = 0.f;
+#pragma unroll
+        for (int w = 0; w < NT / 32; ++w) tot += red[w];
+        const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, (float)norm_count(a)), a.norm_eps)));
+        auto normed = [&](float4 v, float4 w) {
+            return make_float4(__fmul_rn(__fmul_rn(v.x, scale), w.x), __fmul_rn(__fmul_rn(v.y, scale), w.y),
+                               __fmul_rn(__fmul_rn(v.z, scale), w.z), __fmul_rn(__fmul_rn(v.w, scale), w.w));
+        };
+        if (one_pass) {
+#pragma unroll
+            for (int j = 0; j < kPer; ++j) {
+                const int i = tid + j * NT;
+                if (i < nv4) xs_store4<WT>(xs, i << 2, K, normed(xr[j], wr[j]));
+            }
+        } else {
+            for (int i = tid; i < nv4; i += NT)
+                xs_store4<WT>(xs, i << 2, K, normed(load_x4(i), __ldg(reinterpret_cast<const float4*>(a.norm_w) + i)));
+        }
+        consumer_barrier(NT);
     }
-    float ss = 0.f;
-    float4 xr[kPer];
-    if (one_pass) {
-#pragma unroll
-        for (int j = 0; j < kPer; ++j) {
-            const int i = tid + j * NT;
-            if (i < nv4) xr[j] = load_x4(i);
-        }
-#pragma unroll
-        for (int j = 0; j < kPer; ++j) {
-            const int i = tid + j * NT;
-            if (i < nv4) ss = fmaf(xr[j].x, xr[j].x, fmaf(xr[j].y, xr[j].y, fmaf(xr[j].z, xr[j].z, fmaf(xr[j].w, xr[j].w, ss))));
-        }
-    } else {
-        for (int i = tid; i < nv4; i += NT) {
-            const float4 v = load_x4(i);
-            ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
-        }
-    }
-    ss = warp_sum(ss);
-    if ((tid & 31) == 0) red[tid >> 5] = ss;
-    consumer_barrier(NT);
-    float tot = 0.f;
-#pragma unroll
-    for (int w = 0; w < NT / 32; ++w) tot += red[w];
-    const float scale = __fdiv_rn(1.0f, __fsqrt_rn(__fadd_rn(__fdiv_rn(tot, (float)norm_count(a)), a.norm_eps)));
-    auto normed = [&](float4 v, float4 w) {
-        return make_float4(__fmul_rn(__fmul_rn(v.x, scale), w.x), __fmul_rn(__fmul_rn(v.y, scale), w.y),
-                           __fmul_rn(__fmul_rn(v.z, scale), w.z), __fmul_rn(__fmul_rn(v.w, scale), w.w));
-    };
-    if (one_pass) {
-#pragma unroll
-        for (int j = 0; j < kPer; ++j) {
-            const int i = tid + j * NT;
-            if (i < nv4) xs_store4<WT>(xs, i << 2, K, normed(xr[j], wr[j]));
-        }
-    } else {
-        for (int i = tid; i < nv4; i += NT)
-            xs_store4<WT>(xs, i << 2, K, normed(load_x4(i), __ldg(reinterpret_cast<const float4*>(a.norm_w) + i)));
-    }
-    consumer_barrier(NT);
 }
 
-// Staging for grouped rows: inputs of groups first .. first + n - 1 (one per head), K each.  The query projection
-// reads the plain query parts; its last CTA also turns the raw latent of this token into a cache row.  The value
-// projection reads the attended latents, which it puts together from the partial results of the attention splits.
+// Staging for grouped rows: inputs of groups first .. first + n - 1 (one per head), K each.  The query projection reads
+// the plain query parts, the value projection the attended latents, which it puts together from the partial results of
+// the attention splits.
 template <typename WT, int EPI, int NT>
-__device__ __forceinline__ void stage_input_groups(const GemvArgs& a, float* xs, int tid, int first, int n) {
+__device__ __forceinline__ void stage_input_groups(const GemvLatentArgs& a, float* xs, int tid, int first, int n) {
     const int K = a.K, Kx = n * K;
     pdl_wait();
     if (tid == 0) gemv_stamp(a, 1);
     if constexpr (EPI == kEpiLatentQuery) {
-        if (blockIdx.x == gridDim.x - 1) latent_norm_to_cache<NT>(a.lat, a.st, a.seq_len, xs, tid);
         const float4* x4 = reinterpret_cast<const float4*>(a.x + (size_t)first * K);
         for (int i = tid; i < Kx >> 2; i += NT) xs_store4<WT>(xs, i << 2, Kx, __ldcg(x4 + i));
     } else {
@@ -580,7 +592,7 @@ __device__ __forceinline__ void store_rows(const GemvArgs& a, int row, float v0,
 
 // Writes the results of row pair `g` (rows 2g, 2g+1); called by one lane with the warp-reduced sums.
 template <typename WT, int EPI>
-__device__ __forceinline__ void gemv_epilogue(const GemvArgs& a, int g, float v0, float v1) {
+__device__ __forceinline__ void gemv_epilogue(const GemvArgsOf<EPI>& a, int g, float v0, float v1) {
     const int row = g * kRowsPerGroup;
     if constexpr (EPI == kEpiStore) {
         store_rows(a, row, v0, v1);
@@ -636,12 +648,20 @@ __device__ __forceinline__ void gemv_epilogue(const GemvArgs& a, int g, float v0
     }
 }
 
+// CTAs of the launch that rows are dealt to.  The query GEMV of latent attention has one more, the last one, which norms the
+// latent of this token into its cache row while the others run.
+template <int EPI>
+__device__ __forceinline__ int row_ctas() {
+    return EPI == kEpiLatentQuery ? (int)gridDim.x - 1 : (int)gridDim.x;
+}
+
 // ------------------------------------------------------------------ ring (bulk async copy) variant
 
-// Body of the ring kernel.  Returns true on the consumer threads once all of this CTA's rows are
+// Body of the ring kernel (LN: the prologue's norm is a LayerNorm; a template argument because code that a kernel does not
+// need still costs it instruction fetches at every launch).  Returns true on the consumer threads once all of this CTA's rows are
 // done (so a caller can append a CTA-level tail), false on the producer warp and after a timeout.
-template <typename WT, int EPI>
-__device__ __forceinline__ bool gemv_ring_body(const GemvArgs& a, unsigned char* smem) {
+template <typename WT, int EPI, bool LN>
+__device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigned char* smem) {
     uint64_t* full = reinterpret_cast<uint64_t*>(smem);                // [consumer warp][kGemvMaxStages]
     uint64_t* empty = full + kGemvConsumerWarps * kGemvMaxStages;      // [consumer warp][kGemvMaxStages]
     float* red = reinterpret_cast<float*>(smem + kGemvBarrierBytes);   // 8 floats
@@ -653,8 +673,9 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgs& a, unsigned char*
     const int NS = a.n_stages;  // slots per consumer warp
     const int groups = a.n_rows / kRowsPerGroup;
     // this CTA's row pairs, then this warp's (or producer lane's) contiguous share of them
-    const int g0 = (int)(((long long)blockIdx.x * groups) / gridDim.x);
-    const int g1 = (int)(((long long)(blockIdx.x + 1) * groups) / gridDim.x);
+    const int n_cta = row_ctas<EPI>();
+    const int g0 = (int)(((long long)min((int)blockIdx.x, n_cta) * groups) / n_cta);
+    const int g1 = (int)(((long long)min((int)blockIdx.x + 1, n_cta) * groups) / n_cta);
     const int ng = g1 - g0;
     const int w = (warp == kGemvConsumerWarps) ? lane : warp;  // pipeline index
     const int p0 = g0 + (w < kGemvConsumerWarps ? (ng * w) / kGemvConsumerWarps : 0);
@@ -759,12 +780,17 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgs& a, unsigned char*
     // grouped rows: the inputs of the groups this CTA's row pairs belong to are staged back to back
     int first_group = 0, Kx = a.K;
     if constexpr (EPI == kEpiLatentQuery || EPI == kEpiLatentValue) {
+        if (EPI == kEpiLatentQuery && g0 >= g1) {  // the CTA without rows
+            pdl_wait();
+            latent_norm_to_cache<kGemvConsumerWarps * 32>(a.lat, a.st, a.seq_len, red, tid);
+            return true;
+        }
         first_group = g0 / a.group_pairs;
         const int n_groups = (g1 - 1) / a.group_pairs - first_group + 1;
         Kx = n_groups * a.K;
         stage_input_groups<WT, EPI, kGemvConsumerWarps * 32>(a, xs, tid, first_group, n_groups);
     } else {
-        stage_input<WT, kGemvConsumerWarps * 32>(a, xs, red, tid);
+        stage_input<WT, kGemvConsumerWarps * 32, LN>(a, xs, red, tid);
     }
     // where the inputs of row pair p start among the staged ones
     auto input_offset = [&](int p) -> int {
@@ -852,10 +878,10 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgs& a, unsigned char*
     return true;
 }
 
-template <typename WT, int EPI>
-__global__ void __launch_bounds__(kGemvRingThreads) gemv_ring_kernel(const GemvArgs a) {
+template <typename WT, int EPI, bool LN>
+__global__ void __launch_bounds__(kGemvRingThreads) gemv_ring_kernel(const GemvArgsOf<EPI> a) {
     extern __shared__ __align__(128) unsigned char smem[];
-    const bool consumer = gemv_ring_body<WT, EPI>(a, smem);
+    const bool consumer = gemv_ring_body<WT, EPI, LN>(a, smem);
     if constexpr (EPI == kEpiResid) {
         // tensor-parallel exchange: this CTA's rows are on their way, tell every rank (a hint, see GemvArgs)
         if (consumer && a.tp_size > 1 && a.tp_hint_out[0]) {
@@ -871,25 +897,31 @@ __global__ void __launch_bounds__(kGemvRingThreads) gemv_ring_kernel(const GemvA
 //
 // Same partition and epilogues; weights go global -> registers with 128-bit streaming loads.  Kept
 // as the measured alternative to the ring (see profiles/).
-template <typename WT, int EPI>
-__global__ void __launch_bounds__(kGemvLdgThreads) gemv_ldg_kernel(const GemvArgs a) {
+template <typename WT, int EPI, bool LN = false>
+__global__ void __launch_bounds__(kGemvLdgThreads) gemv_ldg_kernel(const GemvArgsOf<EPI> a) {
     extern __shared__ __align__(128) unsigned char smem[];
     float* red = reinterpret_cast<float*>(smem);
     float* xs = reinterpret_cast<float*>(smem + 128);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int groups = a.n_rows / kRowsPerGroup;
-    const int g0 = (int)(((long long)blockIdx.x * groups) / gridDim.x);
-    const int g1 = (int)(((long long)(blockIdx.x + 1) * groups) / gridDim.x);
+    const int n_cta = row_ctas<EPI>();
+    const int g0 = (int)(((long long)min((int)blockIdx.x, n_cta) * groups) / n_cta);
+    const int g1 = (int)(((long long)min((int)blockIdx.x + 1, n_cta) * groups) / n_cta);
     constexpr int NW = kGemvLdgThreads / 32;
 
     int first_group = 0, Kx = a.K;
     if constexpr (EPI == kEpiLatentQuery || EPI == kEpiLatentValue) {
+        if (EPI == kEpiLatentQuery && g0 >= g1) {  // the CTA without rows
+            pdl_wait();
+            latent_norm_to_cache<kGemvLdgThreads>(a.lat, a.st, a.seq_len, red, tid);
+            return;
+        }
         first_group = g0 / a.group_pairs;
         const int n_groups = (g1 - 1) / a.group_pairs - first_group + 1;
         Kx = n_groups * a.K;
         stage_input_groups<WT, EPI, kGemvLdgThreads>(a, xs, tid, first_group, n_groups);
     } else {
-        stage_input<WT, kGemvLdgThreads>(a, xs, red, tid);
+        stage_input<WT, kGemvLdgThreads, LN>(a, xs, red, tid);
     }
     const unsigned char* W = reinterpret_cast<const unsigned char*>(a.W);
     const size_t row_bytes = (size_t)a.K * sizeof(WT);

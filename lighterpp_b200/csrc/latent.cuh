@@ -11,7 +11,7 @@
 //   1. input GEMV   rows  plain queries | rotated queries | latent | rotated key part | gates  (all read the same
 //                   normed input): plain queries and raw latent to FP32 buffers, rotated parts turned and stored where
 //                   they belong, gates through the sigmoid
-//   2. query GEMV   per head: W_uk^T q_plain into the head's query row; one CTA norms the latent into the cache row
+//   2. query GEMV   per head: W_uk^T q_plain into the head's query row; one more CTA norms the latent into the cache row
 //   3. attention    splits over the keys of the window, partial results with their maximum and sum
 //   4. value GEMV   per head: puts the splits together, W_uv times the result, times the head's gate
 //   5. output GEMV  with the residual, like every other mixer

@@ -112,9 +112,6 @@ __device__ __forceinline__ void mma_f16_16816(float (&d)[4], uint32_t a0, uint32
                  : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void ldmatrix_x2(uint32_t addr, uint32_t& r0, uint32_t& r1) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
-}
 __device__ __forceinline__ void ldmatrix_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
 }
@@ -263,11 +260,14 @@ __device__ __forceinline__ void umma_epilogue(const PrefillGemmArgs& a, int spli
     } else if constexpr (EPI == kPfLatentValue) {
         T* p = reinterpret_cast<T*>(a.hb) + (size_t)t0 * a.hb_pitch + (size_t)group * a.n_valid + row;
         const float* gate = a.gate + (size_t)t0 * a.groups + group;
+        float gt[32];  // requested together: one round trip, not one per token
+#pragma unroll
+        for (int i = 0; i < 32; ++i) gt[i] = i < nt ? gate[(size_t)i * a.groups] : 0.f;
 #pragma unroll
         for (int i = 0; i < 32; ++i)
             if (row < a.n_valid && i < nt) {
                 T hi, lo;
-                split_pair(v[i] * gate[(size_t)i * a.groups], hi, lo);
+                split_pair(v[i] * gt[i], hi, lo);
                 p[(size_t)i * a.hb_pitch] = hi;
                 p[(size_t)(kPrefillTokens + i) * a.hb_pitch] = lo;
             }
