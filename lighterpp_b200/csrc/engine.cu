@@ -232,19 +232,32 @@ struct lpp_engine {
 static size_t align_up(size_t v, size_t a) { return (v + a - 1) / a * a; }
 
 template <typename... KArgs, typename... Args>
-static cudaError_t launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s,
-                                 bool pdl, Args... args) {
+static cudaError_t launch_clusters(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s,
+                                   bool pdl, int cluster_x, Args... args) {
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = block;
     cfg.dynamicSmemBytes = smem;
     cfg.stream = s;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cudaLaunchAttribute attr[2];
     cfg.attrs = attr;
-    cfg.numAttrs = pdl ? 1 : 0;
+    cfg.numAttrs = 0;
+    if (pdl) {
+        attr[cfg.numAttrs].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[cfg.numAttrs++].val.programmaticStreamSerializationAllowed = 1;
+    }
+    if (cluster_x > 0) {  // CTAs of a cluster, along x
+        attr[cfg.numAttrs].id = cudaLaunchAttributeClusterDimension;
+        attr[cfg.numAttrs].val.clusterDim.x = (unsigned)cluster_x;
+        attr[cfg.numAttrs].val.clusterDim.y = 1;
+        attr[cfg.numAttrs++].val.clusterDim.z = 1;
+    }
     return cudaLaunchKernelEx(&cfg, kernel, args...);
+}
+template <typename... KArgs, typename... Args>
+static cudaError_t launch_kernel(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t s,
+                                 bool pdl, Args... args) {
+    return launch_clusters(kernel, grid, block, smem, s, pdl, 0, args...);
 }
 
 // ---- GEMV dispatch
@@ -407,40 +420,63 @@ static bool attn_mma_supported(const lpp_engine* e) {
 
 // ---- latent attention: the tensor-core kernel where query and key tiles fit shared memory, else the CUDA-core kernel
 
-constexpr int kLatMinChunk = 64;  // fewest keys worth a split of their own
-// Splits the step launches: as many as the window (or the cache) can fill.
-static int latent_decode_splits(const lpp_engine* e, const LatentLayer& y) {
-    const int keys = y.d.window > 0 ? std::min(y.d.window, e->c.seq_len) : e->c.seq_len;
-    return std::max(1, std::min(kLatentMaxSplits, (keys + kLatMinChunk - 1) / kLatMinChunk));
-}
+constexpr int kLatStepWarps = 8, kLatBlockWarps = 16;  // warps of an attention CTA: one token, prompt block
+constexpr int kLatMinChunk = 64;       // fewest keys worth a split of their own when splits are left apart
+constexpr int kLatClusterChunk = 32;   // ... when they meet in a cluster (prompt blocks)
+constexpr int kLatClusterKeys = 8192;  // spans beyond this take more splits than a cluster holds
+
 static bool latent_mma_supported(const lpp_engine* e, const LatentLayer& y) {
-    return e->c.kv_dtype == LPP_F16 && y.rank_pitch <= 512 && (size_t)latent_mma_smem<2>(y.row_width) <= e->smem_optin &&
+    return e->c.kv_dtype == LPP_F16 && y.rank_pitch <= 512 && (size_t)latent_mma_smem<1, kLatBlockWarps>(y.row_width) <= e->smem_optin &&
            !(e->c.flags & LPP_FLAG_LATENT_CUDA_CORES);
 }
-static int latent_tile_rows(int rows) { return rows <= 16 ? 16 : 32; }
-template <int MT, int NT>
+// How an attention launch of n_tokens is laid out: rows per tile, splits of the keys, whether the splits are a cluster.
+struct LatentPlan {
+    bool mma;
+    int tile_rows, splits, min_chunk;
+    bool cluster;
+};
+static LatentPlan latent_plan(const lpp_engine* e, const LatentLayer& y, int n_tokens) {
+    LatentPlan p = {};
+    const int rows = n_tokens * y.d.heads;
+    p.mma = latent_mma_supported(e, y);
+    // one token: tiles of 16 heads, so that as many CTAs as possible share the keys; a prompt block: 32 rows
+    p.tile_rows = !p.mma ? 1 : (n_tokens == 1 || rows <= 16 || (size_t)latent_mma_smem<2, kLatBlockWarps>(y.row_width) > e->smem_optin) ? 16 : 32;
+    const int tiles = (rows + p.tile_rows - 1) / p.tile_rows;
+    const int tile_tokens = n_tokens == 1 ? 1 : std::min(n_tokens, (p.tile_rows - 1) / y.d.heads + 2);
+    const int keys = std::min(e->c.seq_len, y.d.window > 0 ? y.d.window + tile_tokens - 1 : e->c.seq_len);
+    p.cluster = p.mma && n_tokens > 1 && keys <= kLatClusterKeys;
+    p.min_chunk = p.cluster ? kLatClusterChunk : kLatMinChunk;
+    const int fill = n_tokens == 1 ? kLatentMaxSplits : std::max(1, e->num_sms / tiles);
+    p.splits = std::max(1, std::min({kLatentMaxSplits, (keys + p.min_chunk - 1) / p.min_chunk, fill}));
+    if (p.cluster) p.splits = p.splits >= kLatentMaxCluster ? kLatentMaxCluster : p.splits >= 4 ? 4 : p.splits >= 2 ? 2 : 1;
+    return p;
+}
+
+template <int MT, int NT, int NW>
 static cudaError_t launch_latent_mma(lpp_engine* e, const LatentAttnArgs& a, int splits, bool pdl, cudaStream_t s) {
     static bool attr_done[64] = {};
     if (!attr_done[e->c.device & 63]) {
-        const cudaError_t r = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)e->smem_optin);
+        const cudaError_t r = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, NT, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)e->smem_optin);
         if (r != cudaSuccess) return r;
         attr_done[e->c.device & 63] = true;
     }
     const dim3 grid(splits, (a.n_tokens * a.heads + 16 * MT - 1) / (16 * MT));
-    return launch_kernel(latent_attn_mma_kernel<MT, NT>, grid, dim3(kLatentThreads), (size_t)latent_mma_smem<MT>(a.row_width), s, pdl, a);
+    return launch_clusters(latent_attn_mma_kernel<MT, NT, NW>, grid, dim3(32 * NW), (size_t)latent_mma_smem<MT, NW>(a.row_width), s, pdl,
+                           a.cluster ? splits : 0, a);
 }
-static cudaError_t launch_latent_attn(lpp_engine* e, const LatentLayer& y, const LatentAttnArgs& a, bool pdl, cudaStream_t s) {
-    const int splits = a.max_splits, rp = a.rank_pitch;
-    if (latent_mma_supported(e, y)) {
-        if (latent_tile_rows(a.n_tokens * a.heads) == 16)
-            return rp <= 128   ? launch_latent_mma<1, 2>(e, a, splits, pdl, s)
-                   : rp <= 256 ? launch_latent_mma<1, 4>(e, a, splits, pdl, s)
-                               : launch_latent_mma<1, 8>(e, a, splits, pdl, s);
-        return rp <= 128   ? launch_latent_mma<2, 4>(e, a, splits, pdl, s)
-               : rp <= 256 ? launch_latent_mma<2, 8>(e, a, splits, pdl, s)
-                           : launch_latent_mma<2, 16>(e, a, splits, pdl, s);
+static cudaError_t launch_latent_attn(lpp_engine* e, const LatentPlan& p, const LatentAttnArgs& a, bool pdl, cudaStream_t s) {
+    const int rp = a.rank_pitch;
+    if (p.mma) {
+        constexpr int S = kLatStepWarps, B = kLatBlockWarps;
+        if (a.n_tokens == 1)
+            return rp <= 128   ? launch_latent_mma<1, 2, S>(e, a, p.splits, pdl, s)
+                   : rp <= 256 ? launch_latent_mma<1, 4, S>(e, a, p.splits, pdl, s)
+                               : launch_latent_mma<1, 8, S>(e, a, p.splits, pdl, s);
+        if (p.tile_rows == 16)
+            return rp <= 256 ? launch_latent_mma<1, 2, B>(e, a, p.splits, pdl, s) : launch_latent_mma<1, 4, B>(e, a, p.splits, pdl, s);
+        return rp <= 256 ? launch_latent_mma<2, 2, B>(e, a, p.splits, pdl, s) : launch_latent_mma<2, 4, B>(e, a, p.splits, pdl, s);
     }
-    const dim3 grid(splits, a.heads, a.n_tokens);
+    const dim3 grid(p.splits, a.heads, a.n_tokens);
     const size_t smem = (size_t)(a.row_width + kLatentTile) * 4;
     if (e->c.kv_dtype == LPP_F32) return launch_kernel(latent_attn_kernel<float>, grid, dim3(kLatentThreads), smem, s, pdl, a);
     return launch_kernel(latent_attn_kernel<__half>, grid, dim3(kLatentThreads), smem, s, pdl, a);
@@ -469,13 +505,16 @@ static LatentArgs latent_args(const lpp_engine* e, const LatentLayer& y) {
     L.norm_w = y.lat_w;
     L.norm_eps = e->norm_eps;
     L.part = e->lat_part;
+    const LatentPlan p = latent_plan(e, y, 1);
     L.window = y.d.window;
-    L.max_splits = latent_decode_splits(e, y);
-    L.min_chunk = kLatMinChunk;
+    L.max_splits = p.splits;
+    L.min_chunk = p.min_chunk;
     return L;
 }
-static LatentAttnArgs latent_attn_args(const lpp_engine* e, const LatentLayer& y) {
+static LatentAttnArgs latent_attn_args(const lpp_engine* e, const LatentLayer& y, const LatentPlan& p) {
     LatentAttnArgs a = {};
+    a.cluster = p.cluster;
+    a.plane_pitch = y.val_pitch;
     a.q = e->lat_query;
     a.cache = y.cache;
     a.part = e->lat_part;
@@ -486,8 +525,8 @@ static LatentAttnArgs latent_attn_args(const lpp_engine* e, const LatentLayer& y
     a.rank_pitch = y.rank_pitch;
     a.row_width = y.row_width;
     a.window = y.d.window;
-    a.max_splits = latent_decode_splits(e, y);
-    a.min_chunk = kLatMinChunk;
+    a.max_splits = p.splits;
+    a.min_chunk = p.min_chunk;
     a.seq_len = e->c.seq_len;
     a.scale = y.d.scale;
     return a;
@@ -847,8 +886,9 @@ static void record_latent_mixer(Recorder& R, int l, float* cur) {
     q.group_pairs = y.rank_pitch / kRowsPerGroup;
     record_gemv(R, kLatQuery, kEpiLatentQuery, q);
     if (!kind_skipped(e, kAttn)) {
+        const LatentPlan p = latent_plan(e, y, 1);
         R.mark(kAttn);
-        R.check(launch_latent_attn(e, y, latent_attn_args(e, y), R.pdl(), R.s), "latent attention launch");
+        R.check(launch_latent_attn(e, p, latent_attn_args(e, y, p), R.pdl(), R.s), "latent attention launch");
         R.mark(-1);
         R.prev_kernel = true;
         R.kernels++;
@@ -1869,14 +1909,6 @@ static lpp_status allow_gemm_smem() {
     return LPP_OK;
 }
 
-// Key splits of a prompt block's attention: enough CTAs for about one wave.
-static int latent_prefill_splits(const lpp_engine* e, const LatentLayer& y, int tokens) {
-    const int rows = tokens * y.d.heads;
-    const int tiles = latent_mma_supported(e, y) ? (rows + latent_tile_rows(rows) - 1) / latent_tile_rows(rows) : rows;
-    const int keys = std::min(e->c.seq_len, y.d.window > 0 ? y.d.window + latent_tile_rows(rows) / y.d.heads + 1 : e->c.seq_len);
-    return std::max(1, std::min({kLatentMaxSplits, (keys + kLatMinChunk - 1) / kLatMinChunk, e->num_sms / tiles}));
-}
-
 static lpp_status prefill_setup(lpp_engine* e) {
     if (e->pf_ready) return LPP_OK;
     const lpp_config& c = e->c;
@@ -1893,8 +1925,10 @@ static lpp_status prefill_setup(lpp_engine* e) {
         qn_n = std::max(qn_n, H * y.dim_pitch);
         olat_n = std::max(olat_n, H * y.val_pitch);
         lq_n = std::max(lq_n, H * y.row_width);
-        for (size_t t = 1; t <= T; ++t)
-            lpart_n = std::max(lpart_n, t * H * latent_prefill_splits(e, y, (int)t) * (y.rank_pitch + kLatentPartTail));
+        for (size_t t = 1; t <= T; ++t) {
+            const LatentPlan p = latent_plan(e, y, (int)t);
+            if (!p.cluster) lpart_n = std::max(lpart_n, t * H * p.splits * (y.rank_pitch + kLatentPartTail));
+        }
         gate_n = std::max(gate_n, H);
     }
     TRY(zeroed(e, &e->pf_x, T * D * 4));
@@ -2088,15 +2122,16 @@ static lpp_status prefill_latent_mixer(lpp_engine* e, int l, int n, int start_po
     q.lat_query = e->pf_lq;
     q.lat_pitch = y.row_width;
     CU((launch_prefill_gemm_t<T, kPfLatentQuery>(e, y.m_uk, y.x_qn, q)));
-    LatentAttnArgs a = latent_attn_args(e, y);
+    const LatentPlan p = latent_plan(e, y, n);
+    LatentAttnArgs a = latent_attn_args(e, y, p);
     a.q = e->pf_lq;
     a.part = e->pf_lpart;
     a.start_pos = start_pos;
     a.n_tokens = n;
-    a.max_splits = latent_prefill_splits(e, y, n);
-    CU(launch_latent_attn(e, y, a, true, e->stream));
-    const int tile_rows = latent_mma_supported(e, y) ? latent_tile_rows(n * H) : 0;
-    CU(launch_kernel(prefill_latent_combine_kernel<T>, dim3(n * H), dim3(128), 0, e->stream, true, a, tile_rows, (T*)e->pf_olat, y.val_pitch));
+    a.planes = (T*)e->pf_olat;
+    CU(launch_latent_attn(e, p, a, true, e->stream));
+    if (!p.cluster)
+        CU(launch_kernel(prefill_latent_combine_kernel<T>, dim3(n * H), dim3(128), 0, e->stream, true, a, p.tile_rows, (T*)e->pf_olat, y.val_pitch));
     PrefillGemmArgs v = prefill_gemm_args(e, y.vdim_rows, y.val_pitch, n, start_pos);
     v.groups = H;
     v.group_stride = y.vdim_rows;

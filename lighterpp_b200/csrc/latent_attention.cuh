@@ -24,8 +24,13 @@ struct LatentAttnArgs {
     int window, max_splits, min_chunk;
     int seq_len;
     float scale;
+    // Tensor-core kernel: the splits of a row tile form a cluster and put themselves together
+    int cluster;             // 0 = partial results to `part`
+    __nv_bfloat16* planes;   // then the result goes here: [2 planes][kPrefillTokens][heads * plane_pitch]
+    int plane_pitch;
 };
 
+constexpr int kLatentMaxCluster = 8;
 constexpr int kLatentTile = 64;        // keys per shared-memory tile
 constexpr int kLatentThreads = 256;
 
@@ -104,27 +109,60 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(cons
     }
 }
 
-// ---- tensor cores, FP16 rows.  grid: (splits, row tiles of 16 MT).
+// ---- tensor cores, FP16 rows.  grid: (splits, row tiles of 16 MT); with `cluster` set the splits of a row tile are one
+// thread-block cluster.
 //
-// Eight warps, MT along the query rows times WN = 8 / MT along the other direction of each product.  Query tile and
-// 64-key tiles (double buffered, 16-byte asynchronous copies) lie in shared memory in rows padded by 16 bytes.  Per tile:
-// scores by mma.sync m16n8k16 over the row width into shared memory (FP32); mask, running maximum, exponentials and sum
-// in FP32, a few rows per warp; probabilities (FP16) times the latent part of the same tile, a warp holding 16 rows x
-// NT * 8 columns of the result.
-template <int MT, int NT>
-static __global__ void __launch_bounds__(kLatentThreads) latent_attn_mma_kernel(const LatentAttnArgs a) {
-    constexpr int kRows = 16 * MT, WN = 8 / MT, kTilesW = 8 / WN;  // kTilesW: 8-key tiles of the scores per warp
-    constexpr int kScPitch = kLatentTile + 4, kPPitch = kLatentTile + 8;
+// Query tile and 64-key tiles (double buffered, 16-byte asynchronous copies) lie in shared memory in rows padded by 16
+// bytes.  Per tile: scores by mma.sync m16n8k16, the NW warps taking 16 keys (four groups) and one of NW / 4 parts of the row
+// width each, the parts to shared memory (FP32); sum of the parts, mask, running maximum, exponentials and sum in FP32, a
+// few rows per warp; probabilities (FP16) times the latent part of the same tile, every warp holding all query rows of
+// NT * 8 columns of the result.  Every key row is read from shared memory once per product, the query tile four times.
+//
+// The splits meet in one of two ways.  Prompt block: every CTA leaves its unnormalised result in its own shared memory, and
+// after a cluster barrier each adds up a share of the row tile over all CTAs through distributed shared memory; the
+// finished rows go out as hi + lo operands.  One token: partial results to part, as the CUDA-core kernel does (for 17
+// splits of 64 keys the cluster's gang launch and two barriers cost 4 us more than the value GEMV needs to add them up).
+__device__ __forceinline__ void cluster_barrier() {
+    asm volatile("barrier.cluster.arrive.release;\n\tbarrier.cluster.wait.acquire;" ::: "memory");
+}
+__device__ __forceinline__ uint32_t cluster_map(uint32_t smem_addr, uint32_t rank) {
+    uint32_t r;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(smem_addr), "r"(rank));
+    return r;
+}
+// (volatile keeps these between the barriers, which are volatile too; no memory clobber, so several are in flight at once)
+__device__ __forceinline__ float4 cluster_load4(uint32_t addr) {
+    float4 v;
+    asm volatile("ld.shared::cluster.v4.f32 {%0,%1,%2,%3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr));
+    return v;
+}
+__device__ __forceinline__ float cluster_load(uint32_t addr) {
+    float v;
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr));
+    return v;
+}
+
+constexpr int kLatScPitch = kLatentTile + 4, kLatPPitch = kLatentTile + 8;
+template <int MT, int NW>
+constexpr int latent_mma_smem(int row_width) {
+    return (16 * MT + 2 * kLatentTile) * (row_width * 2 + 16) + 16 * MT * (NW / 4 * kLatScPitch * 4 + kLatPPitch * 2 + 12 + kLatentMaxCluster * 4);
+}
+
+template <int MT, int NT, int NW>
+static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const LatentAttnArgs a) {
+    constexpr int kRows = 16 * MT, kThreads = NW * 32, kParts = NW / 4, kRowsPerWarp = kRows / NW;
     static_assert(NT % 2 == 0, "column tiles go in pairs");
+    static_assert(NW % 4 == 0 && kRows % NW == 0, "warps share the rows evenly");
     extern __shared__ __align__(128) unsigned char lm_smem[];
     const int pitch = a.row_width * 2 + 16;
     unsigned char* qs = lm_smem;
     unsigned char* kt = qs + kRows * pitch;
-    float* sc = reinterpret_cast<float*>(kt + 2 * kLatentTile * pitch);
-    __half* ps = reinterpret_cast<__half*>(sc + kRows * kScPitch);
-    float* s_m = reinterpret_cast<float*>(ps + kRows * kPPitch);
+    float* sc = reinterpret_cast<float*>(kt + 2 * kLatentTile * pitch);          // [kParts][kRows][kLatScPitch]
+    __half* ps = reinterpret_cast<__half*>(sc + kParts * kRows * kLatScPitch);  // [kRows][kLatPPitch]
+    float* s_m = reinterpret_cast<float*>(ps + kRows * kLatPPitch);
     float* s_l = s_m + kRows;
     float* s_f = s_l + kRows;
+    float* s_w = s_f + kRows;  // [kRows][kLatentMaxCluster] weights of the cluster's CTAs
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     pdl_launch_dependents();
     // the position was written by the previous step's sampler (or comes with the launch)
@@ -136,36 +174,40 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_mma_kernel(
     if (base >= 0 && base + a.n_tokens <= a.seq_len)
         sp = latent_span(base + t_lo, base + t_hi, a.window, a.max_splits, a.min_chunk);
     const int split = blockIdx.x;
-    if (split >= sp.n_eff || r0 >= n_rows) {
+    const bool active = split < sp.n_eff;
+    if (!active && !a.cluster) {
         pdl_wait();
         return;
     }
     const int k_begin = sp.first + split * sp.chunk, k_end = min(k_begin + sp.chunk, base + t_hi + 1);
-    const int n_tiles = (k_end - k_begin + kLatentTile - 1) / kLatentTile;
+    const int n_tiles = active ? (k_end - k_begin + kLatentTile - 1) / kLatentTile : 0;
     const unsigned char* cache = reinterpret_cast<const unsigned char*>(a.cache);
     const size_t row_bytes = (size_t)a.row_width * 2;
     const int pieces = a.row_width / 8;
 
-    // rows of the tile in [lo, hi); rows at or beyond k_end are filled with zeros when `fill` is set
+    // rows of the tile in [lo, hi); with `fill` the rows between k_end and the next multiple of 16 become zero
     auto load_keys = [&](int tile, int lo, int hi, bool fill) {
         unsigned char* dst = kt + (size_t)(tile & 1) * kLatentTile * pitch;
         const int p0 = k_begin + tile * kLatentTile;
-        for (int c = tid; c < kLatentTile * pieces; c += kLatentThreads) {
-            const int r = c / pieces, col = c - r * pieces, p = p0 + r;
-            const bool in = p >= lo && p < hi, out = p >= k_end;
-            if (in || (out && fill))
-                cp_async_16(dst + (size_t)r * pitch + col * 16, in ? cache + (size_t)p * row_bytes + col * 16 : cache, in);
+        const int rows = min(kLatentTile, (k_end - p0 + 15) & ~15);
+        for (int r = warp; r < rows; r += NW) {
+            const int p = p0 + r;
+            const bool in = p >= lo && p < hi;
+            if (!in && !(fill && p >= k_end)) continue;
+            const unsigned char* src = in ? cache + (size_t)p * row_bytes : cache;
+            for (int col = lane; col < pieces; col += 32) cp_async_16(dst + r * pitch + col * 16, src + (in ? col * 16 : 0), in);
         }
     };
     // cache rows of earlier steps and blocks do not depend on the preceding kernels
-    load_keys(0, k_begin, min(k_end, base), false);
+    if (active) load_keys(0, k_begin, min(k_end, base), false);
     pdl_wait();
-    load_keys(0, max(k_begin, base), k_end, true);
-    for (int c = tid; c < kRows * pieces; c += kLatentThreads) {
-        const int r = c / pieces, col = c - r * pieces;
-        const bool in = r0 + r < n_rows;
-        cp_async_16(qs + (size_t)r * pitch + col * 16,
-                    reinterpret_cast<const unsigned char*>(a.q) + (in ? (size_t)(r0 + r) * row_bytes + col * 16 : 0), in);
+    if (active) {
+        load_keys(0, max(k_begin, base), k_end, true);
+        for (int r = warp; r < kRows; r += NW) {
+            const bool in = r0 + r < n_rows;
+            const unsigned char* src = reinterpret_cast<const unsigned char*>(a.q) + (in ? (size_t)(r0 + r) * row_bytes : 0);
+            for (int col = lane; col < pieces; col += 32) cp_async_16(qs + r * pitch + col * 16, src + (in ? col * 16 : 0), in);
+        }
     }
     cp_async_commit();
     if (tid < kRows) {
@@ -173,131 +215,215 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_mma_kernel(
         s_l[tid] = 0.f;
     }
 
-    const int mw = warp / WN, nw = warp % WN;
     const int g = lane >> 2, tq = lane & 3, mi = lane >> 3, mr = lane & 7;
-    float o[NT][4];
+    float o[MT][NT][4];
 #pragma unroll
-    for (int i = 0; i < NT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-    const uint32_t q_addr = smem_u32(qs) + (uint32_t)((mw * 16 + (mi & 1) * 8 + mr) * pitch + (mi >> 1) * 16);
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int i = 0; i < NT; ++i) o[m][i][0] = o[m][i][1] = o[m][i][2] = o[m][i][3] = 0.f;
     const int k_steps = a.row_width / 16;
+    const int key16 = warp & 3, part = warp >> 2;  // scores: this warp's 16 keys and its share of the k-steps
+    const int ks0 = part * k_steps / kParts, ks1 = (part + 1) * k_steps / kParts;
+    const uint32_t q_addr = smem_u32(qs) + (uint32_t)(((mi & 1) * 8 + mr) * pitch + (mi >> 1) * 16);
+    const uint32_t p_addr = smem_u32(ps) + (uint32_t)((((mi & 1) * 8 + mr) * kLatPPitch + (mi >> 1) * 8) * 2);
 
     for (int tile = 0; tile < n_tiles; ++tile) {
+        cp_async_wait<0>();
+        __syncthreads();  // this tile is here, and nobody reads the other buffer any more
         if (tile + 1 < n_tiles) {
             load_keys(tile + 1, k_begin, k_end, true);
             cp_async_commit();
-            cp_async_wait<1>();
-        } else {
-            cp_async_wait<0>();
         }
-        __syncthreads();
         const uint32_t ks = smem_u32(kt) + (uint32_t)((tile & 1) * kLatentTile * pitch);
-        {  // scores: 16 rows x kTilesW * 8 keys per warp, two accumulators per key tile (even and odd k-steps)
-            float c[kTilesW][2][4];
+        const int p0 = k_begin + tile * kLatentTile;
+        const int groups = min(kLatentTile / 16, (k_end - p0 + 15) >> 4);  // 16-key groups with keys in them
+        if (key16 < groups) {
+            float c[MT][2][4];
 #pragma unroll
-            for (int j = 0; j < kTilesW; ++j)
+            for (int m = 0; m < MT; ++m)
 #pragma unroll
-                for (int e = 0; e < 2; ++e) c[j][e][0] = c[j][e][1] = c[j][e][2] = c[j][e][3] = 0.f;
-            auto step = [&](int kk, int e) {
-                uint32_t qa[4];
-                ldmatrix_x4(q_addr + (uint32_t)kk * 32u, qa[0], qa[1], qa[2], qa[3]);
-                if constexpr (kTilesW == 1) {
-                    uint32_t b0, b1;
-                    ldmatrix_x2(ks + (uint32_t)((nw * 8 + mr) * pitch + kk * 32 + (mi & 1) * 16), b0, b1);
-                    mma_f16_16816(c[0][e], qa[0], qa[1], qa[2], qa[3], b0, b1);
-                } else {
+                for (int j = 0; j < 2; ++j) c[m][j][0] = c[m][j][1] = c[m][j][2] = c[m][j][3] = 0.f;
+            const uint32_t b_addr = ks + (uint32_t)((key16 * 16 + (mi >> 1) * 8 + mr) * pitch + (mi & 1) * 16);
+#pragma unroll 3
+            for (int kk = ks0; kk < ks1; ++kk) {
+                uint32_t b[4], qa[MT][4];
+                ldmatrix_x4(b_addr + (uint32_t)kk * 32u, b[0], b[1], b[2], b[3]);
 #pragma unroll
-                    for (int j = 0; j < kTilesW; j += 2) {
-                        uint32_t b[4];
-                        ldmatrix_x4(ks + (uint32_t)(((nw * kTilesW + j) * 8 + (mi >> 1) * 8 + mr) * pitch + kk * 32 + (mi & 1) * 16),
-                                    b[0], b[1], b[2], b[3]);
-                        mma_f16_16816(c[j][e], qa[0], qa[1], qa[2], qa[3], b[0], b[1]);
-                        mma_f16_16816(c[j + 1][e], qa[0], qa[1], qa[2], qa[3], b[2], b[3]);
-                    }
+                for (int m = 0; m < MT; ++m)
+                    ldmatrix_x4(q_addr + (uint32_t)(m * 16 * pitch) + (uint32_t)kk * 32u, qa[m][0], qa[m][1], qa[m][2], qa[m][3]);
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    mma_f16_16816(c[m][0], qa[m][0], qa[m][1], qa[m][2], qa[m][3], b[0], b[1]);
+                    mma_f16_16816(c[m][1], qa[m][0], qa[m][1], qa[m][2], qa[m][3], b[2], b[3]);
                 }
-            };
-            int kk = 0;
-#pragma unroll 4
-            for (; kk + 1 < k_steps; kk += 2) {
-                step(kk, 0);
-                step(kk + 1, 1);
             }
-            if (kk < k_steps) step(kk, 0);
 #pragma unroll
-            for (int j = 0; j < kTilesW; ++j) {
-                float* s = sc + (mw * 16 + g) * kScPitch + (nw * kTilesW + j) * 8 + 2 * tq;
-                *reinterpret_cast<float2*>(s) = make_float2(c[j][0][0] + c[j][1][0], c[j][0][1] + c[j][1][1]);
-                *reinterpret_cast<float2*>(s + 8 * kScPitch) = make_float2(c[j][0][2] + c[j][1][2], c[j][0][3] + c[j][1][3]);
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int j = 0; j < 2; ++j) {
+                    float* d = sc + (part * kRows + m * 16 + g) * kLatScPitch + key16 * 16 + j * 8 + 2 * tq;
+                    *reinterpret_cast<float2*>(d) = make_float2(c[m][j][0], c[m][j][1]);
+                    *reinterpret_cast<float2*>(d + 8 * kLatScPitch) = make_float2(c[m][j][2], c[m][j][3]);
+                }
+        }
+        __syncthreads();
+        {  // mask and online softmax: kRowsPerWarp rows per warp, two keys per lane
+            const int p = p0 + lane;
+            float x0[kRowsPerWarp], x1[kRowsPerWarp], m_old[kRowsPerWarp], m_new[kRowsPerWarp], l[kRowsPerWarp];
+#pragma unroll
+            for (int i = 0; i < kRowsPerWarp; ++i) {
+                const int r = warp * kRowsPerWarp + i;
+                const int last = base + min(r0 + r, n_rows - 1) / a.heads, lo = a.window > 0 ? last - a.window + 1 : 0;
+                const float* s0 = sc + r * kLatScPitch + lane;
+                float v0 = 0.f, v1 = 0.f;
+#pragma unroll
+                for (int q = 0; q < kParts; ++q) {
+                    v0 += s0[q * kRows * kLatScPitch];
+                    v1 += s0[q * kRows * kLatScPitch + 32];
+                }
+                x0[i] = (p >= lo && p <= last && p < k_end) ? v0 * a.scale : -INFINITY;
+                x1[i] = (p + 32 >= lo && p + 32 <= last && p + 32 < k_end) ? v1 * a.scale : -INFINITY;
+                m_old[i] = s_m[r];
+                m_new[i] = fmaxf(x0[i], x1[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < kRowsPerWarp; ++i) m_new[i] = fmaxf(m_old[i], warp_max(m_new[i]));
+#pragma unroll
+            for (int i = 0; i < kRowsPerWarp; ++i) {
+                const float u = m_new[i] == -INFINITY ? 0.f : m_new[i];  // nothing visible to this row yet
+                x0[i] = __expf(x0[i] - u);
+                x1[i] = __expf(x1[i] - u);
+                m_old[i] = __expf(m_old[i] - u);  // what earlier tiles are rescaled by; exp(-inf) = 0
+                l[i] = x0[i] + x1[i];
+            }
+#pragma unroll
+            for (int i = 0; i < kRowsPerWarp; ++i) l[i] = warp_sum(l[i]);
+#pragma unroll
+            for (int i = 0; i < kRowsPerWarp; ++i) {
+                const int r = warp * kRowsPerWarp + i;
+                ps[r * kLatPPitch + lane] = __float2half_rn(x0[i]);
+                ps[r * kLatPPitch + lane + 32] = __float2half_rn(x1[i]);
+                if (lane == 0) {
+                    s_f[r] = m_old[i];
+                    s_l[r] = s_l[r] * m_old[i] + l[i];
+                    s_m[r] = m_new[i];
+                }
             }
         }
         __syncthreads();
-        // mask and online softmax: 2 MT rows per warp, two keys per lane
-        const int p = k_begin + tile * kLatentTile + lane;
 #pragma unroll
-        for (int i = 0; i < 2 * MT; ++i) {
-            const int r = warp * 2 * MT + i;
-            const int row = min(r0 + r, n_rows - 1);
-            const int last = base + row / a.heads, lo = a.window > 0 ? last - a.window + 1 : 0;
-            const float x0 = (p >= lo && p <= last && p < k_end) ? sc[r * kScPitch + lane] * a.scale : -INFINITY;
-            const float x1 = (p + 32 >= lo && p + 32 <= last && p + 32 < k_end) ? sc[r * kScPitch + lane + 32] * a.scale : -INFINITY;
-            const float m_old = s_m[r], m = fmaxf(m_old, warp_max(fmaxf(x0, x1)));
-            const float u = m == -INFINITY ? 0.f : m;  // nothing visible to this row yet
-            const float p0 = __expf(x0 - u), p1 = __expf(x1 - u);
-            const float l = warp_sum(p0 + p1);
-            ps[r * kPPitch + lane] = __float2half_rn(p0);
-            ps[r * kPPitch + lane + 32] = __float2half_rn(p1);
-            __syncwarp();
-            if (lane == 0) {
-                const float f = __expf(m_old - u);  // exp(-inf) = 0
-                s_f[r] = f;
-                s_l[r] = s_l[r] * f + l;
-                s_m[r] = m;
+        for (int m = 0; m < MT; ++m) {
+            const float f0 = s_f[m * 16 + g], f1 = s_f[m * 16 + g + 8];
+#pragma unroll
+            for (int i = 0; i < NT; ++i) {
+                o[m][i][0] *= f0;
+                o[m][i][1] *= f0;
+                o[m][i][2] *= f1;
+                o[m][i][3] *= f1;
             }
-        }
-        __syncthreads();
-        const float f0 = s_f[mw * 16 + g], f1 = s_f[mw * 16 + g + 8];
-#pragma unroll
-        for (int i = 0; i < NT; ++i) {
-            o[i][0] *= f0;
-            o[i][1] *= f0;
-            o[i][2] *= f1;
-            o[i][3] *= f1;
         }
 #pragma unroll
         for (int kk = 0; kk < kLatentTile / 16; ++kk) {
-            uint32_t pa[4];
-            ldmatrix_x4(smem_u32(ps) + (uint32_t)(((mw * 16 + (mi & 1) * 8 + mr) * kPPitch + kk * 16 + (mi >> 1) * 8) * 2), pa[0], pa[1],
-                        pa[2], pa[3]);
+            if (kk >= groups) break;
+            uint32_t pa[MT][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+                ldmatrix_x4(p_addr + (uint32_t)((m * 16 * kLatPPitch + kk * 16) * 2), pa[m][0], pa[m][1], pa[m][2], pa[m][3]);
 #pragma unroll
             for (int dp = 0; dp < NT / 2; ++dp) {
-                const int col = nw * NT * 8 + dp * 16;
+                const int col = warp * NT * 8 + dp * 16;
                 if (col < a.rank_pitch) {  // the same for the whole warp
                     uint32_t b[4];
                     ldmatrix_x4_trans(b, ks + (uint32_t)((kk * 16 + (mi & 1) * 8 + mr) * pitch + (col + (mi >> 1) * 8) * 2));
-                    mma_f16_16816(o[2 * dp], pa[0], pa[1], pa[2], pa[3], b[0], b[1]);
-                    mma_f16_16816(o[2 * dp + 1], pa[0], pa[1], pa[2], pa[3], b[2], b[3]);
+#pragma unroll
+                    for (int m = 0; m < MT; ++m) {
+                        mma_f16_16816(o[m][2 * dp], pa[m][0], pa[m][1], pa[m][2], pa[m][3], b[0], b[1]);
+                        mma_f16_16816(o[m][2 * dp + 1], pa[m][0], pa[m][1], pa[m][2], pa[m][3], b[2], b[3]);
+                    }
                 }
             }
         }
-        __syncthreads();  // the buffer is refilled by the copy issued in the next iteration
     }
-    const int stride = a.rank_pitch + kLatentPartTail;
+    __syncthreads();
+    if (!a.cluster) {
+        const int stride = a.rank_pitch + kLatentPartTail;
 #pragma unroll
-    for (int half = 0; half < 2; ++half) {
-        const int r = mw * 16 + g + 8 * half;
-        if (r0 + r >= n_rows) continue;
-        float* dst = a.part + ((size_t)(r0 + r) * a.max_splits + split) * stride;
+        for (int m = 0; m < MT; ++m)
 #pragma unroll
-        for (int i = 0; i < NT; ++i) {
-            const int col = nw * NT * 8 + i * 8 + 2 * tq;
-            if (col < a.rank_pitch) *reinterpret_cast<float2*>(dst + col) = make_float2(o[i][2 * half], o[i][2 * half + 1]);
+            for (int half = 0; half < 2; ++half) {
+                const int r = m * 16 + g + 8 * half;
+                if (r0 + r >= n_rows) continue;
+                float* dst = a.part + ((size_t)(r0 + r) * a.max_splits + split) * stride;
+#pragma unroll
+                for (int i = 0; i < NT; ++i) {
+                    const int col = warp * NT * 8 + i * 8 + 2 * tq;
+                    if (col < a.rank_pitch) *reinterpret_cast<float2*>(dst + col) = make_float2(o[m][i][2 * half], o[m][i][2 * half + 1]);
+                }
+                if (warp == 0 && tq == 0) *reinterpret_cast<float2*>(dst + a.rank_pitch) = make_float2(s_m[r], s_l[r]);
+            }
+        return;
+    }
+    // this CTA's result over the key tiles (nobody reads them any more), rows of rank_pitch + 4 floats: that fits, as
+    // 16 MT rows of 4 bytes are no more than 2 x 64 rows of 2 bytes
+    float* os = reinterpret_cast<float*>(kt);
+    const int o_pitch = a.rank_pitch + 4;
+    if (active) {
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                float* dst = os + (m * 16 + g + 8 * half) * o_pitch;
+#pragma unroll
+                for (int i = 0; i < NT; ++i) {
+                    const int col = warp * NT * 8 + i * 8 + 2 * tq;
+                    if (col < a.rank_pitch) *reinterpret_cast<float2*>(dst + col) = make_float2(o[m][i][2 * half], o[m][i][2 * half + 1]);
+                }
+            }
+    }
+    cluster_barrier();
+    const int n_cta = gridDim.x, n_eff = sp.n_eff;
+    // weights of the CTAs, eight lanes per row: exp(m_c - max m) / sum of l
+    for (int i = tid; i < kRows * kLatentMaxCluster; i += kThreads) {
+        const int r = i / kLatentMaxCluster, c = i % kLatentMaxCluster;
+        float m = -INFINITY, l = 0.f;
+        if (c < n_eff) {
+            m = cluster_load(cluster_map(smem_u32(s_m + r), c));
+            l = cluster_load(cluster_map(smem_u32(s_l + r), c));
         }
-        if (nw == 0 && tq == 0) *reinterpret_cast<float2*>(dst + a.rank_pitch) = make_float2(s_m[r], s_l[r]);
+        float mm = m;
+#pragma unroll
+        for (int d = kLatentMaxCluster / 2; d > 0; d >>= 1) mm = fmaxf(mm, __shfl_xor_sync(0xffffffffu, mm, d));
+        const float e = c < n_eff ? __expf(m - mm) : 0.f;
+        float sum = e * l;
+#pragma unroll
+        for (int d = kLatentMaxCluster / 2; d > 0; d >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, d);
+        s_w[i] = __fdiv_rn(e, sum);
     }
-}
-
-template <int MT>
-constexpr int latent_mma_smem(int row_width) {
-    return (16 * MT + 2 * kLatentTile) * (row_width * 2 + 16) + 16 * MT * ((kLatentTile + 4) * 4 + (kLatentTile + 8) * 2 + 12);
+    __syncthreads();
+    const int q4 = a.rank_pitch >> 2, rows_here = min(kRows, n_rows - r0);
+    for (int i = split * kThreads + tid; i < rows_here * q4; i += n_cta * kThreads) {
+        const int r = i / q4, col = (i - r * q4) << 2;
+        const uint32_t at = smem_u32(os + r * o_pitch + col);
+        float4 x[kLatentMaxCluster];
+        float y[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int c = 0; c < kLatentMaxCluster; ++c)
+            if (c < n_eff) x[c] = cluster_load4(cluster_map(at, c));
+#pragma unroll
+        for (int c = 0; c < kLatentMaxCluster; ++c)
+            if (c < n_eff) {
+                const float w = s_w[r * kLatentMaxCluster + c];
+                y[0] = fmaf(w, x[c].x, y[0]); y[1] = fmaf(w, x[c].y, y[1]); y[2] = fmaf(w, x[c].z, y[2]); y[3] = fmaf(w, x[c].w, y[3]);
+            }
+        const int t = (r0 + r) / a.heads, h = r0 + r - t * a.heads;
+        __nv_bfloat16* d = a.planes + (size_t)t * a.heads * a.plane_pitch + (size_t)h * a.plane_pitch + col;
+        __align__(8) __nv_bfloat16 hi[4], lo[4];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) split_pair(y[c], hi[c], lo[c]);
+        *reinterpret_cast<uint2*>(d) = *reinterpret_cast<const uint2*>(hi);
+        *reinterpret_cast<uint2*>(d + (size_t)kPrefillTokens * a.heads * a.plane_pitch) = *reinterpret_cast<const uint2*>(lo);
+    }
+    cluster_barrier();  // every CTA's shared memory stays until all have read it
 }
 
 // ---- prompt block: the splits of every query row put together, as hi + lo MMA operands of the value GEMM.
@@ -309,8 +435,7 @@ static __global__ void __launch_bounds__(128) prefill_latent_combine_kernel(cons
     pdl_wait();
     const int row = blockIdx.x, t = row / a.heads, h = row - t * a.heads;
     const int n_rows = a.n_tokens * a.heads;
-    // the row's tile in the attention launch (0 = the kernel that takes one row at a time)
-    const int r0 = tile_rows > 0 ? row / tile_rows * tile_rows : row, r1 = tile_rows > 0 ? min(r0 + tile_rows, n_rows) - 1 : row;
+    const int r0 = row / tile_rows * tile_rows, r1 = min(r0 + tile_rows, n_rows) - 1;  // the row's tile in the attention launch
     const LatentSpan sp = latent_span(a.start_pos + r0 / a.heads, a.start_pos + r1 / a.heads, a.window, a.max_splits, a.min_chunk);
     const int stride = a.rank_pitch + kLatentPartTail, lane = threadIdx.x & 31;
     const float* p = a.part + (size_t)row * a.max_splits * stride;

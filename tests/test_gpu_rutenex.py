@@ -250,17 +250,17 @@ def test_needle_at_the_edge_of_the_window(E, dtype, window):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_far_key_without_a_window(E, dtype):
+@pytest.mark.parametrize("n,seq_len", [(700, 700), (700, 9000), (2500, 2500)])
+def test_far_key_without_a_window(E, dtype, n, seq_len):
+    """Splits that meet in a cluster, splits left apart (a long cache), and more keys than splits of the smallest size."""
     cfg, W = needle_model(0)
-    n = 700
     toks = np.random.default_rng(0).integers(0, 79, n).astype(np.int32)
     toks[3] = 79
     want = R.forward(cfg, W, toks)
-    e = engine(E, cfg, W, dtype, seq_len=n)
-    e.extend(toks[:640], 0)
-    got = e.extend(toks[640:690], 640, range(50))
-    check(got, want[640:690], dtype)
-    check(np.stack([e.step_logits(int(toks[p]), p) for p in range(690, n)]), want[690:], dtype)
+    e = engine(E, cfg, W, dtype, seq_len=seq_len)
+    e.extend(toks[:n - 60], 0)
+    check(e.extend(toks[n - 60:n - 10], n - 60, range(50)), want[n - 60:n - 10], dtype)
+    check(np.stack([e.step_logits(int(toks[p]), p) for p in range(n - 10, n)]), want[n - 10:], dtype)
     e.close()
 
 
