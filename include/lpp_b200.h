@@ -56,7 +56,8 @@ typedef enum {
     /* Engines made by lpp_engine_create_layers only (no counterpart in the reference).  H heads with dim plain
      * and rot rotated query/key dimensions and vdim value dimensions each, latent size rank; the shared ids above keep
      * their meaning (RMS_ATT / RMS_FFN / RMS_FINAL are the norm weights before the mixer, before the feed-forward and
-     * before the classifier, WO is [D][H*vdim], W1 / W2 / W3 are gate / down / up). */
+     * before the classifier, WQ / WK are [H*dim][D] and [G*dim][D] for G key/value heads, WO is [D][mixer output], W1 / W2 /
+     * W3 are gate / down / up). */
     LPP_T_NORM1_B = 12,     /* LayerNorm bias before the mixer         [D]                    per layer */
     LPP_T_NORM2_B = 13,     /* LayerNorm bias before the feed-forward  [D]                    per layer */
     LPP_T_NORM_FINAL_B = 14,/* LayerNorm bias before the classifier    [D]                              */
@@ -66,7 +67,20 @@ typedef enum {
     LPP_T_LAT_UK = 18,      /* latent -> plain keys, head by head      [H*dim][rank]          per layer */
     LPP_T_LAT_UV = 19,      /* latent -> values, head by head          [H*vdim][rank]         per layer */
     LPP_T_LAT_G = 20,       /* output gates, one per head              [H][D]                 per layer */
-    LPP_T_COUNT = 21
+    LPP_T_WQ_B = 21,        /* bias of wq                              [H*dim]                per layer */
+    LPP_T_WK_B = 22,        /* bias of wk                              [G*dim]                per layer */
+    LPP_T_WO_B = 23,        /* bias of wo                              [D]                    per layer */
+    LPP_T_WG = 24,          /* output gates, one per element           [H*dim][D]             per layer */
+    LPP_T_SCAN_IN = 25,     /* x, then z                               [2*inner][D]           per layer */
+    LPP_T_SCAN_CONV = 26,   /* convolution of x, last = current token  [inner][conv]          per layer */
+    LPP_T_SCAN_CONV_B = 27, /* its bias                                [inner]                per layer */
+    LPP_T_SCAN_LOW = 28,    /* step (low rank), B, C                   [dt_rank+2*state][inner] per layer */
+    LPP_T_SCAN_DT = 29,     /* step of every channel                   [inner][dt_rank]       per layer */
+    LPP_T_SCAN_DT_B = 30,   /* its bias                                [inner]                per layer */
+    LPP_T_SCAN_A_LOG = 31,  /* log(-A)                                 [inner][state]         per layer */
+    LPP_T_SCAN_D = 32,      /* skip of every channel                   [inner]                per layer */
+    LPP_T_LOOP_STEP = 33,   /* added before every pass of the loop     [times][D]                       */
+    LPP_T_COUNT = 34
 } lpp_tensor;
 
 /* Engine flags (lpp_config.flags). */
@@ -103,7 +117,7 @@ typedef struct {
 
 /* A model as a list of layers, for designs whose layers differ from the reference's (or from one another).  A layer
  * is  x += mixer(norm(x)),  then  x += W2 (act(W1 norm(x)) * (W3 norm(x)))  when it has a feed-forward. */
-typedef enum { LPP_MIXER_LATENT = 1 } lpp_mixer;
+typedef enum { LPP_MIXER_LATENT = 1, LPP_MIXER_SHARED_KV = 2, LPP_MIXER_MAMBA = 3 } lpp_mixer;
 typedef enum { LPP_NORM_RMS = 0, LPP_NORM_LAYER = 1 } lpp_norm;
 typedef enum { LPP_ACT_SILU = 0, LPP_ACT_GELU_TANH = 1 } lpp_act;
 
@@ -122,6 +136,15 @@ typedef struct {
     double yarn_factor, yarn_original, yarn_fast, yarn_slow;
     int32_t ff;        /* width of the feed-forward, 0 = the layer has none */
     int32_t act;       /* lpp_act */
+    /* LPP_MIXER_SHARED_KV: grouped-query attention whose values are its keys before rotation (heads, dim, scale, window and
+     * the rotation as above; the first rot_dims dimensions of a head turn, rot_dim is not used) */
+    int32_t kv_heads;  /* divides heads; query head h takes key/value head h / (heads / kv_heads) */
+    int32_t bias;      /* 1 = biases on queries, keys and output */
+    int32_t gate;      /* 1 = the result is multiplied element by element with sigmoid(wg h) */
+    float softcap;     /* > 0: a scaled score s becomes softcap * tanh(s / softcap); 0 = none */
+    /* LPP_MIXER_MAMBA: selective scan over `inner` channels with `state` elements each, step sizes through a low-rank
+     * projection, a causal convolution over `conv` tokens before it.  Its state is recurrent: see lpp_extend. */
+    int32_t inner, state, conv, dt_rank;
 } lpp_layer_desc;
 
 typedef struct {
@@ -133,6 +156,11 @@ typedef struct {
     int32_t device;
     uint32_t flags;
     int32_t ring_kb, wait_ms;
+    float emb_scale;   /* factor of the embedding rows */
+    float logit_scale; /* factor of the logits */
+    /* Layers loop_start .. loop_stop - 1 run loop_times times in a row, each pass with a cache or state of its own and with
+     * row t of LPP_T_LOOP_STEP added to the residual stream before pass t.  loop_stop == loop_start: no loop. */
+    int32_t loop_start, loop_stop, loop_times;
 } lpp_model_desc;
 
 /* Sampling parameters of one step: forward()'s temperature / penalty arguments
@@ -211,7 +239,11 @@ lpp_status lpp_prefill(lpp_engine* e, const int* h_tokens, int n, int start_pos,
 /* One portion of a sequence with logits: runs the n tokens at positions start_pos .. from the cache that earlier calls
  * left (portions may be cut anywhere) and writes the logits of the n_want tokens want[0] < want[1] < ... (indices into
  * h_tokens) to h_logits[n_want][vocab_size].  n_want may be 0.  Single tokens go through the step graph, longer portions
- * through the batched path where the engine has one. */
+ * through the batched path where the engine has one.
+ *
+ * Models with recurrent layers: their state goes on from where it stands, so start_pos (here and in every other call that
+ * runs tokens) is the number of tokens the sequence has so far, or 0 for a new sequence; anything else, and every position
+ * but 0 after a failed or a profiling call, is LPP_ERR_INVALID_ARG. */
 lpp_status lpp_extend(lpp_engine* e, const int* h_tokens, int n, int start_pos, const int* want, int n_want, float* h_logits,
                       float* device_ms);
 
@@ -227,7 +259,8 @@ lpp_status lpp_kv_prefill(lpp_engine* e, int layer, const void* k, const void* v
                           int memkind);
 /* Read one cache row (this rank's kv heads only) as FP32; h_k / h_v hold head_size floats. */
 lpp_status lpp_kv_read(lpp_engine* e, int layer, int kv_head, int pos, float* h_k, float* h_v);
-/* Latent attention: one cache row as FP32, kv_rank latent values then rot_dim rotated key values. */
+/* Latent attention: one cache row as FP32, kv_rank latent values then rot_dim rotated key values.  layer counts layer runs in
+ * their order of execution (a layer inside a loop has one cache per pass). */
 lpp_status lpp_latent_read(lpp_engine* e, int layer, int pos, float* h_row);
 /* Element offset, inside this engine's K (or V) cache allocation, of element `off` of kv head
  * `kv_head` (rank-local numbering) at `pos`: the reference's scatter index. */
@@ -246,9 +279,9 @@ int64_t lpp_step_bytes(const lpp_engine* e, int pos);
 /* Per-kernel-kind timing of one step at `pos`: the step is captured with a CUDA event-record node
  * before and after every kernel and replayed iters times (isolated kernel durations, no programmatic
  * overlap, no host launch latency).  kinds: 0 qkv gemv, 1 attention, 2 o_proj gemv, 3 gate|up gemv, 4 down gemv,
- * 5 lm-head gemv, 6 sampler, 7 all-reduce, 8 latent query gemv, 9 latent value gemv
- * (0 is the input gemv of a latent layer).  ms[10] total device ms per step per
- * kind, launches[10] launches per step, bytes[10] algorithmic bytes per step.  The sampler runs with the
+ * 5 lm-head gemv, 6 sampler, 7 all-reduce, 8 latent query gemv, 9 latent value gemv, 10 scan's low-rank gemv, 11 selective
+ * scan (0 is the input gemv of every layer described layer by layer, 2 its output gemv).  ms[12] total device ms per step per
+ * kind, launches[12] launches per step, bytes[12] algorithmic bytes per step.  The sampler runs with the
  * temperature and penalty given in *sp (NULL = temperature 0, no penalty). */
 lpp_status lpp_profile_step(lpp_engine* e, int pos, int iters, const lpp_sample_params* sp, float* ms, int* launches,
                             int64_t* bytes);

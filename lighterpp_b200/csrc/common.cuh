@@ -106,8 +106,18 @@ __device__ __forceinline__ T from_float(float v) {
         return v;
 }
 
-// ------------------------------------------------------------------ activations of the gated feed-forward
+// What the epilogue of a row needs besides the product, fetched ahead of it.
+struct RowPrep {
+    float x = 0.f, y = 0.f, z = 0.f, w = 0.f;
+};
 
+// ------------------------------------------------------------------ activations
+
+__device__ __forceinline__ float sigmoid_f(float v) { return __fdiv_rn(1.0f, 1.0f + expf(-v)); }
+__device__ __forceinline__ float silu_f(float v) { return __fdiv_rn(v, 1.0f + expf(-v)); }
+__device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+
+// of the gated feed-forward
 enum Act : int { kActSilu = 0, kActGeluTanh = 1 };
 
 // Argument of the sigmoid that either activation multiplies its input with: silu(z) = z sigmoid(z), and because

@@ -15,8 +15,9 @@
 //   K, V cache [L][KVHl][S][hs]   FP16 (or FP32), the reference's index order
 //   rope [S][hs/2] (cos, sin)     built on the host with libm so rotations match the CPU path bit
 //                                 for bit
-// Engines made by lpp_engine_create_layers keep one allocation per matrix and layer (LatentLayer below): layers may
-// differ in every size, rows are padded with zeros to a multiple of 64 inputs.
+// Engines made by lpp_engine_create_layers keep one allocation per matrix and layer (ModelLayer below): layers may
+// differ in mixer and in every size, rows are padded with zeros to a multiple of 64 inputs.  What a sequence leaves behind
+// (cache rows, recurrent state) belongs to a run of a layer (LayerRun): a layer inside the loop has one per pass.
 #include <cuda_runtime.h>
 #include <cuda_fp16.h>
 #include <dlfcn.h>
@@ -35,10 +36,13 @@
 #include "common.cuh"
 #include "gemv.cuh"
 #include "latent_attention.cuh"
+#include "mamba.cuh"
 #include "ops.cuh"
 #include "prefill.cuh"
+#include "prefill_mixers.cuh"
 #include "sampler.cuh"
 #include "sampler_exact.cuh"
+#include "shared_kv.cuh"
 
 using namespace lpp;
 
@@ -126,23 +130,47 @@ static bool load() {
 
 // ------------------------------------------------------------------ engine
 
-enum Kind { kQkv = 0, kAttn = 1, kOproj = 2, kGateUp = 3, kDown = 4, kLmHead = 5, kSampler = 6, kAllReduce = 7, kLatQuery = 8, kLatValue = 9, kKinds = 10 };
+enum Kind { kQkv = 0, kAttn = 1, kOproj = 2, kGateUp = 3, kDown = 4, kLmHead = 5, kSampler = 6, kAllReduce = 7, kLatQuery = 8, kLatValue = 9, kScanIn = 10, kScan = 11, kKinds = 12 };
 
-// One layer of latent attention with its feed-forward (latent.cuh).  Weight matrices: rows x pitch, pitch = inputs rounded
-// up to 64, zero padded; element type = weight_dtype.
-struct LatentLayer {
+// One layer of an engine described layer by layer.  Weight matrices: rows x pitch, pitch = inputs rounded up to 64, zero
+// padded; element type = weight_dtype.
+struct ModelLayer {
     lpp_layer_desc d;
-    int rank_pitch, row_width;  // query / cache rows: latent part, whole
+    int in_rows;                // rows of the input matrix: everything the mixer projects its input with
+    int o_in, o_pitch, ff_pitch;  // inputs of the output projection, and of it and the down projection with padding
+    void *w_in = nullptr, *wo = nullptr, *w13 = nullptr, *w2 = nullptr;
+    float *n1w = nullptr, *n1b = nullptr, *n2w = nullptr, *n2b = nullptr, *o_b = nullptr;
+    CUtensorMap m_in, m_wo, m_w13, m_w2, x_att, x_hb;   // weights, activation blocks with this layer's widths (batched path)
+    // attention over shared rows (latent_attention.cuh): heads of a group, groups, value part and whole of a row
+    int group_heads = 0, groups = 0, rank_pitch = 0, row_width = 0;
+    const float2* rope = nullptr;
+    // latent attention (latent.cuh)
     int dim_pitch, val_pitch;   // inputs per head of the query and of the value matrix
     int vdim_rows;              // rows per head of the value matrix
-    int o_pitch, ff_pitch;      // inputs of the output projection and of the down projection
-    int q_plain_rows, q_rot_rows, latent_rows, in_rows;
-    void *w_in = nullptr, *w_uk = nullptr, *w_uv = nullptr, *wo = nullptr, *w13 = nullptr, *w2 = nullptr;
-    float *n1w = nullptr, *n1b = nullptr, *n2w = nullptr, *n2b = nullptr, *lat_w = nullptr;
-    const float2* rope = nullptr;
-    void* cache = nullptr;      // [seq_len][row_width]
-    CUtensorMap m_in, m_uk, m_uv, m_wo, m_w13, m_w2;    // weights (batched path)
-    CUtensorMap x_qn, x_olat, x_att, x_hb;              // activation blocks with this layer's widths
+    int q_plain_rows, q_rot_rows, latent_rows;
+    void *w_uk = nullptr, *w_uv = nullptr;
+    float* lat_w = nullptr;
+    CUtensorMap m_uk, m_uv, x_qn, x_olat;
+    // attention whose values are its keys (shared_kv.cuh)
+    int head_rows, q_rows, k_rows;
+    float* qk_b = nullptr;
+    // selective scan (mamba.cuh)
+    int inner_rows, inner_pitch, low_rows, dt_pitch, state_pitch;
+    void *w_low = nullptr, *w_dt = nullptr;
+    float *conv_w = nullptr, *conv_b = nullptr, *dt_b = nullptr, *A = nullptr, *skip = nullptr;
+    CUtensorMap m_low, x_low;
+};
+// A layer in its place in the order of execution, with what it keeps of the sequence.
+struct LayerRun {
+    int layer;
+    int step_row = -1;          // row of the loop's vectors that is added before this run, -1 = none
+    void* cache = nullptr;      // [groups][seq_len][row_width]
+    float* ring = nullptr;      // convolution inputs [taps - 1][inner_rows]
+    float* S = nullptr;         // recurrent state [inner][state_pitch]
+    // vectors added with the output and with the down projection: the output's bias, and the loop's vector that comes before
+    // the next run (with the last of the two products); nullptr = none
+    const float *o_add = nullptr, *down_add = nullptr;
+    float* sum_add = nullptr;   // storage of their sum where there are both
 };
 
 struct lpp_engine {
@@ -163,7 +191,17 @@ struct lpp_engine {
     bool layer_norm = false;
     float norm_eps = 1e-5f;  // src/ops.cpp:20-32
     // layers of lpp_engine_create_layers (empty for the reference's own architecture), buffers their steps share
-    std::vector<LatentLayer> lat;
+    std::vector<ModelLayer> layers;
+    std::vector<LayerRun> runs;
+    float emb_scale = 1.f, logit_scale = 1.f;  // the latter is part of the final norm's weight and bias on the device
+    float* loop_vec = nullptr;                 // [loop_rows][Dp]
+    int loop_rows = 0;
+    // Tokens of the sequence that the recurrent state has seen (a cache can be rewritten from any position, a state goes on
+    // from where it stands or starts anew), -1 = unknown.  Stays 0 without recurrent layers.
+    bool recurrent = false;
+    int state_len = 0;
+    float *scan_x = nullptr, *scan_z = nullptr, *scan_low = nullptr;
+    unsigned int* row_counters = nullptr;
     std::vector<std::pair<lpp_layer_desc, float2*>> rope_tables;
     float *lat_qplain = nullptr, *lat_raw = nullptr, *lat_gate = nullptr, *lat_part = nullptr;
     void* lat_query = nullptr;
@@ -213,6 +251,8 @@ struct lpp_engine {
     void *pf_qn = nullptr, *pf_olat = nullptr;      // latent attention: plain queries, attended latents (hi + lo operands)
     __half* pf_lq = nullptr;                        // query rows
     float *pf_lpart = nullptr, *pf_gate = nullptr;  // attention partials, gates
+    float *pf_sx = nullptr, *pf_sz = nullptr, *pf_tail = nullptr;  // selective scan: convolved x, z, last convolution inputs
+    void* pf_sxp = nullptr;                                        // x as hi + lo operands
     CUtensorMap pf_map_wqkv, pf_map_wo, pf_map_w13, pf_map_w2, pf_map_xn, pf_map_att, pf_map_hb;
     bool pf_ready = false;
 
@@ -355,6 +395,8 @@ static cudaError_t launch_gemv(lpp_engine* e, int epi, int w_dtype, GemvArgs& a,
         LPP_GEMV_CASE(kEpiStore)
         LPP_GEMV_CASE(kEpiResid)
         LPP_GEMV_CASE(kEpiSwiglu)
+        case kEpiResidBias:
+            return w_dtype == LPP_BF16 ? launch_gemv_t<__nv_bfloat16, kEpiResidBias>(e, a, pdl, s) : launch_gemv_t<float, kEpiResidBias>(e, a, pdl, s);
         case kEpiQkv:
             return w_dtype == LPP_F16 ? launch_gemv_t<__half, kEpiQkv>(e, a, pdl, s) : launch_gemv_t<float, kEpiQkv>(e, a, pdl, s);
     }
@@ -374,6 +416,19 @@ static cudaError_t launch_gemv(lpp_engine* e, int epi, int w_dtype, GemvLatentAr
         case kEpiLatentValue: return launch_latent_gemv<kEpiLatentValue, false>(e, w_dtype, a, pdl, s);
     }
     return cudaErrorInvalidValue;
+}
+// Input projections with a row epilogue.
+template <int EPI>
+static cudaError_t launch_row_gemv(lpp_engine* e, int w_dtype, GemvArgsOf<EPI>& a, bool pdl, cudaStream_t s) {
+    if (w_dtype == LPP_BF16)
+        return a.norm_b ? launch_gemv_t<__nv_bfloat16, EPI, true>(e, a, pdl, s) : launch_gemv_t<__nv_bfloat16, EPI, false>(e, a, pdl, s);
+    return a.norm_b ? launch_gemv_t<float, EPI, true>(e, a, pdl, s) : launch_gemv_t<float, EPI, false>(e, a, pdl, s);
+}
+static cudaError_t launch_gemv(lpp_engine* e, int, int w_dtype, GemvSharedKvArgs& a, bool pdl, cudaStream_t s) {
+    return launch_row_gemv<kEpiSharedKvIn>(e, w_dtype, a, pdl, s);
+}
+static cudaError_t launch_gemv(lpp_engine* e, int, int w_dtype, GemvMambaArgs& a, bool pdl, cudaStream_t s) {
+    return launch_row_gemv<kEpiMambaIn>(e, w_dtype, a, pdl, s);
 }
 
 // ---- attention dispatch
@@ -425,7 +480,7 @@ constexpr int kLatMinChunk = 64;       // fewest keys worth a split of their own
 constexpr int kLatClusterChunk = 32;   // ... when they meet in a cluster (prompt blocks)
 constexpr int kLatClusterKeys = 8192;  // spans beyond this take more splits than a cluster holds
 
-static bool latent_mma_supported(const lpp_engine* e, const LatentLayer& y) {
+static bool latent_mma_supported(const lpp_engine* e, const ModelLayer& y) {
     return e->c.kv_dtype == LPP_F16 && y.rank_pitch <= 512 && (size_t)latent_mma_smem<1, kLatBlockWarps>(y.row_width) <= e->smem_optin &&
            !(e->c.flags & LPP_FLAG_LATENT_CUDA_CORES);
 }
@@ -435,18 +490,18 @@ struct LatentPlan {
     int tile_rows, splits, min_chunk;
     bool cluster;
 };
-static LatentPlan latent_plan(const lpp_engine* e, const LatentLayer& y, int n_tokens) {
+static LatentPlan latent_plan(const lpp_engine* e, const ModelLayer& y, int n_tokens) {
     LatentPlan p = {};
-    const int rows = n_tokens * y.d.heads;
+    const int heads = y.group_heads, rows = n_tokens * heads;  // of a group
     p.mma = latent_mma_supported(e, y);
     // one token: tiles of 16 heads, so that as many CTAs as possible share the keys; a prompt block: 32 rows
     p.tile_rows = !p.mma ? 1 : (n_tokens == 1 || rows <= 16 || (size_t)latent_mma_smem<2, kLatBlockWarps>(y.row_width) > e->smem_optin) ? 16 : 32;
-    const int tiles = (rows + p.tile_rows - 1) / p.tile_rows;
-    const int tile_tokens = n_tokens == 1 ? 1 : std::min(n_tokens, (p.tile_rows - 1) / y.d.heads + 2);
+    const int tiles = (rows + p.tile_rows - 1) / p.tile_rows * y.groups;
+    const int tile_tokens = n_tokens == 1 ? 1 : std::min(n_tokens, (p.tile_rows - 1) / heads + 2);
     const int keys = std::min(e->c.seq_len, y.d.window > 0 ? y.d.window + tile_tokens - 1 : e->c.seq_len);
     p.cluster = p.mma && n_tokens > 1 && keys <= kLatClusterKeys;
     p.min_chunk = p.cluster ? kLatClusterChunk : kLatMinChunk;
-    const int fill = n_tokens == 1 ? kLatentMaxSplits : std::max(1, e->num_sms / tiles);
+    const int fill = n_tokens > 1 ? std::max(1, e->num_sms / tiles) : y.groups == 1 ? kLatentMaxSplits : std::max(1, 2 * e->num_sms / tiles);
     p.splits = std::max(1, std::min({kLatentMaxSplits, (keys + p.min_chunk - 1) / p.min_chunk, fill}));
     if (p.cluster) p.splits = p.splits >= kLatentMaxCluster ? kLatentMaxCluster : p.splits >= 4 ? 4 : p.splits >= 2 ? 2 : 1;
     return p;
@@ -460,7 +515,7 @@ static cudaError_t launch_latent_mma(lpp_engine* e, const LatentAttnArgs& a, int
         if (r != cudaSuccess) return r;
         attr_done[e->c.device & 63] = true;
     }
-    const dim3 grid(splits, (a.n_tokens * a.heads + 16 * MT - 1) / (16 * MT));
+    const dim3 grid(splits, (a.n_tokens * a.heads + 16 * MT - 1) / (16 * MT), a.all_heads / a.heads);
     return launch_clusters(latent_attn_mma_kernel<MT, NT, NW>, grid, dim3(32 * NW), (size_t)latent_mma_smem<MT, NW>(a.row_width), s, pdl,
                            a.cluster ? splits : 0, a);
 }
@@ -476,12 +531,12 @@ static cudaError_t launch_latent_attn(lpp_engine* e, const LatentPlan& p, const 
             return rp <= 256 ? launch_latent_mma<1, 2, B>(e, a, p.splits, pdl, s) : launch_latent_mma<1, 4, B>(e, a, p.splits, pdl, s);
         return rp <= 256 ? launch_latent_mma<2, 2, B>(e, a, p.splits, pdl, s) : launch_latent_mma<2, 4, B>(e, a, p.splits, pdl, s);
     }
-    const dim3 grid(p.splits, a.heads, a.n_tokens);
+    const dim3 grid(p.splits, a.all_heads, a.n_tokens);
     const size_t smem = (size_t)(a.row_width + kLatentTile) * 4;
     if (e->c.kv_dtype == LPP_F32) return launch_kernel(latent_attn_kernel<float>, grid, dim3(kLatentThreads), smem, s, pdl, a);
     return launch_kernel(latent_attn_kernel<__half>, grid, dim3(kLatentThreads), smem, s, pdl, a);
 }
-static LatentArgs latent_args(const lpp_engine* e, const LatentLayer& y) {
+static LatentArgs latent_args(const lpp_engine* e, const ModelLayer& y, const LayerRun& r) {
     LatentArgs L = {};
     L.heads = y.d.heads;
     L.dim = y.d.dim;
@@ -501,7 +556,7 @@ static LatentArgs latent_args(const lpp_engine* e, const LatentLayer& y) {
     L.latent = e->lat_raw;
     L.gate = e->lat_gate;
     L.query = e->lat_query;
-    L.cache = y.cache;
+    L.cache = r.cache;
     L.norm_w = y.lat_w;
     L.norm_eps = e->norm_eps;
     L.part = e->lat_part;
@@ -511,19 +566,33 @@ static LatentArgs latent_args(const lpp_engine* e, const LatentLayer& y) {
     L.min_chunk = p.min_chunk;
     return L;
 }
-static LatentAttnArgs latent_attn_args(const lpp_engine* e, const LatentLayer& y, const LatentPlan& p) {
+// For one token; a prompt block overrides what differs.
+static LatentAttnArgs latent_attn_args(const lpp_engine* e, const ModelLayer& y, const LayerRun& r, const LatentPlan& p) {
     LatentAttnArgs a = {};
     a.cluster = p.cluster;
-    a.plane_pitch = y.val_pitch;
     a.q = e->lat_query;
-    a.cache = y.cache;
+    a.cache = r.cache;
     a.part = e->lat_part;
     a.st = e->st;
     a.start_pos = -1;
     a.n_tokens = 1;
-    a.heads = y.d.heads;
+    a.heads = y.group_heads;
+    a.all_heads = y.group_heads * y.groups;
     a.rank_pitch = y.rank_pitch;
     a.row_width = y.row_width;
+    if (y.d.mixer == LPP_MIXER_LATENT) {
+        a.plane_pitch = y.val_pitch;
+        a.plane_cols = y.rank_pitch;
+        a.plane_row = y.d.heads * y.val_pitch;
+    } else {  // finished rows are the output projection's input
+        a.plane_pitch = a.plane_cols = a.out_cols = y.d.dim;
+        a.plane_row = y.o_pitch;
+        a.score_skip = y.d.rot_dims / 16;
+        a.softcap = y.d.softcap;
+        a.out = e->att_out;
+        a.gate = y.d.gate ? e->lat_gate : nullptr;
+        a.counters = e->row_counters;
+    }
     a.window = y.d.window;
     a.max_splits = p.splits;
     a.min_chunk = p.min_chunk;
@@ -531,6 +600,94 @@ static LatentAttnArgs latent_attn_args(const lpp_engine* e, const LatentLayer& y
     a.scale = y.d.scale;
     return a;
 }
+
+// ---- attention whose values are its keys, selective scan
+
+// Constants and state may be read ahead of a step kernel's dependency wait when steps are separate graph launches: what
+// earlier steps wrote is then complete.
+static int step_early(const lpp_engine* e) { return (e->c.flags & LPP_FLAG_NO_GRAPH) ? 0 : 1; }
+
+static SharedKvArgs shared_kv_args(const lpp_engine* e, const ModelLayer& y, const LayerRun& r) {
+    SharedKvArgs s = {};
+    s.heads = y.d.heads;
+    s.kv_heads = y.d.kv_heads;
+    s.dim = y.d.dim;
+    s.rot = y.d.rot_dims;
+    s.head_rows = y.head_rows;
+    s.q_rows = y.q_rows;
+    s.k_rows = y.k_rows;
+    s.rank_pitch = y.rank_pitch;
+    s.row_width = y.row_width;
+    s.cache_f32 = e->c.kv_dtype == LPP_F32;
+    s.early = step_early(e);
+    s.bias = y.qk_b;
+    s.rope = y.rope;
+    s.query = e->lat_query;
+    s.cache = r.cache;
+    s.gate = e->lat_gate;
+    return s;
+}
+static MambaScanArgs mamba_scan_args(const lpp_engine* e, const ModelLayer& y, const LayerRun& r) {
+    MambaScanArgs a = {};
+    a.inner = y.d.inner;
+    a.state = y.d.state;
+    a.dt_rank = y.d.dt_rank;
+    a.state_pitch = y.state_pitch;
+    a.dt_pitch = y.dt_pitch;
+    a.low_rows = y.low_rows;
+    a.low = e->scan_low;
+    a.w_dt = y.w_dt;
+    a.dt_b = y.dt_b;
+    a.A = y.A;
+    a.D = y.skip;
+    a.S = r.S;
+    a.x = e->scan_x;
+    a.z = e->scan_z;
+    a.out = e->att_out;
+    a.st = e->st;
+    a.seq_len = e->c.seq_len;
+    a.early = step_early(e);
+    a.taps = y.d.conv;
+    a.ring = r.ring;
+    a.ring_pitch = y.inner_rows;
+    return a;
+}
+// Limits of a selective-scan layer (registers and shared memory of the scan kernels); lanes per channel and pieces of four
+// state elements per lane by the state's size.
+constexpr int kScanMaxState = 4 * 32 * 8, kScanMaxTaps = 64, kScanMaxRank = 1536;
+#define LPP_SCAN_DISPATCH(n, F)         \
+    do {                                \
+        if ((n) <= 16) return F(4, 1);  \
+        if ((n) <= 32) return F(4, 2);  \
+        if ((n) <= 64) return F(8, 2);  \
+        if ((n) <= 128) return F(16, 2);\
+        if ((n) <= 256) return F(32, 2);\
+        return F(32, 8);                \
+    } while (0)
+template <typename WT>
+static cudaError_t launch_mamba_step(const MambaScanArgs& a, bool pdl, cudaStream_t s) {
+    const size_t smem = (size_t)(a.dt_pitch + 2 * a.state_pitch) * 4;
+#define LPP_SCAN(L_, NS_)                                                                                                      \
+    launch_kernel(mamba_step_kernel<WT, L_, NS_>, dim3((a.inner + kScanStepThreads / L_ - 1) / (kScanStepThreads / L_)), \
+                  dim3(kScanStepThreads), smem, s, pdl, a)
+    LPP_SCAN_DISPATCH(a.state_pitch, LPP_SCAN);
+#undef LPP_SCAN
+}
+template <int L, int NS>
+static cudaError_t launch_mamba_scan_t(const lpp_engine* e, MambaScanArgs a, cudaStream_t s) {
+    a.tile_tokens = kPrefillTokens;
+    while (a.tile_tokens > 1 && (size_t)mamba_scan_smem<L>(a.dt_pitch, a.state_pitch, a.tile_tokens) > e->smem_optin) a.tile_tokens /= 2;
+    const size_t smem = (size_t)mamba_scan_smem<L>(a.dt_pitch, a.state_pitch, a.tile_tokens);
+    const cudaError_t r = cudaFuncSetAttribute(mamba_scan_kernel<L, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)e->smem_optin);
+    if (r != cudaSuccess) return r;
+    return launch_kernel(mamba_scan_kernel<L, NS>, dim3((a.inner + kScanChannels<L> - 1) / kScanChannels<L>), dim3(kScanThreads), smem, s, true, a);
+}
+static cudaError_t launch_mamba_scan(const lpp_engine* e, const MambaScanArgs& a, cudaStream_t s) {
+#define LPP_SCAN(L_, NS_) launch_mamba_scan_t<L_, NS_>(e, a, s)
+    LPP_SCAN_DISPATCH(a.state_pitch, LPP_SCAN);
+#undef LPP_SCAN
+}
+static int conv_smem(int taps) { return (kConvTokens + taps - 1) * kConvChannels * 4; }
 
 // ---- one decode step as a sequence of launches (captured into the graph, or run directly)
 
@@ -592,6 +749,7 @@ static void record_gemv(Recorder& R, int kind, int epi, Args a) {
     a.seq_len = e->c.seq_len;
     a.norm_eps = e->norm_eps;
     a.norm_n = e->c.dim;
+    a.emb_scale = e->emb_scale;
     R.mark(kind);
     R.check(launch_gemv(e, epi, e->c.weight_dtype, a, R.pdl(), R.s), "gemv launch");
     R.mark(-1);
@@ -786,17 +944,27 @@ static __global__ void tp_bump_kernel(unsigned int* epoch) {
 struct LayerView {
     const void *wo, *w13, *w2;
     const float *norm2_w, *norm2_b;
+    const float *o_add, *down_add;  // added with the output and the down projection, nullptr = nothing
     int o_k, ff, ff_k;  // inputs of the output projection; feed-forward width (0 = none), inputs of the down projection
     int act;
 };
-static LayerView layer_view(const lpp_engine* e, int l) {
-    if (!e->lat.empty()) {
-        const LatentLayer& y = e->lat[l];
-        return {y.wo, y.w13, y.w2, y.n2w, y.n2b, y.o_pitch, y.d.ff, y.ff_pitch, y.d.act == LPP_ACT_GELU_TANH ? kActGeluTanh : kActSilu};
+static LayerView layer_view(const lpp_engine* e, int l) {  // l: layer, or run of one
+    if (!e->layers.empty()) {
+        const LayerRun& r = e->runs[l];
+        const ModelLayer& y = e->layers[r.layer];
+        return {y.wo, y.w13, y.w2, y.n2w, y.n2b, r.o_add, r.down_add, y.o_pitch, y.d.ff, y.ff_pitch,
+                y.d.act == LPP_ACT_GELU_TANH ? kActGeluTanh : kActSilu};
     }
     const size_t D = e->c.dim, esz = e->esz;
     return {(const char*)e->wo + (size_t)l * D * e->Dq * esz, (const char*)e->w13 + (size_t)l * 2 * e->Fl * D * esz,
-            (const char*)e->w2 + (size_t)l * D * e->Fl * esz, e->rms_ffn + (size_t)l * D, nullptr, e->Dq, e->Fl, e->Fl, kActSilu};
+            (const char*)e->w2 + (size_t)l * D * e->Fl * esz, e->rms_ffn + (size_t)l * D, nullptr, nullptr, nullptr, e->Dq, e->Fl, e->Fl, kActSilu};
+}
+
+// Steps of the recorded order: layers, or their runs.
+static int n_runs(const lpp_engine* e) { return e->layers.empty() ? e->c.n_layers : (int)e->runs.size(); }
+// The loop's vector that is added before the first run, nullptr = none.
+static const float* first_add(const lpp_engine* e) {
+    return !e->runs.empty() && e->runs[0].step_row >= 0 ? e->loop_vec + (size_t)e->runs[0].step_row * e->Dp : nullptr;
 }
 
 // Grouped-query attention of the reference: fused norm + QKV GEMV + RoPE + KV scatter, split-KV flash decode.
@@ -859,12 +1027,8 @@ static void record_gqa_mixer(Recorder& R, int l, float* cur) {
     R.kernels++;
 }
 
-// Latent attention: input GEMV, query GEMV, attention over the window, value GEMV (latent.cuh).
-static void record_latent_mixer(Recorder& R, int l, float* cur) {
-    lpp_engine* e = R.e;
-    const LatentLayer& y = e->lat[l];
-    GemvLatentArgs a = {};
-    a.lat = latent_args(e, y);
+// The input projection of run l: normed residual stream (the embedding row in the first run) times the layer's input matrix.
+static void set_mixer_input(const lpp_engine* e, GemvArgs& a, const ModelLayer& y, int l, float* cur) {
     a.W = y.w_in;
     a.n_rows = y.in_rows;
     a.K = e->Dp;
@@ -872,10 +1036,75 @@ static void record_latent_mixer(Recorder& R, int l, float* cur) {
     a.norm_b = y.n1b;
     if (l == 0) {
         a.emb = e->emb;
+        a.emb_add = first_add(e);
         a.x_store = cur;
     } else {
         a.x = cur;
     }
+}
+
+template <typename F>
+static void record_launch(Recorder& R, int kind, const char* what, F launch) {
+    if (kind_skipped(R.e, kind)) return;
+    R.mark(kind);
+    R.check(launch(R.pdl()), what);
+    R.mark(-1);
+    R.prev_kernel = true;
+    R.kernels++;
+}
+
+// Attention whose values are its keys: input GEMV, attention over the window (shared_kv.cuh).
+static void record_shared_kv_mixer(Recorder& R, int l, float* cur) {
+    lpp_engine* e = R.e;
+    const LayerRun& r = e->runs[l];
+    const ModelLayer& y = e->layers[r.layer];
+    GemvSharedKvArgs a = {};
+    a.kv = shared_kv_args(e, y, r);
+    set_mixer_input(e, a, y, l, cur);
+    record_gemv(R, kQkv, kEpiSharedKvIn, a);
+    const LatentPlan p = latent_plan(e, y, 1);
+    record_launch(R, kAttn, "shared-row attention launch",
+                  [&](bool pdl) { return launch_latent_attn(e, p, latent_attn_args(e, y, r, p), pdl, R.s); });
+}
+
+// Selective scan: input GEMV with the convolution, GEMV of dt | B | C, scan (mamba.cuh).
+static void record_mamba_mixer(Recorder& R, int l, float* cur) {
+    lpp_engine* e = R.e;
+    const LayerRun& r = e->runs[l];
+    const ModelLayer& y = e->layers[r.layer];
+    GemvMambaArgs a = {};
+    a.mb.inner = y.d.inner;
+    a.mb.inner_rows = y.inner_rows;
+    a.mb.taps = y.d.conv;
+    a.mb.early = step_early(e);
+    a.mb.conv_w = y.conv_w;
+    a.mb.conv_b = y.conv_b;
+    a.mb.ring = r.ring;
+    a.mb.x = e->scan_x;
+    a.mb.z = e->scan_z;
+    set_mixer_input(e, a, y, l, cur);
+    record_gemv(R, kQkv, kEpiMambaIn, a);
+    GemvArgs g = {};
+    g.W = y.w_low;
+    g.n_rows = y.low_rows;
+    g.K = y.inner_pitch;
+    g.x = e->scan_x;
+    g.out = e->scan_low;
+    record_gemv(R, kScanIn, kEpiStore, g);
+    const MambaScanArgs m = mamba_scan_args(e, y, r);
+    record_launch(R, kScan, "selective scan launch", [&](bool pdl) {
+        return e->c.weight_dtype == LPP_BF16 ? launch_mamba_step<__nv_bfloat16>(m, pdl, R.s) : launch_mamba_step<float>(m, pdl, R.s);
+    });
+}
+
+// Latent attention: input GEMV, query GEMV, attention over the window, value GEMV (latent.cuh).
+static void record_latent_mixer(Recorder& R, int l, float* cur) {
+    lpp_engine* e = R.e;
+    const LayerRun& r = e->runs[l];
+    const ModelLayer& y = e->layers[r.layer];
+    GemvLatentArgs a = {};
+    a.lat = latent_args(e, y, r);
+    set_mixer_input(e, a, y, l, cur);
     record_gemv(R, kQkv, kEpiLatentIn, a);
     GemvLatentArgs q = {};
     q.lat = a.lat;
@@ -885,14 +1114,9 @@ static void record_latent_mixer(Recorder& R, int l, float* cur) {
     q.x = e->lat_qplain;
     q.group_pairs = y.rank_pitch / kRowsPerGroup;
     record_gemv(R, kLatQuery, kEpiLatentQuery, q);
-    if (!kind_skipped(e, kAttn)) {
-        const LatentPlan p = latent_plan(e, y, 1);
-        R.mark(kAttn);
-        R.check(launch_latent_attn(e, p, latent_attn_args(e, y, p), R.pdl(), R.s), "latent attention launch");
-        R.mark(-1);
-        R.prev_kernel = true;
-        R.kernels++;
-    }
+    const LatentPlan p = latent_plan(e, y, 1);
+    record_launch(R, kAttn, "latent attention launch",
+                  [&](bool pdl) { return launch_latent_attn(e, p, latent_attn_args(e, y, r, p), pdl, R.s); });
     GemvLatentArgs v = {};
     v.lat = a.lat;
     v.W = y.w_uv;
@@ -906,17 +1130,22 @@ static void record_latent_mixer(Recorder& R, int l, float* cur) {
 static void record_step(Recorder& R, bool with_sampler) {
     lpp_engine* e = R.e;
     const lpp_config& c = e->c;
-    const int D = e->Dp, L = c.n_layers;
+    const int D = e->Dp, L = n_runs(e);
     const size_t esz = e->esz;
     const bool tp = c.tp_size > 1;
     const bool peers = tp_peer_path(e);  // fused exchange over peer memory instead of an NCCL all-reduce
     float* cur = e->xa;
     float* oth = e->xb;
     for (int l = 0; l < L; ++l) {
-        if (!e->lat.empty())
-            record_latent_mixer(R, l, cur);
-        else
+        if (e->layers.empty()) {
             record_gqa_mixer(R, l, cur);
+        } else {
+            switch (e->layers[e->runs[l].layer].d.mixer) {
+                case LPP_MIXER_LATENT: record_latent_mixer(R, l, cur); break;
+                case LPP_MIXER_SHARED_KV: record_shared_kv_mixer(R, l, cur); break;
+                case LPP_MIXER_MAMBA: record_mamba_mixer(R, l, cur); break;
+            }
+        }
         const LayerView v = layer_view(e, l);
         {  // o_proj + residual
             GemvArgs a = {};
@@ -927,8 +1156,9 @@ static void record_step(Recorder& R, bool with_sampler) {
             a.resid = (!tp || c.tp_rank == 0) ? cur : nullptr;
             a.out = tp ? oth : cur;
             if (peers) tp_set_producer(e, a, 2 * l);
+            a.bias = v.o_add;
             set_prefetch(e, a, kOproj, l);
-            record_gemv(R, kOproj, kEpiResid, a);
+            record_gemv(R, kOproj, v.o_add ? kEpiResidBias : kEpiResid, a);
             if (tp && !peers) {
                 record_allreduce(R, oth, D);
                 std::swap(cur, oth);
@@ -958,8 +1188,9 @@ static void record_step(Recorder& R, bool with_sampler) {
             a.resid = (!tp || c.tp_rank == 0) ? cur : nullptr;
             a.out = tp ? oth : cur;
             if (peers) tp_set_producer(e, a, 2 * l + 1);
+            a.bias = v.down_add;
             set_prefetch(e, a, kDown, l);
-            record_gemv(R, kDown, kEpiResid, a);
+            record_gemv(R, kDown, v.down_add ? kEpiResidBias : kEpiResid, a);
             if (tp && !peers) {
                 record_allreduce(R, oth, D);
                 std::swap(cur, oth);
@@ -1301,15 +1532,85 @@ static lpp_status zeroed(lpp_engine* e, T** p, size_t bytes) {
     return zeroed(e, reinterpret_cast<void**>(p), bytes);
 }
 
-static lpp_status setup_latent_layer(lpp_engine* e, LatentLayer& y) {
+static bool layer_has_loop(const lpp_model_desc* m) { return m->loop_times > 0 && m->loop_stop > m->loop_start; }
+
+static lpp_status check_layer(const lpp_layer_desc& d, int l) {
+    if (d.ff < 0 || d.window < 0 || d.rot_dims < 0) return fail(LPP_ERR_INVALID_ARG, "layer %d: bad size", l);
+    if (d.act != LPP_ACT_SILU && d.act != LPP_ACT_GELU_TANH) return fail(LPP_ERR_INVALID_ARG, "layer %d: unknown activation %d", l, d.act);
+    int turnable = 0;  // dimensions of a row that can turn, columns of a cache row's value part
+    int cols = 0;
+    switch (d.mixer) {
+        case LPP_MIXER_LATENT:
+            if (d.heads <= 0 || d.dim <= 0 || d.rot_dim < 0 || d.rot_dim % 2 || d.vdim <= 0 || d.kv_rank <= 0) return fail(LPP_ERR_INVALID_ARG, "layer %d: bad size", l);
+            turnable = d.rot_dim;
+            cols = d.kv_rank;
+            break;
+        case LPP_MIXER_SHARED_KV:
+            if (d.heads <= 0 || d.kv_heads <= 0 || d.heads % d.kv_heads || d.dim <= 0 || !(d.softcap >= 0.f))
+                return fail(LPP_ERR_INVALID_ARG, "layer %d: bad size", l);
+            turnable = cols = d.dim;
+            break;
+        case LPP_MIXER_MAMBA:
+            if (d.inner <= 0 || d.state <= 0 || d.conv <= 0 || d.dt_rank <= 0) return fail(LPP_ERR_INVALID_ARG, "layer %d: bad size", l);
+            if (d.state > kScanMaxState || d.conv > kScanMaxTaps || d.dt_rank > kScanMaxRank)
+                return fail(LPP_ERR_TOO_LARGE, "layer %d: state %d, convolution %d or step rank %d", l, d.state, d.conv, d.dt_rank);
+            return LPP_OK;
+        default: return fail(LPP_ERR_INVALID_ARG, "layer %d: unknown mixer %d", l, d.mixer);
+    }
+    if (d.rot_dims % 2 || d.rot_dims > turnable) return fail(LPP_ERR_INVALID_ARG, "layer %d: rotation of %d of %d dimensions", l, d.rot_dims, turnable);
+    if (d.rot_dims > 0 && !(d.rot_base > 0.0)) return fail(LPP_ERR_INVALID_ARG, "layer %d: bad rotation base", l);
+    if (d.yarn_factor != 0.0 && !(d.yarn_factor > 0.0 && d.yarn_original > 0.0 && d.yarn_fast > 0.0 && d.yarn_slow > 0.0))
+        return fail(LPP_ERR_INVALID_ARG, "layer %d: bad rotation scaling", l);
+    if (cols > kLatentMaxPerThread * kLatentThreads) return fail(LPP_ERR_TOO_LARGE, "layer %d: %d value columns", l, cols);
+    return LPP_OK;
+}
+
+// The engine's sizes of a layer from its description.
+static void size_layer(ModelLayer& y) {
+    lpp_layer_desc& d = y.d;
+    y.ff_pitch = (int)align_up(d.ff, 64);
+    if (d.mixer == LPP_MIXER_MAMBA) {
+        y.inner_rows = (int)align_up(d.inner, 2);
+        y.inner_pitch = (int)align_up(d.inner, 64);
+        y.low_rows = (int)align_up((size_t)d.dt_rank + 2 * d.state, 2);
+        y.dt_pitch = (int)align_up(d.dt_rank, 8);
+        y.state_pitch = (int)align_up(d.state, 4);
+        y.in_rows = 2 * y.inner_rows;
+        y.o_in = d.inner;
+    } else if (d.mixer == LPP_MIXER_SHARED_KV) {
+        d.rot_dim = d.rot_dims;  // only what turns has a column of its own
+        y.group_heads = d.heads / d.kv_heads;
+        y.groups = d.kv_heads;
+        y.rank_pitch = (int)align_up(d.dim, 16);
+        y.row_width = y.rank_pitch + (int)align_up(d.rot_dim, 16);
+        y.head_rows = (int)align_up(d.dim, 2);
+        y.q_rows = d.heads * y.head_rows;
+        y.k_rows = d.kv_heads * y.head_rows;
+        y.in_rows = y.q_rows + y.k_rows + (d.gate ? y.q_rows : 0);
+        y.o_in = d.heads * d.dim;
+    } else {
+        y.group_heads = d.heads;
+        y.groups = 1;
+        y.rank_pitch = (int)align_up(d.kv_rank, 16);
+        y.row_width = y.rank_pitch + (int)align_up(d.rot_dim, 16);
+        y.dim_pitch = (int)align_up(d.dim, 64);
+        y.val_pitch = (int)align_up(d.kv_rank, 64);
+        y.vdim_rows = (int)align_up(d.vdim, 2);
+        y.q_plain_rows = (int)align_up((size_t)d.heads * d.dim, 2);
+        y.q_rot_rows = d.heads * d.rot_dim;
+        y.latent_rows = (int)align_up(d.kv_rank, 2);
+        y.in_rows = y.q_plain_rows + y.q_rot_rows + y.latent_rows + d.rot_dim + (int)align_up(d.heads, 2);
+        y.o_in = d.heads * d.vdim;
+    }
+    y.o_pitch = (int)align_up(y.o_in, 64);
+}
+
+static lpp_status setup_layer(lpp_engine* e, ModelLayer& y) {
     const lpp_layer_desc& d = y.d;
     const size_t D2 = align_up(e->c.dim, 2), Dp = e->Dp, esz = e->esz;
     TRY(zeroed(e, &y.w_in, (size_t)y.in_rows * Dp * esz));
-    TRY(zeroed(e, &y.w_uk, (size_t)d.heads * y.rank_pitch * y.dim_pitch * esz));
-    TRY(zeroed(e, &y.w_uv, (size_t)d.heads * y.vdim_rows * y.val_pitch * esz));
     TRY(zeroed(e, &y.wo, D2 * y.o_pitch * esz));
     TRY(zeroed(e, &y.n1w, Dp * 4));
-    TRY(zeroed(e, &y.lat_w, (size_t)y.rank_pitch * 4));
     if (e->layer_norm) TRY(zeroed(e, &y.n1b, Dp * 4));
     if (d.ff > 0) {
         TRY(zeroed(e, &y.w13, (size_t)2 * d.ff * Dp * esz));
@@ -1317,8 +1618,58 @@ static lpp_status setup_latent_layer(lpp_engine* e, LatentLayer& y) {
         TRY(zeroed(e, &y.n2w, Dp * 4));
         if (e->layer_norm) TRY(zeroed(e, &y.n2b, Dp * 4));
     }
-    TRY(zeroed(e, &y.cache, (size_t)e->c.seq_len * y.row_width * e->kvesz));
+    if (d.mixer == LPP_MIXER_MAMBA) {
+        TRY(zeroed(e, &y.w_low, (size_t)y.low_rows * y.inner_pitch * esz));
+        TRY(zeroed(e, &y.w_dt, (size_t)d.inner * y.dt_pitch * esz));
+        TRY(zeroed(e, &y.conv_w, (size_t)d.conv * y.inner_rows * 4));
+        TRY(zeroed(e, &y.conv_b, (size_t)y.inner_rows * 4));
+        TRY(zeroed(e, &y.dt_b, (size_t)d.inner * 4));
+        TRY(zeroed(e, &y.A, (size_t)d.inner * y.state_pitch * 4));
+        TRY(zeroed(e, &y.skip, (size_t)d.inner * 4));
+        return LPP_OK;
+    }
+    if (d.mixer == LPP_MIXER_LATENT) {
+        TRY(zeroed(e, &y.w_uk, (size_t)d.heads * y.rank_pitch * y.dim_pitch * esz));
+        TRY(zeroed(e, &y.w_uv, (size_t)d.heads * y.vdim_rows * y.val_pitch * esz));
+        TRY(zeroed(e, &y.lat_w, (size_t)y.rank_pitch * 4));
+    } else {
+        TRY(zeroed(e, &y.qk_b, (size_t)(y.q_rows + y.k_rows) * 4));
+        if (d.bias) TRY(zeroed(e, &y.o_b, Dp * 4));
+    }
     return rope_table(e, d, &y.rope);
+}
+static lpp_status setup_run(lpp_engine* e, LayerRun& r) {
+    const ModelLayer& y = e->layers[r.layer];
+    if (y.d.mixer == LPP_MIXER_MAMBA) {
+        TRY(zeroed(e, &r.ring, (size_t)(y.d.conv - 1) * y.inner_rows * 4));
+        return zeroed(e, &r.S, (size_t)y.d.inner * y.state_pitch * 4);
+    }
+    return zeroed(e, &r.cache, (size_t)y.groups * e->c.seq_len * y.row_width * e->kvesz);
+}
+
+// What every run adds to the residual stream besides its products: the output's bias, and before a pass of the loop the
+// loop's vector, which the run before it adds with its last product.
+static lpp_status set_run_adds(lpp_engine* e) {
+    for (size_t i = 0; i < e->runs.size(); ++i) {
+        LayerRun& r = e->runs[i];
+        const ModelLayer& y = e->layers[r.layer];
+        const int row = i + 1 < e->runs.size() ? e->runs[i + 1].step_row : -1;
+        const float* next = row >= 0 ? e->loop_vec + (size_t)row * e->Dp : nullptr;
+        r.o_add = y.o_b;
+        r.down_add = nullptr;
+        if (!next) continue;
+        if (y.d.ff > 0) {
+            r.down_add = next;
+        } else if (!y.o_b) {
+            r.o_add = next;
+        } else {
+            if (!r.sum_add) TRY(zeroed(e, &r.sum_add, (size_t)e->Dp * 4));
+            residual_add_kernel<<<(e->Dp + 255) / 256, 256, 0, e->stream>>>(r.sum_add, y.o_b, next, e->Dp);
+            CU(cudaGetLastError());
+            r.o_add = r.sum_add;
+        }
+    }
+    return LPP_OK;
 }
 
 extern "C" lpp_status lpp_engine_create_layers(const lpp_model_desc* m, const lpp_layer_desc* layers, lpp_engine** out) {
@@ -1329,19 +1680,10 @@ extern "C" lpp_status lpp_engine_create_layers(const lpp_model_desc* m, const lp
     if (!((m->weight_dtype == LPP_BF16 && m->kv_dtype == LPP_F16) || (m->weight_dtype == LPP_F32 && m->kv_dtype == LPP_F32)))
         return fail(LPP_ERR_INVALID_ARG, "weights / cache must be BF16 / F16 or F32 / F32");
     if (m->norm != LPP_NORM_RMS && m->norm != LPP_NORM_LAYER) return fail(LPP_ERR_INVALID_ARG, "unknown norm %d", m->norm);
-    for (int l = 0; l < m->n_layers; ++l) {
-        const lpp_layer_desc& d = layers[l];
-        if (d.mixer != LPP_MIXER_LATENT) return fail(LPP_ERR_INVALID_ARG, "layer %d: unknown mixer %d", l, d.mixer);
-        if (d.heads <= 0 || d.dim <= 0 || d.rot_dim < 0 || d.vdim <= 0 || d.kv_rank <= 0 || d.window < 0 || d.ff < 0)
-            return fail(LPP_ERR_INVALID_ARG, "layer %d: bad size", l);
-        if (d.rot_dim % 2 || d.rot_dims % 2 || d.rot_dims < 0 || d.rot_dims > d.rot_dim)
-            return fail(LPP_ERR_INVALID_ARG, "layer %d: rotation of %d of %d dimensions", l, d.rot_dims, d.rot_dim);
-        if (d.rot_dims > 0 && !(d.rot_base > 0.0)) return fail(LPP_ERR_INVALID_ARG, "layer %d: bad rotation base", l);
-        if (d.yarn_factor != 0.0 && !(d.yarn_factor > 0.0 && d.yarn_original > 0.0 && d.yarn_fast > 0.0 && d.yarn_slow > 0.0))
-            return fail(LPP_ERR_INVALID_ARG, "layer %d: bad rotation scaling", l);
-        if (d.act != LPP_ACT_SILU && d.act != LPP_ACT_GELU_TANH) return fail(LPP_ERR_INVALID_ARG, "layer %d: unknown activation %d", l, d.act);
-        if (d.kv_rank > kLatentMaxPerThread * kLatentThreads) return fail(LPP_ERR_TOO_LARGE, "layer %d: kv_rank %d", l, d.kv_rank);
-    }
+    if (m->loop_times < 0 || m->loop_start < 0 || m->loop_stop < m->loop_start || m->loop_stop > m->n_layers ||
+        (m->loop_times == 0 && m->loop_stop > m->loop_start))
+        return fail(LPP_ERR_INVALID_ARG, "layers %d .. %d, %d times: not a loop of %d layers", m->loop_start, m->loop_stop, m->loop_times, m->n_layers);
+    for (int l = 0; l < m->n_layers; ++l) TRY(check_layer(layers[l], l));
     cudaDeviceProp prop;
     TRY(open_device(m->device, &prop));
     lpp_engine* e = new lpp_engine();
@@ -1366,6 +1708,8 @@ extern "C" lpp_status lpp_engine_create_layers(const lpp_model_desc* m, const lp
     e->Vp = (int)align_up(c.vocab_size, 2);
     e->layer_norm = m->norm == LPP_NORM_LAYER;
     e->norm_eps = m->norm_eps;
+    e->emb_scale = m->emb_scale;
+    e->logit_scale = m->logit_scale;
     e->sample_blocks = (c.vocab_size + kSampleChunk - 1) / kSampleChunk;
     e->got.assign((size_t)LPP_T_COUNT * c.n_layers, 0);
     auto bail = [&](lpp_status s) {
@@ -1374,29 +1718,36 @@ extern "C" lpp_status lpp_engine_create_layers(const lpp_model_desc* m, const lp
     };
     if (e->sample_blocks > kSampleMaxBlocks)
         return bail(fail(LPP_ERR_TOO_LARGE, "vocab_size %d exceeds the sampler's %d", c.vocab_size, kSampleMaxBlocks * kSampleChunk));
-    e->lat.resize(c.n_layers);
-    size_t att_n = 64, hb_n = 64, qplain_n = 0, raw_n = 0, gate_n = 0, query_n = 0, part_n = 0;
+    // order of execution: the layers before the loop, its passes, the rest
+    const bool loop = layer_has_loop(m);
+    for (int l = 0; l < (loop ? m->loop_start : c.n_layers); ++l) e->runs.push_back({l});
+    if (loop) {
+        for (int t = 0; t < m->loop_times; ++t)
+            for (int l = m->loop_start; l < m->loop_stop; ++l) e->runs.push_back({l, l == m->loop_start ? t : -1});
+        for (int l = m->loop_stop; l < c.n_layers; ++l) e->runs.push_back({l});
+    }
+    e->layers.resize(c.n_layers);
+    size_t att_n = 64, hb_n = 64, qplain_n = 0, raw_n = 0, gate_n = 0, query_n = 0, part_n = 0, heads_n = 0, scan_n = 0, low_n = 0;
     for (int l = 0; l < c.n_layers; ++l) {
-        LatentLayer& y = e->lat[l];
-        const lpp_layer_desc& d = y.d = layers[l];
-        y.rank_pitch = (int)align_up(d.kv_rank, 16);
-        y.row_width = y.rank_pitch + (int)align_up(d.rot_dim, 16);
-        y.dim_pitch = (int)align_up(d.dim, 64);
-        y.val_pitch = (int)align_up(d.kv_rank, 64);
-        y.vdim_rows = (int)align_up(d.vdim, 2);
-        y.o_pitch = (int)align_up((size_t)d.heads * d.vdim, 64);
-        y.ff_pitch = (int)align_up(d.ff, 64);
-        y.q_plain_rows = (int)align_up((size_t)d.heads * d.dim, 2);
-        y.q_rot_rows = d.heads * d.rot_dim;
-        y.latent_rows = (int)align_up(d.kv_rank, 2);
-        y.in_rows = y.q_plain_rows + y.q_rot_rows + y.latent_rows + d.rot_dim + (int)align_up(d.heads, 2);
+        ModelLayer& y = e->layers[l];
+        const lpp_layer_desc& d = y.d;
+        y.d = layers[l];
+        size_layer(y);
         att_n = std::max(att_n, (size_t)y.o_pitch);
         hb_n = std::max(hb_n, (size_t)y.ff_pitch);
-        qplain_n = std::max(qplain_n, (size_t)d.heads * y.dim_pitch);
-        raw_n = std::max(raw_n, (size_t)y.latent_rows);
-        gate_n = std::max(gate_n, align_up(d.heads, 2));
+        if (d.mixer == LPP_MIXER_MAMBA) {
+            e->recurrent = true;
+            scan_n = std::max(scan_n, (size_t)y.inner_pitch);
+            low_n = std::max(low_n, (size_t)y.low_rows);
+            continue;
+        }
         query_n = std::max(query_n, (size_t)d.heads * y.row_width);
         part_n = std::max(part_n, (size_t)d.heads * kLatentMaxSplits * (y.rank_pitch + kLatentPartTail));
+        heads_n = std::max(heads_n, (size_t)d.heads);
+        gate_n = std::max(gate_n, d.mixer == LPP_MIXER_LATENT ? align_up(d.heads, 2) : (size_t)d.heads * d.dim);
+        if (d.mixer != LPP_MIXER_LATENT) continue;
+        qplain_n = std::max(qplain_n, (size_t)d.heads * y.dim_pitch);
+        raw_n = std::max(raw_n, (size_t)y.latent_rows);
     }
     auto setup = [&]() -> lpp_status {
         TRY(alloc_step_buffers(e, att_n, hb_n));
@@ -1409,7 +1760,14 @@ extern "C" lpp_status lpp_engine_create_layers(const lpp_model_desc* m, const lp
         TRY(zeroed(e, &e->lat_gate, gate_n * 4));
         TRY(zeroed(e, &e->lat_query, query_n * e->kvesz));
         TRY(zeroed(e, &e->lat_part, part_n * 4));
-        for (LatentLayer& y : e->lat) TRY(setup_latent_layer(e, y));
+        TRY(zeroed(e, &e->row_counters, heads_n * sizeof(unsigned int)));
+        TRY(zeroed(e, &e->scan_x, scan_n * 4));
+        TRY(zeroed(e, &e->scan_z, scan_n * 4));
+        TRY(zeroed(e, &e->scan_low, low_n * 4));
+        if (loop) TRY(zeroed(e, &e->loop_vec, (size_t)m->loop_times * Dp * 4));
+        e->loop_rows = loop ? m->loop_times : 0;
+        for (ModelLayer& y : e->layers) TRY(setup_layer(e, y));
+        for (LayerRun& r : e->runs) TRY(setup_run(e, r));
         CU(cudaStreamSynchronize(e->stream));
         return LPP_OK;
     };
@@ -1438,11 +1796,15 @@ extern "C" lpp_status lpp_engine_destroy(lpp_engine* e) {
                     e->r_values, e->out_tokens, e->st, e->rope, e->stage, e->gtrace, e->pf_x, e->pf_q, e->pf_part, e->pf_xn, e->pf_att, e->pf_hb,
                     e->pf_tokens, e->ex_sync, e->ex_block_sum, e->ex_entry_count, e->ex_entries, e->ex_scalars, e->final_b, e->lat_qplain,
                     e->lat_raw, e->lat_gate, e->lat_query, e->lat_part, e->pf_rows, e->pf_logits, e->pf_qn, e->pf_olat, e->pf_lq,
-                    e->pf_lpart, e->pf_gate};
+                    e->pf_lpart, e->pf_gate, e->loop_vec, e->scan_x, e->scan_z, e->scan_low, e->row_counters, e->pf_sx, e->pf_sz, e->pf_tail, e->pf_sxp};
     for (void* p : bufs)
         if (p) cudaFree(p);
-    for (const LatentLayer& y : e->lat)
-        for (void* p : {y.w_in, y.w_uk, y.w_uv, y.wo, y.w13, y.w2, (void*)y.n1w, (void*)y.n1b, (void*)y.n2w, (void*)y.n2b, (void*)y.lat_w, y.cache})
+    for (const ModelLayer& y : e->layers)
+        for (void* p : {y.w_in, y.w_uk, y.w_uv, y.wo, y.w13, y.w2, (void*)y.n1w, (void*)y.n1b, (void*)y.n2w, (void*)y.n2b, (void*)y.lat_w, (void*)y.o_b,
+                        (void*)y.qk_b, y.w_low, y.w_dt, (void*)y.conv_w, (void*)y.conv_b, (void*)y.dt_b, (void*)y.A, (void*)y.skip})
+            if (p) cudaFree(p);
+    for (const LayerRun& r : e->runs)
+        for (void* p : {r.cache, (void*)r.ring, (void*)r.S, (void*)r.sum_add})
             if (p) cudaFree(p);
     for (auto& t : e->rope_tables) cudaFree(t.second);
     if (e->h_st) cudaFreeHost(e->h_st);
@@ -1533,10 +1895,23 @@ static lpp_status put_block(lpp_engine* e, void* dst, size_t dst_pitch, int dst_
     return put_shape(e, dst, dst_dtype, (const char*)src + (r0 * src_pitch + c0) * dtype_size(src_dtype), src_dtype, memkind, b);
 }
 
-// A tensor of an engine described layer by layer, into the padded layouts of LatentLayer.
-static lpp_status upload_latent(lpp_engine* e, int which, int l, const void* src, int dt, int memkind) {
+static bool tensor_expected(const lpp_engine* e, int t, int l);
+static __global__ void scale_kernel(float* p, int n, float f) {
+    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) p[i] *= f;
+}
+// p <- -exp(p) for a block of rows x cols
+static __global__ void neg_exp_kernel(float* p, int rows, int cols, int pitch) {
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (long long)rows * cols) return;
+    float* v = p + i / cols * pitch + i % cols;
+    *v = (float)-exp((double)*v);
+}
+
+// A tensor of an engine described layer by layer, into the padded layouts of ModelLayer.
+static lpp_status upload_layered(lpp_engine* e, int which, int l, const void* src, int dt, int memkind) {
     const lpp_config& c = e->c;
-    LatentLayer& y = e->lat[l];
+    ModelLayer& y = e->layers[l];
     const lpp_layer_desc& d = y.d;
     const int D = c.dim, wd = c.weight_dtype;
     const size_t Dp = e->Dp, esz = e->esz;
@@ -1547,6 +1922,18 @@ static lpp_status upload_latent(lpp_engine* e, int which, int l, const void* src
     if (norm_bias && !e->layer_norm) return fail(LPP_ERR_INVALID_ARG, "this model's norms have no bias");
     const bool ff = which == LPP_T_RMS_FFN || which == LPP_T_NORM2_B || which == LPP_T_W1 || which == LPP_T_W2 || which == LPP_T_W3;
     if (ff && d.ff == 0) return fail(LPP_ERR_INVALID_ARG, "layer %d has no feed-forward", l);
+    if (which != LPP_T_W_CLS && !tensor_expected(e, which, l)) return fail(LPP_ERR_INVALID_ARG, "tensor id %d does not belong to this model", which);
+    auto final_vec = [&](float* dst) -> lpp_status {  // logits are linear in the last norm's output: their factor goes into its weights
+        TRY(vec(dst, D));
+        scale_kernel<<<(D + 255) / 256, 256, 0, e->stream>>>(dst, D, e->logit_scale);
+        CU(cudaGetLastError());
+        return LPP_OK;
+    };
+    // rows of heads (dim each) into sections of the input matrix, head_rows apart
+    auto heads = [&](size_t r0, int n) -> lpp_status {
+        for (int h = 0; h < n; ++h) TRY(put_block(e, in_row(r0 + (size_t)h * y.head_rows), Dp, wd, src, D, (size_t)h * d.dim, 0, d.dim, D, dt, memkind));
+        return LPP_OK;
+    };
     switch (which) {
         case LPP_T_TOK_EMB: return mat(e->emb, Dp, c.vocab_size, D);
         case LPP_T_W_CLS:
@@ -1555,8 +1942,8 @@ static lpp_status upload_latent(lpp_engine* e, int which, int l, const void* src
                 e->wcls_owned = true;
             }
             return mat(e->wcls, Dp, c.vocab_size, D);
-        case LPP_T_RMS_FINAL: return vec(e->rms_final, D);
-        case LPP_T_NORM_FINAL_B: return vec(e->final_b, D);
+        case LPP_T_RMS_FINAL: return final_vec(e->rms_final);
+        case LPP_T_NORM_FINAL_B: return final_vec(e->final_b);
         case LPP_T_RMS_ATT: return vec(y.n1w, D);
         case LPP_T_NORM1_B: return vec(y.n1b, D);
         case LPP_T_RMS_FFN: return vec(y.n2w, D);
@@ -1600,7 +1987,38 @@ static lpp_status upload_latent(lpp_engine* e, int which, int l, const void* src
                 TRY(put_block(e, (char*)y.w_uv + (size_t)h * y.vdim_rows * y.val_pitch * esz, y.val_pitch, wd, src, d.kv_rank,
                               (size_t)h * d.vdim, 0, d.vdim, d.kv_rank, dt, memkind));
             return LPP_OK;
-        case LPP_T_WO: return mat(y.wo, y.o_pitch, D, d.heads * d.vdim);
+        case LPP_T_WO: return mat(y.wo, y.o_pitch, D, y.o_in);
+        case LPP_T_LOOP_STEP: return put_block(e, e->loop_vec, Dp, LPP_F32, src, D, 0, 0, e->loop_rows, D, dt, memkind);
+        case LPP_T_WQ: return heads(0, d.heads);
+        case LPP_T_WK: return heads(y.q_rows, d.kv_heads);
+        case LPP_T_WG: return heads((size_t)y.q_rows + y.k_rows, d.heads);
+        case LPP_T_WQ_B: return put_block(e, y.qk_b, y.head_rows, LPP_F32, src, d.dim, 0, 0, d.heads, d.dim, dt, memkind);
+        case LPP_T_WK_B: return put_block(e, y.qk_b + y.q_rows, y.head_rows, LPP_F32, src, d.dim, 0, 0, d.kv_heads, d.dim, dt, memkind);
+        case LPP_T_WO_B: return vec(y.o_b, D);
+        case LPP_T_SCAN_IN:
+            TRY(put_block(e, y.w_in, Dp, wd, src, D, 0, 0, d.inner, D, dt, memkind));
+            return put_block(e, in_row(y.inner_rows), Dp, wd, src, D, d.inner, 0, d.inner, D, dt, memkind);
+        case LPP_T_SCAN_CONV: {  // [inner][taps] -> [taps][inner_rows]
+            BlockShape b;
+            b.rows = d.inner;
+            b.cols = d.conv;
+            b.src_pitch = d.conv;
+            b.dst_row = 1;
+            b.dst_col = y.inner_rows;
+            return put_shape(e, y.conv_w, LPP_F32, src, dt, memkind, b);
+        }
+        case LPP_T_SCAN_CONV_B: return vec(y.conv_b, d.inner);
+        case LPP_T_SCAN_LOW: return mat(y.w_low, y.inner_pitch, d.dt_rank + 2 * d.state, d.inner);
+        case LPP_T_SCAN_DT: return mat(y.w_dt, y.dt_pitch, d.inner, d.dt_rank);
+        case LPP_T_SCAN_DT_B: return vec(y.dt_b, d.inner);
+        case LPP_T_SCAN_D: return vec(y.skip, d.inner);
+        case LPP_T_SCAN_A_LOG: {
+            TRY(put_block(e, y.A, y.state_pitch, LPP_F32, src, d.state, 0, 0, d.inner, d.state, dt, memkind));
+            const long long n = (long long)d.inner * d.state;
+            neg_exp_kernel<<<(unsigned int)((n + 255) / 256), 256, 0, e->stream>>>(y.A, d.inner, d.state, y.state_pitch);
+            CU(cudaGetLastError());
+            return LPP_OK;
+        }
         case LPP_T_W1: return put_block(e, y.w13, 2 * Dp, wd, src, D, 0, 0, d.ff, D, dt, memkind);                      // gate -> even rows
         case LPP_T_W3: return put_block(e, (char*)y.w13 + Dp * esz, 2 * Dp, wd, src, D, 0, 0, d.ff, D, dt, memkind);  // up -> odd rows
         case LPP_T_W2: return mat(y.w2, y.ff_pitch, D, d.ff);
@@ -1610,16 +2028,28 @@ static lpp_status upload_latent(lpp_engine* e, int which, int l, const void* src
 // Whether layer l of the model has tensor t.
 static bool tensor_expected(const lpp_engine* e, int t, int l) {
     if (t == LPP_T_W_CLS) return false;  // optional
-    if (e->lat.empty()) return t < LPP_T_NORM1_B;
+    if (e->layers.empty()) return t < LPP_T_NORM1_B;
+    const lpp_layer_desc& d = e->layers[l].d;
     switch (t) {
-        case LPP_T_WQ: case LPP_T_WK: case LPP_T_WV: return false;
+        case LPP_T_TOK_EMB: case LPP_T_RMS_FINAL: case LPP_T_RMS_ATT: case LPP_T_WO: return true;
         case LPP_T_NORM1_B: case LPP_T_NORM_FINAL_B: return e->layer_norm;
-        case LPP_T_NORM2_B: return e->layer_norm && e->lat[l].d.ff > 0;
-        case LPP_T_RMS_FFN: case LPP_T_W1: case LPP_T_W2: case LPP_T_W3: return e->lat[l].d.ff > 0;
+        case LPP_T_NORM2_B: return e->layer_norm && d.ff > 0;
+        case LPP_T_RMS_FFN: case LPP_T_W1: case LPP_T_W2: case LPP_T_W3: return d.ff > 0;
+        case LPP_T_LOOP_STEP: return e->loop_rows > 0;
+        case LPP_T_LAT_Q: case LPP_T_LAT_DKV: case LPP_T_LAT_NORM: case LPP_T_LAT_UK: case LPP_T_LAT_UV: case LPP_T_LAT_G:
+            return d.mixer == LPP_MIXER_LATENT;
+        case LPP_T_WQ: case LPP_T_WK: return d.mixer == LPP_MIXER_SHARED_KV;
+        case LPP_T_WQ_B: case LPP_T_WK_B: case LPP_T_WO_B: return d.mixer == LPP_MIXER_SHARED_KV && d.bias;
+        case LPP_T_WG: return d.mixer == LPP_MIXER_SHARED_KV && d.gate;
+        case LPP_T_SCAN_IN: case LPP_T_SCAN_CONV: case LPP_T_SCAN_CONV_B: case LPP_T_SCAN_LOW: case LPP_T_SCAN_DT: case LPP_T_SCAN_DT_B:
+        case LPP_T_SCAN_A_LOG: case LPP_T_SCAN_D:
+            return d.mixer == LPP_MIXER_MAMBA;
     }
-    return true;
+    return false;
 }
-static bool tensor_stacked(int t) { return !(t == LPP_T_TOK_EMB || t == LPP_T_RMS_FINAL || t == LPP_T_W_CLS || t == LPP_T_NORM_FINAL_B); }
+static bool tensor_stacked(int t) {
+    return !(t == LPP_T_TOK_EMB || t == LPP_T_RMS_FINAL || t == LPP_T_W_CLS || t == LPP_T_NORM_FINAL_B || t == LPP_T_LOOP_STEP);
+}
 
 extern "C" lpp_status lpp_upload_tensor(lpp_engine* e, int which, int layer, const void* src, int src_dtype,
                                         int memkind) {
@@ -1633,8 +2063,8 @@ extern "C" lpp_status lpp_upload_tensor(lpp_engine* e, int which, int layer, con
     if (!stacked) layer = 0;
     CU(cudaSetDevice(c.device));
     TRACE("upload tensor %d layer %d", which, layer);
-    if (!e->lat.empty()) {
-        TRY(upload_latent(e, which, layer, src, src_dtype, memkind));
+    if (!e->layers.empty()) {
+        TRY(upload_layered(e, which, layer, src, src_dtype, memkind));
         e->got[(size_t)which * c.n_layers + layer] = 1;
         e->finalized = false;
         return LPP_OK;
@@ -1706,7 +2136,8 @@ extern "C" lpp_status lpp_finalize(lpp_engine* e) {
     const lpp_config& c = e->c;
     CU(cudaSetDevice(c.device));
     static const char* names[LPP_T_COUNT] = {"tok_emb", "rms_att", "wq", "wk", "wv", "wo", "rms_ffn", "w1", "w2", "w3", "rms_final", "w_cls",
-                                              "norm1_b", "norm2_b", "norm_final_b", "lat_q", "lat_dkv", "lat_norm", "lat_uk", "lat_uv", "lat_g"};
+                                              "norm1_b", "norm2_b", "norm_final_b", "lat_q", "lat_dkv", "lat_norm", "lat_uk", "lat_uv", "lat_g", "wq_b", "wk_b", "wo_b", "wg",
+                                              "scan_in", "scan_conv", "scan_conv_b", "scan_low", "scan_dt", "scan_dt_b", "scan_a_log", "scan_d", "loop_step"};
     for (int t = 0; t < LPP_T_COUNT; ++t) {
         const int n = tensor_stacked(t) ? c.n_layers : 1;
         for (int l = 0; l < n; ++l)
@@ -1723,6 +2154,8 @@ extern "C" lpp_status lpp_finalize(lpp_engine* e) {
         e->stage = nullptr;
         e->stage_bytes = 0;
     }
+    TRY(set_run_adds(e));
+    e->state_len = e->recurrent ? -1 : 0;
     for (int v = 0; v < 2; ++v) {
         if (e->g_full[v]) cudaGraphExecDestroy(e->g_full[v]), e->g_full[v] = nullptr;
         if (e->g_logits[v]) cudaGraphExecDestroy(e->g_logits[v]), e->g_logits[v] = nullptr;
@@ -1740,7 +2173,10 @@ extern "C" lpp_status lpp_finalize(lpp_engine* e) {
         TRACE("finalize: graphs captured (%d kernels per long-context step)", e->kernels_full);
     } else {
         e->kernels_full = 2 + (tp_cls_sharded(e) ? 1 : 0);
-        for (int l = 0; l < c.n_layers; ++l) e->kernels_full += (e->lat.empty() ? 2 : 4) + 1 + (layer_view(e, l).ff > 0 ? 2 : 0);
+        for (int l = 0; l < n_runs(e); ++l) {
+            const int mixer = e->layers.empty() ? 0 : e->layers[e->runs[l].layer].d.mixer;
+            e->kernels_full += (mixer == LPP_MIXER_LATENT ? 4 : mixer == LPP_MIXER_MAMBA ? 3 : 2) + 1 + (layer_view(e, l).ff > 0 ? 2 : 0);
+        }
     }
     e->finalized = true;
     return LPP_OK;
@@ -1783,6 +2219,21 @@ static lpp_status pull_result(lpp_engine* e, int* token) {
     return LPP_OK;
 }
 
+// n tokens at positions start_pos .. are about to run: a recurrent state must stand at start_pos (or start anew at 0).  Until
+// state_ran confirms that they have run, the state counts as unknown.
+static lpp_status state_runs(lpp_engine* e, int start_pos) {
+    if (!e->recurrent) return LPP_OK;
+    if (start_pos != 0 && start_pos != e->state_len)
+        return e->state_len < 0 ? fail(LPP_ERR_INVALID_ARG, "position %d: the recurrent state is not that of a sequence, start at position 0", start_pos)
+                                : fail(LPP_ERR_INVALID_ARG, "position %d: the recurrent state stands at position %d", start_pos, e->state_len);
+    e->state_len = -1;
+    return LPP_OK;
+}
+static lpp_status state_ran(lpp_engine* e, int end_pos) {
+    if (e->recurrent) e->state_len = end_pos;
+    return LPP_OK;
+}
+
 #define NEED_READY(e)                                                              \
     do {                                                                           \
         if (!(e)) return fail(LPP_ERR_INVALID_ARG, "null engine");                 \
@@ -1795,17 +2246,21 @@ extern "C" lpp_status lpp_step(lpp_engine* e, int token, int pos, const lpp_samp
     NEED_READY(e);
     if (!sp || !next_token) return fail(LPP_ERR_INVALID_ARG, "null argument");
     TRY(push_state(e, token, pos, sp, h_history, history_len, r, 0, 0));
+    TRY(state_runs(e, pos));
     TRY(run_step(e, true, pos));
-    return pull_result(e, next_token);
+    TRY(pull_result(e, next_token));
+    return state_ran(e, pos + 1);
 }
 
 extern "C" lpp_status lpp_step_logits(lpp_engine* e, int token, int pos, float* h_logits) {
     NEED_READY(e);
     if (!h_logits) return fail(LPP_ERR_INVALID_ARG, "null argument");
     TRY(push_state(e, token, pos, nullptr, nullptr, 0, 0.f, 0, 0));
+    TRY(state_runs(e, pos));
     TRY(run_step(e, false, pos));
     CU(cudaMemcpyAsync(h_logits, e->logits, (size_t)e->c.vocab_size * 4, cudaMemcpyDeviceToHost, e->stream));
-    return pull_result(e, nullptr);
+    TRY(pull_result(e, nullptr));
+    return state_ran(e, pos + 1);
 }
 
 extern "C" lpp_status lpp_decode(lpp_engine* e, int first_token, int start_pos, int n, const lpp_sample_params* sp,
@@ -1820,11 +2275,13 @@ extern "C" lpp_status lpp_decode(lpp_engine* e, int first_token, int start_pos, 
     if (sp->temperature != 0.0f && !h_r) return fail(LPP_ERR_INVALID_ARG, "temperature > 0 needs h_r");
     TRY(push_state(e, first_token, start_pos, sp, h_history, history_len, 0.f, 1, history_window));
     if (h_r) CU(cudaMemcpyAsync(e->r_values, h_r, (size_t)n * 4, cudaMemcpyHostToDevice, e->stream));
+    TRY(state_runs(e, start_pos));
     CU(cudaEventRecord(e->ev0, e->stream));
     for (int i = 0; i < n; ++i) TRY(run_step(e, true, start_pos + i));
     CU(cudaEventRecord(e->ev1, e->stream));
     CU(cudaMemcpyAsync(h_out_tokens, e->out_tokens, (size_t)n * 4, cudaMemcpyDeviceToHost, e->stream));
     TRY(pull_result(e, nullptr));
+    TRY(state_ran(e, start_pos + n));
     if (device_ms) CU(cudaEventElapsedTime(device_ms, e->ev0, e->ev1));
     return LPP_OK;
 }
@@ -1896,7 +2353,7 @@ static lpp_status make_activation_map(CUtensorMap* m, const void* base, size_t t
 // The tensor-core path takes 16-bit weights, an FP16 cache and a single GPU; everything else is fed token by token.
 static bool prefill_batched(const lpp_engine* e) {
     if (e->c.flags & LPP_FLAG_NO_PREFILL_GEMM) return false;
-    if (!e->lat.empty()) return e->c.weight_dtype == LPP_BF16 && e->c.kv_dtype == LPP_F16;
+    if (!e->layers.empty()) return e->c.weight_dtype == LPP_BF16 && e->c.kv_dtype == LPP_F16;
     return e->c.tp_size == 1 && e->c.weight_dtype == LPP_F16 && e->c.kv_dtype == LPP_F16 && e->hs <= 128 && e->gqa <= 8 &&
            e->c.dim % 64 == 0 && e->Dq % 64 == 0 && e->Fl % 64 == 0;
 }
@@ -1913,23 +2370,31 @@ static lpp_status prefill_setup(lpp_engine* e) {
     if (e->pf_ready) return LPP_OK;
     const lpp_config& c = e->c;
     const size_t D = e->Dp, L = c.n_layers, T = kPrefillTokens;
-    const bool latent = !e->lat.empty();
-    size_t part_rows = D, att_n = e->Dq, hb_n = e->Fl, qn_n = 0, olat_n = 0, lq_n = 0, lpart_n = 0, gate_n = 0;
-    const size_t qkv_rows = latent ? 0 : e->Dq + 2 * (size_t)e->KVd;
+    const bool layered = !e->layers.empty();
+    size_t part_rows = D, att_n = e->Dq, hb_n = e->Fl, qn_n = 0, olat_n = 0, lq_n = 0, lpart_n = 0, gate_n = 0, scan_n = 0, tail_n = 0;
+    const size_t qkv_rows = layered ? 0 : e->Dq + 2 * (size_t)e->KVd;
     part_rows = std::max(part_rows, qkv_rows);
-    for (const LatentLayer& y : e->lat) {
+    for (const ModelLayer& y : e->layers) {
         const size_t H = y.d.heads;
         part_rows = std::max(part_rows, (size_t)y.in_rows);
         att_n = std::max(att_n, (size_t)y.o_pitch);
         hb_n = std::max(hb_n, (size_t)y.ff_pitch);
-        qn_n = std::max(qn_n, H * y.dim_pitch);
-        olat_n = std::max(olat_n, H * y.val_pitch);
+        if (y.d.mixer == LPP_MIXER_MAMBA) {
+            part_rows = std::max(part_rows, (size_t)y.low_rows);
+            scan_n = std::max(scan_n, (size_t)y.inner_pitch);
+            tail_n = std::max(tail_n, (size_t)(y.d.conv - 1) * y.inner_rows);
+            continue;
+        }
+        if (y.d.mixer == LPP_MIXER_LATENT) {
+            qn_n = std::max(qn_n, H * y.dim_pitch);
+            olat_n = std::max(olat_n, H * y.val_pitch);
+        }
         lq_n = std::max(lq_n, H * y.row_width);
         for (size_t t = 1; t <= T; ++t) {
             const LatentPlan p = latent_plan(e, y, (int)t);
             if (!p.cluster) lpart_n = std::max(lpart_n, t * H * p.splits * (y.rank_pitch + kLatentPartTail));
         }
-        gate_n = std::max(gate_n, H);
+        gate_n = std::max(gate_n, y.d.mixer == LPP_MIXER_LATENT ? H : H * y.d.dim);
     }
     TRY(zeroed(e, &e->pf_x, T * D * 4));
     TRY(zeroed(e, &e->pf_xn, 2 * T * D * 2));      // hi plane, lo plane
@@ -1938,20 +2403,29 @@ static lpp_status prefill_setup(lpp_engine* e) {
     TRY(zeroed(e, &e->pf_part, (size_t)kPfMaxSplits * T * part_rows * 4));
     TRY(zeroed(e, &e->pf_tokens, T * sizeof(int)));
     TRY(zeroed(e, &e->pf_rows, T * sizeof(int)));
-    if (latent) {
+    if (layered) {
         TRY(zeroed(e, &e->pf_qn, 2 * T * qn_n * 2));
         TRY(zeroed(e, &e->pf_olat, 2 * T * olat_n * 2));
         TRY(zeroed(e, &e->pf_lq, T * lq_n * 2));
         TRY(zeroed(e, &e->pf_lpart, lpart_n * 4));
         TRY(zeroed(e, &e->pf_gate, T * gate_n * 4));
-        for (LatentLayer& y : e->lat) {
+        TRY(zeroed(e, &e->pf_sx, T * scan_n * 4));
+        TRY(zeroed(e, &e->pf_sz, T * scan_n * 4));
+        TRY(zeroed(e, &e->pf_sxp, 2 * T * scan_n * 2));
+        TRY(zeroed(e, &e->pf_tail, tail_n * 4));
+        for (ModelLayer& y : e->layers) {
             const size_t H = y.d.heads, D2 = align_up(c.dim, 2);
             TRY(make_weight_map(&y.m_in, y.w_in, y.in_rows, D, kUmmaM));
-            TRY(make_weight_map(&y.m_uk, y.w_uk, H * y.rank_pitch, y.dim_pitch, kUmmaM));
-            TRY(make_weight_map(&y.m_uv, y.w_uv, H * y.vdim_rows, y.val_pitch, kUmmaM));
+            if (y.d.mixer == LPP_MIXER_LATENT) {
+                TRY(make_weight_map(&y.m_uk, y.w_uk, H * y.rank_pitch, y.dim_pitch, kUmmaM));
+                TRY(make_weight_map(&y.m_uv, y.w_uv, H * y.vdim_rows, y.val_pitch, kUmmaM));
+                TRY(make_activation_map(&y.x_qn, e->pf_qn, T, H * y.dim_pitch, kPrefillTokens));
+                TRY(make_activation_map(&y.x_olat, e->pf_olat, T, H * y.val_pitch, kPrefillTokens));
+            } else if (y.d.mixer == LPP_MIXER_MAMBA) {
+                TRY(make_weight_map(&y.m_low, y.w_low, y.low_rows, y.inner_pitch, kUmmaM));
+                TRY(make_activation_map(&y.x_low, e->pf_sxp, T, y.inner_pitch, kPrefillTokens));
+            }
             TRY(make_weight_map(&y.m_wo, y.wo, D2, y.o_pitch, kUmmaM));
-            TRY(make_activation_map(&y.x_qn, e->pf_qn, T, H * y.dim_pitch, kPrefillTokens));
-            TRY(make_activation_map(&y.x_olat, e->pf_olat, T, H * y.val_pitch, kPrefillTokens));
             TRY(make_activation_map(&y.x_att, e->pf_att, T, y.o_pitch, kPrefillTokens));
             if (y.d.ff > 0) {
                 TRY(make_weight_map(&y.m_w13, y.w13, 2 * (size_t)y.d.ff, D, kUmmaM));
@@ -2012,12 +2486,15 @@ static PrefillGemmArgs prefill_gemm_args(const lpp_engine* e, int n_rows, int K,
     return a;
 }
 
-// x_rows -> normalised operands; `parts` > 1: the previous residual GEMM's partial sums are added to x first.
-static lpp_status prefill_norm(lpp_engine* e, int n, const float* w, const float* b, bool embed, int parts, const int* rows, bool pdl) {
+// x_rows -> normalised operands; `parts` > 1: the previous residual GEMM's partial sums are added to x first, and so is `add`
+// (nullptr = nothing).
+static lpp_status prefill_norm(lpp_engine* e, int n, const float* w, const float* b, bool embed, const float* add, int parts, const int* rows, bool pdl) {
     PrefillNormArgs a = {};
     a.x = e->pf_x;
     a.tokens = e->pf_tokens;
     a.emb = embed ? e->emb : nullptr;
+    a.emb_scale = e->emb_scale;
+    a.add = add;
     a.vocab = e->c.vocab_size;
     a.rows = rows;
     a.norm_w = w;
@@ -2089,27 +2566,50 @@ static lpp_status prefill_gqa_mixer(lpp_engine* e, int l, int n, int start_pos, 
     return LPP_OK;
 }
 
+// W . in of a block as partial sums over ranges of K, [range][token][row] in pf_part; *splits = the number of ranges.
+static lpp_status prefill_partial_sums(lpp_engine* e, const CUtensorMap& wm, const CUtensorMap& xm, int n_rows, int K, int n, int start_pos, int* splits) {
+    PrefillGemmArgs g = prefill_gemm_args(e, n_rows, K, n, start_pos);
+    g.out = e->pf_part;
+    g.out_pitch = n_rows;
+    g.splits = *splits = prefill_splits(e, n_rows, K);
+    CU((launch_prefill_gemm_t<__nv_bfloat16, kPfStore>(e, wm, xm, g)));
+    return LPP_OK;
+}
+
+// Attention over shared rows of a prompt block: queries pf_lq, finished rows to `planes` as hi + lo operands.
+static lpp_status prefill_row_attention(lpp_engine* e, const ModelLayer& y, const LayerRun& r, int n, int start_pos, void* planes) {
+    const LatentPlan p = latent_plan(e, y, n);
+    LatentAttnArgs a = latent_attn_args(e, y, r, p);
+    a.q = e->pf_lq;
+    a.part = e->pf_lpart;
+    a.start_pos = start_pos;
+    a.n_tokens = n;
+    a.planes = (__nv_bfloat16*)planes;
+    a.out = nullptr;
+    if (a.gate) a.gate = e->pf_gate;
+    CU(launch_latent_attn(e, p, a, true, e->stream));
+    if (!p.cluster)
+        CU(launch_kernel(prefill_latent_combine_kernel, dim3(n * a.all_heads), dim3(128), 0, e->stream, true, a, p.tile_rows));
+    return LPP_OK;
+}
+
 // Latent attention of a prompt block: input GEMM (cut along K) and its finishing kernel, per-head query GEMM, attention in
 // key splits, their combination, per-head value GEMM with the gates.
 static lpp_status prefill_latent_mixer(lpp_engine* e, int l, int n, int start_pos, bool cache_only) {
     typedef __nv_bfloat16 T;
-    const LatentLayer& y = e->lat[l];
+    const LayerRun& r = e->runs[l];
+    const ModelLayer& y = e->layers[r.layer];
     const int H = y.d.heads;
-    PrefillGemmArgs g = prefill_gemm_args(e, y.in_rows, e->Dp, n, start_pos);
-    g.out = e->pf_part;
-    g.out_pitch = y.in_rows;
-    g.splits = prefill_splits(e, y.in_rows, e->Dp);
-    CU((launch_prefill_gemm_t<T, kPfStore>(e, y.m_in, e->pf_map_xn, g)));
     PrefillLatentFinishArgs f = {};
+    TRY(prefill_partial_sums(e, y.m_in, e->pf_map_xn, y.in_rows, e->Dp, n, start_pos, &f.splits));
     f.part = e->pf_part;
     f.n_rows = y.in_rows;
-    f.splits = g.splits;
     f.start_pos = start_pos;
     f.seq_len = e->c.seq_len;
     f.qn = e->pf_qn;
     f.gate = e->pf_gate;
     f.st = e->st;
-    f.lat = latent_args(e, y);
+    f.lat = latent_args(e, y, r);
     f.lat.query = e->pf_lq;
     const int q_sections = cache_only ? 0 : (y.q_plain_rows + y.q_rot_rows + 2 * kLatFinishThreads - 1) / (2 * kLatFinishThreads);
     CU(launch_kernel(prefill_latent_finish_kernel<T>, dim3(n, 1 + q_sections), dim3(kLatFinishThreads), (size_t)y.latent_rows * 4, e->stream,
@@ -2122,16 +2622,7 @@ static lpp_status prefill_latent_mixer(lpp_engine* e, int l, int n, int start_po
     q.lat_query = e->pf_lq;
     q.lat_pitch = y.row_width;
     CU((launch_prefill_gemm_t<T, kPfLatentQuery>(e, y.m_uk, y.x_qn, q)));
-    const LatentPlan p = latent_plan(e, y, n);
-    LatentAttnArgs a = latent_attn_args(e, y, p);
-    a.q = e->pf_lq;
-    a.part = e->pf_lpart;
-    a.start_pos = start_pos;
-    a.n_tokens = n;
-    a.planes = (T*)e->pf_olat;
-    CU(launch_latent_attn(e, p, a, true, e->stream));
-    if (!p.cluster)
-        CU(launch_kernel(prefill_latent_combine_kernel<T>, dim3(n * H), dim3(128), 0, e->stream, true, a, p.tile_rows, (T*)e->pf_olat, y.val_pitch));
+    TRY(prefill_row_attention(e, y, r, n, start_pos, e->pf_olat));
     PrefillGemmArgs v = prefill_gemm_args(e, y.vdim_rows, y.val_pitch, n, start_pos);
     v.groups = H;
     v.group_stride = y.vdim_rows;
@@ -2144,39 +2635,107 @@ static lpp_status prefill_latent_mixer(lpp_engine* e, int l, int n, int start_po
     return LPP_OK;
 }
 
+// Attention whose values are its keys, of a prompt block: input GEMM (cut along K) and its finishing kernel, attention.
+static lpp_status prefill_shared_kv_mixer(lpp_engine* e, int l, int n, int start_pos, bool cache_only) {
+    const LayerRun& r = e->runs[l];
+    const ModelLayer& y = e->layers[r.layer];
+    PrefillSharedKvArgs f = {};
+    TRY(prefill_partial_sums(e, y.m_in, e->pf_map_xn, y.in_rows, e->Dp, n, start_pos, &f.splits));
+    f.part = e->pf_part;
+    f.n_rows = y.in_rows;
+    f.start_pos = start_pos;
+    f.seq_len = e->c.seq_len;
+    f.keys_only = cache_only;
+    f.st = e->st;
+    f.kv = shared_kv_args(e, y, r);
+    f.kv.query = e->pf_lq;
+    f.kv.gate = e->pf_gate;
+    CU(launch_kernel(prefill_shared_kv_finish_kernel, dim3(n, (y.in_rows / 2 + 255) / 256), dim3(256), 0, e->stream, true, f));
+    return cache_only ? LPP_OK : prefill_row_attention(e, y, r, n, start_pos, e->pf_att);
+}
+
+// Selective scan of a prompt block: input GEMM (cut along K), convolution, GEMM of dt | B | C (cut along K), recurrence.
+static lpp_status prefill_mamba_mixer(lpp_engine* e, int l, int n, int start_pos) {
+    const LayerRun& r = e->runs[l];
+    const ModelLayer& y = e->layers[r.layer];
+    MambaConvArgs v = {};
+    TRY(prefill_partial_sums(e, y.m_in, e->pf_map_xn, y.in_rows, e->Dp, n, start_pos, &v.splits));
+    v.part = e->pf_part;
+    v.n_tokens = n;
+    v.start_pos = start_pos;
+    v.seq_len = e->c.seq_len;
+    v.inner = y.d.inner;
+    v.inner_rows = y.inner_rows;
+    v.taps = y.d.conv;
+    v.conv_w = y.conv_w;
+    v.conv_b = y.conv_b;
+    v.ring = r.ring;
+    v.tail = e->pf_tail;
+    v.x = e->pf_sx;
+    v.z = e->pf_sz;
+    v.x_pitch = y.inner_pitch;
+    v.planes = (__nv_bfloat16*)e->pf_sxp;
+    v.st = e->st;
+    const dim3 grid((y.d.inner + kConvChannels - 1) / kConvChannels, (n + kConvTokens - 1) / kConvTokens, 2);
+    CU(launch_kernel(mamba_conv_kernel, grid, dim3(kConvChannels), (size_t)conv_smem(y.d.conv), e->stream, true, v));
+    MambaScanArgs a = mamba_scan_args(e, y, r);
+    TRY(prefill_partial_sums(e, y.m_low, y.x_low, y.low_rows, y.inner_pitch, n, start_pos, &a.splits));
+    a.low = e->pf_part;
+    a.n_tokens = n;
+    a.start_pos = start_pos;
+    a.x = e->pf_sx;
+    a.z = e->pf_sz;
+    a.x_pitch = y.inner_pitch;
+    a.tail = e->pf_tail;
+    a.planes = (__nv_bfloat16*)e->pf_att;
+    a.plane_row = y.o_pitch;
+    CU(launch_mamba_scan(e, a, e->stream));
+    return LPP_OK;
+}
+
 // One block of n <= kPrefillTokens prompt tokens at positions start_pos ...  Without wanted logits the last layer stops
 // after its cache rows are written (nothing downstream of them is needed); otherwise the n_want rows `want` of the block go
 // through the final norm and the classifier and their logits are copied to h_logits.
 static lpp_status prefill_block(lpp_engine* e, const int* h_tokens, int n, int start_pos, const int* want, int n_want, float* h_logits) {
     const lpp_config& c = e->c;
-    const int L = c.n_layers;
-    const bool latent = !e->lat.empty();
+    const int L = n_runs(e);
+    const bool layered = !e->layers.empty();
     CU(cudaMemcpyAsync(e->pf_tokens, h_tokens, (size_t)n * sizeof(int), cudaMemcpyHostToDevice, e->stream));
     if (n_want > 0) CU(cudaMemcpyAsync(e->pf_rows, want, (size_t)n_want * sizeof(int), cudaMemcpyHostToDevice, e->stream));
     int parts = 1;
+    const float* add = first_add(e);  // what the next norm adds to the residual stream first
     for (int l = 0; l < L; ++l) {
         const bool cache_only = l == L - 1 && n_want == 0;
         const LayerView v = layer_view(e, l);
+        const ModelLayer* y = layered ? &e->layers[e->runs[l].layer] : nullptr;
         // layer 0 takes the embedding rows; later layers first add the previous residual GEMM's partial sums
-        TRY(prefill_norm(e, n, latent ? e->lat[l].n1w : e->rms_att + (size_t)l * c.dim, latent ? e->lat[l].n1b : nullptr, l == 0, parts,
-                         nullptr, l > 0));
-        TRY(latent ? prefill_latent_mixer(e, l, n, start_pos, cache_only) : prefill_gqa_mixer(e, l, n, start_pos, cache_only));
+        TRY(prefill_norm(e, n, layered ? y->n1w : e->rms_att + (size_t)l * c.dim, layered ? y->n1b : nullptr, l == 0, add, parts, nullptr, l > 0));
+        if (!layered)
+            TRY(prefill_gqa_mixer(e, l, n, start_pos, cache_only));
+        else if (y->d.mixer == LPP_MIXER_LATENT)
+            TRY(prefill_latent_mixer(e, l, n, start_pos, cache_only));
+        else if (y->d.mixer == LPP_MIXER_SHARED_KV)
+            TRY(prefill_shared_kv_mixer(e, l, n, start_pos, cache_only));
+        else
+            TRY(prefill_mamba_mixer(e, l, n, start_pos));
         if (cache_only) return LPP_OK;
-        TRY(prefill_resid(e, latent ? e->lat[l].m_wo : e->pf_map_wo, latent ? 0 : l * c.dim, latent ? e->lat[l].x_att : e->pf_map_att, v.o_k, n,
-                          start_pos, &parts));
+        TRY(prefill_resid(e, layered ? y->m_wo : e->pf_map_wo, layered ? 0 : l * c.dim, layered ? y->x_att : e->pf_map_att, v.o_k, n, start_pos,
+                          &parts));
+        add = v.o_add;
         if (v.ff == 0) continue;  // a layer without a feed-forward
-        TRY(prefill_norm(e, n, v.norm2_w, v.norm2_b, false, parts, nullptr, true));
+        TRY(prefill_norm(e, n, v.norm2_w, v.norm2_b, false, add, parts, nullptr, true));
         PrefillGemmArgs u = prefill_gemm_args(e, 2 * v.ff, e->Dp, n, start_pos);
-        u.row0 = latent ? 0 : l * 2 * v.ff;
+        u.row0 = layered ? 0 : l * 2 * v.ff;
         u.hb = e->pf_hb;
         u.hb_pitch = v.ff_k;
         u.act = v.act;
-        CU(launch_prefill_gemm<kPfSwiglu>(e, latent ? e->lat[l].m_w13 : e->pf_map_w13, e->pf_map_xn, u));
-        TRY(prefill_resid(e, latent ? e->lat[l].m_w2 : e->pf_map_w2, latent ? 0 : l * c.dim, latent ? e->lat[l].x_hb : e->pf_map_hb, v.ff_k, n,
-                          start_pos, &parts));
+        CU(launch_prefill_gemm<kPfSwiglu>(e, layered ? y->m_w13 : e->pf_map_w13, e->pf_map_xn, u));
+        TRY(prefill_resid(e, layered ? y->m_w2 : e->pf_map_w2, layered ? 0 : l * c.dim, layered ? y->x_hb : e->pf_map_hb, v.ff_k, n, start_pos,
+                          &parts));
+        add = v.down_add;
     }
     if (!e->pf_logits) CU(cudaMalloc(&e->pf_logits, (size_t)kPrefillTokens * e->Vp * 4));
-    TRY(prefill_norm(e, n_want, e->rms_final, e->final_b, false, parts, e->pf_rows, true));
+    TRY(prefill_norm(e, n_want, e->rms_final, e->final_b, false, add, parts, e->pf_rows, true));
     PrefillGemmArgs g = prefill_gemm_args(e, e->Vp, e->Dp, n_want, start_pos);
     g.out = e->pf_logits;
     g.out_pitch = e->Vp;
@@ -2198,6 +2757,7 @@ extern "C" lpp_status lpp_extend(lpp_engine* e, const int* h_tokens, int n, int 
     const size_t V = e->c.vocab_size;
     int w = 0;  // wanted tokens served so far
     TRY(push_state(e, h_tokens[0], start_pos, nullptr, nullptr, 0, 0.f, 0, 0));  // clears the device status
+    TRY(state_runs(e, start_pos));
     if (prefill_batched(e) && n > 1) {
         TRY(prefill_setup(e));
         CU(cudaEventRecord(e->ev0, e->stream));
@@ -2224,6 +2784,7 @@ extern "C" lpp_status lpp_extend(lpp_engine* e, const int* h_tokens, int n, int 
         CU(cudaEventRecord(e->ev1, e->stream));
     }
     TRY(pull_result(e, nullptr));
+    TRY(state_ran(e, start_pos + n));
     if (device_ms) CU(cudaEventElapsedTime(device_ms, e->ev0, e->ev1));
     return LPP_OK;
 }
@@ -2235,7 +2796,7 @@ extern "C" lpp_status lpp_prefill(lpp_engine* e, const int* h_tokens, int n, int
 // ------------------------------------------------------------------ KV cache access
 
 extern "C" int64_t lpp_kv_index(const lpp_engine* e, int layer, int kv_head, int pos, int off) {
-    if (!e || !e->lat.empty()) return -1;
+    if (!e || !e->layers.empty()) return -1;
     const int64_t kvd = (int64_t)e->KVHl * e->hs, S = e->c.seq_len;
     return (int64_t)layer * (kvd * S) + (int64_t)kv_head * (S * e->hs) + (int64_t)pos * e->hs + off;
 }
@@ -2244,7 +2805,7 @@ extern "C" lpp_status lpp_kv_prefill(lpp_engine* e, int layer, const void* k, co
                                      int memkind) {
     if (!e || !k || !v) return fail(LPP_ERR_INVALID_ARG, "null argument");
     const lpp_config& c = e->c;
-    if (!e->lat.empty()) return fail(LPP_ERR_INVALID_ARG, "this model keeps latents, not keys and values");
+    if (!e->layers.empty()) return fail(LPP_ERR_INVALID_ARG, "this model keeps no separate keys and values");
     if (layer < 0 || layer >= c.n_layers || n_pos < 0 || n_pos > c.seq_len) return fail(LPP_ERR_INVALID_ARG, "layer/n_pos out of range");
     if (src_dtype != LPP_F16 && src_dtype != LPP_F32) return fail(LPP_ERR_INVALID_ARG, "bad src_dtype");
     CU(cudaSetDevice(c.device));
@@ -2267,7 +2828,7 @@ extern "C" lpp_status lpp_kv_prefill(lpp_engine* e, int layer, const void* k, co
 extern "C" lpp_status lpp_kv_read(lpp_engine* e, int layer, int kv_head, int pos, float* h_k, float* h_v) {
     if (!e || !h_k || !h_v) return fail(LPP_ERR_INVALID_ARG, "null argument");
     const lpp_config& c = e->c;
-    if (!e->lat.empty()) return fail(LPP_ERR_INVALID_ARG, "this model keeps latents, not keys and values");
+    if (!e->layers.empty()) return fail(LPP_ERR_INVALID_ARG, "this model keeps no separate keys and values");
     if (layer < 0 || layer >= c.n_layers || kv_head < 0 || kv_head >= e->KVHl || pos < 0 || pos >= c.seq_len)
         return fail(LPP_ERR_INVALID_ARG, "index out of range");
     CU(cudaSetDevice(c.device));
@@ -2291,12 +2852,14 @@ extern "C" lpp_status lpp_kv_read(lpp_engine* e, int layer, int kv_head, int pos
 
 extern "C" lpp_status lpp_latent_read(lpp_engine* e, int layer, int pos, float* h_row) {
     if (!e || !h_row) return fail(LPP_ERR_INVALID_ARG, "null argument");
-    if (layer < 0 || layer >= (int)e->lat.size() || pos < 0 || pos >= e->c.seq_len) return fail(LPP_ERR_INVALID_ARG, "index out of range");
+    if (layer < 0 || layer >= (int)e->runs.size() || pos < 0 || pos >= e->c.seq_len) return fail(LPP_ERR_INVALID_ARG, "index out of range");
+    const LayerRun& r = e->runs[layer];
+    const ModelLayer& y = e->layers[r.layer];
+    if (y.d.mixer != LPP_MIXER_LATENT) return fail(LPP_ERR_INVALID_ARG, "layer run %d keeps no latents", layer);
     CU(cudaSetDevice(e->c.device));
     CU(cudaStreamSynchronize(e->stream));
-    const LatentLayer& y = e->lat[layer];
     std::vector<unsigned char> raw((size_t)y.row_width * e->kvesz);
-    CU(cudaMemcpy(raw.data(), (const char*)y.cache + (size_t)pos * raw.size(), raw.size(), cudaMemcpyDeviceToHost));
+    CU(cudaMemcpy(raw.data(), (const char*)r.cache + (size_t)pos * raw.size(), raw.size(), cudaMemcpyDeviceToHost));
     auto at = [&](int i) { return e->kvesz == 4 ? ((const float*)raw.data())[i] : __half2float(((const __half*)raw.data())[i]); };
     for (int i = 0; i < y.d.kv_rank; ++i) h_row[i] = at(i);
     for (int i = 0; i < y.d.rot_dim; ++i) h_row[y.d.kv_rank + i] = at(y.rank_pitch + i);
@@ -2431,16 +2994,30 @@ static void kind_bytes(const lpp_engine* e, int pos, int64_t* b) {
     const lpp_config& c = e->c;
     const int64_t D = c.dim, L = c.n_layers, V = c.vocab_size, esz = e->esz;
     for (int k = 0; k < kKinds; ++k) b[k] = 0;
-    if (!e->lat.empty()) {
-        for (const LatentLayer& y : e->lat) {
+    if (!e->layers.empty()) {
+        for (const LayerRun& r : e->runs) {
+            const ModelLayer& y = e->layers[r.layer];
             const lpp_layer_desc& d = y.d;
             const int64_t keys = d.window > 0 ? std::min<int64_t>(d.window, pos + 1) : pos + 1;
-            const int64_t row = d.kv_rank + d.rot_dim, H = d.heads;
-            b[kQkv] += (H * (d.dim + d.rot_dim) + row + H) * D * esz + 8 * D;
-            b[kLatQuery] += H * d.dim * d.kv_rank * esz;
-            b[kAttn] += (keys + 1) * row * e->kvesz;
-            b[kLatValue] += H * d.vdim * d.kv_rank * esz;
-            b[kOproj] += D * H * d.vdim * esz;
+            const int64_t H = d.heads;
+            if (d.mixer == LPP_MIXER_LATENT) {
+                const int64_t row = d.kv_rank + d.rot_dim;
+                b[kQkv] += (H * (d.dim + d.rot_dim) + row + H) * D * esz + 8 * D;
+                b[kLatQuery] += H * d.dim * d.kv_rank * esz;
+                b[kAttn] += (keys + 1) * row * e->kvesz;
+                b[kLatValue] += H * d.vdim * d.kv_rank * esz;
+                b[kOproj] += D * H * d.vdim * esz;
+            } else if (d.mixer == LPP_MIXER_SHARED_KV) {
+                b[kQkv] += ((1 + (d.gate ? 1 : 0)) * H + d.kv_heads) * d.dim * D * esz + 4 * D;
+                b[kAttn] += (keys + 1) * d.kv_heads * (d.dim + d.rot_dims) * e->kvesz;
+                b[kOproj] += D * H * d.dim * esz;
+            } else {  // the recurrent state is read and written
+                const int64_t E = d.inner, N = d.state;
+                b[kQkv] += 2 * E * D * esz + 4 * D + E * (d.conv + 1 + d.conv) * 4;
+                b[kScanIn] += (d.dt_rank + 2 * N) * E * esz;
+                b[kScan] += E * d.dt_rank * esz + E * (3 * N + 2) * 4;
+                b[kOproj] += D * E * esz;
+            }
             if (d.ff > 0) {
                 b[kGateUp] += (int64_t)2 * d.ff * D * esz + 8 * D;
                 b[kDown] += D * d.ff * esz;
@@ -2475,6 +3052,7 @@ extern "C" lpp_status lpp_profile_kind(lpp_engine* e, int pos, int kind, int ite
     if (pos < 0 || pos >= e->c.seq_len) return fail(LPP_ERR_INVALID_ARG, "pos out of range");
     *ms_per_launch = 0.f;
     *launches = 0;
+    if (e->recurrent) e->state_len = -1;
     lpp_sample_params sp = {0.8f, 1.1f};
     cudaGraphExec_t gx = nullptr;
     int n_kernels = 0;
@@ -2517,6 +3095,7 @@ extern "C" lpp_status lpp_profile_step(lpp_engine* e, int pos, int iters, const 
     if (pos < 0 || pos >= e->c.seq_len) return fail(LPP_ERR_INVALID_ARG, "pos out of range");
     for (int k = 0; k < kKinds; ++k) ms[k] = 0.f, launches[k] = 0;
     kind_bytes(e, pos, bytes);
+    if (e->recurrent) e->state_len = -1;
     // the sampler that is timed is the one the caller's workload runs (argmax and categorical paths differ)
     const lpp_sample_params sp = spp ? *spp : lpp_sample_params{0.f, 1.f};
     const int hist[3] = {1, 2, 3};

@@ -1,8 +1,8 @@
 // Batch-1 streaming GEMV family: out[n] = W[n,K] . x[K] with FP16, BF16 or FP32 weights, FP32 activations
 // and FP32 accumulation.  One kernel template serves every matrix of the decode step; what differs
 // is the prologue (plain vector, RMSNorm'd or LayerNorm'd vector, embedding row, per-head inputs, combination of
-// attention splits) and the epilogue (store, residual add, gated activation, RoPE + KV-cache scatter, and the
-// three projections of latent attention, latent.cuh).
+// attention splits) and the epilogue (store, residual add, gated activation, RoPE + KV-cache scatter, the
+// three projections of latent attention, latent.cuh, and the input projections of shared_kv.cuh and mamba.cuh).
 //
 // Replaces, from the reference tree: gemv_kernel / gemv_f16_kernel / convert_f32_to_f16_kernel
 // (src/matmul.cu:9-161), rmsnorm (src/RMSNorm.cu:11-71, fused as prologue), swiglu_kernel
@@ -25,6 +25,8 @@
 #pragma once
 #include "common.cuh"
 #include "latent.cuh"
+#include "mamba.cuh"
+#include "shared_kv.cuh"
 
 namespace lpp {
 
@@ -35,7 +37,10 @@ enum GemvEpi : int {
     kEpiQkv = 3,
     kEpiLatentIn = 4,     // query | latent | rotated key part | gate rows of latent attention
     kEpiLatentQuery = 5,  // per head: query in the latent space
-    kEpiLatentValue = 6   // per head: value of the attended latent, times the head's gate
+    kEpiLatentValue = 6,  // per head: value of the attended latent, times the head's gate
+    kEpiResidBias = 7,    // residual add and a bias
+    kEpiSharedKvIn = 8,   // query | key | gate rows of attention whose values are its keys
+    kEpiMambaIn = 9       // x | z rows of a selective-scan layer
 };
 
 constexpr int kGemvConsumerWarps = 8;
@@ -55,6 +60,8 @@ struct GemvArgs {
     const float* x;       // input vector [K] (ignored when emb != nullptr)
     const float* norm_w;  // RMSNorm weight [K], nullptr = no normalisation
     const void* emb;      // embedding table [vocab][K] in the weight dtype, nullptr = use x
+    float emb_scale;      // the embedding row's factor
+    const float* emb_add; // [K] added to the scaled row (nullptr = nothing)
     float* x_store;       // CTA 0 stores the un-normalised input vector here (nullptr = don't)
     StepState* st;        // token / pos / status
     int vocab, seq_len;
@@ -68,6 +75,7 @@ struct GemvArgs {
     float* out;          // Store/Resid: [n_rows]; Swiglu: [n_rows/2]; Qkv: q vector [q_rows]
     int act;             // Swiglu: activation of the gate (Act)
     const float* resid;  // Resid: added to the result when non-null
+    const float* bias;   // ResidBias: [n_rows]
     int q_rows, kv_rows, head_size;  // Qkv: rows are q | k | v
     const float2* rope;              // Qkv: [seq_len][head_size/2] (cos, sin)
     void* k_cache;                   // Qkv: this layer's K cache [kv_heads][seq_len][head_size]
@@ -117,8 +125,22 @@ struct GemvLatentArgs : GemvArgs {
 };
 template <int EPI>
 constexpr bool is_latent_epi = EPI == kEpiLatentIn || EPI == kEpiLatentQuery || EPI == kEpiLatentValue;
+struct GemvSharedKvArgs : GemvArgs {
+    SharedKvArgs kv;
+};
+struct GemvMambaArgs : GemvArgs {
+    MambaInArgs mb;
+};
 template <int EPI>
-using GemvArgsOf = std::conditional_t<is_latent_epi<EPI>, GemvLatentArgs, GemvArgs>;
+using GemvArgsOf = std::conditional_t<is_latent_epi<EPI>, GemvLatentArgs,
+                                      std::conditional_t<EPI == kEpiSharedKvIn, GemvSharedKvArgs, std::conditional_t<EPI == kEpiMambaIn, GemvMambaArgs, GemvArgs>>>;
+template <int EPI>
+constexpr bool is_resid_epi = EPI == kEpiResid || EPI == kEpiResidBias;
+// Epilogues that need several loads of their own per row: done by a lane per row, up to 16 row pairs of a warp together, with
+// what does not depend on the product fetched before it is formed.
+template <int EPI>
+constexpr bool is_row_epi = EPI == kEpiSharedKvIn || EPI == kEpiMambaIn;
+constexpr int kRowEpiPairs = 16;
 
 // ------------------------------------------------------------------ x staging layouts
 //
@@ -349,7 +371,7 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
     if (tid == 0) gemv_stamp(a, 1);
 
     if (a.emb) {
-        // first layer: the input is the embedding row of the device-resident token, widened exactly
+        // first layer: the input is the embedding row of the device-resident token, widened exactly, times its factor
         int tok = a.st->token;
         if (tok < 0 || tok >= a.vocab) {
             if (tid == 0) atomicOr(&a.st->status, kStatusBadToken);
@@ -359,7 +381,8 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
         const bool store = a.x_store && blockIdx.x == 0;
         float ss = 0.f;
         for (int k = tid; k < K; k += NT) {
-            const float v = to_float(erow[k]);
+            float v = to_float(erow[k]) * a.emb_scale;
+            if (a.emb_add) v += __ldg(a.emb_add + k);
             ss = fmaf(v, v, ss);
             if (store) a.x_store[k] = v;
             xs[xs_index<WT>(k, K)] = v;
@@ -596,7 +619,12 @@ __device__ __forceinline__ void gemv_epilogue(const GemvArgsOf<EPI>& a, int g, f
     const int row = g * kRowsPerGroup;
     if constexpr (EPI == kEpiStore) {
         store_rows(a, row, v0, v1);
-    } else if constexpr (EPI == kEpiResid) {
+    } else if constexpr (is_resid_epi<EPI>) {
+        if constexpr (EPI == kEpiResidBias) {
+            const float2 b = __ldg(reinterpret_cast<const float2*>(a.bias + row));
+            v0 += b.x;
+            v1 += b.y;
+        }
         // x += W.xb (src/model.cpp:232, 239); under tensor parallelism only rank 0 passes resid
         if (a.resid) {
             const float2 r = __ldcg(reinterpret_cast<const float2*>(a.resid + row));  // written by an earlier phase
@@ -646,6 +674,36 @@ __device__ __forceinline__ void gemv_epilogue(const GemvArgsOf<EPI>& a, int g, f
                 *reinterpret_cast<__half2*>(reinterpret_cast<__half*>(base) + idx) = __floats2half2_rn(v0, v1);
         }
     }
+}
+
+// The same for a row epilogue: `row` with its product v and that of its pair partner.
+template <int EPI>
+__device__ __forceinline__ RowPrep row_prep(const GemvArgsOf<EPI>& a, int row) {
+    const int pos = a.st->pos;
+    if (row >= a.n_rows || pos < 0 || pos >= a.seq_len) return RowPrep();
+    if constexpr (EPI == kEpiSharedKvIn)
+        return shared_kv_prep(a.kv, pos, row);
+    else
+        return mamba_in_prep(a.mb, pos, row);
+}
+template <int EPI>
+__device__ __forceinline__ void row_epilogue(const GemvArgsOf<EPI>& a, int row, float v, float other, const RowPrep& p) {
+    const int pos = a.st->pos;
+    if (pos < 0 || pos >= a.seq_len) {
+        atomicOr(&a.st->status, kStatusBadPos);
+        return;
+    }
+    if constexpr (EPI == kEpiSharedKvIn)
+        shared_kv_row(a.kv, a.kv.query, a.kv.gate, a.seq_len, pos, row, v, other, p);
+    else
+        mamba_in_row(a.mb, pos, row, v, p);
+}
+template <int EPI>
+__device__ __forceinline__ bool row_early(const GemvArgsOf<EPI>& a) {
+    if constexpr (EPI == kEpiSharedKvIn)
+        return a.kv.early != 0;
+    else
+        return a.mb.early != 0;
 }
 
 // CTAs of the launch that rows are dealt to.  The query GEMV of latent attention has one more, the last one, which norms the
@@ -777,6 +835,30 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
             asm volatile("" ::"f"(cs.x), "f"(cs.y));
         }
     }
+    // row epilogue: lane l looks after row l % 2 of pair l / 2 of the warp's current batch of pairs
+    RowPrep prep;
+    float mine = 0.f, partner = 0.f;
+    if constexpr (is_row_epi<EPI>) {
+        if (!row_early<EPI>(a)) pdl_wait();
+        if (p0 + (lane >> 1) < p1) prep = row_prep<EPI>(a, p0 * kRowsPerGroup + lane);
+    }
+    // the sums of pair p (on every lane) to whoever finishes it
+    auto finish = [&](int p, float v0, float v1) {
+        if constexpr (is_row_epi<EPI>) {
+            const int i = (p - p0) % kRowEpiPairs;
+            if ((lane >> 1) == i) {
+                mine = (lane & 1) ? v1 : v0;
+                partner = (lane & 1) ? v0 : v1;
+            }
+            if (i == kRowEpiPairs - 1 || p + 1 == p1) {
+                const int first = p - i;  // the batch's first pair
+                if ((lane >> 1) <= i) row_epilogue<EPI>(a, first * kRowsPerGroup + lane, mine, partner, prep);
+                if (p + 1 + (lane >> 1) < p1) prep = row_prep<EPI>(a, (p + 1) * kRowsPerGroup + lane);
+            }
+        } else if (lane == 0) {
+            gemv_epilogue<WT, EPI>(a, p, v0, v1);
+        }
+    };
     // grouped rows: the inputs of the groups this CTA's row pairs belong to are staged back to back
     int first_group = 0, Kx = a.K;
     if constexpr (EPI == kEpiLatentQuery || EPI == kEpiLatentValue) {
@@ -821,8 +903,13 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
     // trip runs beside the dot product instead of after it (the weights are usually in the ring
     // already when the input arrives).  The producing kernel has completed: stage_input waited.
     float2 r_first = make_float2(0.f, 0.f);
-    if (EPI == kEpiResid && a.resid && lane == 0 && p0 < p1)
+    if (is_resid_epi<EPI> && a.resid && lane == 0 && p0 < p1)
         r_first = __ldcg(reinterpret_cast<const float2*>(a.resid + (size_t)p0 * kRowsPerGroup));
+    if (EPI == kEpiResidBias && lane == 0 && p0 < p1) {
+        const float2 b = __ldg(reinterpret_cast<const float2*>(a.bias + (size_t)p0 * kRowsPerGroup));
+        r_first.x += b.x;
+        r_first.y += b.y;
+    }
     if (m > 0) {
         for (int p = p0; p < p1 && ok; p += pstep) {
             const int cnt = min(unit, p1 - p);
@@ -838,11 +925,10 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
                 if (!(a.debug & 1)) dot_rows<WT, 2, false>(r0, r0 + row_bytes, xs, Kx, input_offset(p + i), a.K, lane, acc0, acc1);
                 acc0 = warp_sum(acc0);
                 acc1 = warp_sum(acc1);
-                if (lane == 0) {
-                    if (EPI == kEpiResid && p + i == p0)
-                        store_rows(a, p0 * kRowsPerGroup, acc0 + r_first.x, acc1 + r_first.y);
-                    else
-                        gemv_epilogue<WT, EPI>(a, p + i, acc0, acc1);
+                if (is_resid_epi<EPI> && p + i == p0) {
+                    if (lane == 0) store_rows(a, p0 * kRowsPerGroup, acc0 + r_first.x, acc1 + r_first.y);
+                } else {
+                    finish(p + i, acc0, acc1);
                 }
             }
             release();
@@ -866,11 +952,10 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
                 }
             if (!ok) break;
             const float v0 = warp_sum(acc[0]), v1 = warp_sum(acc[1]);
-            if (lane == 0) {
-                if (EPI == kEpiResid && p == p0)
-                    store_rows(a, p0 * kRowsPerGroup, v0 + r_first.x, v1 + r_first.y);
-                else
-                    gemv_epilogue<WT, EPI>(a, p, v0, v1);
+            if (is_resid_epi<EPI> && p == p0) {
+                if (lane == 0) store_rows(a, p0 * kRowsPerGroup, v0 + r_first.x, v1 + r_first.y);
+            } else {
+                finish(p, v0, v1);
             }
         }
     }
@@ -933,7 +1018,12 @@ __global__ void __launch_bounds__(kGemvLdgThreads) gemv_ldg_kernel(const GemvArg
         dot_rows<WT, 2, true>(r0, r0 + row_bytes, xs, Kx, k0, a.K, lane, acc0, acc1);
         acc0 = warp_sum(acc0);
         acc1 = warp_sum(acc1);
-        if (lane == 0) gemv_epilogue<WT, EPI>(a, g, acc0, acc1);
+        if constexpr (is_row_epi<EPI>) {
+            const int row = g * kRowsPerGroup + lane;
+            if (lane < kRowsPerGroup) row_epilogue<EPI>(a, row, lane ? acc1 : acc0, lane ? acc0 : acc1, row_prep<EPI>(a, row));
+        } else if (lane == 0) {
+            gemv_epilogue<WT, EPI>(a, g, acc0, acc1);
+        }
     }
     pdl_launch_dependents();
 }

@@ -68,8 +68,6 @@ __device__ __forceinline__ void latent_put(void* base, int f32, size_t i, float 
         reinterpret_cast<__half*>(base)[i] = __float2half_rn(v);
 }
 
-__device__ __forceinline__ float sigmoid_f(float v) { return __fdiv_rn(1.0f, 1.0f + expf(-v)); }
-
 // Epilogue of the input GEMV: rows row and row + 1 (row even).
 __device__ __forceinline__ void latent_in_rows(const LatentArgs& L, StepState* st, int seq_len, int row, float v0, float v1) {
     const int pos = st->pos;

@@ -1,12 +1,13 @@
-// Attention kernels of latent attention (latent.cuh has the scheme) and the two small kernels around them on the batched
-// prompt path.
+// Attention over shared rows: one cache row per position serves as key and, with its first rank_pitch columns, as value.
+// Latent attention (latent.cuh) has one such row for all heads, attention whose values are its unrotated keys
+// (shared_kv.cuh) one per key/value head.  Also the two small kernels around latent attention on the batched prompt path.
 //
-// In the latent space all heads share one key / value row per position, so the query rows of an attention launch are the
-// (token, head) pairs, row = token * heads + head: one row block for a decode step, n_tokens x heads rows for a prompt
-// block.  A CTA takes a tile of query rows and one of the splits of the keys that the tile's tokens can see (sliding
-// window; a tile's tokens are neighbours, so their windows nearly coincide) and writes the unnormalised weighted sum,
-// its maximum and its sum.  Whoever consumes the result puts the splits together (value GEMV when decoding,
-// prefill_latent_combine_kernel in a prompt block).
+// Heads that share a row form a group.  The query rows of a group in an attention launch are its (token, head) pairs,
+// row = token * heads + head: one row block for a decode step, n_tokens x heads rows for a prompt block.  A CTA takes a
+// tile of query rows and one of the splits of the keys that the tile's tokens can see (sliding window; a tile's tokens
+// are neighbours, so their windows nearly coincide) and writes the unnormalised weighted sum, its maximum and its sum.
+// Whoever consumes the result puts the splits together: the value GEMV of latent attention when decoding, the last CTA
+// of a row tile to finish when `out` is set, prefill_latent_combine_kernel in a prompt block.
 #pragma once
 #include "latent.cuh"
 #include "prefill.cuh"
@@ -14,21 +15,86 @@
 namespace lpp {
 
 struct LatentAttnArgs {
-    const void* q;      // [rows][row_width]
-    const void* cache;  // [positions][row_width], this layer's
-    float* part;        // [rows][max_splits][rank_pitch + kLatentPartTail]
+    const void* q;      // [token][all_heads][row_width]
+    const void* cache;  // [group][positions][row_width], this layer's
+    float* part;        // [token][all_heads][max_splits][rank_pitch + kLatentPartTail]
     const StepState* st;
     int start_pos;      // position of token 0; < 0 = the step's device-resident position
-    int n_tokens, heads;
+    int n_tokens;
+    int heads;          // query heads of a group: they share its cache rows
+    int all_heads;      // heads x groups
+    int score_skip;     // 16-column steps at the start of a row that scores leave out (zero in the queries)
     int rank_pitch, row_width;
     int window, max_splits, min_chunk;
     int seq_len;
     float scale;
+    float softcap;      // > 0: a score s becomes softcap * tanh(s / softcap)
+    // One token, splits put together by the CTA that finishes last: out[head * out_cols + col] = result * gate
+    float* out;              // nullptr = partial results stay in `part`
+    const float* gate;       // [all_heads * out_cols], prompt blocks [token][all_heads * out_cols]; nullptr = none
+    int out_cols;            // valid columns of a result
+    unsigned int* counters;  // one per row tile (or head), zero between launches
     // Tensor-core kernel: the splits of a row tile form a cluster and put themselves together
     int cluster;             // 0 = partial results to `part`
-    __nv_bfloat16* planes;   // then the result goes here: [2 planes][kPrefillTokens][heads * plane_pitch]
-    int plane_pitch;
+    // A prompt block's finished rows, hi + lo: [2 planes][kPrefillTokens][plane_row], head after head of plane_pitch
+    // columns, of which the first plane_cols are written
+    __nv_bfloat16* planes;
+    int plane_pitch, plane_cols, plane_row;
 };
+
+// Global query row of a group's row r.
+__device__ __forceinline__ int latent_row(const LatentAttnArgs& a, int group, int r) {
+    const int t = r / a.heads;
+    return t * a.all_heads + group * a.heads + (r - t * a.heads);
+}
+__device__ __forceinline__ float latent_score(const LatentAttnArgs& a, float dot) {
+    const float s = dot * a.scale;
+    return a.softcap > 0.f ? a.softcap * tanhf(__fdiv_rn(s, a.softcap)) : s;
+}
+// The last of `n` CTAs to get here returns true, with the others' global stores visible.  NT threads, all of the CTA.
+__device__ __forceinline__ bool latent_last_arrival(unsigned int* counter, int n, int* flag, int tid) {
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) *flag = atomicAdd(counter, 1u) == (unsigned int)n - 1u;
+    __syncthreads();
+    if (!*flag) return false;
+    __threadfence();
+    if (tid == 0) *counter = 0u;
+    return true;
+}
+// One column of a query row from its n_eff partial results, p = the row's first one: added up in split order.
+__device__ __forceinline__ float latent_combine1(const LatentAttnArgs& a, const float* p, int n_eff, int col) {
+    const int stride = a.rank_pitch + kLatentPartTail;
+    float mm = -INFINITY, av = 0.f, lv = 0.f;
+    for (int s0 = 0; s0 < n_eff; s0 += 8) {
+        float ms[8], ls[8], as[8], mb = mm;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const bool ok = s0 + i < n_eff;
+            const float* ps = p + (size_t)(s0 + i) * stride;
+            ms[i] = ok ? __ldcg(ps + a.rank_pitch) : -INFINITY;
+            ls[i] = ok ? __ldcg(ps + a.rank_pitch + 1) : 0.f;
+            as[i] = ok ? __ldcg(ps + col) : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < 8; ++i) mb = fmaxf(mb, ms[i]);
+        const float fo = mm == -INFINITY ? 0.f : expf(mm - mb);
+        av *= fo;
+        lv *= fo;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const float f = ms[i] == -INFINITY ? 0.f : expf(ms[i] - mb);
+            av = fmaf(as[i], f, av);
+            lv = fmaf(ls[i], f, lv);
+        }
+        mm = mb;
+    }
+    return __fdiv_rn(av, lv);
+}
+__device__ __forceinline__ void latent_out(const LatentAttnArgs& a, int head, int col, float v) {
+    const int at = head * a.out_cols + col;
+    a.out[at] = a.gate ? v * __ldcg(a.gate + at) : v;
+}
 
 constexpr int kLatentMaxCluster = 8;
 constexpr int kLatentTile = 64;        // keys per shared-memory tile
@@ -40,6 +106,7 @@ template <typename KT>
 static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(const LatentAttnArgs a) {
     extern __shared__ float lat_smem[];  // query row, then scores of a tile
     __shared__ float s_f, s_m, s_l;
+    __shared__ int s_last;
     float* qs = lat_smem;
     float* sc = lat_smem + a.row_width;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -52,9 +119,9 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(cons
     const int split = blockIdx.x;
     if (split >= sp.n_eff) return;
     const int k_begin = sp.first + split * sp.chunk, k_end = min(k_begin + sp.chunk, pos + 1);
-    const size_t row = (size_t)blockIdx.z * a.heads + blockIdx.y;
+    const size_t row = (size_t)blockIdx.z * a.all_heads + blockIdx.y;
     const KT* q = reinterpret_cast<const KT*>(a.q) + row * a.row_width;
-    const KT* kc = reinterpret_cast<const KT*>(a.cache);
+    const KT* kc = reinterpret_cast<const KT*>(a.cache) + (size_t)(blockIdx.y / a.heads) * a.seq_len * a.row_width;
     for (int i = tid; i < a.row_width; i += kLatentThreads) qs[i] = to_float(q[i]);
     if (tid == 0) s_m = -INFINITY, s_l = 0.f;
     float o[kLatentMaxPerThread];
@@ -68,7 +135,7 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(cons
             float s = 0.f;
             for (int i = lane; i < a.row_width; i += 32) s = fmaf(qs[i], to_float(kr[i]), s);
             s = warp_sum(s);
-            if (lane == 0) sc[k] = s * a.scale;
+            if (lane == 0) sc[k] = latent_score(a, s);
         }
         __syncthreads();
         if (warp == 0) {
@@ -99,7 +166,14 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(cons
         }
         __syncthreads();
     }
-    float* p = a.part + (row * a.max_splits + split) * (a.rank_pitch + kLatentPartTail);
+    if (a.out && sp.n_eff == 1) {  // all keys seen
+#pragma unroll
+        for (int j = 0; j < kLatentMaxPerThread; ++j)
+            if (tid + j * kLatentThreads < a.out_cols) latent_out(a, blockIdx.y, tid + j * kLatentThreads, __fdiv_rn(o[j], s_l));
+        return;
+    }
+    float* p0 = a.part + row * a.max_splits * (a.rank_pitch + kLatentPartTail);
+    float* p = p0 + (size_t)split * (a.rank_pitch + kLatentPartTail);
 #pragma unroll
     for (int j = 0; j < kLatentMaxPerThread; ++j)
         if (tid + j * kLatentThreads < a.rank_pitch) p[tid + j * kLatentThreads] = o[j];
@@ -107,9 +181,11 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(cons
         p[a.rank_pitch] = s_m;
         p[a.rank_pitch + 1] = s_l;
     }
+    if (!a.out || !latent_last_arrival(a.counters + blockIdx.y, sp.n_eff, &s_last, tid)) return;
+    for (int i = tid; i < a.out_cols; i += kLatentThreads) latent_out(a, blockIdx.y, i, latent_combine1(a, p0, sp.n_eff, i));
 }
 
-// ---- tensor cores, FP16 rows.  grid: (splits, row tiles of 16 MT); with `cluster` set the splits of a row tile are one
+// ---- tensor cores, FP16 rows.  grid: (splits, row tiles of 16 MT, groups); with `cluster` set the splits of a row tile are one
 // thread-block cluster.
 //
 // Query tile and 64-key tiles (double buffered, 16-byte asynchronous copies) lie in shared memory in rows padded by 16
@@ -121,7 +197,8 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(cons
 // The splits meet in one of two ways.  Prompt block: every CTA leaves its unnormalised result in its own shared memory, and
 // after a cluster barrier each adds up a share of the row tile over all CTAs through distributed shared memory; the
 // finished rows go out as hi + lo operands.  One token: partial results to part, as the CUDA-core kernel does (for 17
-// splits of 64 keys the cluster's gang launch and two barriers cost 4 us more than the value GEMV needs to add them up).
+// splits of 64 keys the cluster's gang launch and two barriers cost 4 us more than the value GEMV needs to add them up);
+// with `out` set the last CTA of a row tile puts them together, and a span of one split goes out at once.
 __device__ __forceinline__ void cluster_barrier() {
     asm volatile("barrier.cluster.arrive.release;\n\tbarrier.cluster.wait.acquire;" ::: "memory");
 }
@@ -140,6 +217,30 @@ __device__ __forceinline__ float cluster_load(uint32_t addr) {
     float v;
     asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(addr));
     return v;
+}
+
+// Columns col .. col + 3 of a finished row of a prompt block, times the gate, as hi + lo operands.
+__device__ __forceinline__ void latent_planes4(const LatentAttnArgs& a, int t, int h, int col, float (&y)[4]) {
+    if (a.gate) {
+        const float* g = a.gate + ((size_t)t * a.all_heads + h) * a.plane_cols + col;
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+            if (col + c < a.plane_cols) y[c] *= __ldcg(g + c);
+    }
+    __nv_bfloat16* d = a.planes + (size_t)t * a.plane_row + (size_t)h * a.plane_pitch + col;
+    __nv_bfloat16* d_lo = d + (size_t)kPrefillTokens * a.plane_row;
+    __align__(8) __nv_bfloat16 hi[4], lo[4];
+#pragma unroll
+    for (int c = 0; c < 4; ++c) split_pair(y[c], hi[c], lo[c]);
+    if (((a.plane_pitch | a.plane_cols) & 3) == 0) {
+        if (col >= a.plane_cols) return;
+        *reinterpret_cast<uint2*>(d) = *reinterpret_cast<const uint2*>(hi);
+        *reinterpret_cast<uint2*>(d_lo) = *reinterpret_cast<const uint2*>(lo);
+        return;
+    }
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+        if (col + c < a.plane_cols) d[c] = hi[c], d_lo[c] = lo[c];
 }
 
 constexpr int kLatScPitch = kLatentTile + 4, kLatPPitch = kLatentTile + 8;
@@ -181,8 +282,9 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
     }
     const int k_begin = sp.first + split * sp.chunk, k_end = min(k_begin + sp.chunk, base + t_hi + 1);
     const int n_tiles = active ? (k_end - k_begin + kLatentTile - 1) / kLatentTile : 0;
-    const unsigned char* cache = reinterpret_cast<const unsigned char*>(a.cache);
     const size_t row_bytes = (size_t)a.row_width * 2;
+    const int group = blockIdx.z;
+    const unsigned char* cache = reinterpret_cast<const unsigned char*>(a.cache) + (size_t)group * a.seq_len * row_bytes;
     const int pieces = a.row_width / 8;
 
     // rows of the tile in [lo, hi); with `fill` the rows between k_end and the next multiple of 16 become zero
@@ -205,7 +307,7 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
         load_keys(0, max(k_begin, base), k_end, true);
         for (int r = warp; r < kRows; r += NW) {
             const bool in = r0 + r < n_rows;
-            const unsigned char* src = reinterpret_cast<const unsigned char*>(a.q) + (in ? (size_t)(r0 + r) * row_bytes : 0);
+            const unsigned char* src = reinterpret_cast<const unsigned char*>(a.q) + (in ? (size_t)latent_row(a, group, r0 + r) * row_bytes : 0);
             for (int col = lane; col < pieces; col += 32) cp_async_16(qs + r * pitch + col * 16, src + (in ? col * 16 : 0), in);
         }
     }
@@ -221,9 +323,9 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
     for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int i = 0; i < NT; ++i) o[m][i][0] = o[m][i][1] = o[m][i][2] = o[m][i][3] = 0.f;
-    const int k_steps = a.row_width / 16;
+    const int k_steps = a.row_width / 16 - a.score_skip;
     const int key16 = warp & 3, part = warp >> 2;  // scores: this warp's 16 keys and its share of the k-steps
-    const int ks0 = part * k_steps / kParts, ks1 = (part + 1) * k_steps / kParts;
+    const int ks0 = a.score_skip + part * k_steps / kParts, ks1 = a.score_skip + (part + 1) * k_steps / kParts;
     const uint32_t q_addr = smem_u32(qs) + (uint32_t)(((mi & 1) * 8 + mr) * pitch + (mi >> 1) * 16);
     const uint32_t p_addr = smem_u32(ps) + (uint32_t)((((mi & 1) * 8 + mr) * kLatPPitch + (mi >> 1) * 8) * 2);
 
@@ -281,8 +383,8 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
                     v0 += s0[q * kRows * kLatScPitch];
                     v1 += s0[q * kRows * kLatScPitch + 32];
                 }
-                x0[i] = (p >= lo && p <= last && p < k_end) ? v0 * a.scale : -INFINITY;
-                x1[i] = (p + 32 >= lo && p + 32 <= last && p + 32 < k_end) ? v1 * a.scale : -INFINITY;
+                x0[i] = (p >= lo && p <= last && p < k_end) ? latent_score(a, v0) : -INFINITY;
+                x1[i] = (p + 32 >= lo && p + 32 <= last && p + 32 < k_end) ? latent_score(a, v1) : -INFINITY;
                 m_old[i] = s_m[r];
                 m_new[i] = fmaxf(x0[i], x1[i]);
             }
@@ -346,6 +448,24 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
     }
     __syncthreads();
     if (!a.cluster) {
+        if (a.out && sp.n_eff == 1) {  // all keys seen: finished rows
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int half = 0; half < 2; ++half) {
+                    const int r = m * 16 + g + 8 * half;
+                    if (r0 + r >= n_rows) continue;
+                    const int head = latent_row(a, group, r0 + r);  // one token: row = head
+                    const float l = s_l[r];
+#pragma unroll
+                    for (int i = 0; i < NT; ++i) {
+                        const int col = warp * NT * 8 + i * 8 + 2 * tq;
+                        if (col < a.out_cols) latent_out(a, head, col, __fdiv_rn(o[m][i][2 * half], l));
+                        if (col + 1 < a.out_cols) latent_out(a, head, col + 1, __fdiv_rn(o[m][i][2 * half + 1], l));
+                    }
+                }
+            return;
+        }
         const int stride = a.rank_pitch + kLatentPartTail;
 #pragma unroll
         for (int m = 0; m < MT; ++m)
@@ -353,7 +473,7 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
             for (int half = 0; half < 2; ++half) {
                 const int r = m * 16 + g + 8 * half;
                 if (r0 + r >= n_rows) continue;
-                float* dst = a.part + ((size_t)(r0 + r) * a.max_splits + split) * stride;
+                float* dst = a.part + ((size_t)latent_row(a, group, r0 + r) * a.max_splits + split) * stride;
 #pragma unroll
                 for (int i = 0; i < NT; ++i) {
                     const int col = warp * NT * 8 + i * 8 + 2 * tq;
@@ -361,6 +481,13 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
                 }
                 if (warp == 0 && tq == 0) *reinterpret_cast<float2*>(dst + a.rank_pitch) = make_float2(s_m[r], s_l[r]);
             }
+        if (!a.out) return;
+        if (!latent_last_arrival(a.counters + group * gridDim.y + blockIdx.y, sp.n_eff, reinterpret_cast<int*>(s_w), tid)) return;
+        const int rows_here = min(kRows, n_rows - r0);
+        for (int i = tid; i < rows_here * a.out_cols; i += kThreads) {
+            const int r = i / a.out_cols, col = i - r * a.out_cols, head = latent_row(a, group, r0 + r);
+            latent_out(a, head, col, latent_combine1(a, a.part + (size_t)head * a.max_splits * stride, sp.n_eff, col));
+        }
         return;
     }
     // this CTA's result over the key tiles (nobody reads them any more), rows of rank_pitch + 4 floats: that fits, as
@@ -415,27 +542,20 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
                 const float w = s_w[r * kLatentMaxCluster + c];
                 y[0] = fmaf(w, x[c].x, y[0]); y[1] = fmaf(w, x[c].y, y[1]); y[2] = fmaf(w, x[c].z, y[2]); y[3] = fmaf(w, x[c].w, y[3]);
             }
-        const int t = (r0 + r) / a.heads, h = r0 + r - t * a.heads;
-        __nv_bfloat16* d = a.planes + (size_t)t * a.heads * a.plane_pitch + (size_t)h * a.plane_pitch + col;
-        __align__(8) __nv_bfloat16 hi[4], lo[4];
-#pragma unroll
-        for (int c = 0; c < 4; ++c) split_pair(y[c], hi[c], lo[c]);
-        *reinterpret_cast<uint2*>(d) = *reinterpret_cast<const uint2*>(hi);
-        *reinterpret_cast<uint2*>(d + (size_t)kPrefillTokens * a.heads * a.plane_pitch) = *reinterpret_cast<const uint2*>(lo);
+        const int t = (r0 + r) / a.heads, h = group * a.heads + (r0 + r - t * a.heads);
+        latent_planes4(a, t, h, col, y);
     }
     cluster_barrier();  // every CTA's shared memory stays until all have read it
 }
 
-// ---- prompt block: the splits of every query row put together, as hi + lo MMA operands of the value GEMM.
-// grid: rows; out: [2 planes][kPrefillTokens][heads * in_pitch], in_pitch >= rank_pitch inputs per head
-template <typename T>
-static __global__ void __launch_bounds__(128) prefill_latent_combine_kernel(const LatentAttnArgs a, int tile_rows, T* out, int in_pitch) {
+// ---- prompt block: the splits of every query row put together (plane_cols columns).  grid: rows
+static __global__ void __launch_bounds__(128) prefill_latent_combine_kernel(const LatentAttnArgs a, int tile_rows) {
     __shared__ float wt[kLatentMaxSplits];
     pdl_launch_dependents();
     pdl_wait();
-    const int row = blockIdx.x, t = row / a.heads, h = row - t * a.heads;
-    const int n_rows = a.n_tokens * a.heads;
-    const int r0 = row / tile_rows * tile_rows, r1 = min(r0 + tile_rows, n_rows) - 1;  // the row's tile in the attention launch
+    const int row = blockIdx.x, t = row / a.all_heads, h = row - t * a.all_heads;
+    const int n_rows = a.n_tokens * a.heads, r = t * a.heads + h % a.heads;  // of the head's group
+    const int r0 = r / tile_rows * tile_rows, r1 = min(r0 + tile_rows, n_rows) - 1;  // the row's tile in the attention launch
     const LatentSpan sp = latent_span(a.start_pos + r0 / a.heads, a.start_pos + r1 / a.heads, a.window, a.max_splits, a.min_chunk);
     const int stride = a.rank_pitch + kLatentPartTail, lane = threadIdx.x & 31;
     const float* p = a.part + (size_t)row * a.max_splits * stride;
@@ -449,23 +569,14 @@ static __global__ void __launch_bounds__(128) prefill_latent_combine_kernel(cons
         wt[lane] = __fdiv_rn(e, sum);
     }
     __syncthreads();
-    T* hi_row = out + (size_t)t * a.heads * in_pitch + (size_t)h * in_pitch;
-    T* lo_row = hi_row + (size_t)kPrefillTokens * a.heads * in_pitch;
-    for (int k = 2 * threadIdx.x; k < a.rank_pitch; k += 256) {
-        float2 v = make_float2(0.f, 0.f);
+    for (int k = 4 * threadIdx.x; k < a.rank_pitch; k += 512) {
+        float y[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 4
         for (int s = 0; s < sp.n_eff; ++s) {
-            const float2 x = __ldcg(reinterpret_cast<const float2*>(p + (size_t)s * stride + k));
-            v.x = fmaf(wt[s], x.x, v.x);
-            v.y = fmaf(wt[s], x.y, v.y);
+            const float4 x = __ldcg(reinterpret_cast<const float4*>(p + (size_t)s * stride + k));
+            y[0] = fmaf(wt[s], x.x, y[0]); y[1] = fmaf(wt[s], x.y, y[1]); y[2] = fmaf(wt[s], x.z, y[2]); y[3] = fmaf(wt[s], x.w, y[3]);
         }
-        T hi[2], lo[2];
-        split_pair(v.x, hi[0], lo[0]);
-        split_pair(v.y, hi[1], lo[1]);
-        hi_row[k] = hi[0];
-        hi_row[k + 1] = hi[1];
-        lo_row[k] = lo[0];
-        lo_row[k + 1] = lo[1];
+        latent_planes4(a, t, h, k, y);
     }
 }
 

@@ -556,7 +556,8 @@ static __global__ void __launch_bounds__(256) prefill_qkv_finish_kernel(const Pr
 }
 
 // Rows of the residual stream -> normalised rows (hi + lo MMA operands): RMSNorm, or LayerNorm when a bias is given.
-// Layer 0 takes the embedding rows of the prompt tokens and also writes them out as the FP32 residual stream.  With a
+// Layer 0 takes the embedding rows of the prompt tokens, times their factor, and also writes them out as the FP32 residual
+// stream.  With a
 // row list, block i takes row rows[i] (the positions whose logits are wanted).  D is the row pitch; the statistics cover
 // the first norm_n inputs, the rest is zero padding with zero weights.  grid: rows.
 constexpr int kPfNormThreads = 512;
@@ -564,6 +565,8 @@ struct PrefillNormArgs {
     float* x;            // [kPrefillTokens][D]
     const int* tokens;   // with emb
     const void* emb;     // [vocab][D], nullptr = the rows of x
+    float emb_scale;     // factor of the embedding rows
+    const float* add;    // [D] added to every row first (nullptr = nothing)
     int vocab;
     const int* rows;     // nullptr = block i takes row i
     const float* norm_w;
@@ -614,7 +617,7 @@ static __global__ void __launch_bounds__(kPfNormThreads) prefill_norm_kernel(con
         if (a.emb) {
             const uint2 h = __ldg(reinterpret_cast<const uint2*>(reinterpret_cast<const T*>(a.emb) + (size_t)tok * D + 4 * (size_t)i));
             const float2 lo = unpack2<T>(h.x), hi = unpack2<T>(h.y);
-            w = make_float4(lo.x, lo.y, hi.x, hi.y);
+            w = make_float4(lo.x * a.emb_scale, lo.y * a.emb_scale, hi.x * a.emb_scale, hi.y * a.emb_scale);
         } else {
             w = xr[i];
         }
@@ -628,7 +631,11 @@ static __global__ void __launch_bounds__(kPfNormThreads) prefill_norm_kernel(con
                     w.x += p[s0].x; w.y += p[s0].y; w.z += p[s0].z; w.w += p[s0].w;
                 }
         }
-        if (a.emb || add_parts) xr[i] = w;  // the residual stream as the next residual GEMM reads it
+        if (a.add) {
+            const float4 p = __ldg(reinterpret_cast<const float4*>(a.add) + i);
+            w.x += p.x; w.y += p.y; w.z += p.z; w.w += p.w;
+        }
+        if (a.emb || a.add || add_parts) xr[i] = w;  // the residual stream as the next residual GEMM reads it
         return w;
     };
     const bool ln = a.norm_b != nullptr;

@@ -13,7 +13,7 @@ from typing import Dict, Iterable, Optional, Sequence, Tuple
 
 import numpy as np
 
-from .formats import LayeredConfig, ModelConfig
+from .formats import LatentMixer, LayeredConfig, MambaMixer, ModelConfig, SharedKvMixer
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "liblpp_b200.so")
@@ -25,13 +25,14 @@ TENSOR_IDS = {"tok_emb": 0, "rms_att": 1, "wq": 2, "wk": 3, "wv": 4, "wo": 5, "r
               "w3": 9, "rms_final": 10, "w_cls": 11,
               # models described layer by layer
               "norm1_b": 12, "norm2_b": 13, "norm_final_b": 14, "lat_q": 15, "lat_dkv": 16, "lat_norm": 17, "lat_uk": 18,
-              "lat_uv": 19, "lat_g": 20}
-_UNSTACKED = ("tok_emb", "rms_final", "w_cls", "norm_final_b")
+              "lat_uv": 19, "lat_g": 20, "wq_b": 21, "wk_b": 22, "wo_b": 23, "wg": 24, "scan_in": 25, "scan_conv": 26,
+              "scan_conv_b": 27, "scan_low": 28, "scan_dt": 29, "scan_dt_b": 30, "scan_a_log": 31, "scan_d": 32, "loop_step": 33}
+_UNSTACKED = ("tok_emb", "rms_final", "w_cls", "norm_final_b", "loop_step")
 TP_HANDLE_BYTES = 64
 FLAG_TP_NCCL, FLAG_TP_LOCAL, FLAG_NO_PREFILL_GEMM, FLAG_LATENT_CUDA_CORES = 32, 64, 128, 256
-MIXERS, NORMS, ACTIVATIONS = {"latent": 1}, {"rms": 0, "layer": 1}, {"silu": 0, "gelu_tanh": 1}
+MIXERS, NORMS, ACTIVATIONS = {LatentMixer: 1, SharedKvMixer: 2, MambaMixer: 3}, {"rms": 0, "layer": 1}, {"silu": 0, "gelu_tanh": 1}
 KINDS = ["qkv_gemv", "attention", "oproj_gemv", "gateup_gemv", "down_gemv", "lmhead_gemv", "sampler", "allreduce",
-         "latent_query_gemv", "latent_value_gemv"]
+         "latent_query_gemv", "latent_value_gemv", "scan_low_gemv", "scan"]
 
 # every symbol include/lpp_b200.h declares; tests check the built library exports all of them
 EXPORTS = [
@@ -63,13 +64,17 @@ class LayerDesc(C.Structure):
     _fields_ = [("mixer", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32), ("rot_dim", C.c_int32), ("vdim", C.c_int32),
                 ("kv_rank", C.c_int32), ("window", C.c_int32), ("scale", C.c_float), ("rot_dims", C.c_int32),
                 ("rot_base", C.c_double), ("yarn_factor", C.c_double), ("yarn_original", C.c_double),
-                ("yarn_fast", C.c_double), ("yarn_slow", C.c_double), ("ff", C.c_int32), ("act", C.c_int32)]
+                ("yarn_fast", C.c_double), ("yarn_slow", C.c_double), ("ff", C.c_int32), ("act", C.c_int32),
+                ("kv_heads", C.c_int32), ("bias", C.c_int32), ("gate", C.c_int32), ("softcap", C.c_float), ("inner", C.c_int32),
+                ("state", C.c_int32), ("conv", C.c_int32), ("dt_rank", C.c_int32)]
 
 
 class ModelDesc(C.Structure):
     _fields_ = [("dim", C.c_int32), ("vocab_size", C.c_int32), ("seq_len", C.c_int32), ("n_layers", C.c_int32),
                 ("norm", C.c_int32), ("norm_eps", C.c_float), ("weight_dtype", C.c_int32), ("kv_dtype", C.c_int32),
-                ("device", C.c_int32), ("flags", C.c_uint32), ("ring_kb", C.c_int32), ("wait_ms", C.c_int32)]
+                ("device", C.c_int32), ("flags", C.c_uint32), ("ring_kb", C.c_int32), ("wait_ms", C.c_int32),
+                ("emb_scale", C.c_float), ("logit_scale", C.c_float), ("loop_start", C.c_int32), ("loop_stop", C.c_int32),
+                ("loop_times", C.c_int32)]
 
 
 class SampleParams(C.Structure):
@@ -175,16 +180,23 @@ class Engine:
     def _create_layers(self, cfg: LayeredConfig, device: int, flags: int, ring_kb: int, wait_ms: int) -> None:
         layers = (LayerDesc * len(cfg.layers))()
         for d, y in zip(layers, cfg.layers):
-            m, r = y.mixer, y.mixer.rotation
-            d.mixer = MIXERS["latent"]
-            d.heads, d.dim, d.rot_dim, d.vdim, d.kv_rank = m.heads, m.dim, m.rot_dim, m.vdim, m.kv_rank
-            d.window, d.scale = m.window, m.scale
+            m = y.mixer
+            d.mixer, d.ff, d.act = MIXERS[type(m)], y.ff, ACTIVATIONS[y.act]
+            if isinstance(m, MambaMixer):
+                d.inner, d.state, d.conv, d.dt_rank = m.inner, m.state, m.conv, m.dt_rank
+                continue
+            d.heads, d.dim, d.window, d.scale = m.heads, m.dim, m.window, m.scale
+            if isinstance(m, LatentMixer):
+                d.rot_dim, d.vdim, d.kv_rank = m.rot_dim, m.vdim, m.kv_rank
+            else:
+                d.kv_heads, d.softcap, d.bias, d.gate = m.kv_heads, m.softcap, m.bias, m.gate
+            r = m.rotation
             d.rot_dims, d.rot_base = r.dims, r.base
             if r.yarn is not None:
                 d.yarn_factor, d.yarn_original, d.yarn_fast, d.yarn_slow = r.yarn.factor, r.yarn.original, r.yarn.fast, r.yarn.slow
-            d.ff, d.act = y.ff, ACTIVATIONS[y.act]
-        m = ModelDesc(cfg.dim, cfg.vocab_size, cfg.seq_len, len(cfg.layers), NORMS[cfg.norm], cfg.norm_eps,
-                      self.weight_dtype, self.kv_dtype, device, flags, ring_kb, wait_ms)
+        loop = (cfg.loop.start, cfg.loop.stop, cfg.loop.times) if cfg.loop else (0, 0, 0)
+        m = ModelDesc(cfg.dim, cfg.vocab_size, cfg.seq_len, len(cfg.layers), NORMS[cfg.norm], cfg.norm_eps, self.weight_dtype,
+                      self.kv_dtype, device, flags, ring_kb, wait_ms, cfg.emb_scale, cfg.logit_scale, *loop)
         h = C.c_void_p()
         _check(self.lib.lpp_engine_create_layers(C.byref(m), layers, C.byref(h)), "lpp_engine_create_layers")
         self.h = h
@@ -314,7 +326,7 @@ class Engine:
         return k, v
 
     def latent_read(self, layer: int, pos: int) -> np.ndarray:
-        """One cache row of a latent-attention layer: normed latent, then the rotated key part."""
+        """One cache row of a latent-attention layer outside a loop's reach: normed latent, then the rotated key part."""
         m = self.cfg.layers[layer].mixer
         row = np.empty(m.kv_rank + m.rot_dim, dtype=np.float32)
         _check(self.lib.lpp_latent_read(self.h, layer, pos, row.ctypes.data_as(C.POINTER(C.c_float))), "lpp_latent_read")
@@ -338,12 +350,12 @@ class Engine:
     def profile_step(self, pos: int, iters: int = 5, temperature: float = 0.0, penalty: float = 1.0
                      ) -> Dict[str, Dict[str, float]]:
         """Isolated per-kernel-kind durations of one step; the sampler runs with the given parameters."""
-        ms = (C.c_float * 10)()
-        n = (C.c_int * 10)()
-        b = (C.c_int64 * 10)()
+        ms = (C.c_float * len(KINDS))()
+        n = (C.c_int * len(KINDS))()
+        b = (C.c_int64 * len(KINDS))()
         sp = SampleParams(temperature, penalty)
         _check(self.lib.lpp_profile_step(self.h, int(pos), int(iters), C.byref(sp), ms, n, b), "lpp_profile_step")
-        return {KINDS[i]: {"ms": float(ms[i]), "launches": int(n[i]), "bytes": int(b[i])} for i in range(10)}
+        return {KINDS[i]: {"ms": float(ms[i]), "launches": int(n[i]), "bytes": int(b[i])} for i in range(len(KINDS))}
 
     def tp_export(self) -> bytes:
         """IPC handle of this rank's exchange buffer (to be gathered over the caller's host channel)."""

@@ -17,7 +17,7 @@ from __future__ import annotations
 import json
 import struct
 from dataclasses import dataclass, asdict, field
-from typing import Dict, Iterable, List, Optional, Tuple
+from typing import Dict, Iterable, List, Optional, Tuple, Union
 
 import numpy as np
 
@@ -83,8 +83,40 @@ class LatentMixer:
 
 
 @dataclass
+class SharedKvMixer:
+    """Grouped-query attention whose values are its keys before rotation.  ``softcap`` 0 = plain scores, ``bias`` on
+    queries, keys and output, ``gate`` = a sigmoid gate per element of the result; ``window`` 0 = all earlier positions."""
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    rotation: Rotation
+    window: int = 0
+    softcap: float = 0.0
+    bias: bool = False
+    gate: bool = False
+
+
+@dataclass
+class MambaMixer:
+    """Selective scan over ``inner`` channels of ``state`` elements, after a causal convolution over ``conv`` tokens."""
+    inner: int
+    state: int
+    conv: int
+    dt_rank: int
+
+
+@dataclass
+class Loop:
+    """Layers start .. stop - 1 run ``times`` times in a row; a vector of its own is added before every pass."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass
 class Layer:
-    mixer: LatentMixer
+    mixer: Union[LatentMixer, SharedKvMixer, MambaMixer]
     ff: int = 0  # 0 = no feed-forward
     act: str = "silu"
 
@@ -98,6 +130,9 @@ class LayeredConfig:
     layers: List[Layer] = field(default_factory=list)
     norm: str = "rms"
     norm_eps: float = 1e-5
+    emb_scale: float = 1.0
+    logit_scale: float = 1.0
+    loop: Optional[Loop] = None
 
     @property
     def n_layers(self) -> int:

@@ -14,7 +14,7 @@ from typing import Callable, Dict, Iterator, NamedTuple, Tuple
 import numpy as np
 
 from .engine import Engine
-from .formats import (Layer, LatentMixer, LayeredConfig, Rotation, Yarn, load_model, read_safetensors)
+from .formats import (Layer, LatentMixer, LayeredConfig, Loop, MambaMixer, Rotation, SharedKvMixer, Yarn, load_model, read_safetensors)
 
 TensorRow = Tuple[str, int, str, Tuple[int, ...]]
 
@@ -32,17 +32,30 @@ def _rotation(rot: dict) -> Rotation:
     return Rotation(int(rot["dims"]), float(rot["base"]), yarn)
 
 
+def _feed_forward(i: int, y: dict) -> int:
+    mlp = y.get("mlp")
+    if mlp and mlp["kind"] != "dense":
+        raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+    return int(mlp["ff"]) if mlp else 0
+
+
+def _feed_forward_tensors(i: int, y: Layer, dim: int) -> Iterator[TensorRow]:
+    if y.ff:
+        yield "rms_ffn", i, f"l{i}.norm2", (dim,)
+        yield "w1", i, f"l{i}.mlp.gate", (y.ff, dim)
+        yield "w3", i, f"l{i}.mlp.up", (y.ff, dim)
+        yield "w2", i, f"l{i}.mlp.down", (dim, y.ff)
+
+
 def rutenex_config(cfg: dict, seq_len: int) -> LayeredConfig:
     layers = []
     for i, y in enumerate(cfg["layers"]):
         if y["type"] != "latent_attention":
             raise ValueError(f"layer {i}: unknown mixer {y['type']!r}")
-        m, mlp, mask = y["mixer"], y.get("mlp"), y["mixer"].get("mask") or {}
-        if mlp and mlp["kind"] != "dense":
-            raise ValueError(f"layer {i}: unknown feed-forward {mlp['kind']!r}")
+        m, mask = y["mixer"], y["mixer"].get("mask") or {}
         layers.append(Layer(LatentMixer(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]),
                                         float(m["scale"]), _rotation(m["rot"]), int(mask.get("size") or 0)),
-                            int(mlp["ff"]) if mlp else 0, "gelu_tanh"))
+                            _feed_forward(i, y), "gelu_tanh"))
     return LayeredConfig(int(cfg["width"]), int(cfg["vocab"]), seq_len, layers, "layer", float(cfg["norm"]["eps"]))
 
 
@@ -60,17 +73,70 @@ def rutenex_tensors(c: LayeredConfig) -> Iterator[TensorRow]:
         yield "lat_uv", i, p + "mix.uv", (m.heads * m.vdim, m.kv_rank)
         yield "lat_g", i, p + "mix.g", (m.heads, D)
         yield "wo", i, p + "mix.o", (D, m.heads * m.vdim)
+        yield from _feed_forward_tensors(i, y, D)
         if y.ff:
-            yield "rms_ffn", i, p + "norm2", (D,)
             yield "norm2_b", i, p + "norm2.b", (D,)
-            yield "w1", i, p + "mlp.gate", (y.ff, D)
-            yield "w3", i, p + "mlp.up", (y.ff, D)
-            yield "w2", i, p + "mlp.down", (D, y.ff)
     yield "rms_final", 0, "final.norm", (D,)
     yield "norm_final_b", 0, "final.norm.b", (D,)
 
 
-ARCHITECTURES: Dict[str, Architecture] = {"Rutenex": Architecture(rutenex_config, rutenex_tensors)}
+# ------------------------------------------------------------------ Kolatar: selective-scan and key-is-value attention layers,
+# some of which run several times
+
+def kolatar_config(cfg: dict, seq_len: int) -> LayeredConfig:
+    layers = []
+    for i, y in enumerate(cfg["layers"]):
+        m = y["mixer"]
+        if y["type"] == "mamba1":
+            mixer = MambaMixer(int(m["inner"]), int(m["state"]), int(m["conv"]), int(m["dt_rank"]))
+        elif y["type"] == "attention":
+            if int(m.get("vdim", m["dim"])) != int(m["dim"]):
+                raise ValueError(f"layer {i}: values of {m['vdim']} dimensions cannot be keys of {m['dim']}")
+            mixer = SharedKvMixer(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), float(m["scale"]), _rotation(m["rot"]),
+                                  int((m.get("mask") or {}).get("size") or 0), float(m.get("softcap") or 0.0), bias=True, gate=True)
+        else:
+            raise ValueError(f"layer {i}: unknown mixer {y['type']!r}")
+        layers.append(Layer(mixer, _feed_forward(i, y), "silu"))
+    loop = cfg.get("loop")
+    return LayeredConfig(int(cfg["width"]), int(cfg["vocab"]), seq_len, layers, "rms", float(cfg["norm"]["eps"]),
+                         float(cfg["embedding"]["scale"]), float(cfg["logit_scale"]),
+                         Loop(int(loop["start"]), int(loop["stop"]), int(loop["times"])) if loop else None)
+
+
+def kolatar_tensors(c: LayeredConfig) -> Iterator[TensorRow]:
+    D = c.dim
+    yield "tok_emb", 0, "embed", (c.vocab_size, D)
+    if c.loop and c.loop.stop > c.loop.start:
+        yield "loop_step", 0, "loop.step", (c.loop.times, D)
+    for i, y in enumerate(c.layers):
+        p, m = f"l{i}.mix.", y.mixer
+        yield "rms_att", i, f"l{i}.norm1", (D,)
+        if isinstance(m, MambaMixer):
+            yield "scan_in", i, p + "in", (2 * m.inner, D)
+            yield "scan_conv", i, p + "conv", (m.inner, m.conv)
+            yield "scan_conv_b", i, p + "conv.b", (m.inner,)
+            yield "scan_low", i, p + "x", (m.dt_rank + 2 * m.state, m.inner)
+            yield "scan_dt", i, p + "dt", (m.inner, m.dt_rank)
+            yield "scan_dt_b", i, p + "dt.b", (m.inner,)
+            yield "scan_a_log", i, p + "A_log", (m.inner, m.state)
+            yield "scan_d", i, p + "D", (m.inner,)
+            yield "wo", i, p + "o", (D, m.inner)
+        else:
+            q, k = m.heads * m.dim, m.kv_heads * m.dim
+            yield "wq", i, p + "q", (q, D)
+            yield "wq_b", i, p + "q.b", (q,)
+            yield "wk", i, p + "k", (k, D)
+            yield "wk_b", i, p + "k.b", (k,)
+            yield "wg", i, p + "g", (q, D)
+            yield "wo", i, p + "o", (D, q)
+            yield "wo_b", i, p + "o.b", (D,)
+        yield from _feed_forward_tensors(i, y, D)
+    yield "rms_final", 0, "final.norm", (D,)
+    yield "w_cls", 0, "head", (c.vocab_size, D)
+
+
+ARCHITECTURES: Dict[str, Architecture] = {"Kolatar": Architecture(kolatar_config, kolatar_tensors),
+                                          "Rutenex": Architecture(rutenex_config, rutenex_tensors)}
 
 # weight / cache types of the two precisions a model folder is served in
 PRECISIONS = {"bfloat16": ("bf16", "f16"), "float32": ("f32", "f32")}
