@@ -46,6 +46,11 @@ LAYERED = {
     "rutenex-1b": (2048, 16, 8192, 32768, dict(heads=16, **_MLA), 1024, (32, 8), 1024),
     "rutenex-8b": (4096, 32, 14336, 32768, dict(heads=32, **_MLA), 4096, (32, 8), 1024),
     "rutenex-300m": (1024, 24, 2816, 32768, dict(heads=16, dim=64, rot_dim=32, vdim=64, kv_rank=256), 512, (16, 4), 1024),
+    # layers: groups of two selective-scan layers and an attention layer with the feed-forward, the first group running twice;
+    # the existing model has as many layers as make its weights per token about as many bytes
+    "kolatar-1b": (2048, 6, 8192, 32768, dict(inner=4096, state=16, conv=4, dt_rank=128, heads=32, kv_heads=8, dim=64), 1024, (32, 8), 1024),
+    "kolatar-8b": (4096, 11, 14336, 32768, dict(inner=8192, state=16, conv=4, dt_rank=256, heads=32, kv_heads=8, dim=128), 4096, (32, 8), 1024),
+    "kolatar-300m": (1024, 8, 2816, 32768, dict(inner=2048, state=16, conv=4, dt_rank=64, heads=16, kv_heads=4, dim=64), 512, (16, 4), 1024),
 }
 
 
@@ -472,33 +477,50 @@ def run_reference(args, rank, world):
             "e2e": {"value": cb["value"], "unit": "tok/s", "h2d_bytes_per_step": 0, "d2h_bytes_per_step": 0}}
 
 
+def layered_config(name):
+    """(architecture, its configuration, that of the existing model beside it)"""
+    from lighterpp_b200.formats import LatentMixer, Layer, LayeredConfig, Loop, MambaMixer, ModelConfig, Rotation, SharedKvMixer, Yarn
+    width, layers, ff, vocab, mix, window, (heads, kv), n_prompt = LAYERED[name]
+    seq, yarn = n_prompt + 1024, Yarn(4.0, 4096, 32.0, 1.0)
+    if name.startswith("rutenex"):
+        m = LatentMixer(scale=(mix["dim"] + mix["rot_dim"]) ** -0.5, window=window, rotation=Rotation(mix["rot_dim"], 1e6, yarn), **mix)
+        cfg = LayeredConfig(width, vocab, seq, [Layer(m, ff, "gelu_tanh") for _ in range(layers)], "layer", 1e-6)
+        return "Rutenex", cfg, ModelConfig(width, ff, layers, heads, kv, vocab, seq, 500000.0)
+    scan = Layer(MambaMixer(mix["inner"], mix["state"], mix["conv"], mix["dt_rank"]))
+    dim = mix["dim"]
+    attn = Layer(SharedKvMixer(mix["heads"], mix["kv_heads"], dim, dim ** -0.5, Rotation(dim // 2, 1e6, yarn), window, 30.0, True, True), ff)
+    cfg = LayeredConfig(width, vocab, seq, [scan, scan, attn] * layers, "rms", 1e-5, 1.0, 1.0, Loop(0, 3, 2))
+    scan_n = width * 3 * mix["inner"] + mix["inner"] * (2 * mix["dt_rank"] + 2 * mix["state"])
+    attn_n = width * dim * (3 * mix["heads"] + mix["kv_heads"]) + 3 * width * ff
+    llama_n = width * (2 * width + 2 * kv * width // heads) + 3 * width * ff
+    return "Kolatar", cfg, ModelConfig(width, ff, round((layers + 1) * (2 * scan_n + attn_n) / llama_n), heads, kv, vocab, seq, 500000.0)
+
+
 def layered_engines(name):
     """(label, engine) of the layered design and of the existing model, random weights, one after the other."""
     import torch
     from lighterpp_b200 import engine as E
-    from lighterpp_b200.formats import LatentMixer, Layer, LayeredConfig, ModelConfig, Rotation, Yarn
     from lighterpp_b200.models import ARCHITECTURES
-    width, layers, ff, vocab, mix, window, (heads, kv), n_prompt = LAYERED[name]
-    seq = n_prompt + 1024
+    arch, cfg, llama = layered_config(name)
     g = torch.Generator(device="cuda")
     g.manual_seed(7)
-    m = LatentMixer(scale=(mix["dim"] + mix["rot_dim"]) ** -0.5, window=window,
-                    rotation=Rotation(mix["rot_dim"], 1e6, Yarn(4.0, 4096, 32.0, 1.0)), **mix)
-    cfg = LayeredConfig(width, vocab, seq, [Layer(m, ff, "gelu_tanh") for _ in range(layers)], "layer", 1e-6)
     eng = E.Engine(cfg, "bf16", "f16")
-    for ours, layer, tensor, shape in ARCHITECTURES["Rutenex"].tensors(cfg):
-        if len(shape) == 1:
+    for ours, layer, tensor, shape in ARCHITECTURES[arch].tensors(cfg):
+        if tensor.endswith("dt.b"):
+            t = torch.full(shape, -3.0, device="cuda")
+        elif tensor.endswith("A_log"):
+            t = torch.log(torch.arange(1, shape[1] + 1, device="cuda").float()).repeat(shape[0], 1)
+        elif len(shape) == 1:
             t = torch.zeros(shape, device="cuda") if tensor.endswith(".b") else torch.ones(shape, device="cuda")
         else:
             t = torch.randn(shape, device="cuda", generator=g) * shape[1] ** -0.5
         eng.upload(ours, t.to(torch.bfloat16), layer)
     eng.finalize()
     torch.cuda.empty_cache()
-    yield "rutenex", eng
+    yield arch.lower(), eng
     eng.close()
-    cfg = ModelConfig(width, ff, layers, heads, kv, vocab, seq, 500000.0)
-    eng = E.Engine(cfg, "f16", "f16")
-    for tensor, l, t in gen_device_weights(cfg, "f16", True, 7):
+    eng = E.Engine(llama, "f16", "f16")
+    for tensor, l, t in gen_device_weights(llama, "f16", True, 7):
         eng.upload(tensor, t, max(l, 0))
     eng.finalize()
     torch.cuda.empty_cache()
@@ -544,7 +566,7 @@ def run_layered(args):
                            "decode_tok_s": round(1e6 / us, 1), "us_per_token": round(us, 1), "step_gbs": round(gbs, 1),
                            "step_frac_of_measured": round(gbs / peak, 3), "kernels_per_step": eng.kernels_per_step, "kernels": kinds}
     line["clocks"] = clk.summary()
-    line["value"] = line["rutenex"]["decode_tok_s"]
+    line["value"] = line[args.layered.split("-")[0]]["decode_tok_s"]
     return line
 
 

@@ -1541,7 +1541,7 @@ static lpp_status check_layer(const lpp_layer_desc& d, int l) {
     int cols = 0;
     switch (d.mixer) {
         case LPP_MIXER_LATENT:
-            if (d.heads <= 0 || d.dim <= 0 || d.rot_dim < 0 || d.rot_dim % 2 || d.vdim <= 0 || d.kv_rank <= 0) return fail(LPP_ERR_INVALID_ARG, "layer %d: bad size", l);
+            if (d.heads <= 0 || d.dim <= 0 || d.rot_dim < 0 || d.vdim <= 0 || d.kv_rank <= 0) return fail(LPP_ERR_INVALID_ARG, "layer %d: bad size", l);
             turnable = d.rot_dim;
             cols = d.kv_rank;
             break;
@@ -1557,7 +1557,7 @@ static lpp_status check_layer(const lpp_layer_desc& d, int l) {
             return LPP_OK;
         default: return fail(LPP_ERR_INVALID_ARG, "layer %d: unknown mixer %d", l, d.mixer);
     }
-    if (d.rot_dims % 2 || d.rot_dims > turnable) return fail(LPP_ERR_INVALID_ARG, "layer %d: rotation of %d of %d dimensions", l, d.rot_dims, turnable);
+    if (d.rot_dims % 2 || (d.mixer == LPP_MIXER_LATENT && d.rot_dim % 2) || d.rot_dims > turnable) return fail(LPP_ERR_INVALID_ARG, "layer %d: rotation of %d of %d dimensions", l, d.rot_dims, turnable);
     if (d.rot_dims > 0 && !(d.rot_base > 0.0)) return fail(LPP_ERR_INVALID_ARG, "layer %d: bad rotation base", l);
     if (d.yarn_factor != 0.0 && !(d.yarn_factor > 0.0 && d.yarn_original > 0.0 && d.yarn_fast > 0.0 && d.yarn_slow > 0.0))
         return fail(LPP_ERR_INVALID_ARG, "layer %d: bad rotation scaling", l);

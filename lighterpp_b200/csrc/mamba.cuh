@@ -83,12 +83,30 @@ struct MambaScanArgs {
     int taps, ring_pitch;
 };
 
-// S <- exp(dt A) S + dx B; returns this lane's share of S . C
+// exp(x) - 1 for x <= 0.  A channel that forgets slowly multiplies its state with a factor just below 1 thousands of times,
+// and always with much the same one: the rounding of the factor itself to 32 bits (2^-25 of it, the same way every time)
+// would add up, so the state is updated with its difference from 1.  Taylor series where it cancels (the first term left
+// out is below 2e-8 of the sum).
+__device__ __forceinline__ float decay_m1(float x) {
+    float p = fmaf(x, 1.f / 40320.f, 1.f / 5040.f);
+    p = fmaf(x, p, 1.f / 720.f);
+    p = fmaf(x, p, 1.f / 120.f);
+    p = fmaf(x, p, 1.f / 24.f);
+    p = fmaf(x, p, 1.f / 6.f);
+    p = fmaf(x, p, 0.5f);
+    p = fmaf(x * x, p, x);
+    return x > -0.5f ? p : expf(x) - 1.f;
+}
+// S <- exp(dt A) S + dx B
+__device__ __forceinline__ void state_update(float& S, float A, float B, float dt, float dx) {
+    S = fmaf(decay_m1(dt * A), S, fmaf(dx, B, S));
+}
+// The same for four elements; returns their share of S . C
 __device__ __forceinline__ float mamba_update(float4& S, const float4& A, const float4& B, const float4& C, float dt, float dx) {
-    S.x = fmaf(expf(dt * A.x), S.x, dx * B.x);
-    S.y = fmaf(expf(dt * A.y), S.y, dx * B.y);
-    S.z = fmaf(expf(dt * A.z), S.z, dx * B.z);
-    S.w = fmaf(expf(dt * A.w), S.w, dx * B.w);
+    state_update(S.x, A.x, B.x, dt, dx);
+    state_update(S.y, A.y, B.y, dt, dx);
+    state_update(S.z, A.z, B.z, dt, dx);
+    state_update(S.w, A.w, B.w, dt, dx);
     return fmaf(S.x, C.x, fmaf(S.y, C.y, fmaf(S.z, C.z, S.w * C.w)));
 }
 template <int L>
