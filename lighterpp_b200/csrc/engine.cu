@@ -252,6 +252,7 @@ struct lpp_engine {
     __half* pf_lq = nullptr;                        // query rows
     float *pf_lpart = nullptr, *pf_gate = nullptr;  // attention partials, gates
     float *pf_sx = nullptr, *pf_sz = nullptr, *pf_tail = nullptr;  // selective scan: convolved x, z, last convolution inputs
+    float* pf_low = nullptr;                                       // dt | B | C rows
     void* pf_sxp = nullptr;                                        // x as hi + lo operands
     CUtensorMap pf_map_wqkv, pf_map_wo, pf_map_w13, pf_map_w2, pf_map_xn, pf_map_att, pf_map_hb;
     bool pf_ready = false;
@@ -507,32 +508,37 @@ static LatentPlan latent_plan(const lpp_engine* e, const ModelLayer& y, int n_to
     return p;
 }
 
-template <int MT, int NT, int NW>
-static cudaError_t launch_latent_mma(lpp_engine* e, const LatentAttnArgs& a, int splits, bool pdl, cudaStream_t s) {
+template <int MT, int NT, int NW, bool SKV>
+static cudaError_t launch_latent_mma_t(lpp_engine* e, const LatentAttnArgs& a, int splits, bool pdl, cudaStream_t s) {
     static bool attr_done[64] = {};
     if (!attr_done[e->c.device & 63]) {
-        const cudaError_t r = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, NT, NW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)e->smem_optin);
+        const cudaError_t r = cudaFuncSetAttribute(latent_attn_mma_kernel<MT, NT, NW, SKV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)e->smem_optin);
         if (r != cudaSuccess) return r;
         attr_done[e->c.device & 63] = true;
     }
     const dim3 grid(splits, (a.n_tokens * a.heads + 16 * MT - 1) / (16 * MT), a.all_heads / a.heads);
-    return launch_clusters(latent_attn_mma_kernel<MT, NT, NW>, grid, dim3(32 * NW), (size_t)latent_mma_smem<MT, NW>(a.row_width), s, pdl,
+    return launch_clusters(latent_attn_mma_kernel<MT, NT, NW, SKV>, grid, dim3(32 * NW), (size_t)latent_mma_smem<MT, NW>(a.row_width), s, pdl,
                            a.cluster ? splits : 0, a);
 }
-static cudaError_t launch_latent_attn(lpp_engine* e, const LatentPlan& p, const LatentAttnArgs& a, bool pdl, cudaStream_t s) {
+template <int MT, int NT, int NW>
+static cudaError_t launch_latent_mma(lpp_engine* e, const LatentAttnArgs& a, int splits, bool skv, bool pdl, cudaStream_t s) {
+    return skv ? launch_latent_mma_t<MT, NT, NW, true>(e, a, splits, pdl, s) : launch_latent_mma_t<MT, NT, NW, false>(e, a, splits, pdl, s);
+}
+static cudaError_t launch_latent_attn(lpp_engine* e, const LatentPlan& p, const LatentAttnArgs& a, bool skv, bool pdl, cudaStream_t s) {
     const int rp = a.rank_pitch;
     if (p.mma) {
         constexpr int S = kLatStepWarps, B = kLatBlockWarps;
         if (a.n_tokens == 1)
-            return rp <= 128   ? launch_latent_mma<1, 2, S>(e, a, p.splits, pdl, s)
-                   : rp <= 256 ? launch_latent_mma<1, 4, S>(e, a, p.splits, pdl, s)
-                               : launch_latent_mma<1, 8, S>(e, a, p.splits, pdl, s);
+            return rp <= 128   ? launch_latent_mma<1, 2, S>(e, a, p.splits, skv, pdl, s)
+                   : rp <= 256 ? launch_latent_mma<1, 4, S>(e, a, p.splits, skv, pdl, s)
+                               : launch_latent_mma<1, 8, S>(e, a, p.splits, skv, pdl, s);
         if (p.tile_rows == 16)
-            return rp <= 256 ? launch_latent_mma<1, 2, B>(e, a, p.splits, pdl, s) : launch_latent_mma<1, 4, B>(e, a, p.splits, pdl, s);
-        return rp <= 256 ? launch_latent_mma<2, 2, B>(e, a, p.splits, pdl, s) : launch_latent_mma<2, 4, B>(e, a, p.splits, pdl, s);
+            return rp <= 256 ? launch_latent_mma<1, 2, B>(e, a, p.splits, skv, pdl, s) : launch_latent_mma<1, 4, B>(e, a, p.splits, skv, pdl, s);
+        return rp <= 256 ? launch_latent_mma<2, 2, B>(e, a, p.splits, skv, pdl, s) : launch_latent_mma<2, 4, B>(e, a, p.splits, skv, pdl, s);
     }
     const dim3 grid(p.splits, a.all_heads, a.n_tokens);
-    const size_t smem = (size_t)(a.row_width + kLatentTile) * 4;
+    // query row and scores of a tile, or what one row's combination needs
+    const size_t smem = (size_t)std::max(a.row_width + kLatentTile, kLatentMaxSplits + 4 * kLatentThreads) * 4;
     if (e->c.kv_dtype == LPP_F32) return launch_kernel(latent_attn_kernel<float>, grid, dim3(kLatentThreads), smem, s, pdl, a);
     return launch_kernel(latent_attn_kernel<__half>, grid, dim3(kLatentThreads), smem, s, pdl, a);
 }
@@ -589,6 +595,7 @@ static LatentAttnArgs latent_attn_args(const lpp_engine* e, const ModelLayer& y,
         a.plane_row = y.o_pitch;
         a.score_skip = y.d.rot_dims / 16;
         a.softcap = y.d.softcap;
+        a.cap_rate = y.d.softcap > 0.f ? 2.f / y.d.softcap : 0.f;
         a.out = e->att_out;
         a.gate = y.d.gate ? e->lat_gate : nullptr;
         a.counters = e->row_counters;
@@ -676,7 +683,7 @@ static cudaError_t launch_mamba_step(const MambaScanArgs& a, bool pdl, cudaStrea
 template <int L, int NS>
 static cudaError_t launch_mamba_scan_t(const lpp_engine* e, MambaScanArgs a, cudaStream_t s) {
     a.tile_tokens = kPrefillTokens;
-    while (a.tile_tokens > 1 && (size_t)mamba_scan_smem<L>(a.dt_pitch, a.state_pitch, a.tile_tokens) > e->smem_optin) a.tile_tokens /= 2;
+    while (a.tile_tokens > 4 && (size_t)mamba_scan_smem<L>(a.dt_pitch, a.state_pitch, a.tile_tokens) > e->smem_optin) a.tile_tokens /= 2;
     const size_t smem = (size_t)mamba_scan_smem<L>(a.dt_pitch, a.state_pitch, a.tile_tokens);
     const cudaError_t r = cudaFuncSetAttribute(mamba_scan_kernel<L, NS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)e->smem_optin);
     if (r != cudaSuccess) return r;
@@ -687,7 +694,17 @@ static cudaError_t launch_mamba_scan(const lpp_engine* e, const MambaScanArgs& a
     LPP_SCAN_DISPATCH(a.state_pitch, LPP_SCAN);
 #undef LPP_SCAN
 }
-static int conv_smem(int taps) { return (kConvTokens + taps - 1) * kConvChannels * 4; }
+static cudaError_t launch_mamba_conv(const MambaConvArgs& a, cudaStream_t s) {
+    const dim3 grid((a.inner + 2 * kConvThreads - 1) / (2 * kConvThreads), (a.n_tokens + kConvTokens - 1) / kConvTokens, 2), block(kConvThreads);
+    switch (a.taps) {
+        case 2: return launch_kernel(mamba_conv_kernel<2>, grid, block, 0, s, true, a);
+        case 3: return launch_kernel(mamba_conv_kernel<3>, grid, block, 0, s, true, a);
+        case 4: return launch_kernel(mamba_conv_kernel<4>, grid, block, 0, s, true, a);
+    }
+    const size_t smem = (size_t)(kConvTokens + a.taps - 1) * kConvThreads * sizeof(float2);
+    const cudaError_t r = cudaFuncSetAttribute(mamba_conv_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max<size_t>(smem, 49152));
+    return r != cudaSuccess ? r : launch_kernel(mamba_conv_kernel<0>, grid, block, smem, s, true, a);
+}
 
 // ---- one decode step as a sequence of launches (captured into the graph, or run directly)
 
@@ -1064,7 +1081,7 @@ static void record_shared_kv_mixer(Recorder& R, int l, float* cur) {
     record_gemv(R, kQkv, kEpiSharedKvIn, a);
     const LatentPlan p = latent_plan(e, y, 1);
     record_launch(R, kAttn, "shared-row attention launch",
-                  [&](bool pdl) { return launch_latent_attn(e, p, latent_attn_args(e, y, r, p), pdl, R.s); });
+                  [&](bool pdl) { return launch_latent_attn(e, p, latent_attn_args(e, y, r, p), true, pdl, R.s); });
 }
 
 // Selective scan: input GEMV with the convolution, GEMV of dt | B | C, scan (mamba.cuh).
@@ -1116,7 +1133,7 @@ static void record_latent_mixer(Recorder& R, int l, float* cur) {
     record_gemv(R, kLatQuery, kEpiLatentQuery, q);
     const LatentPlan p = latent_plan(e, y, 1);
     record_launch(R, kAttn, "latent attention launch",
-                  [&](bool pdl) { return launch_latent_attn(e, p, latent_attn_args(e, y, r, p), pdl, R.s); });
+                  [&](bool pdl) { return launch_latent_attn(e, p, latent_attn_args(e, y, r, p), false, pdl, R.s); });
     GemvLatentArgs v = {};
     v.lat = a.lat;
     v.W = y.w_uv;
@@ -1796,7 +1813,7 @@ extern "C" lpp_status lpp_engine_destroy(lpp_engine* e) {
                     e->r_values, e->out_tokens, e->st, e->rope, e->stage, e->gtrace, e->pf_x, e->pf_q, e->pf_part, e->pf_xn, e->pf_att, e->pf_hb,
                     e->pf_tokens, e->ex_sync, e->ex_block_sum, e->ex_entry_count, e->ex_entries, e->ex_scalars, e->final_b, e->lat_qplain,
                     e->lat_raw, e->lat_gate, e->lat_query, e->lat_part, e->pf_rows, e->pf_logits, e->pf_qn, e->pf_olat, e->pf_lq,
-                    e->pf_lpart, e->pf_gate, e->loop_vec, e->scan_x, e->scan_z, e->scan_low, e->row_counters, e->pf_sx, e->pf_sz, e->pf_tail, e->pf_sxp};
+                    e->pf_lpart, e->pf_gate, e->loop_vec, e->scan_x, e->scan_z, e->scan_low, e->row_counters, e->pf_sx, e->pf_sz, e->pf_tail, e->pf_sxp, e->pf_low};
     for (void* p : bufs)
         if (p) cudaFree(p);
     for (const ModelLayer& y : e->layers)
@@ -2371,7 +2388,7 @@ static lpp_status prefill_setup(lpp_engine* e) {
     const lpp_config& c = e->c;
     const size_t D = e->Dp, L = c.n_layers, T = kPrefillTokens;
     const bool layered = !e->layers.empty();
-    size_t part_rows = D, att_n = e->Dq, hb_n = e->Fl, qn_n = 0, olat_n = 0, lq_n = 0, lpart_n = 0, gate_n = 0, scan_n = 0, tail_n = 0;
+    size_t part_rows = D, att_n = e->Dq, hb_n = e->Fl, qn_n = 0, olat_n = 0, lq_n = 0, lpart_n = 0, gate_n = 0, scan_n = 0, tail_n = 0, low_n = 0;
     const size_t qkv_rows = layered ? 0 : e->Dq + 2 * (size_t)e->KVd;
     part_rows = std::max(part_rows, qkv_rows);
     for (const ModelLayer& y : e->layers) {
@@ -2380,7 +2397,8 @@ static lpp_status prefill_setup(lpp_engine* e) {
         att_n = std::max(att_n, (size_t)y.o_pitch);
         hb_n = std::max(hb_n, (size_t)y.ff_pitch);
         if (y.d.mixer == LPP_MIXER_MAMBA) {
-            part_rows = std::max(part_rows, (size_t)y.low_rows);
+            part_rows = std::max(part_rows, (size_t)y.low_rows * kLowMaxSplits / kPfMaxSplits);
+            low_n = std::max(low_n, (size_t)mamba_low_pitch(y.dt_pitch, y.state_pitch));
             scan_n = std::max(scan_n, (size_t)y.inner_pitch);
             tail_n = std::max(tail_n, (size_t)(y.d.conv - 1) * y.inner_rows);
             continue;
@@ -2413,6 +2431,7 @@ static lpp_status prefill_setup(lpp_engine* e) {
         TRY(zeroed(e, &e->pf_sz, T * scan_n * 4));
         TRY(zeroed(e, &e->pf_sxp, 2 * T * scan_n * 2));
         TRY(zeroed(e, &e->pf_tail, tail_n * 4));
+        TRY(zeroed(e, &e->pf_low, T * low_n * 4));
         for (ModelLayer& y : e->layers) {
             const size_t H = y.d.heads, D2 = align_up(c.dim, 2);
             TRY(make_weight_map(&y.m_in, y.w_in, y.in_rows, D, kUmmaM));
@@ -2456,9 +2475,9 @@ static lpp_status prefill_setup(lpp_engine* e) {
 }
 
 // Ranges of K a GEMM is cut into so that its row tiles (128 weight rows: the weight maps' box) fill the GPU.
-static int prefill_splits(const lpp_engine* e, int n_rows, int K) {
+static int prefill_splits(const lpp_engine* e, int n_rows, int K, int max_splits = kPfMaxSplits) {
     const int tiles = (n_rows + kUmmaM - 1) / kUmmaM, n_kc = (K + kPfKc - 1) / kPfKc;
-    return tiles < e->num_sms ? std::max(1, std::min({kPfMaxSplits, n_kc, (e->num_sms + tiles - 1) / tiles})) : 1;
+    return tiles < e->num_sms ? std::max(1, std::min({max_splits, n_kc, (e->num_sms + tiles - 1) / tiles})) : 1;
 }
 
 // A GEMM whose row tiles do not fill the GPU is also cut along K (a.splits); its partial sums go to pf_part and are added
@@ -2567,11 +2586,12 @@ static lpp_status prefill_gqa_mixer(lpp_engine* e, int l, int n, int start_pos, 
 }
 
 // W . in of a block as partial sums over ranges of K, [range][token][row] in pf_part; *splits = the number of ranges.
-static lpp_status prefill_partial_sums(lpp_engine* e, const CUtensorMap& wm, const CUtensorMap& xm, int n_rows, int K, int n, int start_pos, int* splits) {
+static lpp_status prefill_partial_sums(lpp_engine* e, const CUtensorMap& wm, const CUtensorMap& xm, int n_rows, int K, int n, int start_pos, int* splits,
+                                       int max_splits = kPfMaxSplits) {
     PrefillGemmArgs g = prefill_gemm_args(e, n_rows, K, n, start_pos);
     g.out = e->pf_part;
     g.out_pitch = n_rows;
-    g.splits = *splits = prefill_splits(e, n_rows, K);
+    g.splits = *splits = prefill_splits(e, n_rows, K, max_splits);
     CU((launch_prefill_gemm_t<__nv_bfloat16, kPfStore>(e, wm, xm, g)));
     return LPP_OK;
 }
@@ -2587,7 +2607,7 @@ static lpp_status prefill_row_attention(lpp_engine* e, const ModelLayer& y, cons
     a.planes = (__nv_bfloat16*)planes;
     a.out = nullptr;
     if (a.gate) a.gate = e->pf_gate;
-    CU(launch_latent_attn(e, p, a, true, e->stream));
+    CU(launch_latent_attn(e, p, a, y.d.mixer == LPP_MIXER_SHARED_KV, true, e->stream));
     if (!p.cluster)
         CU(launch_kernel(prefill_latent_combine_kernel, dim3(n * a.all_heads), dim3(128), 0, e->stream, true, a, p.tile_rows));
     return LPP_OK;
@@ -2676,11 +2696,12 @@ static lpp_status prefill_mamba_mixer(lpp_engine* e, int l, int n, int start_pos
     v.x_pitch = y.inner_pitch;
     v.planes = (__nv_bfloat16*)e->pf_sxp;
     v.st = e->st;
-    const dim3 grid((y.d.inner + kConvChannels - 1) / kConvChannels, (n + kConvTokens - 1) / kConvTokens, 2);
-    CU(launch_kernel(mamba_conv_kernel, grid, dim3(kConvChannels), (size_t)conv_smem(y.d.conv), e->stream, true, v));
+    CU(launch_mamba_conv(v, e->stream));
     MambaScanArgs a = mamba_scan_args(e, y, r);
-    TRY(prefill_partial_sums(e, y.m_low, y.x_low, y.low_rows, y.inner_pitch, n, start_pos, &a.splits));
-    a.low = e->pf_part;
+    int splits;
+    TRY(prefill_partial_sums(e, y.m_low, y.x_low, y.low_rows, y.inner_pitch, n, start_pos, &splits, kLowMaxSplits));
+    CU(launch_kernel(mamba_low_kernel, dim3(n), dim3(kLowThreads), 0, e->stream, true, a, (const float*)e->pf_part, splits, e->pf_low));
+    a.low = e->pf_low;
     a.n_tokens = n;
     a.start_pos = start_pos;
     a.x = e->pf_sx;

@@ -29,6 +29,7 @@ struct LatentAttnArgs {
     int seq_len;
     float scale;
     float softcap;      // > 0: a score s becomes softcap * tanh(s / softcap)
+    float cap_rate;     // 2 / softcap
     // One token, splits put together by the CTA that finishes last: out[head * out_cols + col] = result * gate
     float* out;              // nullptr = partial results stay in `part`
     const float* gate;       // [all_heads * out_cols], prompt blocks [token][all_heads * out_cols]; nullptr = none
@@ -47,64 +48,102 @@ __device__ __forceinline__ int latent_row(const LatentAttnArgs& a, int group, in
     const int t = r / a.heads;
     return t * a.all_heads + group * a.heads + (r - t * a.heads);
 }
-__device__ __forceinline__ float latent_score(const LatentAttnArgs& a, float dot) {
-    const float s = dot * a.scale;
-    return a.softcap > 0.f ? a.softcap * tanhf(__fdiv_rn(s, a.softcap)) : s;
+// softcap * tanh(s / softcap) as softcap - 2 softcap / (1 + exp(2 s / softcap)): an absolute error of a few 1e-7 softcap.
+__device__ __forceinline__ float capped_score(const LatentAttnArgs& a, float s) {
+    return a.softcap - __fdividef(2.f * a.softcap, 1.f + __expf(s * a.cap_rate));
 }
-// The last of `n` CTAs to get here returns true, with the others' global stores visible.  NT threads, all of the CTA.
-__device__ __forceinline__ bool latent_last_arrival(unsigned int* counter, int n, int* flag, int tid) {
-    __threadfence();
+// The last of `n` CTAs to get here returns true, with the others' global stores visible.  Called by all threads of the CTA; the
+// barriers put every thread's accesses before and after the counter's release and acquire.
+__device__ __forceinline__ bool latent_last_arrival(unsigned int* counter, unsigned int n, int* flag, int tid) {
     __syncthreads();
-    if (tid == 0) *flag = atomicAdd(counter, 1u) == (unsigned int)n - 1u;
-    __syncthreads();
-    if (!*flag) return false;
-    __threadfence();
-    if (tid == 0) *counter = 0u;
-    return true;
-}
-// One column of a query row from its n_eff partial results, p = the row's first one: added up in split order.
-__device__ __forceinline__ float latent_combine1(const LatentAttnArgs& a, const float* p, int n_eff, int col) {
-    const int stride = a.rank_pitch + kLatentPartTail;
-    float mm = -INFINITY, av = 0.f, lv = 0.f;
-    for (int s0 = 0; s0 < n_eff; s0 += 8) {
-        float ms[8], ls[8], as[8], mb = mm;
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const bool ok = s0 + i < n_eff;
-            const float* ps = p + (size_t)(s0 + i) * stride;
-            ms[i] = ok ? __ldcg(ps + a.rank_pitch) : -INFINITY;
-            ls[i] = ok ? __ldcg(ps + a.rank_pitch + 1) : 0.f;
-            as[i] = ok ? __ldcg(ps + col) : 0.f;
-        }
-#pragma unroll
-        for (int i = 0; i < 8; ++i) mb = fmaxf(mb, ms[i]);
-        const float fo = mm == -INFINITY ? 0.f : expf(mm - mb);
-        av *= fo;
-        lv *= fo;
-#pragma unroll
-        for (int i = 0; i < 8; ++i) {
-            const float f = ms[i] == -INFINITY ? 0.f : expf(ms[i] - mb);
-            av = fmaf(as[i], f, av);
-            lv = fmaf(ls[i], f, lv);
-        }
-        mm = mb;
+    if (tid == 0) {
+        unsigned int ticket;
+        asm volatile("atom.add.acq_rel.gpu.global.u32 %0, [%1], 1;" : "=r"(ticket) : "l"(counter) : "memory");
+        *flag = ticket == n - 1u;
+        if (ticket == n - 1u) *counter = 0u;
     }
-    return __fdiv_rn(av, lv);
+    __syncthreads();
+    return *flag;
 }
 __device__ __forceinline__ void latent_out(const LatentAttnArgs& a, int head, int col, float v) {
     const int at = head * a.out_cols + col;
     a.out[at] = a.gate ? v * __ldcg(a.gate + at) : v;
 }
-
+__device__ __forceinline__ void latent_out4(const LatentAttnArgs& a, int head, int col, float4 v) {
+    const int at = head * a.out_cols + col;
+    if ((a.out_cols & 3) == 0) {
+        if (col >= a.out_cols) return;
+        if (a.gate) {
+            const float4 g = __ldcg(reinterpret_cast<const float4*>(a.gate + at));
+            v.x *= g.x; v.y *= g.y; v.z *= g.z; v.w *= g.w;
+        }
+        *reinterpret_cast<float4*>(a.out + at) = v;
+        return;
+    }
+    const float y[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int c = 0; c < 4; ++c)
+        if (col + c < a.out_cols) latent_out(a, head, col + c, y[c]);
+}
 constexpr int kLatentMaxCluster = 8;
 constexpr int kLatentTile = 64;        // keys per shared-memory tile
 constexpr int kLatentThreads = 256;
+
+// Heads `head` .. head + n - 1 of a token from their n_eff partial results: added up in split order and finished.  NT threads;
+// scratch: n * kLatentMaxSplits + 4 NT floats.  A thread takes four columns of a head and, where there are threads to
+// spare, half of the splits.  Kept short: this code is fetched by a few CTAs at the end of every launch.
+template <int NT>
+__device__ __forceinline__ void latent_combine_heads(const LatentAttnArgs& a, int head, int n, int n_eff, float* scratch, int tid) {
+    float* wt = scratch;                                                       // [n][kLatentMaxSplits]
+    float4* half = reinterpret_cast<float4*>(scratch + n * kLatentMaxSplits);  // [NT]
+    const int stride = a.rank_pitch + kLatentPartTail, warp = tid >> 5, lane = tid & 31;
+    const int q4 = a.rank_pitch >> 2, slots = n * q4;
+    const int halves = 2 * slots <= NT ? 2 : 1, per = NT / halves, part = tid >= per ? 1 : 0;
+    const int s_half = halves == 2 ? (n_eff + 1) >> 1 : n_eff, s_begin = part ? s_half : 0, s_end = part ? n_eff : s_half;
+    const float* p0 = a.part + (size_t)head * a.max_splits * stride;
+    // weights of the splits: exp(m_s - max m) / sum of l
+    auto weights = [&]() {
+        for (int k = warp; k < n; k += NT / 32) {
+            const float2 ml = lane < n_eff ? __ldcg(reinterpret_cast<const float2*>(p0 + ((size_t)k * a.max_splits + lane) * stride + a.rank_pitch))
+                                           : make_float2(-INFINITY, 0.f);
+            const float e = expf(ml.x - warp_max(ml.x));
+            wt[k * kLatentMaxSplits + lane] = __fdiv_rn(e, warp_sum(e * ml.y));
+        }
+        __syncthreads();
+    };
+    for (int base = 0; base < slots; base += per) {
+        const int slot = min(base + tid - part * per, slots - 1), r = slot / q4, col = (slot - r * q4) << 2;
+        const bool mine = base + tid - part * per < slots;
+        const float* p = p0 + (size_t)r * a.max_splits * stride + col;
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int s0 = s_begin, first = base == 0; s0 < s_end || first; s0 += 8, first = 0) {
+            float4 v[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] = __ldcg(reinterpret_cast<const float4*>(p + (size_t)min(s0 + i, n_eff - 1) * stride));
+            if (first) weights();  // beside the first loads
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float w = s0 + i < s_end ? wt[r * kLatentMaxSplits + s0 + i] : 0.f;
+                acc.x = fmaf(w, v[i].x, acc.x); acc.y = fmaf(w, v[i].y, acc.y); acc.z = fmaf(w, v[i].z, acc.z); acc.w = fmaf(w, v[i].w, acc.w);
+            }
+        }
+        if (halves == 2) {
+            half[tid] = acc;
+            __syncthreads();
+            if (part) return;
+            const float4 b = half[tid + per];
+            acc.x += b.x; acc.y += b.y; acc.z += b.z; acc.w += b.w;
+        }
+        if (!mine) continue;
+        latent_out4(a, head + r, col, acc);
+    }
+}
 
 // ---- any sizes, FP32 or FP16 rows, FP32 arithmetic.  grid: (splits, heads, tokens)
 constexpr int kLatentMaxPerThread = 8;  // latent elements of one thread: ranks up to 2048
 template <typename KT>
 static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(const LatentAttnArgs a) {
-    extern __shared__ float lat_smem[];  // query row, then scores of a tile
+    extern __shared__ __align__(16) float lat_smem[];  // query row, then scores of a tile
     __shared__ float s_f, s_m, s_l;
     __shared__ int s_last;
     float* qs = lat_smem;
@@ -135,7 +174,7 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(cons
             float s = 0.f;
             for (int i = lane; i < a.row_width; i += 32) s = fmaf(qs[i], to_float(kr[i]), s);
             s = warp_sum(s);
-            if (lane == 0) sc[k] = latent_score(a, s);
+            if (lane == 0) sc[k] = a.softcap > 0.f ? a.softcap * tanhf(__fdiv_rn(s * a.scale, a.softcap)) : s * a.scale;
         }
         __syncthreads();
         if (warp == 0) {
@@ -172,8 +211,7 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(cons
             if (tid + j * kLatentThreads < a.out_cols) latent_out(a, blockIdx.y, tid + j * kLatentThreads, __fdiv_rn(o[j], s_l));
         return;
     }
-    float* p0 = a.part + row * a.max_splits * (a.rank_pitch + kLatentPartTail);
-    float* p = p0 + (size_t)split * (a.rank_pitch + kLatentPartTail);
+    float* p = a.part + (row * a.max_splits + split) * (a.rank_pitch + kLatentPartTail);
 #pragma unroll
     for (int j = 0; j < kLatentMaxPerThread; ++j)
         if (tid + j * kLatentThreads < a.rank_pitch) p[tid + j * kLatentThreads] = o[j];
@@ -182,7 +220,7 @@ static __global__ void __launch_bounds__(kLatentThreads) latent_attn_kernel(cons
         p[a.rank_pitch + 1] = s_l;
     }
     if (!a.out || !latent_last_arrival(a.counters + blockIdx.y, sp.n_eff, &s_last, tid)) return;
-    for (int i = tid; i < a.out_cols; i += kLatentThreads) latent_out(a, blockIdx.y, i, latent_combine1(a, p0, sp.n_eff, i));
+    latent_combine_heads<kLatentThreads>(a, blockIdx.y, 1, sp.n_eff, lat_smem, tid);
 }
 
 // ---- tensor cores, FP16 rows.  grid: (splits, row tiles of 16 MT, groups); with `cluster` set the splits of a row tile are one
@@ -220,8 +258,9 @@ __device__ __forceinline__ float cluster_load(uint32_t addr) {
 }
 
 // Columns col .. col + 3 of a finished row of a prompt block, times the gate, as hi + lo operands.
+template <bool GATED>
 __device__ __forceinline__ void latent_planes4(const LatentAttnArgs& a, int t, int h, int col, float (&y)[4]) {
-    if (a.gate) {
+    if (GATED && a.gate) {
         const float* g = a.gate + ((size_t)t * a.all_heads + h) * a.plane_cols + col;
 #pragma unroll
         for (int c = 0; c < 4; ++c)
@@ -232,7 +271,7 @@ __device__ __forceinline__ void latent_planes4(const LatentAttnArgs& a, int t, i
     __align__(8) __nv_bfloat16 hi[4], lo[4];
 #pragma unroll
     for (int c = 0; c < 4; ++c) split_pair(y[c], hi[c], lo[c]);
-    if (((a.plane_pitch | a.plane_cols) & 3) == 0) {
+    if (!GATED || ((a.plane_pitch | a.plane_cols) & 3) == 0) {  // (rows of latents are padded)
         if (col >= a.plane_cols) return;
         *reinterpret_cast<uint2*>(d) = *reinterpret_cast<const uint2*>(hi);
         *reinterpret_cast<uint2*>(d_lo) = *reinterpret_cast<const uint2*>(lo);
@@ -249,7 +288,9 @@ constexpr int latent_mma_smem(int row_width) {
     return (16 * MT + 2 * kLatentTile) * (row_width * 2 + 16) + 16 * MT * (NW / 4 * kLatScPitch * 4 + kLatPPitch * 2 + 12 + kLatentMaxCluster * 4);
 }
 
-template <int MT, int NT, int NW>
+// SKV: attention of shared_kv.cuh (groups, score cap, gates, `out`); an argument because latent attention should not fetch its
+// code.
+template <int MT, int NT, int NW, bool SKV>
 static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const LatentAttnArgs a) {
     constexpr int kRows = 16 * MT, kThreads = NW * 32, kParts = NW / 4, kRowsPerWarp = kRows / NW;
     static_assert(NT % 2 == 0, "column tiles go in pairs");
@@ -283,7 +324,12 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
     const int k_begin = sp.first + split * sp.chunk, k_end = min(k_begin + sp.chunk, base + t_hi + 1);
     const int n_tiles = active ? (k_end - k_begin + kLatentTile - 1) / kLatentTile : 0;
     const size_t row_bytes = (size_t)a.row_width * 2;
-    const int group = blockIdx.z;
+    const int group = SKV ? blockIdx.z : 0;
+    auto row_of = [&](int r) -> int { return SKV ? latent_row(a, group, r) : r; };  // global row of the group's row r
+    auto score = [&](float dot) -> float {
+        const float s = dot * a.scale;
+        return SKV && a.softcap > 0.f ? capped_score(a, s) : s;
+    };
     const unsigned char* cache = reinterpret_cast<const unsigned char*>(a.cache) + (size_t)group * a.seq_len * row_bytes;
     const int pieces = a.row_width / 8;
 
@@ -307,7 +353,7 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
         load_keys(0, max(k_begin, base), k_end, true);
         for (int r = warp; r < kRows; r += NW) {
             const bool in = r0 + r < n_rows;
-            const unsigned char* src = reinterpret_cast<const unsigned char*>(a.q) + (in ? (size_t)latent_row(a, group, r0 + r) * row_bytes : 0);
+            const unsigned char* src = reinterpret_cast<const unsigned char*>(a.q) + (in ? (size_t)row_of(r0 + r) * row_bytes : 0);
             for (int col = lane; col < pieces; col += 32) cp_async_16(qs + r * pitch + col * 16, src + (in ? col * 16 : 0), in);
         }
     }
@@ -323,9 +369,9 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
     for (int m = 0; m < MT; ++m)
 #pragma unroll
         for (int i = 0; i < NT; ++i) o[m][i][0] = o[m][i][1] = o[m][i][2] = o[m][i][3] = 0.f;
-    const int k_steps = a.row_width / 16 - a.score_skip;
+    const int skip = SKV ? a.score_skip : 0, k_steps = a.row_width / 16 - skip;
     const int key16 = warp & 3, part = warp >> 2;  // scores: this warp's 16 keys and its share of the k-steps
-    const int ks0 = a.score_skip + part * k_steps / kParts, ks1 = a.score_skip + (part + 1) * k_steps / kParts;
+    const int ks0 = skip + part * k_steps / kParts, ks1 = skip + (part + 1) * k_steps / kParts;
     const uint32_t q_addr = smem_u32(qs) + (uint32_t)(((mi & 1) * 8 + mr) * pitch + (mi >> 1) * 16);
     const uint32_t p_addr = smem_u32(ps) + (uint32_t)((((mi & 1) * 8 + mr) * kLatPPitch + (mi >> 1) * 8) * 2);
 
@@ -383,8 +429,8 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
                     v0 += s0[q * kRows * kLatScPitch];
                     v1 += s0[q * kRows * kLatScPitch + 32];
                 }
-                x0[i] = (p >= lo && p <= last && p < k_end) ? latent_score(a, v0) : -INFINITY;
-                x1[i] = (p + 32 >= lo && p + 32 <= last && p + 32 < k_end) ? latent_score(a, v1) : -INFINITY;
+                x0[i] = (p >= lo && p <= last && p < k_end) ? score(v0) : -INFINITY;
+                x1[i] = (p + 32 >= lo && p + 32 <= last && p + 32 < k_end) ? score(v1) : -INFINITY;
                 m_old[i] = s_m[r];
                 m_new[i] = fmaxf(x0[i], x1[i]);
             }
@@ -448,14 +494,14 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
     }
     __syncthreads();
     if (!a.cluster) {
-        if (a.out && sp.n_eff == 1) {  // all keys seen: finished rows
+        if (SKV && a.out && sp.n_eff == 1) {  // all keys seen: finished rows
 #pragma unroll
             for (int m = 0; m < MT; ++m)
 #pragma unroll
                 for (int half = 0; half < 2; ++half) {
                     const int r = m * 16 + g + 8 * half;
                     if (r0 + r >= n_rows) continue;
-                    const int head = latent_row(a, group, r0 + r);  // one token: row = head
+                    const int head = group * a.heads + r0 + r;  // one token
                     const float l = s_l[r];
 #pragma unroll
                     for (int i = 0; i < NT; ++i) {
@@ -473,7 +519,7 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
             for (int half = 0; half < 2; ++half) {
                 const int r = m * 16 + g + 8 * half;
                 if (r0 + r >= n_rows) continue;
-                float* dst = a.part + ((size_t)latent_row(a, group, r0 + r) * a.max_splits + split) * stride;
+                float* dst = a.part + ((size_t)row_of(r0 + r) * a.max_splits + split) * stride;
 #pragma unroll
                 for (int i = 0; i < NT; ++i) {
                     const int col = warp * NT * 8 + i * 8 + 2 * tq;
@@ -481,12 +527,11 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
                 }
                 if (warp == 0 && tq == 0) *reinterpret_cast<float2*>(dst + a.rank_pitch) = make_float2(s_m[r], s_l[r]);
             }
-        if (!a.out) return;
-        if (!latent_last_arrival(a.counters + group * gridDim.y + blockIdx.y, sp.n_eff, reinterpret_cast<int*>(s_w), tid)) return;
-        const int rows_here = min(kRows, n_rows - r0);
-        for (int i = tid; i < rows_here * a.out_cols; i += kThreads) {
-            const int r = i / a.out_cols, col = i - r * a.out_cols, head = latent_row(a, group, r0 + r);
-            latent_out(a, head, col, latent_combine1(a, a.part + (size_t)head * a.max_splits * stride, sp.n_eff, col));
+        if constexpr (SKV) {
+            // scratch over the scores, whose space is larger: [kParts][kRows][kLatScPitch] floats
+            static_assert(MT > 1 || kParts * kRows * kLatScPitch >= kRows * kLatentMaxSplits + 4 * kThreads, "scratch of the combination");
+            if (MT == 1 && a.out && latent_last_arrival(a.counters + group * gridDim.y + blockIdx.y, sp.n_eff, reinterpret_cast<int*>(s_w), tid))
+                latent_combine_heads<kThreads>(a, group * a.heads + r0, min(kRows, n_rows - r0), sp.n_eff, sc, tid);
         }
         return;
     }
@@ -542,8 +587,8 @@ static __global__ void __launch_bounds__(NW * 32) latent_attn_mma_kernel(const L
                 const float w = s_w[r * kLatentMaxCluster + c];
                 y[0] = fmaf(w, x[c].x, y[0]); y[1] = fmaf(w, x[c].y, y[1]); y[2] = fmaf(w, x[c].z, y[2]); y[3] = fmaf(w, x[c].w, y[3]);
             }
-        const int t = (r0 + r) / a.heads, h = group * a.heads + (r0 + r - t * a.heads);
-        latent_planes4(a, t, h, col, y);
+        const int t = (r0 + r) / a.heads, h = (SKV ? group * a.heads : 0) + (r0 + r - t * a.heads);
+        latent_planes4<SKV>(a, t, h, col, y);
     }
     cluster_barrier();  // every CTA's shared memory stays until all have read it
 }
@@ -576,7 +621,7 @@ static __global__ void __launch_bounds__(128) prefill_latent_combine_kernel(cons
             const float4 x = __ldcg(reinterpret_cast<const float4*>(p + (size_t)s * stride + k));
             y[0] = fmaf(wt[s], x.x, y[0]); y[1] = fmaf(wt[s], x.y, y[1]); y[2] = fmaf(wt[s], x.z, y[2]); y[3] = fmaf(wt[s], x.w, y[3]);
         }
-        latent_planes4(a, t, h, k, y);
+        latent_planes4<true>(a, t, h, k, y);
     }
 }
 

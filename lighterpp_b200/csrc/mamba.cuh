@@ -64,7 +64,7 @@ struct MambaScanArgs {
     int inner, state, dt_rank;
     int state_pitch, dt_pitch;  // elements per channel of S and A (multiple of 4), of w_dt (multiple of 8)
     int low_rows;               // row of `low`: dt | B | C, even
-    const float* low;           // step: [low_rows]; prompt block: partial sums [splits][kPrefillTokens][low_rows]
+    const float* low;           // step: [low_rows]; prompt block: [kPrefillTokens][mamba_low_pitch], padded
     const void* w_dt;           // [inner][dt_pitch], weight type
     const float *dt_b, *A, *D;  // [inner], [inner][state_pitch] (negative), [inner]
     float* S;                   // [inner][state_pitch]
@@ -74,8 +74,8 @@ struct MambaScanArgs {
     int seq_len;
     int early;                  // step: weights and state may be read before the dependency wait
     // prompt block
-    int splits, n_tokens, start_pos, x_pitch;
-    int tile_tokens;            // tokens whose dt | B | C rows fit shared memory together
+    int n_tokens, start_pos, x_pitch;
+    int tile_tokens;            // tokens whose rows fit shared memory together (a multiple of 4)
     __nv_bfloat16* planes;      // [2 planes][kPrefillTokens][plane_row]
     int plane_row;
     const float* tail;          // convolution inputs of the block's last tokens, laid out like the ring
@@ -95,7 +95,7 @@ __device__ __forceinline__ float decay_m1(float x) {
     p = fmaf(x, p, 1.f / 6.f);
     p = fmaf(x, p, 0.5f);
     p = fmaf(x * x, p, x);
-    return x > -0.5f ? p : expf(x) - 1.f;
+    return x > -0.5f ? p : __expf(x) - 1.f;
 }
 // S <- exp(dt A) S + dx B
 __device__ __forceinline__ void state_update(float& S, float A, float B, float dt, float dx) {
@@ -115,7 +115,7 @@ __device__ __forceinline__ float lane_group_sum(float v) {
     for (int o = L / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
 }
-// dt | B | C of one token in shared memory: dt padded to dt_pitch, B and C to state_pitch, with zeros.
+// Element i of a token's dt | B | C row with dt padded to dt_pitch, B and C to state_pitch, with zeros.
 __device__ __forceinline__ float mamba_low(const MambaScanArgs& a, const float* src, int i) {
     int n = a.dt_rank, from = 0;
     if (i >= a.dt_pitch) {

@@ -20,17 +20,6 @@ __device__ __forceinline__ float2 prefill_sum2(const float* part, int n_rows, in
         }
     return v;
 }
-// One row alone.
-__device__ __forceinline__ float prefill_sum1(const float* part, int n_rows, int splits, int t, int row) {
-    float p[kPfMaxSplits], v = 0.f;
-#pragma unroll
-    for (int s = 0; s < kPfMaxSplits; ++s)
-        if (s < splits) p[s] = part[((size_t)s * kPrefillTokens + t) * n_rows + row];
-#pragma unroll
-    for (int s = 0; s < kPfMaxSplits; ++s)
-        if (s < splits) v += p[s];
-    return v;
-}
 
 // ---- attention whose values are its keys (shared_kv.cuh): after the input GEMM (partial sums over ranges of K, added in
 // range order), one row pair per thread.
@@ -68,9 +57,10 @@ static __global__ void __launch_bounds__(256) prefill_shared_kv_finish_kernel(co
 
 // Convolution of a prompt block after the input GEMM (partial sums added in range order): x convolved, as FP32 rows and as
 // hi + lo operands of the next GEMM; z through the silu.  The inputs of the last taps - 1 tokens go to `tail`; the scan
-// copies them to the ring once every CTA of this launch has read it.
-// grid: (ceil(inner / 128), ceil(tokens / 8), 2: x, z); shared memory (x): (8 + taps - 1) * 128 floats
-constexpr int kConvChannels = 128, kConvTokens = 8;
+// copies them to the ring once every CTA of this launch has read it.  A thread takes two channels of kConvTokens tokens;
+// TAPS = the number of taps (inputs in registers), or 0 = any (inputs in shared memory).
+// grid: (ceil(inner / 256), ceil(tokens / kConvTokens), 2: x, z); shared memory (TAPS 0): (kConvTokens + taps - 1) * 256 floats
+constexpr int kConvThreads = 128, kConvTokens = 4;
 struct MambaConvArgs {
     const float* part;  // [splits][kPrefillTokens][2 * inner_rows]
     int splits, n_tokens, start_pos, seq_len;
@@ -82,61 +72,139 @@ struct MambaConvArgs {
     __nv_bfloat16* planes;  // [2 planes][kPrefillTokens][x_pitch]
     StepState* st;
 };
-static __global__ void __launch_bounds__(kConvChannels) mamba_conv_kernel(const MambaConvArgs a) {
-    extern __shared__ float cv_in[];  // [kConvTokens + taps - 1][kConvChannels]; a thread reads back only what it wrote
+template <int TAPS>
+static __global__ void __launch_bounds__(kConvThreads) mamba_conv_kernel(const MambaConvArgs a) {
+    extern __shared__ float2 cv_in[];  // [kConvTokens + taps - 1][kConvThreads]; a thread reads back only what it wrote
     pdl_launch_dependents();
-    const int tid = threadIdx.x, c = blockIdx.x * kConvChannels + tid;
-    const int t0 = blockIdx.y * kConvTokens, t1 = min(t0 + kConvTokens, a.n_tokens);
-    const int n_rows = 2 * a.inner_rows, slots = a.taps - 1;
+    const int tid = threadIdx.x, c = 2 * ((int)blockIdx.x * kConvThreads + tid);
+    const int t0 = blockIdx.y * kConvTokens, n_rows = 2 * a.inner_rows, slots = TAPS > 0 ? TAPS - 1 : a.taps - 1;
+    const bool in = c < a.inner, ok = a.start_pos >= 0 && a.start_pos + a.n_tokens <= a.seq_len;
+    float2 w[TAPS > 0 ? TAPS : 1], bias = make_float2(0.f, 0.f);
+    if (in && blockIdx.z == 0) {  // constants: ahead of the dependency wait
+        bias = __ldg(reinterpret_cast<const float2*>(a.conv_b + c));
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[j] = __ldg(reinterpret_cast<const float2*>(a.conv_w + (size_t)j * a.inner_rows + c));
+    }
     pdl_wait();
-    if (a.start_pos < 0 || a.start_pos + a.n_tokens > a.seq_len) {
-        if (tid == 0) atomicOr(&a.st->status, kStatusBadPos);
-        return;
-    }
-    if (c >= a.inner) return;
+    if (!ok && tid == 0) atomicOr(&a.st->status, kStatusBadPos);
+    if (!ok || !in) return;
     if (blockIdx.z == 1) {
-#pragma unroll 4
-        for (int t = t0; t < t1; ++t) a.z[(size_t)t * a.x_pitch + c] = silu_f(prefill_sum1(a.part, n_rows, a.splits, t, a.inner_rows + c));
+        float2 v[kConvTokens];
+#pragma unroll
+        for (int i = 0; i < kConvTokens; ++i)
+            if (t0 + i < a.n_tokens) v[i] = prefill_sum2(a.part, n_rows, a.splits, t0 + i, a.inner_rows + c);
+#pragma unroll
+        for (int i = 0; i < kConvTokens; ++i)
+            if (t0 + i < a.n_tokens) *reinterpret_cast<float2*>(a.z + (size_t)(t0 + i) * a.x_pitch + c) = make_float2(silu_f(v[i].x), silu_f(v[i].y));
         return;
     }
-#pragma unroll 4
-    for (int t = t0 - slots; t < t1; ++t) {
-        float v = 0.f;
+    // input i of the thread: token t0 - slots + i; zero before the first position
+    auto input = [&](int i) -> float2 {
+        const int t = t0 - slots + i;
+        if (t >= a.n_tokens) return make_float2(0.f, 0.f);
+        float2 v = make_float2(0.f, 0.f);
         if (t >= 0)
-            v = prefill_sum1(a.part, n_rows, a.splits, t, c);
+            v = prefill_sum2(a.part, n_rows, a.splits, t, c);
         else if (a.start_pos + t >= 0)
-            v = __ldcg(a.ring + (size_t)((a.start_pos + t) % slots) * a.inner_rows + c);
-        cv_in[(t - t0 + slots) * kConvChannels + tid] = v;
-        if (t >= t0 && t >= a.n_tokens - slots) a.tail[(size_t)((a.start_pos + t) % slots) * a.inner_rows + c] = v;
-    }
-    const float bias = __ldg(a.conv_b + c);
-    for (int t = t0; t < t1; ++t) {
-        float v = bias;
-#pragma unroll 4
-        for (int j = 0; j < a.taps; ++j) v = fmaf(__ldg(a.conv_w + (size_t)j * a.inner_rows + c), cv_in[(t - t0 + j) * kConvChannels + tid], v);
-        v = silu_f(v);
-        a.x[(size_t)t * a.x_pitch + c] = v;
-        __nv_bfloat16 hi, lo;
-        split_pair(v, hi, lo);
-        a.planes[(size_t)t * a.x_pitch + c] = hi;
-        a.planes[(size_t)(kPrefillTokens + t) * a.x_pitch + c] = lo;
+            v = __ldcg(reinterpret_cast<const float2*>(a.ring + (size_t)((a.start_pos + t) % slots) * a.inner_rows + c));
+        return v;
+    };
+    auto keep = [&](int i, float2 v) {
+        const int t = t0 - slots + i;
+        if (t >= t0 && t >= a.n_tokens - slots && t < a.n_tokens)
+            *reinterpret_cast<float2*>(a.tail + (size_t)((a.start_pos + t) % slots) * a.inner_rows + c) = v;
+    };
+    auto put = [&](int i, float2 v) {
+        const int t = t0 + i;
+        if (t >= a.n_tokens) return;
+        v = make_float2(silu_f(v.x), silu_f(v.y));
+        *reinterpret_cast<float2*>(a.x + (size_t)t * a.x_pitch + c) = v;
+        __align__(4) __nv_bfloat16 hi[2], lo[2];
+        split_pair(v.x, hi[0], lo[0]);
+        split_pair(v.y, hi[1], lo[1]);
+        *reinterpret_cast<uint32_t*>(a.planes + (size_t)t * a.x_pitch + c) = *reinterpret_cast<const uint32_t*>(hi);
+        *reinterpret_cast<uint32_t*>(a.planes + (size_t)(kPrefillTokens + t) * a.x_pitch + c) = *reinterpret_cast<const uint32_t*>(lo);
+    };
+    if constexpr (TAPS > 0) {
+        constexpr int N = kConvTokens + TAPS - 1;
+        float2 v[N];
+#pragma unroll
+        for (int i = 0; i < N; ++i) v[i] = input(i);
+        if constexpr (TAPS > 1)
+#pragma unroll
+            for (int i = 0; i < N; ++i) keep(i, v[i]);
+#pragma unroll
+        for (int i = 0; i < kConvTokens; ++i) {
+            float2 s = bias;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) s = make_float2(fmaf(w[j].x, v[i + j].x, s.x), fmaf(w[j].y, v[i + j].y, s.y));
+            put(i, s);
+        }
+    } else {
+        for (int i = 0; i < kConvTokens + slots; ++i) {
+            const float2 v = input(i);
+            keep(i, v);
+            cv_in[i * kConvThreads + tid] = v;
+        }
+        for (int i = 0; i < kConvTokens; ++i) {
+            float2 s = bias;
+            for (int j = 0; j <= slots; ++j) {
+                const float2 wj = __ldg(reinterpret_cast<const float2*>(a.conv_w + (size_t)j * a.inner_rows + c)), v = cv_in[(i + j) * kConvThreads + tid];
+                s = make_float2(fmaf(wj.x, v.x, s.x), fmaf(wj.y, v.y, s.y));
+            }
+            put(i, s);
+        }
     }
 }
 
-// The recurrence over a prompt block.  A CTA owns kScanThreads / L channels and walks the block in tiles of tile_tokens:
-// dt | B | C rows to shared memory (partial sums of the W_x GEMM added in range order), dt = softplus(W_dt . + bias) for all
-// tokens and channels of the tile, then token by token with the state in registers.
-constexpr int kScanThreads = 128;
-template <int L>
-constexpr int kScanChannels = kScanThreads / L;
-// floats per token row in shared memory, an odd number of 16-byte pieces (rows on different banks)
+// dt | B | C rows after their GEMM, whose row tiles are few and whose K is therefore cut into up to kLowMaxSplits ranges:
+// partial sums added in range order, sections padded with zeros to dt_pitch and state_pitch.  grid: tokens
+constexpr int kLowMaxSplits = 32, kLowThreads = 256;
+// floats per row, an odd number of 16-byte pieces (rows on different banks of shared memory)
 __host__ __device__ inline int mamba_low_pitch(int dt_pitch, int state_pitch) {
     const int n = dt_pitch + 2 * state_pitch;
     return (n / 4) % 2 ? n : n + 4;
 }
+static __global__ void __launch_bounds__(kLowThreads) mamba_low_kernel(const MambaScanArgs a, const float* part, int splits, float* out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t = blockIdx.x, n_low = a.dt_pitch + 2 * a.state_pitch;
+    for (int i = threadIdx.x; i < n_low; i += kLowThreads) {
+        float v[kLowMaxSplits], sum = 0.f;
+#pragma unroll
+        for (int s = 0; s < kLowMaxSplits; ++s)
+            if (s < splits) v[s] = mamba_low(a, part + ((size_t)s * kPrefillTokens + t) * a.low_rows, i);
+#pragma unroll
+        for (int s = 0; s < kLowMaxSplits; ++s)
+            if (s < splits) sum += v[s];
+        out[(size_t)t * mamba_low_pitch(a.dt_pitch, a.state_pitch) + i] = sum;
+    }
+}
+
+// The recurrence over a prompt block.  A CTA owns kScanThreads / L channels and walks the block in tiles of tile_tokens:
+// dt | B | C rows, x and z to shared memory, dt = softplus(W_dt . + bias) for all tokens and channels of the tile, then
+// four tokens at a time with the state in registers.
+constexpr int kScanThreads = 128;
+template <int L>
+constexpr int kScanChannels = kScanThreads / L;
 template <int L>
 __host__ __device__ inline int mamba_scan_smem(int dt_pitch, int state_pitch, int tile_tokens) {
-    return (tile_tokens * (mamba_low_pitch(dt_pitch, state_pitch) + 2 * kScanChannels<L>) + kScanChannels<L> * (dt_pitch + 4)) * 4;
+    return (tile_tokens * (mamba_low_pitch(dt_pitch, state_pitch) + 3 * kScanChannels<L>) + kScanChannels<L> * (dt_pitch + 4)) * 4;
+}
+// Sums over the L lanes of a channel of four values each (one per token); lane ln gets that of token scan_token(ln).
+__device__ __forceinline__ int scan_token(int ln) { return ((ln & 1) << 1) | ((ln >> 1) & 1); }
+template <int L>
+__device__ __forceinline__ float lane_group_sum4(const float (&y)[4], int ln) {
+    static_assert(L >= 4, "four tokens to four lanes");
+    const bool b0 = ln & 1, b1 = ln & 2;
+    float p = b0 ? y[2] : y[0], q = b0 ? y[3] : y[1];
+    p += __shfl_xor_sync(0xffffffffu, b0 ? y[0] : y[2], 1);
+    q += __shfl_xor_sync(0xffffffffu, b0 ? y[1] : y[3], 1);
+    float r = b1 ? q : p;
+    r += __shfl_xor_sync(0xffffffffu, b1 ? p : q, 2);
+#pragma unroll
+    for (int o = 4; o < L; o <<= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
+    return r;
 }
 template <int L, int NS>
 static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const MambaScanArgs a) {
@@ -146,8 +214,9 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
     const int LP = mamba_low_pitch(a.dt_pitch, a.state_pitch), WP = a.dt_pitch + 4;
     float* low = sm_scan;                       // [tile_tokens][LP]
     float* wd = low + a.tile_tokens * LP;       // [CH][WP]
-    float* dts = wd + CH * WP;                  // [tile_tokens][CH]
-    float* xs = dts + a.tile_tokens * CH;       // [tile_tokens][CH]: x, then y
+    float* xs = wd + CH * WP;                   // [tile_tokens][CH]: x, then y
+    float* zs = xs + a.tile_tokens * CH;        // [tile_tokens][CH]
+    float* dts = zs + a.tile_tokens * CH;       // [tile_tokens][CH]
     const int tid = threadIdx.x, ln = tid % L, cl = tid / L, c0 = blockIdx.x * CH, c = c0 + cl;
     const bool in = c < a.inner;
     const int pieces = a.state_pitch / 4;
@@ -173,38 +242,33 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
     for (int j = 0; j < CPT; ++j) bias[j] = c0 + tx + j * TX < a.inner ? __ldg(a.dt_b + c0 + tx + j * TX) : 0.f;
     pdl_wait();
     if (a.start_pos < 0 || a.start_pos + a.n_tokens > a.seq_len) return;
-#pragma unroll
-    for (int i = 0; i < NS; ++i)
-        S[i] = in && a.start_pos > 0 && ln + i * L < pieces ? __ldcg(reinterpret_cast<const float4*>(a.S + (size_t)c * a.state_pitch) + ln + i * L) : zero;
-    // the convolution inputs that the next portion needs
-    if (a.taps > 1) {
-        const int slots = a.taps - 1, keep = min(slots, a.n_tokens);
-        for (int i = tid; i < keep * CH; i += kScanThreads) {
-            const int k = i / CH, ch = c0 + i - k * CH;
-            const size_t at = (size_t)((a.start_pos + a.n_tokens - 1 - k) % slots) * a.ring_pitch + ch;
-            if (ch < a.inner) a.ring[at] = __ldcg(a.tail + at);
-        }
-    }
     for (int t0 = 0; t0 < a.n_tokens; t0 += a.tile_tokens) {
         const int nt = min(a.tile_tokens, a.n_tokens - t0);
         if (t0 > 0) __syncthreads();
-        // dt | B | C rows
-        const int n_low = a.dt_pitch + 2 * a.state_pitch;
-        for (int i = tid; i < nt * n_low; i += kScanThreads) {
-            const int t = i / n_low, k = i - t * n_low;
-            float v[kPfMaxSplits], sum = 0.f;
-#pragma unroll
-            for (int s = 0; s < kPfMaxSplits; ++s)
-                if (s < a.splits) v[s] = mamba_low(a, a.low + ((size_t)s * kPrefillTokens + t0 + t) * a.low_rows, k);
-#pragma unroll
-            for (int s = 0; s < kPfMaxSplits; ++s)
-                if (s < a.splits) sum += v[s];
-            low[t * LP + k] = sum;
+        for (int i = tid; i < nt * (LP / 4); i += kScanThreads) cp_async_16(low + 4 * i, a.low + (size_t)t0 * LP + 4 * i, true);
+        for (int i = tid; i < nt * (CH / 4); i += kScanThreads) {  // x_pitch is a multiple of 64: no row ends inside a piece
+            const int t = i / (CH / 4), k = 4 * (i - t * (CH / 4));
+            const size_t at = (size_t)(t0 + t) * a.x_pitch + c0 + k;
+            const bool have = c0 + k < a.x_pitch;
+            cp_async_16(xs + t * CH + k, a.x + (have ? at : 0), have);
+            cp_async_16(zs + t * CH + k, a.z + (have ? at : 0), have);
         }
-        for (int i = tid; i < nt * CH; i += kScanThreads) {
-            const int t = i / CH, ch = i - t * CH;
-            xs[i] = c0 + ch < a.inner ? __ldcg(a.x + (size_t)(t0 + t) * a.x_pitch + c0 + ch) : 0.f;
+        cp_async_commit();
+        if (t0 == 0) {
+#pragma unroll
+            for (int i = 0; i < NS; ++i)
+                S[i] = in && a.start_pos > 0 && ln + i * L < pieces ? __ldcg(reinterpret_cast<const float4*>(a.S + (size_t)c * a.state_pitch) + ln + i * L) : zero;
+            // the convolution inputs that the next portion needs
+            if (a.taps > 1) {
+                const int slots = a.taps - 1, keep = min(slots, a.n_tokens);
+                for (int i = tid; i < keep * CH; i += kScanThreads) {
+                    const int k = i / CH, ch = c0 + i - k * CH;
+                    const size_t at = (size_t)((a.start_pos + a.n_tokens - 1 - k) % slots) * a.ring_pitch + ch;
+                    if (ch < a.inner) a.ring[at] = __ldcg(a.tail + at);
+                }
+            }
         }
+        cp_async_wait<0>();
         __syncthreads();
         for (int tb = 0; tb < nt; tb += TPT * TY) {
             float acc[TPT][CPT];
@@ -214,7 +278,7 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
                 for (int j = 0; j < CPT; ++j) acc[i][j] = 0.f;
             int at[TPT];
 #pragma unroll
-            for (int i = 0; i < TPT; ++i) at[i] = min(tb + ty + i * TY, nt - 1) * LP;  // beyond the tile: not stored
+            for (int i = 0; i < TPT; ++i) at[i] = min(tb + ty + i * TY, nt - 1) * LP;  // beyond the tile: not used
             for (int k = 0; k < a.dt_pitch; k += 4) {
                 float4 l[TPT], w[CPT];
 #pragma unroll
@@ -231,35 +295,40 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
             for (int i = 0; i < TPT; ++i) {
                 const int t = tb + ty + i * TY;
 #pragma unroll
-                for (int j = 0; j < CPT; ++j)
-                    if (t < nt) dts[t * CH + tx + j * TX] = softplus_f(acc[i][j] + bias[j]);
+                for (int j = 0; j < CPT; ++j)  // a step of size 0 leaves the state alone: what fills up the last four tokens
+                    if (t < a.tile_tokens) dts[t * CH + tx + j * TX] = t < nt ? softplus_f(acc[i][j] + bias[j]) : 0.f;
             }
         }
         __syncthreads();
-#pragma unroll 4
-        for (int t = 0; t < nt; ++t) {
-            const float dt = dts[t * CH + cl], x = xs[t * CH + cl];
-            const float4* B = reinterpret_cast<const float4*>(low + t * LP + a.dt_pitch);
-            float y = 0.f;
+        for (int t = 0; t < nt; t += 4) {
+            float y[4];
 #pragma unroll
-            for (int i = 0; i < NS; ++i) {
-                const int q = ln + i * L;
-                if (q < pieces) y += mamba_update(S[i], A[i], B[q], B[pieces + q], dt, dt * x);
+            for (int k = 0; k < 4; ++k) {
+                const int tk = min(t + k, nt - 1);
+                const float dt = dts[(t + k) * CH + cl], dx = dt * xs[tk * CH + cl];
+                const float4* B = reinterpret_cast<const float4*>(low + tk * LP + a.dt_pitch);
+                y[k] = 0.f;
+#pragma unroll
+                for (int i = 0; i < NS; ++i) {
+                    const int q = ln + i * L;
+                    if (q < pieces) y[k] += mamba_update(S[i], A[i], B[q], B[pieces + q], dt, dx);
+                }
             }
-            y = lane_group_sum<L>(y);
+            const float sum = lane_group_sum4<L>(y, ln);
+            const int mine = t + scan_token(ln);
             __syncwarp();  // the channel's lanes have read x
-            if (ln == 0) xs[t * CH + cl] = fmaf(D, x, y);
+            if (ln < 4 && mine < nt) xs[mine * CH + cl] = fmaf(D, xs[mine * CH + cl], sum);
         }
         __syncthreads();
-        for (int i = tid; i < nt * CH; i += kScanThreads) {
-            const int t = i / CH, ch = i - t * CH;
+        for (int i = tid; i < nt * (CH / 2); i += kScanThreads) {
+            const int t = i / (CH / 2), ch = 2 * (i - t * (CH / 2));
             if (c0 + ch >= a.inner) continue;
-            const float v = xs[i] * __ldcg(a.z + (size_t)(t0 + t) * a.x_pitch + c0 + ch);
-            __nv_bfloat16 hi, lo;
-            split_pair(v, hi, lo);
+            __align__(4) __nv_bfloat16 hi[2], lo[2];
+            split_pair(xs[t * CH + ch] * zs[t * CH + ch], hi[0], lo[0]);
+            split_pair(c0 + ch + 1 < a.inner ? xs[t * CH + ch + 1] * zs[t * CH + ch + 1] : 0.f, hi[1], lo[1]);
             __nv_bfloat16* d = a.planes + (size_t)(t0 + t) * a.plane_row + c0 + ch;
-            d[0] = hi;
-            d[(size_t)kPrefillTokens * a.plane_row] = lo;
+            *reinterpret_cast<uint32_t*>(d) = *reinterpret_cast<const uint32_t*>(hi);
+            *reinterpret_cast<uint32_t*>(d + (size_t)kPrefillTokens * a.plane_row) = *reinterpret_cast<const uint32_t*>(lo);
         }
     }
     if (!in) return;
