@@ -501,7 +501,7 @@ def layered_engines(name):
     import torch
     from lighterpp_b200 import engine as E
     from lighterpp_b200.models import ARCHITECTURES
-    arch, cfg, llama = layered_config(name)
+    arch, cfg, _ = layered_config(name)
     g = torch.Generator(device="cuda")
     g.manual_seed(7)
     eng = E.Engine(cfg, "bf16", "f16")
@@ -519,6 +519,13 @@ def layered_engines(name):
     torch.cuda.empty_cache()
     yield arch.lower(), eng
     eng.close()
+    yield from llama_engine(name)
+
+
+def llama_engine(name):
+    import torch
+    from lighterpp_b200 import engine as E
+    llama = layered_config(name)[2]
     eng = E.Engine(llama, "f16", "f16")
     for tensor, l, t in gen_device_weights(llama, "f16", True, 7):
         eng.upload(tensor, t, max(l, 0))

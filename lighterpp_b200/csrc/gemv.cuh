@@ -136,6 +136,14 @@ using GemvArgsOf = std::conditional_t<is_latent_epi<EPI>, GemvLatentArgs,
                                       std::conditional_t<EPI == kEpiSharedKvIn, GemvSharedKvArgs, std::conditional_t<EPI == kEpiMambaIn, GemvMambaArgs, GemvArgs>>>;
 template <int EPI>
 constexpr bool is_resid_epi = EPI == kEpiResid || EPI == kEpiResidBias;
+// What a kernel never does is left out of it: a step's kernels follow each other in microseconds, and their code is fetched
+// anew at every launch once it no longer fits the instruction caches together.
+template <typename WT>
+constexpr bool may_be_tp = !std::is_same<WT, __nv_bfloat16>::value;  // engines described layer by layer run on one GPU
+template <int EPI>
+constexpr bool may_embed = EPI == kEpiQkv || EPI == kEpiLatentIn || EPI == kEpiSharedKvIn || EPI == kEpiMambaIn;  // a layer's first kernel
+template <int EPI>
+constexpr bool may_norm = !is_resid_epi<EPI>;
 // Epilogues that need several loads of their own per row: done by a lane per row, up to 16 row pairs of a warp together, with
 // what does not depend on the product fetched before it is formed.
 template <int EPI>
@@ -155,6 +163,9 @@ __device__ __forceinline__ int xs_index(int k, int K) {
         return k;
 }
 
+// Timing experiments exist in builds with LPP_TIMING_AIDS only.
+#ifdef LPP_TIMING_AIDS
+__device__ __forceinline__ int gemv_debug(const GemvArgs& a) { return a.debug; }
 __device__ __forceinline__ void gemv_stamp(const GemvArgs& a, int k) {
     if (a.trace) {
         unsigned long long t;
@@ -162,6 +173,10 @@ __device__ __forceinline__ void gemv_stamp(const GemvArgs& a, int k) {
         a.trace[(size_t)blockIdx.x * 8 + k] = t;
     }
 }
+#else
+__device__ __forceinline__ constexpr int gemv_debug(const GemvArgs&) { return 0; }
+__device__ __forceinline__ void gemv_stamp(const GemvArgs&, int) {}
+#endif
 
 // Stores four consecutive inputs x[k..k+3] (k % 4 == 0) into the staging layout.
 template <typename WT>
@@ -341,14 +356,14 @@ __device__ __forceinline__ void stage_input_peers(const GemvArgs& a, float* xs, 
 // RMS-normalises it (ss = 1/sqrt(mean(x^2) + 1e-5); out = x*ss*w, src/ops.cpp:20-32) and leaves it
 // in shared memory in the layout xs_index<WT> describes.  Executed by `NT` threads (tid 0..NT-1).
 // The norm weights are constants, so their loads are issued before the dependency wait.
-template <typename WT, int NT, bool LN>
+template <typename WT, int EPI, int NT, bool LN>
 __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float* red, int tid) {
     const int K = a.K;
     const int nv4 = K >> 2;
     constexpr int kPer = 4;  // float4 per thread and pass: one pass covers 4*4*NT inputs
     const bool one_pass = nv4 <= kPer * NT;
     float4 wr[kPer], br[kPer];
-    if (a.norm_w && one_pass) {
+    if (may_norm<EPI> && a.norm_w && one_pass) {
 #pragma unroll
         for (int j = 0; j < kPer; ++j) {
             const int i = tid + j * NT;
@@ -361,7 +376,7 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
     // rank's own slot included): its flags can only be complete once every rank's producing GEMV has
     // stored all its rows, which in turn follows everything earlier in the step, so that case does not
     // wait for the local kernel to drain its peer stores and exit.
-    if constexpr (!LN) {
+    if constexpr (!LN && may_be_tp<WT> && !is_resid_epi<EPI>) {
         if (a.tp_in != nullptr) {
             stage_input_peers<WT, NT>(a, xs, red, tid);
             return;
@@ -370,7 +385,7 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
     pdl_wait();  // activations / KV / step state come from the previous kernel
     if (tid == 0) gemv_stamp(a, 1);
 
-    if (a.emb) {
+    if (may_embed<EPI> && a.emb) {
         // first layer: the input is the embedding row of the device-resident token, widened exactly, times its factor
         int tok = a.st->token;
         if (tok < 0 || tok >= a.vocab) {
@@ -451,7 +466,7 @@ __device__ __forceinline__ void stage_input(const GemvArgs& a, float* xs, float*
         consumer_barrier(NT);
         return;
     } else {
-        if (!a.norm_w) {
+        if (!may_norm<EPI> || !a.norm_w) {
             for (int i = tid; i < nv4; i += NT) xs_store4<WT>(xs, i << 2, K, load_x4(i));
             consumer_barrier(NT);
             return;
@@ -600,8 +615,9 @@ __device__ __forceinline__ void dot_rows(const unsigned char* row0, const unsign
 
 // Store of a finished row pair: locally, or as {value, flag} words into this rank's slot (residual GEMVs) or
 // row range (vocabulary-sharded classifier) on every rank of the tensor-parallel group.
+template <typename WT>
 __device__ __forceinline__ void store_rows(const GemvArgs& a, int row, float v0, float v1) {
-    if (a.tp_out[0]) {
+    if (may_be_tp<WT> && a.tp_out[0]) {
         const unsigned long long flag = (unsigned long long)(*a.tp_epoch + 1u) << 32;
         const unsigned long long w0 = flag | __float_as_uint(v0), w1 = flag | __float_as_uint(v1);
 #pragma unroll
@@ -618,7 +634,7 @@ template <typename WT, int EPI>
 __device__ __forceinline__ void gemv_epilogue(const GemvArgsOf<EPI>& a, int g, float v0, float v1) {
     const int row = g * kRowsPerGroup;
     if constexpr (EPI == kEpiStore) {
-        store_rows(a, row, v0, v1);
+        store_rows<WT>(a, row, v0, v1);
     } else if constexpr (is_resid_epi<EPI>) {
         if constexpr (EPI == kEpiResidBias) {
             const float2 b = __ldg(reinterpret_cast<const float2*>(a.bias + row));
@@ -631,7 +647,7 @@ __device__ __forceinline__ void gemv_epilogue(const GemvArgsOf<EPI>& a, int g, f
             v0 += r.x;
             v1 += r.y;
         }
-        store_rows(a, row, v0, v1);
+        store_rows<WT>(a, row, v0, v1);
     } else if constexpr (EPI == kEpiSwiglu) {
         // rows are interleaved (gate_i, up_i); hb = (h1*sigmoid(h1))*h3 (src/ops.cpp:78-87), or the tanh form of
         // GELU in place of h1*sigmoid(h1)
@@ -748,7 +764,7 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
     // The dependent kernel is released for launch at once: its CTAs take over an SM as soon as one of
     // this kernel's CTAs leaves it and start streaming their own weights while the rest of this grid
     // finishes (they still wait for this grid's completion before touching activations).
-    if (tid == 0 && !(a.debug & 4)) pdl_launch_dependents();
+    if (tid == 0 && !(gemv_debug(a) & 4)) pdl_launch_dependents();
     if (tid < kGemvConsumerWarps * NS) {
         const int bw = tid / NS, sl = tid - bw * NS;
         mbar_init(&full[bw * kGemvMaxStages + sl], 1);
@@ -768,16 +784,16 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
             bool alive = true;
             // streamed weights are marked evict-first in L2: they are used once per token and would
             // otherwise push the K/V cache and the activations out (debug bit 8 turns the hint off)
-            const unsigned long long policy = !(a.debug & 8) ? l2_policy_evict_first() : 0ull;
+            const unsigned long long policy = !(gemv_debug(a) & 8) ? l2_policy_evict_first() : 0ull;
             auto issue = [&](const unsigned char* src, uint32_t bytes) -> bool {
                 // trip p > 0 reuses a slot once its release number p-1 has happened
                 if (pass > 0 && !mbar_wait_bounded(&myempty[slot], (uint32_t)(pass - 1) & 1u, a.st))
                     return false;
-                if (a.debug & 2) {
+                if (gemv_debug(a) & 2) {
                     mbar_arrive(&myfull[slot]);
                 } else {
                     mbar_arrive_expect_tx(&myfull[slot], bytes);
-                    if (!(a.debug & 8))
+                    if (!(gemv_debug(a) & 8))
                         bulk_g2s_hint(myring + (size_t)slot * a.stage_bytes, src, bytes, &myfull[slot], policy);
                     else
                         bulk_g2s(myring + (size_t)slot * a.stage_bytes, src, bytes, &myfull[slot]);
@@ -807,7 +823,7 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
             if (lane == 0) gemv_stamp(a, 6);
             // this lane's HBM requests are all queued: pull its share of the next kernel's weights
             // towards L2 so the memory system stays busy across the kernel boundary
-            if (a.pf && alive) {
+            if (may_be_tp<WT> && a.pf && alive) {
                 const unsigned int lanes = gridDim.x * kGemvConsumerWarps;
                 unsigned int slice = (a.pf_bytes + lanes - 1) / lanes;
                 slice = (slice + 15u) & ~15u;
@@ -820,7 +836,7 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
         }
         __syncwarp();
         // all of this CTA's copies are issued: the next kernel may start launching
-        if (lane == 0 && (a.debug & 4)) pdl_launch_dependents();
+        if (lane == 0 && (gemv_debug(a) & 4)) pdl_launch_dependents();
         return false;
     }
 
@@ -872,7 +888,7 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
         Kx = n_groups * a.K;
         stage_input_groups<WT, EPI, kGemvConsumerWarps * 32>(a, xs, tid, first_group, n_groups);
     } else {
-        stage_input<WT, kGemvConsumerWarps * 32, LN>(a, xs, red, tid);
+        stage_input<WT, EPI, kGemvConsumerWarps * 32, LN>(a, xs, red, tid);
     }
     // where the inputs of row pair p start among the staged ones
     auto input_offset = [&](int p) -> int {
@@ -922,11 +938,11 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
             for (int i = 0; i < cnt; ++i) {
                 float acc0 = 0.f, acc1 = 0.f;
                 const unsigned char* r0 = st + (size_t)i * kRowsPerGroup * row_bytes;
-                if (!(a.debug & 1)) dot_rows<WT, 2, false>(r0, r0 + row_bytes, xs, Kx, input_offset(p + i), a.K, lane, acc0, acc1);
+                if (!(gemv_debug(a) & 1)) dot_rows<WT, 2, false>(r0, r0 + row_bytes, xs, Kx, input_offset(p + i), a.K, lane, acc0, acc1);
                 acc0 = warp_sum(acc0);
                 acc1 = warp_sum(acc1);
                 if (is_resid_epi<EPI> && p + i == p0) {
-                    if (lane == 0) store_rows(a, p0 * kRowsPerGroup, acc0 + r_first.x, acc1 + r_first.y);
+                    if (lane == 0) store_rows<WT>(a, p0 * kRowsPerGroup, acc0 + r_first.x, acc1 + r_first.y);
                 } else {
                     finish(p + i, acc0, acc1);
                 }
@@ -947,13 +963,13 @@ __device__ __forceinline__ bool gemv_ring_body(const GemvArgsOf<EPI>& a, unsigne
                     const int klen = min(a.kc, a.K - k0);
                     const unsigned char* st = myring + (size_t)slot * a.stage_bytes;
                     float dummy = 0.f;
-                    if (!(a.debug & 1)) dot_rows<WT, 1, false>(st, st, xs, Kx, input_offset(p) + k0, klen, lane, acc[r], dummy);
+                    if (!(gemv_debug(a) & 1)) dot_rows<WT, 1, false>(st, st, xs, Kx, input_offset(p) + k0, klen, lane, acc[r], dummy);
                     release();
                 }
             if (!ok) break;
             const float v0 = warp_sum(acc[0]), v1 = warp_sum(acc[1]);
             if (is_resid_epi<EPI> && p == p0) {
-                if (lane == 0) store_rows(a, p0 * kRowsPerGroup, v0 + r_first.x, v1 + r_first.y);
+                if (lane == 0) store_rows<WT>(a, p0 * kRowsPerGroup, v0 + r_first.x, v1 + r_first.y);
             } else {
                 finish(p, v0, v1);
             }
@@ -967,7 +983,7 @@ template <typename WT, int EPI, bool LN>
 __global__ void __launch_bounds__(kGemvRingThreads) gemv_ring_kernel(const GemvArgsOf<EPI> a) {
     extern __shared__ __align__(128) unsigned char smem[];
     const bool consumer = gemv_ring_body<WT, EPI, LN>(a, smem);
-    if constexpr (EPI == kEpiResid) {
+    if constexpr (EPI == kEpiResid && may_be_tp<WT>) {
         // tensor-parallel exchange: this CTA's rows are on their way, tell every rank (a hint, see GemvArgs)
         if (consumer && a.tp_size > 1 && a.tp_hint_out[0]) {
             consumer_barrier(kGemvConsumerWarps * 32);
@@ -1006,7 +1022,7 @@ __global__ void __launch_bounds__(kGemvLdgThreads) gemv_ldg_kernel(const GemvArg
         Kx = n_groups * a.K;
         stage_input_groups<WT, EPI, kGemvLdgThreads>(a, xs, tid, first_group, n_groups);
     } else {
-        stage_input<WT, kGemvLdgThreads, LN>(a, xs, red, tid);
+        stage_input<WT, EPI, kGemvLdgThreads, LN>(a, xs, red, tid);
     }
     const unsigned char* W = reinterpret_cast<const unsigned char*>(a.W);
     const size_t row_bytes = (size_t)a.K * sizeof(WT);
