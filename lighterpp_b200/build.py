@@ -10,7 +10,7 @@ LIB_PATH = os.path.join(_HERE, "liblpp_b200.so")
 
 
 def ensure_built() -> str:
-    """Path of the library; builds it (about a minute) when it is missing.  Callers that race for it wait for the one
+    """Path of the library; builds it (one or two minutes) when it is missing.  Callers that race for it wait for the one
     that builds, and the finished library appears under its name in one step."""
     if os.path.exists(LIB_PATH):
         return LIB_PATH

@@ -660,8 +660,9 @@ static MambaScanArgs mamba_scan_args(const lpp_engine* e, const ModelLayer& y, c
     return a;
 }
 // Limits of a selective-scan layer (registers and shared memory of the scan kernels); lanes per channel and pieces of four
-// state elements per lane by the state's size.
+// state elements per lane by the state's size, and with them the elements a channel has in memory.
 constexpr int kScanMaxState = 4 * 32 * 8, kScanMaxTaps = 64, kScanMaxRank = 1536;
+static int scan_state_pitch(int n) { return n <= 16 ? 16 : n <= 32 ? 32 : n <= 64 ? 64 : n <= 128 ? 128 : n <= 256 ? 256 : kScanMaxState; }
 #define LPP_SCAN_DISPATCH(n, F)         \
     do {                                \
         if ((n) <= 16) return F(4, 1);  \
@@ -695,13 +696,13 @@ static cudaError_t launch_mamba_scan(const lpp_engine* e, const MambaScanArgs& a
 #undef LPP_SCAN
 }
 static cudaError_t launch_mamba_conv(const MambaConvArgs& a, cudaStream_t s) {
-    const dim3 grid((a.inner + 2 * kConvThreads - 1) / (2 * kConvThreads), (a.n_tokens + kConvTokens - 1) / kConvTokens, 2), block(kConvThreads);
+    const dim3 grid((a.inner + 4 * kConvThreads - 1) / (4 * kConvThreads), (a.n_tokens + kConvTokens - 1) / kConvTokens, 2), block(kConvThreads);
     switch (a.taps) {
         case 2: return launch_kernel(mamba_conv_kernel<2>, grid, block, 0, s, true, a);
         case 3: return launch_kernel(mamba_conv_kernel<3>, grid, block, 0, s, true, a);
         case 4: return launch_kernel(mamba_conv_kernel<4>, grid, block, 0, s, true, a);
     }
-    const size_t smem = (size_t)(kConvTokens + a.taps - 1) * kConvThreads * sizeof(float2);
+    const size_t smem = (size_t)(kConvTokens + a.taps - 1) * kConvThreads * sizeof(float4);
     const cudaError_t r = cudaFuncSetAttribute(mamba_conv_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max<size_t>(smem, 49152));
     return r != cudaSuccess ? r : launch_kernel(mamba_conv_kernel<0>, grid, block, smem, s, true, a);
 }
@@ -1587,11 +1588,11 @@ static void size_layer(ModelLayer& y) {
     lpp_layer_desc& d = y.d;
     y.ff_pitch = (int)align_up(d.ff, 64);
     if (d.mixer == LPP_MIXER_MAMBA) {
-        y.inner_rows = (int)align_up(d.inner, 2);
+        y.inner_rows = (int)align_up(d.inner, 4);
         y.inner_pitch = (int)align_up(d.inner, 64);
         y.low_rows = (int)align_up((size_t)d.dt_rank + 2 * d.state, 2);
         y.dt_pitch = (int)align_up(d.dt_rank, 8);
-        y.state_pitch = (int)align_up(d.state, 4);
+        y.state_pitch = scan_state_pitch(d.state);
         y.in_rows = 2 * y.inner_rows;
         y.o_in = d.inner;
     } else if (d.mixer == LPP_MIXER_SHARED_KV) {

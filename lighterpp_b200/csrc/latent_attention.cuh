@@ -272,14 +272,15 @@ __device__ __forceinline__ void latent_planes4(const LatentAttnArgs& a, int t, i
 #pragma unroll
     for (int c = 0; c < 4; ++c) split_pair(y[c], hi[c], lo[c]);
     if (!GATED || ((a.plane_pitch | a.plane_cols) & 3) == 0) {  // (rows of latents are padded)
-        if (col >= a.plane_cols) return;
-        *reinterpret_cast<uint2*>(d) = *reinterpret_cast<const uint2*>(hi);
-        *reinterpret_cast<uint2*>(d_lo) = *reinterpret_cast<const uint2*>(lo);
-        return;
-    }
+        if (col < a.plane_cols) {
+            *reinterpret_cast<uint2*>(d) = *reinterpret_cast<const uint2*>(hi);
+            *reinterpret_cast<uint2*>(d_lo) = *reinterpret_cast<const uint2*>(lo);
+        }
+    } else {
 #pragma unroll
-    for (int c = 0; c < 4; ++c)
-        if (col + c < a.plane_cols) d[c] = hi[c], d_lo[c] = lo[c];
+        for (int c = 0; c < 4; ++c)
+            if (col + c < a.plane_cols) d[c] = hi[c], d_lo[c] = lo[c];
+    }
 }
 
 constexpr int kLatScPitch = kLatentTile + 4, kLatPPitch = kLatentTile + 8;

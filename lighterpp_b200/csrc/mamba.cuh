@@ -21,7 +21,7 @@ namespace lpp {
 // ---- input projection of a step: rows  x [inner_rows] | z [inner_rows]
 
 struct MambaInArgs {
-    int inner, inner_rows;  // channels, rounded up to even
+    int inner, inner_rows;  // channels, rounded up to a multiple of 4
     int taps;
     int early;              // weights and state may be read before the dependency wait (and so may the position)
     const float* conv_w;    // [taps][inner_rows]
@@ -58,11 +58,12 @@ __device__ __forceinline__ void mamba_in_row(const MambaInArgs& m, int pos, int 
 }
 
 // ---- the recurrence.  A channel's state belongs to L neighbouring lanes, each of which holds NS pieces of four elements
-// (piece q of the channel to lane q % L).
+// (piece q of the channel to lane q % L).  In memory a channel has 4 L NS elements, the ones beyond its state zero: they stay
+// zero, because the same holds for A, B and C.
 
 struct MambaScanArgs {
     int inner, state, dt_rank;
-    int state_pitch, dt_pitch;  // elements per channel of S and A (multiple of 4), of w_dt (multiple of 8)
+    int state_pitch, dt_pitch;  // elements per channel of S and A (4 L NS), of w_dt (multiple of 8)
     int low_rows;               // row of `low`: dt | B | C, even
     const float* low;           // step: [low_rows]; prompt block: [kPrefillTokens][mamba_low_pitch], padded
     const void* w_dt;           // [inner][dt_pitch], weight type
@@ -83,31 +84,67 @@ struct MambaScanArgs {
     int taps, ring_pitch;
 };
 
+// Pairs of floats in one 64-bit register: sm_100 multiplies and adds both with one instruction.
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack_f2(float lo, float hi) {
+    f32x2 r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ float2 unpack_f2(f32x2 v) {
+    float2 r;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(r.x), "=f"(r.y) : "l"(v));
+    return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+    f32x2 r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+    f32x2 r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ f32x2 both(float v) { return pack_f2(v, v); }
+__device__ __forceinline__ float exp2_approx(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+
 // exp(x) - 1 for x <= 0.  A channel that forgets slowly multiplies its state with a factor just below 1 thousands of times,
 // and always with much the same one: the rounding of the factor itself to 32 bits (2^-25 of it, the same way every time)
 // would add up, so the state is updated with its difference from 1.  Taylor series where it cancels (the first term left
-// out is below 2e-8 of the sum).
-__device__ __forceinline__ float decay_m1(float x) {
-    float p = fmaf(x, 1.f / 40320.f, 1.f / 5040.f);
-    p = fmaf(x, p, 1.f / 720.f);
-    p = fmaf(x, p, 1.f / 120.f);
-    p = fmaf(x, p, 1.f / 24.f);
-    p = fmaf(x, p, 1.f / 6.f);
-    p = fmaf(x, p, 0.5f);
-    p = fmaf(x * x, p, x);
-    return x > -0.5f ? p : __expf(x) - 1.f;
+// out is below 5e-8 of the sum).
+__device__ __forceinline__ f32x2 decay_m1(f32x2 x) {
+    f32x2 p = fma2(x, both(1.f / 720.f), both(1.f / 120.f));
+    p = fma2(x, p, both(1.f / 24.f));
+    p = fma2(x, p, both(1.f / 6.f));
+    p = fma2(x, p, both(0.5f));
+    p = fma2(mul2(x, x), p, x);
+    const float2 v = unpack_f2(x), series = unpack_f2(p), t = unpack_f2(mul2(x, both(1.4426950408889634f)));
+    return pack_f2(v.x > -0.25f ? series.x : exp2_approx(t.x) - 1.f, v.y > -0.25f ? series.y : exp2_approx(t.y) - 1.f);
 }
-// S <- exp(dt A) S + dx B
-__device__ __forceinline__ void state_update(float& S, float A, float B, float dt, float dx) {
-    S = fmaf(decay_m1(dt * A), S, fmaf(dx, B, S));
+// Four elements of a channel, as two pairs.
+struct ScanPiece {
+    f32x2 lo, hi;
+};
+__device__ __forceinline__ ScanPiece scan_piece(const float4& v) { return {pack_f2(v.x, v.y), pack_f2(v.z, v.w)}; }
+__device__ __forceinline__ float4 scan_float4(const ScanPiece& p) {
+    const float2 a = unpack_f2(p.lo), b = unpack_f2(p.hi);
+    return make_float4(a.x, a.y, b.x, b.y);
 }
-// The same for four elements; returns their share of S . C
-__device__ __forceinline__ float mamba_update(float4& S, const float4& A, const float4& B, const float4& C, float dt, float dx) {
-    state_update(S.x, A.x, B.x, dt, dx);
-    state_update(S.y, A.y, B.y, dt, dx);
-    state_update(S.z, A.z, B.z, dt, dx);
-    state_update(S.w, A.w, B.w, dt, dx);
-    return fmaf(S.x, C.x, fmaf(S.y, C.y, fmaf(S.z, C.z, S.w * C.w)));
+// S <- exp(dt A) S + dx B for four elements; y gains their S C, pair by pair.
+__device__ __forceinline__ void mamba_update(ScanPiece& S, const ScanPiece& A, const ScanPiece& B, const ScanPiece& C, f32x2 dt, f32x2 dx, f32x2& y) {
+    S.lo = fma2(decay_m1(mul2(dt, A.lo)), S.lo, fma2(dx, B.lo, S.lo));
+    S.hi = fma2(decay_m1(mul2(dt, A.hi)), S.hi, fma2(dx, B.hi, S.hi));
+    y = fma2(S.lo, C.lo, y);
+    y = fma2(S.hi, C.hi, y);
+}
+__device__ __forceinline__ float pair_sum(f32x2 v) {
+    const float2 f = unpack_f2(v);
+    return f.x + f.y;
 }
 template <int L>
 __device__ __forceinline__ float lane_group_sum(float v) {
@@ -139,15 +176,16 @@ static __global__ void __launch_bounds__(kScanStepThreads) mamba_step_kernel(con
     if (!a.early) pdl_wait();
     const int pos = a.st->pos;
     const bool ok = pos >= 0 && pos < a.seq_len;
-    const int pieces = a.state_pitch / 4, vecs = a.dt_pitch / kVec;
+    constexpr int pieces = L * NS;
+    const int vecs = a.dt_pitch / kVec;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
-    float4 A[NS], S[NS];
+    const float4* A4 = reinterpret_cast<const float4*>(a.A) + (size_t)(in ? c : 0) * pieces + ln;
+    float4* S4 = reinterpret_cast<float4*>(a.S) + (size_t)(in ? c : 0) * pieces + ln;
+    ScanPiece A[NS], S[NS];
 #pragma unroll
     for (int i = 0; i < NS; ++i) {
-        const int q = ln + i * L;
-        const bool have = in && q < pieces;
-        A[i] = have ? __ldg(reinterpret_cast<const float4*>(a.A + (size_t)c * a.state_pitch) + q) : zero;
-        S[i] = have && pos > 0 ? __ldcg(reinterpret_cast<const float4*>(a.S + (size_t)c * a.state_pitch) + q) : zero;
+        A[i] = scan_piece(__ldg(A4 + i * L));
+        S[i] = scan_piece(pos > 0 ? __ldcg(S4 + i * L) : zero);
     }
     const uint4* w = reinterpret_cast<const uint4*>(reinterpret_cast<const WT*>(a.w_dt) + (size_t)(in ? c : 0) * a.dt_pitch);
     uint4 wv[kAhead];
@@ -181,17 +219,13 @@ static __global__ void __launch_bounds__(kScanStepThreads) mamba_step_kernel(con
     const float dt = softplus_f(lane_group_sum<L>(dot) + bias);
     const float4* B = reinterpret_cast<const float4*>(sc_low + a.dt_pitch);
     const float4* C = B + pieces;
-    float y = 0.f;
+    f32x2 y2 = both(0.f);
 #pragma unroll
-    for (int i = 0; i < NS; ++i) {
-        const int q = ln + i * L;
-        if (q < pieces) y += mamba_update(S[i], A[i], B[q], C[q], dt, dt * x);
-    }
-    y = lane_group_sum<L>(y);
+    for (int i = 0; i < NS; ++i) mamba_update(S[i], A[i], scan_piece(B[ln + i * L]), scan_piece(C[ln + i * L]), both(dt), both(dt * x), y2);
+    const float y = lane_group_sum<L>(pair_sum(y2));
     if (!in || !ok) return;
 #pragma unroll
-    for (int i = 0; i < NS; ++i)
-        if (ln + i * L < pieces) *(reinterpret_cast<float4*>(a.S + (size_t)c * a.state_pitch) + ln + i * L) = S[i];
+    for (int i = 0; i < NS; ++i) S4[i * L] = scan_float4(S[i]);
     if (ln == 0) a.out[c] = fmaf(D, x, y) * z;
 }
 

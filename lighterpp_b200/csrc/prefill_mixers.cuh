@@ -57,10 +57,10 @@ static __global__ void __launch_bounds__(256) prefill_shared_kv_finish_kernel(co
 
 // Convolution of a prompt block after the input GEMM (partial sums added in range order): x convolved, as FP32 rows and as
 // hi + lo operands of the next GEMM; z through the silu.  The inputs of the last taps - 1 tokens go to `tail`; the scan
-// copies them to the ring once every CTA of this launch has read it.  A thread takes two channels of kConvTokens tokens;
+// copies them to the ring once every CTA of this launch has read it.  A thread takes four channels of kConvTokens tokens;
 // TAPS = the number of taps (inputs in registers), or 0 = any (inputs in shared memory).
 // grid: (ceil(inner / 256), ceil(tokens / kConvTokens), 2: x, z); shared memory (TAPS 0): (kConvTokens + taps - 1) * 256 floats
-constexpr int kConvThreads = 128, kConvTokens = 4;
+constexpr int kConvThreads = 64, kConvTokens = 4;
 struct MambaConvArgs {
     const float* part;  // [splits][kPrefillTokens][2 * inner_rows]
     int splits, n_tokens, start_pos, seq_len;
@@ -72,86 +72,111 @@ struct MambaConvArgs {
     __nv_bfloat16* planes;  // [2 planes][kPrefillTokens][x_pitch]
     StepState* st;
 };
+// N tokens' sums of the partial sums of rows row .. row + 3, tokens t0 .. (clamped to the block: no branches, so the loads of
+// a range of K are in flight together), in range order.
+template <int N>
+__device__ __forceinline__ void prefill_sums(const float* part, int n_rows, int splits, int n_tokens, int t0, int row, float4 (&v)[N]) {
+    const float4* p[N];
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        p[i] = reinterpret_cast<const float4*>(part + (size_t)min(max(t0 + i, 0), n_tokens - 1) * n_rows + row);
+        v[i] = *p[i];
+    }
+#pragma unroll 2
+    for (int s = 1; s < splits; ++s)
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const float4 w = p[i][(size_t)s * kPrefillTokens * n_rows / 4];
+            v[i].x += w.x; v[i].y += w.y; v[i].z += w.z; v[i].w += w.w;
+        }
+}
+// With the fast exponential and division, like the gated feed-forward's activation on this path.
+__device__ __forceinline__ float4 silu4(const float4& v) {
+    return make_float4(__fdividef(v.x, 1.f + __expf(-v.x)), __fdividef(v.y, 1.f + __expf(-v.y)), __fdividef(v.z, 1.f + __expf(-v.z)),
+                       __fdividef(v.w, 1.f + __expf(-v.w)));
+}
+__device__ __forceinline__ float4 fma4(const float4& a, const float4& b, const float4& c) {
+    return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w));
+}
 template <int TAPS>
 static __global__ void __launch_bounds__(kConvThreads) mamba_conv_kernel(const MambaConvArgs a) {
-    extern __shared__ float2 cv_in[];  // [kConvTokens + taps - 1][kConvThreads]; a thread reads back only what it wrote
+    extern __shared__ float4 cv_in[];  // [kConvTokens + taps - 1][kConvThreads]; a thread reads back only what it wrote
     pdl_launch_dependents();
-    const int tid = threadIdx.x, c = 2 * ((int)blockIdx.x * kConvThreads + tid);
+    const int tid = threadIdx.x, c = 4 * ((int)blockIdx.x * kConvThreads + tid);
     const int t0 = blockIdx.y * kConvTokens, n_rows = 2 * a.inner_rows, slots = TAPS > 0 ? TAPS - 1 : a.taps - 1;
     const bool in = c < a.inner, ok = a.start_pos >= 0 && a.start_pos + a.n_tokens <= a.seq_len;
-    float2 w[TAPS > 0 ? TAPS : 1], bias = make_float2(0.f, 0.f);
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 w[TAPS > 0 ? TAPS : 1], bias = zero;
     if (in && blockIdx.z == 0) {  // constants: ahead of the dependency wait
-        bias = __ldg(reinterpret_cast<const float2*>(a.conv_b + c));
+        bias = __ldg(reinterpret_cast<const float4*>(a.conv_b + c));
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) w[j] = __ldg(reinterpret_cast<const float2*>(a.conv_w + (size_t)j * a.inner_rows + c));
+        for (int j = 0; j < TAPS; ++j) w[j] = __ldg(reinterpret_cast<const float4*>(a.conv_w + (size_t)j * a.inner_rows + c));
     }
     pdl_wait();
     if (!ok && tid == 0) atomicOr(&a.st->status, kStatusBadPos);
     if (!ok || !in) return;
     if (blockIdx.z == 1) {
-        float2 v[kConvTokens];
+        float4 v[kConvTokens];
+        prefill_sums(a.part, n_rows, a.splits, a.n_tokens, t0, a.inner_rows + c, v);
 #pragma unroll
         for (int i = 0; i < kConvTokens; ++i)
-            if (t0 + i < a.n_tokens) v[i] = prefill_sum2(a.part, n_rows, a.splits, t0 + i, a.inner_rows + c);
-#pragma unroll
-        for (int i = 0; i < kConvTokens; ++i)
-            if (t0 + i < a.n_tokens) *reinterpret_cast<float2*>(a.z + (size_t)(t0 + i) * a.x_pitch + c) = make_float2(silu_f(v[i].x), silu_f(v[i].y));
+            if (t0 + i < a.n_tokens) *reinterpret_cast<float4*>(a.z + (size_t)(t0 + i) * a.x_pitch + c) = silu4(v[i]);
         return;
     }
-    // input i of the thread: token t0 - slots + i; zero before the first position
-    auto input = [&](int i) -> float2 {
-        const int t = t0 - slots + i;
-        if (t >= a.n_tokens) return make_float2(0.f, 0.f);
-        float2 v = make_float2(0.f, 0.f);
-        if (t >= 0)
-            v = prefill_sum2(a.part, n_rows, a.splits, t, c);
-        else if (a.start_pos + t >= 0)
-            v = __ldcg(reinterpret_cast<const float2*>(a.ring + (size_t)((a.start_pos + t) % slots) * a.inner_rows + c));
-        return v;
+    // Input i of the thread is that of token t0 - slots + i: a product, from the ring, or zero before the first position.
+    auto earlier = [&](int i, const float4& v) -> float4 {
+        const int pos = a.start_pos + t0 - slots + i;
+        if (t0 - slots + i >= 0) return v;
+        return pos < 0 ? zero : __ldcg(reinterpret_cast<const float4*>(a.ring + (size_t)(pos % slots) * a.inner_rows + c));
     };
-    auto keep = [&](int i, float2 v) {
+    auto keep = [&](int i, const float4& v) {
         const int t = t0 - slots + i;
         if (t >= t0 && t >= a.n_tokens - slots && t < a.n_tokens)
-            *reinterpret_cast<float2*>(a.tail + (size_t)((a.start_pos + t) % slots) * a.inner_rows + c) = v;
+            *reinterpret_cast<float4*>(a.tail + (size_t)((a.start_pos + t) % slots) * a.inner_rows + c) = v;
     };
-    auto put = [&](int i, float2 v) {
+    auto put = [&](int i, const float4& sum) {
         const int t = t0 + i;
         if (t >= a.n_tokens) return;
-        v = make_float2(silu_f(v.x), silu_f(v.y));
-        *reinterpret_cast<float2*>(a.x + (size_t)t * a.x_pitch + c) = v;
-        __align__(4) __nv_bfloat16 hi[2], lo[2];
-        split_pair(v.x, hi[0], lo[0]);
-        split_pair(v.y, hi[1], lo[1]);
-        *reinterpret_cast<uint32_t*>(a.planes + (size_t)t * a.x_pitch + c) = *reinterpret_cast<const uint32_t*>(hi);
-        *reinterpret_cast<uint32_t*>(a.planes + (size_t)(kPrefillTokens + t) * a.x_pitch + c) = *reinterpret_cast<const uint32_t*>(lo);
+        const float4 v = silu4(sum);
+        *reinterpret_cast<float4*>(a.x + (size_t)t * a.x_pitch + c) = v;
+        const float x[4] = {v.x, v.y, v.z, v.w};
+        __align__(8) __nv_bfloat16 hi[4], lo[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) split_pair(x[k], hi[k], lo[k]);
+        *reinterpret_cast<uint2*>(a.planes + (size_t)t * a.x_pitch + c) = *reinterpret_cast<const uint2*>(hi);
+        *reinterpret_cast<uint2*>(a.planes + (size_t)(kPrefillTokens + t) * a.x_pitch + c) = *reinterpret_cast<const uint2*>(lo);
     };
     if constexpr (TAPS > 0) {
         constexpr int N = kConvTokens + TAPS - 1;
-        float2 v[N];
+        float4 v[N];
+        prefill_sums(a.part, n_rows, a.splits, a.n_tokens, t0 - slots, c, v);
+        if constexpr (TAPS > 1) {
+            if (t0 < slots)
 #pragma unroll
-        for (int i = 0; i < N; ++i) v[i] = input(i);
-        if constexpr (TAPS > 1)
+                for (int i = 0; i < TAPS - 1; ++i) v[i] = earlier(i, v[i]);
+            if (t0 + kConvTokens > a.n_tokens - slots)
 #pragma unroll
-            for (int i = 0; i < N; ++i) keep(i, v[i]);
+                for (int i = 0; i < N; ++i) keep(i, v[i]);
+        }
 #pragma unroll
         for (int i = 0; i < kConvTokens; ++i) {
-            float2 s = bias;
+            float4 s = bias;
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) s = make_float2(fmaf(w[j].x, v[i + j].x, s.x), fmaf(w[j].y, v[i + j].y, s.y));
+            for (int j = 0; j < TAPS; ++j) s = fma4(w[j], v[i + j], s);
             put(i, s);
         }
     } else {
         for (int i = 0; i < kConvTokens + slots; ++i) {
-            const float2 v = input(i);
-            keep(i, v);
-            cv_in[i * kConvThreads + tid] = v;
+            float4 v[1];
+            prefill_sums(a.part, n_rows, a.splits, a.n_tokens, t0 - slots + i, c, v);
+            v[0] = earlier(i, v[0]);
+            if (slots > 0) keep(i, v[0]);
+            cv_in[i * kConvThreads + tid] = v[0];
         }
         for (int i = 0; i < kConvTokens; ++i) {
-            float2 s = bias;
-            for (int j = 0; j <= slots; ++j) {
-                const float2 wj = __ldg(reinterpret_cast<const float2*>(a.conv_w + (size_t)j * a.inner_rows + c)), v = cv_in[(i + j) * kConvThreads + tid];
-                s = make_float2(fmaf(wj.x, v.x, s.x), fmaf(wj.y, v.y, s.y));
-            }
+            float4 s = bias;
+            for (int j = 0; j <= slots; ++j)
+                s = fma4(__ldg(reinterpret_cast<const float4*>(a.conv_w + (size_t)j * a.inner_rows + c)), cv_in[(i + j) * kConvThreads + tid], s);
             put(i, s);
         }
     }
@@ -219,8 +244,10 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
     float* dts = zs + a.tile_tokens * CH;       // [tile_tokens][CH]
     const int tid = threadIdx.x, ln = tid % L, cl = tid / L, c0 = blockIdx.x * CH, c = c0 + cl;
     const bool in = c < a.inner;
-    const int pieces = a.state_pitch / 4;
+    constexpr int pieces = L * NS;
     const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4* A4 = reinterpret_cast<const float4*>(a.A) + (size_t)(in ? c : 0) * pieces + ln;
+    float4* S4 = reinterpret_cast<float4*>(a.S) + (size_t)(in ? c : 0) * pieces + ln;
     pdl_launch_dependents();
     // weights: ahead of the dependency wait
     for (int i = tid; i < CH * (a.dt_pitch / 8); i += kScanThreads) {
@@ -232,9 +259,9 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
         *reinterpret_cast<float4*>(d) = make_float4(f0.x, f0.y, f1.x, f1.y);
         *reinterpret_cast<float4*>(d + 4) = make_float4(f2.x, f2.y, f3.x, f3.y);
     }
-    float4 A[NS], S[NS];
+    ScanPiece A[NS], S[NS];
 #pragma unroll
-    for (int i = 0; i < NS; ++i) A[i] = in && ln + i * L < pieces ? __ldg(reinterpret_cast<const float4*>(a.A + (size_t)c * a.state_pitch) + ln + i * L) : zero;
+    for (int i = 0; i < NS; ++i) A[i] = scan_piece(__ldg(A4 + i * L));
     const float D = in ? __ldg(a.D + c) : 0.f;
     const int tx = tid % TX, ty = tid / TX;
     float bias[CPT];
@@ -256,8 +283,7 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
         cp_async_commit();
         if (t0 == 0) {
 #pragma unroll
-            for (int i = 0; i < NS; ++i)
-                S[i] = in && a.start_pos > 0 && ln + i * L < pieces ? __ldcg(reinterpret_cast<const float4*>(a.S + (size_t)c * a.state_pitch) + ln + i * L) : zero;
+            for (int i = 0; i < NS; ++i) S[i] = scan_piece(a.start_pos > 0 ? __ldcg(S4 + i * L) : zero);
             // the convolution inputs that the next portion needs
             if (a.taps > 1) {
                 const int slots = a.taps - 1, keep = min(slots, a.n_tokens);
@@ -271,32 +297,32 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
         cp_async_wait<0>();
         __syncthreads();
         for (int tb = 0; tb < nt; tb += TPT * TY) {
-            float acc[TPT][CPT];
+            f32x2 acc[TPT][CPT];
 #pragma unroll
             for (int i = 0; i < TPT; ++i)
 #pragma unroll
-                for (int j = 0; j < CPT; ++j) acc[i][j] = 0.f;
+                for (int j = 0; j < CPT; ++j) acc[i][j] = both(0.f);
             int at[TPT];
 #pragma unroll
             for (int i = 0; i < TPT; ++i) at[i] = min(tb + ty + i * TY, nt - 1) * LP;  // beyond the tile: not used
+#pragma unroll 2
             for (int k = 0; k < a.dt_pitch; k += 4) {
-                float4 l[TPT], w[CPT];
+                ScanPiece l[TPT], w[CPT];
 #pragma unroll
-                for (int i = 0; i < TPT; ++i) l[i] = *reinterpret_cast<const float4*>(low + at[i] + k);
+                for (int i = 0; i < TPT; ++i) l[i] = scan_piece(*reinterpret_cast<const float4*>(low + at[i] + k));
 #pragma unroll
-                for (int j = 0; j < CPT; ++j) w[j] = *reinterpret_cast<const float4*>(wd + (tx + j * TX) * WP + k);
+                for (int j = 0; j < CPT; ++j) w[j] = scan_piece(*reinterpret_cast<const float4*>(wd + (tx + j * TX) * WP + k));
 #pragma unroll
                 for (int i = 0; i < TPT; ++i)
 #pragma unroll
-                    for (int j = 0; j < CPT; ++j)
-                        acc[i][j] = fmaf(l[i].x, w[j].x, fmaf(l[i].y, w[j].y, fmaf(l[i].z, w[j].z, fmaf(l[i].w, w[j].w, acc[i][j]))));
+                    for (int j = 0; j < CPT; ++j) acc[i][j] = fma2(l[i].hi, w[j].hi, fma2(l[i].lo, w[j].lo, acc[i][j]));
             }
 #pragma unroll
             for (int i = 0; i < TPT; ++i) {
                 const int t = tb + ty + i * TY;
 #pragma unroll
                 for (int j = 0; j < CPT; ++j)  // a step of size 0 leaves the state alone: what fills up the last four tokens
-                    if (t < a.tile_tokens) dts[t * CH + tx + j * TX] = t < nt ? softplus_f(acc[i][j] + bias[j]) : 0.f;
+                    if (t < a.tile_tokens) dts[t * CH + tx + j * TX] = t < nt ? softplus_f(pair_sum(acc[i][j]) + bias[j]) : 0.f;
             }
         }
         __syncthreads();
@@ -307,12 +333,11 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
                 const int tk = min(t + k, nt - 1);
                 const float dt = dts[(t + k) * CH + cl], dx = dt * xs[tk * CH + cl];
                 const float4* B = reinterpret_cast<const float4*>(low + tk * LP + a.dt_pitch);
-                y[k] = 0.f;
+                f32x2 y2 = both(0.f);
 #pragma unroll
-                for (int i = 0; i < NS; ++i) {
-                    const int q = ln + i * L;
-                    if (q < pieces) y[k] += mamba_update(S[i], A[i], B[q], B[pieces + q], dt, dx);
-                }
+                for (int i = 0; i < NS; ++i)
+                    mamba_update(S[i], A[i], scan_piece(B[ln + i * L]), scan_piece(B[pieces + ln + i * L]), both(dt), both(dx), y2);
+                y[k] = pair_sum(y2);
             }
             const float sum = lane_group_sum4<L>(y, ln);
             const int mine = t + scan_token(ln);
@@ -333,8 +358,7 @@ static __global__ void __launch_bounds__(kScanThreads) mamba_scan_kernel(const M
     }
     if (!in) return;
 #pragma unroll
-    for (int i = 0; i < NS; ++i)
-        if (ln + i * L < pieces) *(reinterpret_cast<float4*>(a.S + (size_t)c * a.state_pitch) + ln + i * L) = S[i];
+    for (int i = 0; i < NS; ++i) S4[i * L] = scan_float4(S[i]);
 }
 
 }  // namespace lpp
