@@ -2701,7 +2701,8 @@ static lpp_status prefill_mamba_mixer(lpp_engine* e, int l, int n, int start_pos
     MambaScanArgs a = mamba_scan_args(e, y, r);
     int splits;
     TRY(prefill_partial_sums(e, y.m_low, y.x_low, y.low_rows, y.inner_pitch, n, start_pos, &splits, kLowMaxSplits));
-    CU(launch_kernel(mamba_low_kernel, dim3(n), dim3(kLowThreads), 0, e->stream, true, a, (const float*)e->pf_part, splits, e->pf_low));
+    CU(launch_kernel(mamba_low_kernel, dim3(n, (y.dt_pitch + 2 * y.state_pitch + kLowColumns - 1) / kLowColumns), dim3(kLowThreads), 0, e->stream, true,
+                     a, (const float*)e->pf_part, splits, e->pf_low));
     a.low = e->pf_low;
     a.n_tokens = n;
     a.start_pos = start_pos;

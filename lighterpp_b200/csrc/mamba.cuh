@@ -152,16 +152,14 @@ __device__ __forceinline__ float lane_group_sum(float v) {
     for (int o = L / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
     return v;
 }
-// Element i of a token's dt | B | C row with dt padded to dt_pitch, B and C to state_pitch, with zeros.
-__device__ __forceinline__ float mamba_low(const MambaScanArgs& a, const float* src, int i) {
-    int n = a.dt_rank, from = 0;
-    if (i >= a.dt_pitch) {
-        i -= a.dt_pitch;
-        n = a.state;
-        from = a.dt_rank;
-        if (i >= a.state_pitch) i -= a.state_pitch, from += a.state;
-    }
-    return i < n ? __ldcg(src + from + i) : 0.f;
+// Where element i of a token's padded dt | B | C row (dt to dt_pitch, B and C to state_pitch) lies in the unpadded one; -1 =
+// padding.
+__device__ __forceinline__ int mamba_low_source(const MambaScanArgs& a, int i) {
+    if (i < a.dt_pitch) return i < a.dt_rank ? i : -1;
+    i -= a.dt_pitch;
+    const int from = i < a.state_pitch ? a.dt_rank : a.dt_rank + a.state;
+    if (i >= a.state_pitch) i -= a.state_pitch;
+    return i < a.state ? from + i : -1;
 }
 
 // One token.  grid: ceil(inner / (kScanStepThreads / L)); shared memory: dt_pitch + 2 state_pitch floats
@@ -195,7 +193,11 @@ static __global__ void __launch_bounds__(kScanStepThreads) mamba_step_kernel(con
     const float bias = in ? __ldg(a.dt_b + c) : 0.f, D = in ? __ldg(a.D + c) : 0.f;
     pdl_wait();
     const float x = in ? __ldcg(a.x + c) : 0.f, z = in ? __ldcg(a.z + c) : 0.f;
-    for (int i = tid; i < a.dt_pitch + 2 * a.state_pitch; i += kScanStepThreads) sc_low[i] = mamba_low(a, a.low, i);
+    for (int i = tid; i < a.dt_pitch + 2 * a.state_pitch; i += kScanStepThreads) {
+        const int src = mamba_low_source(a, i);
+        const float v = __ldcg(a.low + max(src, 0));
+        sc_low[i] = src >= 0 ? v : 0.f;
+    }
     __syncthreads();
     float dot = 0.f;
     auto mul = [&](const uint4& u, int v) {

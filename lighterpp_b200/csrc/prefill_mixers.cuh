@@ -183,27 +183,35 @@ static __global__ void __launch_bounds__(kConvThreads) mamba_conv_kernel(const M
 }
 
 // dt | B | C rows after their GEMM, whose row tiles are few and whose K is therefore cut into up to kLowMaxSplits ranges:
-// partial sums added in range order, sections padded with zeros to dt_pitch and state_pitch.  grid: tokens
-constexpr int kLowMaxSplits = 32, kLowThreads = 256;
+// partial sums added in range order (in kLowGroups groups), sections padded with zeros to dt_pitch and state_pitch.
+// grid: (tokens, ceil(row / kLowColumns))
+constexpr int kLowMaxSplits = 32, kLowColumns = 64, kLowGroups = 4, kLowThreads = kLowColumns * kLowGroups;
 // floats per row, an odd number of 16-byte pieces (rows on different banks of shared memory)
 __host__ __device__ inline int mamba_low_pitch(int dt_pitch, int state_pitch) {
     const int n = dt_pitch + 2 * state_pitch;
     return (n / 4) % 2 ? n : n + 4;
 }
 static __global__ void __launch_bounds__(kLowThreads) mamba_low_kernel(const MambaScanArgs a, const float* part, int splits, float* out) {
+    __shared__ float group_sum[kLowGroups][kLowColumns];
     pdl_launch_dependents();
+    const int t = blockIdx.x, tid = threadIdx.x, col = tid % kLowColumns, group = tid / kLowColumns, i = (int)blockIdx.y * kLowColumns + col;
+    const int src = mamba_low_source(a, i);  // -1: padding
+    constexpr int N = kLowMaxSplits / kLowGroups;
+    const int per = (splits + kLowGroups - 1) / kLowGroups, s0 = group * per, n = min(per, splits - s0);
     pdl_wait();
-    const int t = blockIdx.x, n_low = a.dt_pitch + 2 * a.state_pitch;
-    for (int i = threadIdx.x; i < n_low; i += kLowThreads) {
-        float v[kLowMaxSplits], sum = 0.f;
+    const float* p = part + ((size_t)s0 * kPrefillTokens + t) * a.low_rows + max(src, 0);
+    float v[N], sum = 0.f;
 #pragma unroll
-        for (int s = 0; s < kLowMaxSplits; ++s)
-            if (s < splits) v[s] = mamba_low(a, part + ((size_t)s * kPrefillTokens + t) * a.low_rows, i);
+    for (int s = 0; s < N; ++s) v[s] = s < n ? __ldcg(p + (size_t)s * kPrefillTokens * a.low_rows) : 0.f;
 #pragma unroll
-        for (int s = 0; s < kLowMaxSplits; ++s)
-            if (s < splits) sum += v[s];
-        out[(size_t)t * mamba_low_pitch(a.dt_pitch, a.state_pitch) + i] = sum;
-    }
+    for (int s = 0; s < N; ++s) sum += v[s];
+    group_sum[group][col] = sum;
+    __syncthreads();
+    if (group != 0 || i >= a.dt_pitch + 2 * a.state_pitch) return;
+    sum = 0.f;
+#pragma unroll
+    for (int g = 0; g < kLowGroups; ++g) sum += group_sum[g][col];
+    out[(size_t)t * mamba_low_pitch(a.dt_pitch, a.state_pitch) + i] = src >= 0 ? sum : 0.f;
 }
 
 // The recurrence over a prompt block.  A CTA owns kScanThreads / L channels and walks the block in tiles of tile_tokens:
