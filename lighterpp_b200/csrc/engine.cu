@@ -2535,7 +2535,8 @@ static lpp_status prefill_norm(lpp_engine* e, int n, const float* w, const float
 
 // x += W . in  for the block: output and down projection.  Returns the number of partial sums the next norm adds.
 static lpp_status prefill_resid(lpp_engine* e, const CUtensorMap& wm, int row0, const CUtensorMap& xm, int K, int n, int start_pos, int* parts) {
-    PrefillGemmArgs g = prefill_gemm_args(e, (e->c.dim + 1) & ~1, K, n, start_pos);
+    // all Dp columns: beyond dim the products are zero (rows outside the map), and so are the partial sums that the norm adds
+    PrefillGemmArgs g = prefill_gemm_args(e, e->Dp, K, n, start_pos);
     g.row0 = row0;
     g.x = e->pf_x;
     g.x_pitch = e->Dp;

@@ -178,6 +178,16 @@ def test_sizes_off_every_grid(E, dtype):
     e.close()
 
 
+@pytest.mark.parametrize("width,ff", [(71, 300), (130, 700)])
+def test_padding_of_narrow_rows_stays_zero(E, width, ff):
+    """Residual products cut along K whose rows are narrower than the row pitch: partial sums of the padding are zero too."""
+    cfg = model([(mixer(heads=9, vdim=24), ff), (mixer(), ff)], width=width)
+    W, toks = R.random_weights(cfg, ff), tokens(cfg, 100, ff)
+    e = engine(E, cfg, W, "bfloat16")
+    check(portions(e, toks, [70, 2, 28]), R.forward(cfg, W, toks), "bfloat16")
+    e.close()
+
+
 @pytest.mark.parametrize("heads,kv_rank,rot_dim,window", [(4, 96, 16, 30), (16, 200, 8, 100), (12, 512, 64, 150), (24, 128, 16, 20),
                                                           (33, 256, 32, 64), (20, 448, 64, 0), (3, 640, 16, 90), (17, 8, 2, 65)])
 def test_attention_instantiations(E, heads, kv_rank, rot_dim, window):
