@@ -557,9 +557,8 @@ static __global__ void __launch_bounds__(256) prefill_qkv_finish_kernel(const Pr
 
 // Rows of the residual stream -> normalised rows (hi + lo MMA operands): RMSNorm, or LayerNorm when a bias is given.
 // Layer 0 takes the embedding rows of the prompt tokens, times their factor, and also writes them out as the FP32 residual
-// stream.  With a
-// row list, block i takes row rows[i] (the positions whose logits are wanted).  D is the row pitch; the statistics cover
-// the first norm_n inputs, the rest is zero padding with zero weights.  grid: rows.
+// stream.  With a row list, block i takes row rows[i] (the positions whose logits are wanted).  D is the row pitch; the
+// statistics cover the first norm_n inputs, the rest is zero padding with zero weights.  grid: rows.
 constexpr int kPfNormThreads = 512;
 struct PrefillNormArgs {
     float* x;            // [kPrefillTokens][D]

@@ -326,7 +326,7 @@ class Engine:
         return k, v
 
     def latent_read(self, layer: int, pos: int) -> np.ndarray:
-        """One cache row of a latent-attention layer outside a loop's reach: normed latent, then the rotated key part."""
+        """One cache row of a latent-attention layer (of a model without a loop): normed latent, then the rotated key part."""
         m = self.cfg.layers[layer].mixer
         row = np.empty(m.kv_rank + m.rot_dim, dtype=np.float32)
         _check(self.lib.lpp_latent_read(self.h, layer, pos, row.ctypes.data_as(C.POINTER(C.c_float))), "lpp_latent_read")

@@ -460,8 +460,7 @@ def test_incomplete_and_wrong_descriptions_are_refused(E, small):
         with pytest.raises(E.LppError):
             e.upload(name, np.zeros((4, 4), np.float32), layer)
     with pytest.raises(E.LppError, match="keeps no latents"):
-        e.latent_read(0, 0) if hasattr(e.cfg.layers[0].mixer, "kv_rank") else E._check(
-            e.lib.lpp_latent_read(e.h, 0, 0, np.zeros(8, np.float32).ctypes.data_as(E.C.POINTER(E.C.c_float))), "lpp_latent_read")
+        E._check(e.lib.lpp_latent_read(e.h, 0, 0, np.zeros(8, np.float32).ctypes.data_as(E.C.POINTER(E.C.c_float))), "lpp_latent_read")
     e.close()
     for change in (lambda c: setattr(c.layers[1].mixer, "kv_heads", 3), lambda c: setattr(c.layers[1].mixer.rotation, "dims", 26),
                    lambda c: setattr(c.layers[1].mixer.rotation, "dims", 7), lambda c: setattr(c.layers[0].mixer, "state", 2000),
